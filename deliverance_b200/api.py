@@ -120,6 +120,10 @@ def build_model(cfg: ModelConfig, device, dtype, tp: TensorParallelContext):
         from .models.gemma4 import Gemma4Model
 
         return Gemma4Model(cfg, device, dtype, tp)
+    if cfg.model_type == "fatotar":
+        from .models.fatotar import FatotarModel
+
+        return FatotarModel(cfg, device, dtype, tp)
     return DecoderModel(cfg, device, dtype, tp)
 
 

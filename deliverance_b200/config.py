@@ -18,8 +18,10 @@ from dataclasses import dataclass, field
 from typing import Any, Optional
 
 SUPPORTED_MODEL_TYPES = (
-    "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert",
+    "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert", "fatotar",
 )
+# designs whose config.json names an architecture instead of a model_type
+_ARCHITECTURE_TYPES = {"fatotar": "fatotar"}
 
 # transformers' Gemma3TextConfig defaults: hub configs of the multimodal checkpoints leave most text fields out
 _GEMMA3_TEXT_DEFAULTS = dict(vocab_size=262208, hidden_size=2304, intermediate_size=9216, num_hidden_layers=26, num_attention_heads=8,
@@ -54,7 +56,7 @@ class ModelConfig:
     attn_softcap: float = 0.0
     final_softcap: float = 0.0
     sliding_window: int = 0
-    layer_types: tuple[str, ...] = ()  # per layer: "attention" | "sliding" | "mamba"
+    layer_types: tuple[str, ...] = ()  # per layer: "attention" | "sliding" | "mamba" | "latent"
     # norms
     norm_weight_offset: float = 0.0  # gemma: (1 + w)
     post_norms: bool = False  # gemma2: post-attention and post-feedforward norms
@@ -188,6 +190,48 @@ def _parse_gemma4(outer: dict) -> ModelConfig:
     return cfg
 
 
+def config_model_type(d: dict) -> Optional[str]:
+    """``model_type`` of a parsed ``config.json``; configs without one are recognised by their ``architecture``."""
+    mt = d.get("model_type")
+    return mt if mt else _ARCHITECTURE_TYPES.get(str(d.get("architecture", "")).lower())
+
+
+def layer_run_order(n_layers: int, loop: Optional[dict]) -> tuple[int, ...]:
+    """Weight-layer index of every layer run: layers ``start .. stop - 1`` run ``times`` times in a row, the rest once."""
+    if not loop:
+        return tuple(range(n_layers))
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not (0 <= start < stop <= n_layers and times >= 1):
+        raise ValueError(f"loop {loop} does not fit {n_layers} layers")
+    return tuple(range(start)) + tuple(range(start, stop)) * times + tuple(range(stop, n_layers))
+
+
+def _parse_fatotar(d: dict) -> ModelConfig:
+    """Fatotar: latent attention and a dense gated feed-forward side by side on one residual stream, LayerNorms, a hashed-bigram
+    embedding, a range of layers that runs several times. Every layer carries its own sizes; ``extra["layers"]`` keeps them as
+    given, ``extra["order"]`` is the weight layer of every layer run (a run has its own cache), and the layer-indexed fields of
+    :class:`ModelConfig` count runs. The context length is not part of the design: ``max_position_embeddings`` bounds what the
+    engine admits."""
+    layers = list(d["layers"])
+    for i, L in enumerate(layers):
+        if L["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: unknown mixer '{L['type']}'")
+        if L.get("mlp") and L["mlp"]["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward '{L['mlp']['kind']}'")
+    order = layer_run_order(len(layers), d.get("loop"))
+    mixers = [L["mixer"] for L in layers]
+    cfg = ModelConfig(
+        model_type="fatotar", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), num_layers=len(order),
+        num_heads=max(int(m["heads"]) for m in mixers), num_kv_heads=1, head_dim=max(int(m["kv_rank"]) for m in mixers),
+        intermediate_size=max([int(L["mlp"]["ff"]) for L in layers if L.get("mlp")] or [0]),
+        max_position_embeddings=int(d.get("max_position_embeddings") or 131072), norm_eps=float(d["norm"]["eps"]), hidden_act="relu",
+        embedding_multiplier=float(d["embedding"].get("scale", 1.0)), bos_token_id=d.get("bos_token_id"), eos_token_ids=_eos(d.get("eos_token_id")),
+        pad_token_id=d.get("pad_token_id"), layer_types=tuple("latent" for _ in order), use_rope=False, add_bos=False, raw=d,
+    )
+    cfg.extra = {"layers": layers, "order": order, "bigram": d["embedding"].get("bigram")}
+    return cfg
+
+
 def _eos(v: Any) -> tuple[int, ...]:
     if v is None:
         return ()
@@ -207,9 +251,11 @@ def _rope(d: dict, default_theta: float) -> tuple[float, float]:
 
 
 def parse_config(d: dict) -> ModelConfig:
-    mt = d.get("model_type")
+    mt = config_model_type(d)
     if mt not in SUPPORTED_MODEL_TYPES:
         raise ValueError(f"unsupported model_type '{mt}' (supported: {', '.join(SUPPORTED_MODEL_TYPES)})")
+    if mt == "fatotar":
+        return _parse_fatotar(d)
     if mt in ("gemma4", "gemma4_text"):
         return _parse_gemma4(d)
     if mt in ("gemma3", "gemma3_text"):

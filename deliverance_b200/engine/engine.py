@@ -57,6 +57,7 @@ class Request:
     fill: Optional[list] = None  # tokens whose KV must be cached before decoding: the prompt, or after a preemption prompt + output[:-1]
     resumed: bool = False  # re-admitted after a preemption: the prefill only rebuilds the cache, nothing is sampled from it
     preemptions: int = 0
+    replay: bool = False  # tokens are given step by step (Engine.replay_step), the scheduler leaves it alone
     t_progress: float = 0.0
 
     def __post_init__(self):
@@ -137,6 +138,7 @@ class Engine:
         # (a family that runs on the PyTorch operator set reads lengths on the host inside its forward: not capturable)
         self.use_graphs = bool(self.config.cuda_graphs and self.device.type == "cuda" and getattr(model, "supports_cuda_graphs", True))
         self.hybrid = mamba_shapes is not None
+        self.needs_prev = bool(getattr(model, "reads_previous_token", False))  # batches carry the token in front of every token
         # one-step lookahead of greedy graph decode: the step in flight whose sampled tokens the host has not read yet
         self._inflight: Optional[dict] = None
         # ("force" runs the same schedule without CUDA graphs: the host-side logic is then testable on a CPU)
@@ -164,6 +166,8 @@ class Engine:
         limit = min(params.ntokens or ctx, ctx)
         if len(prompt) == 0:
             raise ValueError("empty prompt")
+        if any(r.replay for r in self.running):
+            raise RuntimeError("replay and generation do not share an engine at the same time")
         if len(prompt) >= limit:
             raise ValueError(f"prompt has {len(prompt)} tokens, which does not fit ntokens={limit}")
         if min(prompt) < 0 or max(prompt) >= self.cfg.vocab_size:
@@ -371,8 +375,7 @@ class Engine:
                         break
             if r.state != RUNNING or not self._reserve(r, r.computed + n):
                 continue  # preempted by an older request of this step, or waiting for older requests to release pages
-            seqs.append({"tokens": r.fill[r.computed : r.computed + n], "start": r.computed, "pages": r.pages,
-                         "state_slot": max(r.state_slot, 0)})
+            seqs.append(self._portion(r, n))
             chosen.append((r, n))
             budget -= n
         if not seqs:
@@ -406,6 +409,73 @@ class Engine:
             finished = self._sample_and_advance(done_reqs, sub)
         return finished
 
+    def _portion(self, r: Request, n: int) -> dict:
+        """Batch entry of the next ``n`` tokens of ``r.fill``."""
+        s = {"tokens": r.fill[r.computed : r.computed + n], "start": r.computed, "pages": r.pages, "state_slot": max(r.state_slot, 0)}
+        if self.needs_prev:
+            s["prev"] = r.fill[r.computed - 1] if r.computed > 0 else -1
+        return s
+
+    # ------------------------------------------------------------------------------------------------ replay of given tokens
+    def open_replay(self) -> Request:
+        """A request whose tokens are given step by step (:meth:`replay_step`) instead of being sampled. It holds a place, pages and
+        a state slot like any other running request until :meth:`close_replay`."""
+        if self.waiting or self._inflight is not None or any(not r.replay for r in self.running):
+            raise RuntimeError("replay and generation do not share an engine at the same time")
+        if len(self.running) >= self.config.max_seqs:
+            raise MemoryError(f"all {self.config.max_seqs} sequence places are taken")
+        r = Request(self._next_id, [], GeneratorParameters(), state=RUNNING, replay=True)
+        self._next_id += 1
+        if self.hybrid:
+            r.state_slot = self.kv.alloc_state_slot()
+        self.running.append(r)
+        return r
+
+    def close_replay(self, r: Request) -> None:
+        self._finish(r, FinishReason.CANCELLED)
+
+    def replay_step(self, entries: list) -> Optional[torch.Tensor]:
+        """One batch of ``(request, next tokens, wanted places among them)``: prompt portions and single tokens together, exactly the
+        forward passes of a scheduled step (a batch of single tokens of started requests is a decode step, captured graph included).
+        Returns fp32 logits of the wanted places in order, or None when nothing is wanted."""
+        seqs, rows, base = [], [], 0
+        for r, tokens, want in entries:
+            if not tokens:
+                raise ValueError("an entry needs at least one token")
+            if min(tokens) < 0 or max(tokens) >= self.cfg.vocab_size:
+                raise ValueError(f"token ids must lie in [0, {self.cfg.vocab_size})")
+            if any(not 0 <= w < len(tokens) for w in want):
+                raise ValueError("wanted place outside the entry")
+            r.fill.extend(int(t) for t in tokens)
+            if len(r.fill) > self.cfg.max_position_embeddings:
+                raise ValueError(f"more than {self.cfg.max_position_embeddings} tokens")
+            self.kv.ensure_pages(r.pages, len(r.fill))
+            s = self._portion(r, len(tokens))
+            s["rid"] = (r.rid, r.preemptions)
+            seqs.append(s)
+            rows += [base + w for w in want]
+            base += len(tokens)
+        B = len(seqs)
+        decode = all(len(s["tokens"]) == 1 and s["start"] > 0 for s in seqs)
+        self.metrics["decode_steps" if decode else "prefill_steps"] += 1
+        if decode and self.use_graphs and B <= _BUCKETS[-1]:
+            logits = self._graph_decode(seqs)[:B]
+        else:
+            batch = make_batch(seqs, self.page_size, self.device)
+            if decode:
+                batch.decode_splits = self._splits(B)
+            else:
+                batch.logits_rows = torch.tensor(rows, dtype=torch.int64).to(self.device)
+            logits = self.model.forward(batch, self.kv)
+            decode = decode or batch.is_decode
+        for r, tokens, _ in entries:
+            r.computed += len(tokens)
+        if not rows:
+            return None
+        if decode:  # one row per entry; batches of portions return the wanted rows only
+            logits = logits.index_select(0, torch.tensor(rows, dtype=torch.int64, device=logits.device))
+        return self._full(logits)
+
     # ------------------------------------------------------------------------------------------------ decode
     def _decode_inputs(self, reqs: list[Request]):
         seqs = []
@@ -414,6 +484,10 @@ class Engine:
             self.kv.ensure_pages(r.pages, pos + 1)
             seqs.append({"tokens": [r.output[-1] if r.output else 0], "start": pos, "pages": r.pages, "state_slot": max(r.state_slot, 0),
                          "rid": (r.rid, r.preemptions)})
+            if self.needs_prev:
+                # the token in front of the one being fed: with a step in flight that is the newest token the host knows
+                before = len(r.output) - (1 if r.pending == 0 else 0)
+                seqs[-1]["prev"] = r.output[before - 1] if before > 0 else r.prompt[-1]
         return seqs
 
     def _plain_greedy(self, reqs: list[Request]) -> bool:
@@ -574,6 +648,8 @@ class Engine:
                 bt[i, : len(pg)] = torch.tensor(pg, dtype=torch.int32)
         for i in range(n, bucket):
             owners[i] = None
+        if self.needs_prev:
+            h["prev"][:n] = torch.tensor([s["prev"] for s in seqs], dtype=torch.int32)
         if self.hybrid:
             h["st"][:n] = torch.tensor([s["state_slot"] for s in seqs], dtype=torch.int64)
         if n < bucket:
@@ -592,7 +668,9 @@ class Engine:
         b.block_tables[:, :width].copy_(bt[:, :width], non_blocking=True)
         if b.state_slots is not None:
             b.state_slots.copy_(h["st"], non_blocking=True)
-        self.metrics["h2d_bytes"] = self.metrics.get("h2d_bytes", 0) + bucket * (4 + 4 + 8 + 4 + 4 * width)
+        if b.prev_ids is not None:
+            b.prev_ids.copy_(h["prev"], non_blocking=True)
+        self.metrics["h2d_bytes"] = self.metrics.get("h2d_bytes", 0) + bucket * (4 + 4 + 8 + 4 + 4 * width + (4 if b.prev_ids is not None else 0))
         g["graph"].replay()
         self.metrics["graph_replays"] += 1
         self.metrics["kernel_launches"] += g["launches"]
@@ -612,6 +690,7 @@ class Engine:
             logits_rows=torch.arange(bucket, dtype=torch.int64, device=dev),
             decode_splits=self._splits(bucket),
             state_slots=torch.zeros(bucket, dtype=torch.int64, device=dev) if self.hybrid else None,
+            prev_ids=torch.zeros(bucket, dtype=torch.int32, device=dev) if self.needs_prev else None,
         )
         # warm up outside capture (lazy handles, function attributes, scratch), then capture
         side = torch.cuda.Stream(device=dev)
@@ -634,6 +713,7 @@ class Engine:
             "ctx": torch.ones(bucket, dtype=torch.int32, pin_memory=pin),
             "bt": torch.zeros(bucket, self.max_pages_per_seq, dtype=torch.int32, pin_memory=pin),
             "st": torch.zeros(bucket, dtype=torch.int64, pin_memory=pin),
+            "prev": torch.zeros(bucket, dtype=torch.int32, pin_memory=pin),
         } for _ in range(2)]
         g = {"graph": graph, "batch": batch, "logits": logits, "host": host, "launches": launches, "calls": 0,
              "bt_owners": [[None] * bucket, [None] * bucket]}

@@ -13,7 +13,8 @@ whose reference counts are bumped, so a hit costs no copy and no extra memory, a
 (``max_prefix_tokens``) is a setting, not a limit of the data structure.
 
 Layout per attention layer: ``k[pages, KV, page_size, D]`` and ``v[...]`` in the working dtype; page 0 is a scratch page
-that padded batch rows write to. Recurrent (mamba) layers get per-sequence state slots instead of pages.
+that padded batch rows write to. Latent-attention layers use the same pair with one "head": ``k`` holds the compressed vectors, ``v``
+the rotated key parts shared by all heads (a width of its own, ``v_dim_per_layer``). Recurrent (mamba) layers get per-sequence state slots instead of pages.
 """
 from __future__ import annotations
 
@@ -240,6 +241,7 @@ class PagedKVCache:
         # optional per-layer shapes and cache sharing (gemma4: wide global heads, late layers reuse an earlier layer's cache)
         heads = layout.get("kv_heads_per_layer") or [layout["kv_heads"]] * len(kinds)
         dims = layout.get("head_dim_per_layer") or [layout["head_dim"]] * len(kinds)
+        v_dims = layout.get("v_dim_per_layer") or dims
         shared = layout.get("shared_from") or [-1] * len(kinds)
         for i, kind in enumerate(kinds):
             if kind == "mamba":
@@ -249,9 +251,9 @@ class PagedKVCache:
                 self.k.append(self.k[shared[i]])
                 self.v.append(self.v[shared[i]])
             else:
-                shape = (num_pages, heads[i], self.page_size, dims[i])
-                self.k.append(torch.zeros(shape, dtype=dtype, device=self.device))
-                self.v.append(torch.zeros(shape, dtype=dtype, device=self.device))
+                shape = (num_pages, heads[i], self.page_size)
+                self.k.append(torch.zeros(shape + (dims[i],), dtype=dtype, device=self.device))
+                self.v.append(torch.zeros(shape + (v_dims[i],), dtype=dtype, device=self.device))
         self.allocator = PageAllocator(num_pages)
         self.prefix = PrefixCache(self.settings, self.allocator)
         self.prefix.kv = self
@@ -274,8 +276,9 @@ class PagedKVCache:
         heads = layout.get("kv_heads_per_layer") or [layout["kv_heads"]] * len(kinds)
         dims = layout.get("head_dim_per_layer") or [layout["head_dim"]] * len(kinds)
         shared = layout.get("shared_from") or [-1] * len(kinds)
-        rows = sum(heads[i] * dims[i] for i, k in enumerate(kinds) if k != "mamba" and shared[i] < 0)
-        return 2 * rows * page_size * torch.empty((), dtype=dtype).element_size()
+        v_dims = layout.get("v_dim_per_layer") or dims
+        rows = sum(heads[i] * (dims[i] + v_dims[i]) for i, k in enumerate(kinds) if k != "mamba" and shared[i] < 0)
+        return rows * page_size * torch.empty((), dtype=dtype).element_size()
 
     # -- per-sequence page management ---------------------------------------------------------------------------
     def ensure_pages(self, pages: list[int], n_tokens: int) -> None:
@@ -353,7 +356,7 @@ class PagedKVCache:
         idx = torch.tensor(pages[: (n_tokens + self.page_size - 1) // self.page_size], device=self.device, dtype=torch.long)
         kh, hd = self.k[layer].shape[1], self.k[layer].shape[3]
         k = self.k[layer][idx].permute(1, 0, 2, 3).reshape(kh, -1, hd)[:, :n_tokens]
-        v = self.v[layer][idx].permute(1, 0, 2, 3).reshape(kh, -1, hd)[:, :n_tokens]
+        v = self.v[layer][idx].permute(1, 0, 2, 3).reshape(kh, -1, self.v[layer].shape[3])[:, :n_tokens]
         return k, v
 
 

@@ -140,6 +140,11 @@ class MseTurboQuantCodec:
         return e.codes.numel() + e.norms.numel() * 4
 
 
+def _codec_for(codec: MseTurboQuantCodec, dim: int, bits: int) -> MseTurboQuantCodec:
+    """``codec`` when it fits, else one for rows of another width (layers differ in width, and so do the two halves of a latent cache)."""
+    return codec if codec.dim == dim and codec.bits == bits else MseTurboQuantCodec(dim, bits)
+
+
 def snapshot_pages(kv, pages: list[int], n_tokens: int, compression: str = "NONE", bits: int = 3) -> dict:
     """Host copy of the K/V rows of ``pages`` for every attention layer (``NONE`` | ``LZ4`` | ``DEFLATE`` | ``MSE_TURBOQUANT``)."""
     out = {"compression": compression, "n_tokens": n_tokens, "layers": {}}
@@ -150,7 +155,7 @@ def snapshot_pages(kv, pages: list[int], n_tokens: int, compression: str = "NONE
         kk, vv = kv.gather_rows(i, pages, n_tokens)
         if compression == "MSE_TURBOQUANT":
             codec = codec or MseTurboQuantCodec(kk.shape[-1], bits)
-            out["layers"][i] = (codec.encode(kk), codec.encode(vv))
+            out["layers"][i] = (_codec_for(codec, kk.shape[-1], bits).encode(kk), _codec_for(codec, vv.shape[-1], bits).encode(vv))
         elif compression in ("LZ4", "DEFLATE"):
             raw = lambda t: (block_compress(t.cpu().contiguous().view(torch.uint8).numpy().tobytes(), compression), tuple(t.shape), t.dtype)  # noqa: E731
             out["layers"][i] = (raw(kk), raw(vv))
@@ -167,7 +172,7 @@ def restore_pages(kv, snap: dict, pages: list[int]) -> None:
     for i, (ek, ev) in snap["layers"].items():
         if snap["compression"] == "MSE_TURBOQUANT":
             dt = kv.k[i].dtype if kv.k[i].dtype in (torch.float32, torch.bfloat16) else torch.float32
-            kk, vv = snap["codec"].decode(ek, dt, kv.device), snap["codec"].decode(ev, dt, kv.device)
+            kk, vv = (_codec_for(snap["codec"], e.shape[-1], e.bits).decode(e, dt, kv.device) for e in (ek, ev))
         elif snap["compression"] in ("LZ4", "DEFLATE"):
             def un(e):
                 n_out = int(torch.tensor(e[1]).prod().item()) * torch.empty(0, dtype=e[2]).element_size()

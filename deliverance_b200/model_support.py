@@ -67,7 +67,9 @@ def detect_model(model_dir_or_config: str) -> str:
         p = os.path.join(p, "config.json")
     with open(p) as f:
         d = json.load(f)
-    mt = d.get("model_type")
+    from .config import config_model_type
+
+    mt = config_model_type(d)
     if not mt:
         raise ValueError(f"{p} has no model_type")
     return str(mt).lower()

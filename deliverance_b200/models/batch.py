@@ -25,6 +25,8 @@ class ForwardBatch:
     q_len_host: list = field(default_factory=list)
     ctx_len_host: list = field(default_factory=list)
     token_types: Optional[torch.Tensor] = None  # bert
+    prev_ids: Optional[torch.Tensor] = None  # [T] int32 token before each token of its sequence (-1: none), for models that read it
+    plans: dict = field(default_factory=dict)  # per-batch work plans of model mechanisms, built once and shared by the layers
     _tiles: dict = field(default_factory=dict)  # tile height -> (tile_seq, tile_q0) device tensors
 
     def tiles(self, rows: int):
@@ -53,7 +55,8 @@ class ForwardBatch:
 def make_batch(seqs: list[dict], page_size: int, device, max_pages: Optional[int] = None) -> ForwardBatch:
     """Build a batch from host-side sequence descriptions.
 
-    Each entry: ``{"tokens": [new token ids], "start": first position, "pages": [page ids], "state_slot": int}``.
+    Each entry: ``{"tokens": [new token ids], "start": first position, "pages": [page ids], "state_slot": int}``. An entry may
+    carry ``"prev"``, the token in front of its first one (-1 at the start of a sequence): ``prev_ids`` is then filled.
     """
     from ..ops import prefill_tiles
 
@@ -111,9 +114,16 @@ def make_batch(seqs: list[dict], page_size: int, device, max_pages: Optional[int
     state_slots = None
     if any("state_slot" in s for s in seqs):
         state_slots = t([int(s.get("state_slot", 0)) for s in seqs], torch.int64)
+    prev_ids = None
+    if any("prev" in s for s in seqs):
+        prev = []
+        for s in seqs:
+            prev.append(int(s.get("prev", -1)))
+            prev.extend(int(x) for x in s["tokens"][:-1])
+        prev_ids = t(prev, torch.int32)
     return ForwardBatch(
         token_ids=t(toks, torch.int32), positions=t(pos, torch.int32), slots=t(slots, torch.int64), q_start=t(qs, torch.int32),
         q_len=t(ql, torch.int32), ctx_len=t(cl, torch.int32), block_tables=bt.to(dev, non_blocking=True), is_decode=is_decode,
         logits_rows=t(last, torch.int64), tile_seq=t(ts, torch.int32) if ts else None, tile_q0=t(t0, torch.int32) if ts else None,
-        state_slots=state_slots, q_len_host=ql, ctx_len_host=cl,
+        state_slots=state_slots, q_len_host=ql, ctx_len_host=cl, prev_ids=prev_ids,
     )

@@ -88,8 +88,7 @@ class DecoderModel:
         self.dtype = dtype or (torch.bfloat16 if self.device.type == "cuda" else torch.float32)
         self.tp = tp
         TensorParallelPlanner.validate(cfg, tp.size)
-        if self.device.type == "cuda" and cfg.num_heads and cfg.head_dim not in (64, 128, 256):
-            raise ValueError(f"head_dim {cfg.head_dim} is not supported by the CUDA attention kernels (64, 128, 256)")
+        self._check_kernels()
         self.n_heads = cfg.num_heads // tp.size
         self.n_kv = max(1, cfg.num_kv_heads // tp.size)  # with more ranks than KV heads, size / kv_heads ranks replicate one head
         self.layers: list[LayerWeights] = []
@@ -115,6 +114,11 @@ class DecoderModel:
         self.sp_min_rows: Optional[int] = 256 * tp.size if (tp.enabled and os.environ.get("DLV_TP_SEQ_PARALLEL", "0") == "1") else None
         self._sp = None  # (M, rows per rank, first own row, own rows) while such a forward runs
         self._sp_ordered = False
+
+    def _check_kernels(self) -> None:
+        """Refuse head sizes the family's CUDA attention kernels do not have."""
+        if self.device.type == "cuda" and self.cfg.num_heads and self.cfg.head_dim not in (64, 128, 256):
+            raise ValueError(f"head_dim {self.cfg.head_dim} is not supported by the CUDA attention kernels (64, 128, 256)")
 
     # ------------------------------------------------------------------------------------------------ loading
     def _dev(self, t: torch.Tensor, dtype=None) -> torch.Tensor:

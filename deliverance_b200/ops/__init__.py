@@ -223,6 +223,10 @@ def linear(x: torch.Tensor, w: LinearWeight, out_f32: bool = False, impl: int = 
     """``x [T, K] @ W[N, K]^T (+ bias)``."""
     if _cuda(x):
         _count()
+        if x.dtype == torch.float32:  # models that run in 32-bit: true fp32 FMA, no reduced-precision tensor-core mode
+            if w.q4:
+                raise ValueError("JQ4 weights need bf16 activations")
+            return require_ext().linear_f32(x, w.w, w.bias, out)
         return w.handle().run(x, out, w.bias, out_f32, impl, force_splits)
     if w.q4:
         y = ref.linear_q4(x, w.packed, w.scales, w.bias)
@@ -337,6 +341,35 @@ def embedding(table, ids, scale=1.0, pos_table=None, pos=None, type_table=None, 
     if type_table is not None:
         out = out + (type_table[types.long()].float() if types is not None else type_table[0].float())
     return out.to(dtype or table.dtype)
+
+
+def bigram_embedding(table, bigram, ids, prev, mul_prev: int, mul_cur: int, scale: float = 1.0) -> torch.Tensor:
+    """fp32 ``table[ids] * scale + bigram[row]``; ``row = (prev * mul_prev + ids * mul_cur) mod buckets`` with ``buckets`` = rows of
+    ``bigram`` minus one, and the last row for tokens without a predecessor (``prev < 0``). ``bigram`` None: plain embedding."""
+    if _cuda(table):
+        _count()
+        return require_ext().bigram_embedding(table, bigram, ids.to(torch.int32), prev, mul_prev, mul_cur, scale)
+    return ref.bigram_embedding(table, bigram, ids, prev, mul_prev, mul_cur, scale)
+
+
+def add_layernorm(residual, delta, norm1, norm2, eps, pitch: int, dtype):
+    """fp32 residual stream: ``residual += delta`` in place (``delta`` may be None), then one or two LayerNorms of the same rows from one
+    set of statistics. ``norm1`` / ``norm2``: (weight, bias) in fp32 or None. Outputs are ``[T, pitch]`` (zeros behind the row width)."""
+    w1, b1 = norm1 if norm1 is not None else (None, None)
+    w2, b2 = norm2 if norm2 is not None else (None, None)
+    if _cuda(residual):
+        _count()
+        return tuple(require_ext().add_layernorm(residual, delta, w1, b1, w2, b2, eps, pitch, dtype == torch.float32))
+    return ref.add_layernorm(residual, delta, norm1, norm2, eps, pitch, dtype)
+
+
+def gated_act_into(gate_up, act: str, out) -> None:
+    """``out = act(gate) * up`` for ``gate_up [T, 2 I]``; ``out`` is an ``[T, I]`` column range of a wider row."""
+    if _cuda(gate_up):
+        _count()
+        require_ext().gated_act(gate_up, act, out)
+    else:
+        out.copy_(ref.act_mul(gate_up, act))
 
 
 def _check_full_rotary(cos, D: int) -> None:

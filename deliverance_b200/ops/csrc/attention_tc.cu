@@ -22,6 +22,14 @@
 // Every wait is bounded (common.cuh); on expiry the CTA records a status word, skips its stores, lets its copies and MMAs drain
 // (bounded), frees tensor memory and returns; CTAs that start after a recorded failure leave at once.
 //
+// Two layouts share the kernel (template parameter LATENT):
+//   paged   q [T, H * D], K and V rows in the paged cache, one head_dim for both, GQA groups;
+//   latent  keys and values expanded from the latent cache into flat rows (latent.cu): per head kn columns of an unrotated key part, one
+//           rotated key part shared by all heads (its own tensor map: it is copied behind the head's columns of every K tile, never
+//           materialised per head), DV columns of value. Key 0 of a sequence is its row kv_row0 of those buffers. The epilogue multiplies
+//           with a sigmoid output gate and stores the dv real columns of every head.
+// Both take DK (query / key columns) and DV (value columns) as multiples of 64.
+//
 // Replaces the reference's packed prefill attention (core/.../generator/CausalSelfAttention.java:458-502: per head QK^T GEMM over
 // the visible pages, causal scaled softmax with optional soft-cap, saxpy with V).
 #include <stdexcept>
@@ -48,6 +56,12 @@ struct AttnTcParams {
   float scale, softcap;
   int window, causal;
   int* status;
+  // latent layout only
+  const int* kv_row0;          // [sequences] row of key 0 in the expanded buffers
+  int kn_blocks;               // 64-column blocks of the per-head key part (the blocks behind it come from the shared part)
+  int dv, out_pitch;           // real value columns per head, row pitch of out
+  const __nv_bfloat16* gate;   // gate logits [T, gate_pitch], head h at column h * dv (nullptr: no gate)
+  int gate_pitch;
 };
 
 // MN-major shared-memory descriptor (128-byte swizzle): the operand tile is stored as rows of the K dimension, each row 64 elements of
@@ -85,19 +99,24 @@ __device__ __forceinline__ void tmem_st_x32(uint32_t taddr, const uint32_t* r) {
 
 constexpr int kAtBM = 128, kAtBN = 64;  // query rows per score tile / keys per tile
 
-template <int D, int QT>
+template <int DK, int DV, int QT>
 struct AttnTcSmem {
-  static constexpr int kSub = D / 64;                  // 64-column sub-tiles per operand tile
-  static constexpr int kTileQ = kAtBM * 128 * kSub;    // bytes of a [128 rows][D] bf16 query tile
-  static constexpr int kTileKV = kAtBN * 128 * kSub;   // bytes of a [64 keys][D] bf16 K or V tile
-  static constexpr int kStages = D <= 128 ? 4 : 2;
+  static constexpr int kSubK = DK / 64, kSubV = DV / 64;  // 64-column sub-tiles per operand tile
+  static constexpr int kTileQ = kAtBM * 128 * kSubK;      // bytes of a [128 rows][DK] bf16 query tile
+  static constexpr int kTileK = kAtBN * 128 * kSubK;      // bytes of a [64 keys][DK] bf16 K tile
+  static constexpr int kTileV = kAtBN * 128 * kSubV;
+  static constexpr int kRoom = 227 * 1024 - 512 - 1024 - QT * kTileQ;  // barriers + alignment slack
+  static constexpr int kFit = kRoom / (kTileK + kTileV);
+  static constexpr int kStages = kFit >= 4 ? 4 : kFit;
   static constexpr int kOffK = QT * kTileQ;
-  static constexpr int kOffV = kOffK + kStages * kTileKV;
-  static constexpr int kOffCtrl = kOffV + kStages * kTileKV;
-  static constexpr int kNeed = kOffCtrl + 512 + 1024;  // barriers + alignment slack
+  static constexpr int kOffV = kOffK + kStages * kTileK;
+  static constexpr int kOffCtrl = kOffV + kStages * kTileV;
+  static constexpr int kNeed = kOffCtrl + 512 + 1024;
   // every CTA allocates all 512 tensor-memory columns, so two CTAs must never share an SM: ask for more than half of its shared memory
   static constexpr int kBytes = kNeed > 118 * 1024 ? kNeed : 118 * 1024;
   static constexpr int kThreads = 128 + 128 * QT;  // warp 0 issues Q K^T, warp 1 the copies, warp 2 issues P V, warp 3 idles, warps 4.. softmax
+  static_assert(kStages >= 2 && DK % 64 == 0 && DV % 64 == 0, "attention tile does not fit");
+  static_assert(256 + QT * DV <= 512, "score slots and accumulators exceed tensor memory");
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -111,13 +130,15 @@ __device__ __forceinline__ float fmax3(float a, float b, float c) {
   return y;
 }
 
-template <int D, int QT>
-__global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
-    prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,  // [T, H * D], box 128 x 64
-                           const __grid_constant__ CUtensorMap map_k,  // [pages * KV * page, D], box min(page, 64) x 64
-                           const __grid_constant__ CUtensorMap map_v, const AttnTcParams p) {
-  using L = AttnTcSmem<D, QT>;
-  constexpr int NS = L::kStages, SUB = L::kSub;
+template <int DK, int DV, int QT, bool LATENT>
+__global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
+    prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,  // [T, H * DK], box 128 x 64
+                           const __grid_constant__ CUtensorMap map_k,  // paged [pages * KV * page, DK], box min(page, 64) x 64; latent [rows, H * kn]
+                           const __grid_constant__ CUtensorMap map_v,  // paged as K; latent [rows, H * DV], box 64 x 64
+                           const __grid_constant__ CUtensorMap map_r,  // latent: shared key part [rows, DK - kn], box 64 x 64 (paged: unused)
+                           const AttnTcParams p) {
+  using L = AttnTcSmem<DK, DV, QT>;
+  constexpr int NS = L::kStages, SUBK = L::kSubK, SUBV = L::kSubV;
   constexpr int kProducer = 1, kIssuer = 0, kIssuerPV = 2;
   extern __shared__ uint8_t at_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(at_raw) + 1023) & ~uintptr_t(1023));
@@ -181,6 +202,7 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
     tma_prefetch_desc(&map_q);
     tma_prefetch_desc(&map_k);
     tma_prefetch_desc(&map_v);
+    if (LATENT) tma_prefetch_desc(&map_r);
   }
   constexpr uint32_t kTmemCols = 512;
   if (warp == kIssuer) tmem_alloc(smem_u32(tmem_slot), kTmemCols);
@@ -188,7 +210,7 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  constexpr uint32_t kColS = 0, kColO = 256;  // score slot b of query tile q at kColS + (2 q + b) 64, accumulator of query tile q at kColO + q D
+  constexpr uint32_t kColS = 0, kColO = 256;  // score slot b of query tile q at kColS + (2 q + b) 64, accumulator of query tile q at kColO + q DV
   pdl_wait();
   pdl_trigger();
 
@@ -199,11 +221,10 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
     if (lane == 0) {
       mbar_expect_tx(smem_u32(bar_q), (two ? 2 : 1) * L::kTileQ);
       for (int q = 0; q < (two ? 2 : 1); ++q)
-        for (int c = 0; c < SUB; ++c)
-          tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * D + c * 64, qs + q0 + q * kAtBM);
+        for (int c = 0; c < SUBK; ++c)
+          tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * DK + c * 64, qs + q0 + q * kAtBM);
     }
     const int box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;  // page_size is 32, 64 or 128
-    const int n_copy = (kAtBN / box_rows) * SUB;
     int issued = 0;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t, ++issued) {
@@ -215,16 +236,29 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
         if (t >= NS) ok = mbar_wait(smem_u32(empty), ((t / NS) - 1) & 1, abort_flag, p.status);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        if (lane == 0) mbar_expect_tx(smem_u32(full), L::kTileKV);
+        if (lane == 0) mbar_expect_tx(smem_u32(full), kv == 0 ? L::kTileK : L::kTileV);
         __syncwarp();
+        uint8_t* dst = smem + (kv == 0 ? L::kOffK + s * L::kTileK : L::kOffV + s * L::kTileV);
+        const int sub = kv == 0 ? SUBK : SUBV;
+        if constexpr (LATENT) {
+          // rows behind the sequence's last key belong to the next sequence, or lie outside the buffer and arrive as zeros
+          const int row = p.kv_row0[seq] + kt * kAtBN;
+          for (int c = lane; c < sub; c += 32) {
+            const bool shared_part = kv == 0 && c >= p.kn_blocks;
+            const int x = shared_part ? (c - p.kn_blocks) * 64 : (kv == 0 ? h * p.kn_blocks + c : h * SUBV + c) * 64;
+            tma_load_2d(smem_u32(dst + c * (kAtBN * 128)), shared_part ? &map_r : (kv == 0 ? &map_k : &map_v), smem_u32(full), x, row);
+          }
+          continue;
+        }
+        const int n_copy = (kAtBN / box_rows) * sub;
         for (int i = lane; i < n_copy; i += 32) {
-          const int pg = i / SUB, c = i - pg * SUB;
+          const int pg = i / sub, c = i - pg * sub;
           const int key0 = kt * kAtBN + pg * box_rows;
           // pages past the context are never read by an unmasked score; the scratch page 0 keeps the copy inside the cache
           const int page = key0 < ctx ? p.block_tables[static_cast<long long>(seq) * p.bt_stride + key0 / p.page_size] : 0;
           const int row = (page * p.KV + kvh) * p.page_size + (key0 % p.page_size);
           const uint32_t off = c * (kAtBN * 128) + pg * box_rows * 128;
-          tma_load_2d(smem_u32(smem + (kv == 0 ? L::kOffK : L::kOffV) + s * L::kTileKV + off), kv == 0 ? &map_k : &map_v, smem_u32(full), c * 64, row);
+          tma_load_2d(smem_u32(dst + off), kv == 0 ? &map_k : &map_v, smem_u32(full), c * 64, row);
         }
       }
       if (!ok) break;
@@ -250,7 +284,7 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
     // issues the P V of every item once its probabilities are written and its V tile has landed. While one of them waits, the other
     // feeds the pipe. Everything the two depend on travels through mbarriers; tcgen05.commit covers the MMAs of its own thread.
     constexpr uint32_t idesc_s = umma_idesc_bf16(kAtBM, kAtBN);
-    constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(kAtBM, D);
+    constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(kAtBM, DV);
     auto valid = [&](int j, int q) { return q == 0 ? (j >= a0 && j < b0) : (j >= a1 && j < b1); };
     auto advance = [&](int& j, int& q) {  // next valid item; j == hi when there is none
       do {
@@ -279,10 +313,10 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
           if (!ok) break;
           tc_fence_after();
           const uint64_t desc_q = desc_q0 + static_cast<uint64_t>((q * L::kTileQ) >> 4);
-          const uint64_t desc_k = desc_k0 + static_cast<uint64_t>((s * L::kTileKV) >> 4);
+          const uint64_t desc_k = desc_k0 + static_cast<uint64_t>((s * L::kTileK) >> 4);
           const uint32_t d_s = tmem_base + kColS + slot * kAtBN;
 #pragma unroll
-          for (int k16 = 0; k16 < D / 16; ++k16) {
+          for (int k16 = 0; k16 < DK / 16; ++k16) {
             const uint64_t adv_q = static_cast<uint64_t>(((k16 >> 2) * (kAtBM * 128) + (k16 & 3) * 32) >> 4);
             const uint64_t adv_k = static_cast<uint64_t>(((k16 >> 2) * (kAtBN * 128) + (k16 & 3) * 32) >> 4);
             umma_bf16(d_s, desc_q + adv_q, desc_k + adv_k, idesc_s, k16 > 0 ? 1u : 0u);
@@ -301,8 +335,8 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
                mbar_wait(smem_u32(&bar_v_full[s]), ((j - lo) / NS) & 1, abort_flag, p.status);
           if (!ok) break;
           tc_fence_after();
-          const uint32_t tmem_p = tmem_base + kColS + slot * kAtBN, d_o = tmem_base + kColO + q * D;
-          const uint64_t desc_v0 = umma_desc_mn_sw128(v_base + s * L::kTileKV, kAtBN * 128, 1024);
+          const uint32_t tmem_p = tmem_base + kColS + slot * kAtBN, d_o = tmem_base + kColO + q * DV;
+          const uint64_t desc_v0 = umma_desc_mn_sw128(v_base + s * L::kTileV, kAtBN * 128, 1024);
 #pragma unroll
           for (int k16 = 0; k16 < kAtBN / 16; ++k16) {
             // 16 keys = two 8-row swizzle atoms (2048 bytes) further down the V tile; the 64-column blocks of D are kAtBN * 128 bytes apart
@@ -392,13 +426,13 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
         if (!ok) break;
         tc_fence_after();
 #pragma unroll 1
-        for (int c0 = 0; c0 < D; c0 += 32) {
+        for (int c0 = 0; c0 < DV; c0 += 32) {
           uint32_t v[32];
-          tmem_ld_x32(lane_addr + kColO + q * D + c0, v);
+          tmem_ld_x32(lane_addr + kColO + q * DV + c0, v);
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
-          tmem_st_x32(lane_addr + kColO + q * D + c0, v);
+          tmem_st_x32(lane_addr + kColO + q * DV + c0, v);
         }
         l_run *= alpha;
       }
@@ -434,18 +468,49 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
     if (ok) {
       tc_fence_after();
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* orow = p.out + static_cast<size_t>(qs + q0 + q * kAtBM + r) * (static_cast<size_t>(p.H) * D) + static_cast<size_t>(h) * D;
+      const size_t trow = static_cast<size_t>(qs + q0 + q * kAtBM + r);
+      __nv_bfloat16* orow = p.out + (LATENT ? trow * p.out_pitch + static_cast<size_t>(h) * p.dv : trow * (static_cast<size_t>(p.H) * DV) + static_cast<size_t>(h) * DV);
+      const __nv_bfloat16* grow = LATENT && p.gate != nullptr ? p.gate + trow * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
 #pragma unroll 1
-      for (int c0 = 0; c0 < D; c0 += 32) {
+      for (int c0 = 0; c0 < DV; c0 += 32) {
         uint32_t v[32];
         if (jb > ja) {
-          tmem_ld_x32(lane_addr + kColO + q * D + c0, v);
+          tmem_ld_x32(lane_addr + kColO + q * DV + c0, v);
           tmem_ld_wait();
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = 0u;
         }
-        if (r < my_rows) {
+        if (LATENT) {
+          if (r < my_rows) {
+            const bool vec = (p.dv & 7) == 0;  // (then rows, heads and the gate are 16-byte aligned as well)
+#pragma unroll
+            for (int i = 0; i < 32; i += 8) {
+              if (c0 + i >= p.dv) break;
+              float w[8];
+#pragma unroll
+              for (int e = 0; e < 8; ++e) w[e] = __uint_as_float(v[i + e]) * inv;
+              if (vec) {
+                if (grow != nullptr) {
+                  const uint4 gv = *reinterpret_cast<const uint4*>(grow + c0 + i);
+                  const uint32_t* gu = reinterpret_cast<const uint32_t*>(&gv);
+#pragma unroll
+                  for (int e = 0; e < 4; ++e) {
+                    const float2 g2 = unpack_bf162(gu[e]);
+                    w[2 * e] /= 1.f + __expf(-g2.x);
+                    w[2 * e + 1] /= 1.f + __expf(-g2.y);
+                  }
+                }
+                *reinterpret_cast<uint4*>(orow + c0 + i) =
+                    make_uint4(pack_bf162(w[0], w[1]), pack_bf162(w[2], w[3]), pack_bf162(w[4], w[5]), pack_bf162(w[6], w[7]));
+              } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+                  if (c0 + i + e < p.dv) orow[c0 + i + e] = f2bf(grow != nullptr ? w[e] / (1.f + __expf(-bf2f(grow[c0 + i + e]))) : w[e]);
+              }
+            }
+          }
+        } else if (r < my_rows) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             uint4 o;
@@ -467,20 +532,15 @@ __global__ void __launch_bounds__(AttnTcSmem<D, QT>::kThreads, 1)
   }
 }
 
-template <int D, int QT>
-static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
-                               int num_tiles, cudaStream_t st) {
-  using L = AttnTcSmem<D, QT>;
+template <int DK, int DV, int QT, bool LATENT>
+static int launch_prefill_tc_maps(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr, const AttnTcParams& p,
+                                  int num_tiles, cudaStream_t st) {
+  using L = AttnTcSmem<DK, DV, QT>;
   static PerDeviceOnce attr_once;
   if (attr_once.first()) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel<D, QT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel<DK, DV, QT, LATENT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
     if (e != cudaSuccess) throw std::runtime_error(std::string("prefill attention (tcgen05): cudaFuncSetAttribute: ") + cudaGetErrorString(e));
   }
-  CUtensorMap mq, mk, mv;
-  encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * D, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
-  const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
-  encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
-  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(num_tiles, p.H);
   cfg.blockDim = dim3(L::kThreads);
@@ -491,9 +551,72 @@ static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, c
   attr[0].val.programmaticStreamSerializationAllowed = g_pdl_enabled ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_attn_tc_kernel<D, QT>, mq, mk, mv, p);
+  cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_attn_tc_kernel<DK, DV, QT, LATENT>, mq, mk, mv, mr, p);
   if (e != cudaSuccess) throw std::runtime_error(std::string("prefill attention (tcgen05) launch: ") + cudaGetErrorString(e));
   return 0;
+}
+
+template <int D, int QT>
+static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
+                               int num_tiles, cudaStream_t st) {
+  CUtensorMap mq, mk, mv;
+  encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * D, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
+  const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
+  encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
+  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
+  return launch_prefill_tc_maps<D, D, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
+}
+
+// ---- latent layout -----------------------------------------------------------------------------------------------------
+// Operand widths the kernel is instantiated for: the value columns of a head are padded to the returned width (0: not available,
+// dk = 64-padded unrotated + rotated columns must be one of 128, 192, 256 and dv at most 256).
+int prefill_latent_tc_dv(int dk, int dv) {
+  if (dk != 128 && dk != 192 && dk != 256) return 0;
+  if (dv <= 64 && dk == 128) return 64;
+  if (dv <= 128) return 128;
+  if (dv <= 256 && dk == 256) return 256;
+  return 0;
+}
+int prefill_latent_tc_tile_rows(int dv_padded) { return dv_padded <= 128 ? 256 : 128; }
+
+int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
+  if (a.num_tiles == 0) return 0;
+  const int DV = prefill_latent_tc_dv(a.dk, a.dv);
+  if (DV == 0 || a.kn % 64 != 0 || a.kn <= 0 || a.kn >= a.dk) return 1;
+  AttnTcParams p = {};
+  p.q_start = a.q_start;
+  p.q_len = a.q_len;
+  p.ctx_lens = a.ctx;
+  p.tile_seq = a.tile_seq;
+  p.tile_q0 = a.tile_q0;
+  p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.H = p.KV = a.H;
+  p.page_size = kAtBN;
+  p.scale = a.scale;
+  p.window = a.window;
+  p.causal = 1;
+  p.status = a.status;
+  p.kv_row0 = a.kv_row0;
+  p.kn_blocks = a.kn / 64;
+  p.dv = a.dv;
+  p.out_pitch = a.out_pitch;
+  p.gate = static_cast<const __nv_bfloat16*>(a.gate);
+  p.gate_pitch = a.gate_pitch;
+  CUtensorMap mq, mk, mv, mr;
+  const uint64_t H = static_cast<uint64_t>(a.H), rows = static_cast<uint64_t>(a.kv_rows);
+  encode_map_2d(&mq, 0, a.q, static_cast<uint64_t>(a.T), H * a.dk, static_cast<uint64_t>(a.q_pitch) * 2, kAtBM, 64, 128);
+  encode_map_2d(&mk, 0, a.k, rows, H * a.kn, static_cast<uint64_t>(a.kv_pitch) * 2, kAtBN, 64, 128);
+  encode_map_2d(&mv, 0, a.v, rows, H * DV, static_cast<uint64_t>(a.kv_pitch) * 2, kAtBN, 64, 128);
+  encode_map_2d(&mr, 0, a.kr, rows, static_cast<uint64_t>(a.dk - a.kn), static_cast<uint64_t>(a.kr_pitch) * 2, kAtBN, 64, 128);
+#define DLV_LAT(DKV, DVV, QTV) \
+  if (a.dk == DKV && DV == DVV) return launch_prefill_tc_maps<DKV, DVV, QTV, true>(mq, mk, mv, mr, p, a.num_tiles, st)
+  DLV_LAT(128, 64, 2);
+  DLV_LAT(128, 128, 2);
+  DLV_LAT(192, 128, 2);
+  DLV_LAT(256, 128, 2);
+  DLV_LAT(256, 256, 1);
+#undef DLV_LAT
+  return 1;
 }
 
 // Query rows one CTA of the tcgen05 prefill kernel covers: two 128-row tiles share the K / V tiles where their two accumulators fit

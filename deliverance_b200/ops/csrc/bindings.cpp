@@ -811,6 +811,8 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
   return out;
 }
 
+#include "bindings_latent.inc"
+
 // ---- sampling ---------------------------------------------------------------------------------------------------------
 std::vector<Tensor> argmax(const Tensor& logits, c10::optional<Tensor> mask, double softcap, double inv_scale) {
   TORCH_CHECK(logits.is_cuda() && logits.scalar_type() == at::kFloat && logits.dim() == 2 && logits.stride(1) == 1, "logits must be fp32 [B, V]");
@@ -1522,6 +1524,17 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("prefill_attention", &prefill_attention);
   m.def("prefill_attention_tc", &prefill_attention_tc);
   m.def("prefill_tc_tile_rows", &dlv::prefill_attention_tc_tile_rows);
+  m.def("linear_f32", &linear_f32);
+  m.def("bigram_embedding", &bigram_embedding);
+  m.def("add_layernorm", &add_layernorm);
+  m.def("gated_act", &gated_act);
+  m.def("latent_prepare", &latent_prepare);
+  m.def("latent_decode", &latent_decode);
+  m.def("latent_gather", &latent_gather);
+  m.def("latent_prefill", &latent_prefill);
+  m.def("latent_rows_f32", &latent_rows_f32);
+  m.def("latent_prefill_dv", [](int64_t dk, int64_t dv) { return dlv::prefill_latent_tc_dv(static_cast<int>(dk), static_cast<int>(dv)); });
+  m.def("latent_prefill_tile_rows", [](int64_t dv) { return dlv::prefill_latent_tc_tile_rows(static_cast<int>(dv)); });
   m.def("gemv_simt_only", [](bool on) { dlv::g_gemv_simt_only = on; });
   m.def("gemv_dense", [](bool on) { dlv::g_gemv_dense = on; });
   m.def(

@@ -288,6 +288,102 @@ __global__ void __launch_bounds__(256) rope_kv_kernel(__nv_bfloat16* __restrict_
   }
 }
 
+// ------------------------------------------------------------------------------------------------ fp32 residual stream
+// Models that keep the residual stream in fp32: embedding with a hashed-bigram table, residual add + one or two LayerNorms of the same
+// row, gated activation with row pitches. TIO: bf16 or fp32 activations.
+__device__ __forceinline__ float io_ld(const __nv_bfloat16* p) { return bf2f(*p); }
+__device__ __forceinline__ float io_ld(const float* p) { return *p; }
+__device__ __forceinline__ void io_st(__nv_bfloat16* p, float v) { *p = f2bf(v); }
+__device__ __forceinline__ void io_st(float* p, float v) { *p = v; }
+
+// out[t] = table[ids[t]] * scale + bigram[row]; row = (prev * mul_prev + id * mul_cur) mod buckets, or `buckets` (the extra last row) when the
+// token has no predecessor (prev < 0)
+template <typename TIO>
+__global__ void __launch_bounds__(128) bigram_embedding_kernel(const TIO* __restrict__ table, const TIO* __restrict__ bigram, const int* __restrict__ ids,
+                                                               const int* __restrict__ prev, float* __restrict__ out, int W, int vocab, int buckets,
+                                                               long long mul_prev, long long mul_cur, float scale) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) id = 0;  // host validates ids; never read out of the table
+  const TIO* src = table + static_cast<size_t>(id) * W;
+  const TIO* bg = nullptr;
+  if (bigram != nullptr) {
+    const long long pv = prev[t];
+    long long row = pv < 0 ? buckets : (pv * mul_prev + static_cast<long long>(id) * mul_cur) % buckets;
+    if (row < 0) row += buckets;
+    bg = bigram + row * W;
+  }
+  for (int i = threadIdx.x; i < W; i += blockDim.x)
+    out[static_cast<size_t>(t) * W + i] = io_ld(src + i) * scale + (bg != nullptr ? io_ld(bg + i) : 0.f);
+}
+
+// residual += delta (when given; written back), then y1 = LayerNorm(residual; w1, b1) and, when w2 is given, y2 = LayerNorm(residual; w2, b2)
+// from the same statistics. Columns W .. y_pitch of the outputs are zeroed. One CTA per row.
+template <typename TIO>
+__global__ void __launch_bounds__(256) add_layernorm_kernel(float* __restrict__ residual, const float* __restrict__ delta, const float* __restrict__ w1,
+                                                            const float* __restrict__ b1, TIO* __restrict__ y1, const float* __restrict__ w2,
+                                                            const float* __restrict__ b2, TIO* __restrict__ y2, int W, int y_pitch, float eps) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ float row[];
+  __shared__ float red[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * W, yb = static_cast<size_t>(blockIdx.x) * y_pitch;
+  float s = 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    float v = residual[base + i];
+    if (delta != nullptr) {
+      v += delta[base + i];
+      residual[base + i] = v;
+    }
+    row[i] = v;
+    s += v;
+  }
+  const float mean = block_sum(s, red) / W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float d = row[i] - mean;
+    ss += d * d;
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / W + eps);
+  for (int i = threadIdx.x; i < y_pitch; i += blockDim.x) {
+    const float n = i < W ? (row[i] - mean) * inv : 0.f;
+    if (y1 != nullptr) io_st(y1 + yb + i, i < W ? n * w1[i] + b1[i] : 0.f);
+    if (y2 != nullptr) io_st(y2 + yb + i, i < W ? n * w2[i] + b2[i] : 0.f);
+  }
+}
+
+// out[t, c] = act(in[t, c]) * in[t, I + c]
+template <typename TIO>
+__global__ void __launch_bounds__(256) gated_act_kernel(const TIO* __restrict__ in, long long ld_in, TIO* __restrict__ out, long long ld_out, int I, int act,
+                                                        long long total) {
+  pdl_wait();
+  pdl_trigger();
+  const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= total) return;
+  const int per_row = I / 8;
+  const long long t = idx / per_row;
+  const int c = static_cast<int>(idx % per_row) * 8;
+  const TIO* g = in + t * ld_in + c;
+  TIO* o = out + t * ld_out + c;
+  if constexpr (sizeof(TIO) == 2) {
+    const uint4 gv = *reinterpret_cast<const uint4*>(g), uv = *reinterpret_cast<const uint4*>(g + I);
+    const uint32_t* gu = reinterpret_cast<const uint32_t*>(&gv);
+    const uint32_t* uu = reinterpret_cast<const uint32_t*>(&uv);
+    uint32_t ou[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 a = unpack_bf162(gu[j]), b = unpack_bf162(uu[j]);
+      ou[j] = pack_bf162(act_apply(a.x, act) * b.x, act_apply(a.y, act) * b.y);
+    }
+    *reinterpret_cast<uint4*>(o) = make_uint4(ou[0], ou[1], ou[2], ou[3]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = act_apply(g[j], act) * g[I + j];
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ launchers
 void launch_rmsnorm(const void* x, void* residual, const void* w, void* y, int T, int H, float eps, float offset,
                     float res_mult, cudaStream_t st) {
@@ -318,6 +414,35 @@ void launch_embedding(const void* table, const int* ids, const void* pos_table, 
   launch_pdl(embedding_kernel, dim3(T), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(table), ids, static_cast<const __nv_bfloat16*>(pos_table), pos,
                                       static_cast<const __nv_bfloat16*>(type_table), types, static_cast<__nv_bfloat16*>(out), H, vocab,
                                       scale);
+}
+void launch_bigram_embedding(const void* table, const void* bigram, const int* ids, const int* prev, float* out, int rows, int W, int vocab, int buckets,
+                             long long mul_prev, long long mul_cur, float scale, bool is_f32, cudaStream_t st) {
+  if (rows == 0) return;
+  if (is_f32)
+    launch_pdl(bigram_embedding_kernel<float>, dim3(rows), dim3(128), 0, st, static_cast<const float*>(table), static_cast<const float*>(bigram), ids, prev,
+               out, W, vocab, buckets, mul_prev, mul_cur, scale);
+  else
+    launch_pdl(bigram_embedding_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(table),
+               static_cast<const __nv_bfloat16*>(bigram), ids, prev, out, W, vocab, buckets, mul_prev, mul_cur, scale);
+}
+void launch_add_layernorm(float* residual, const float* delta, const float* w1, const float* b1, void* y1, const float* w2, const float* b2, void* y2,
+                          int rows, int W, int y_pitch, float eps, bool is_f32, cudaStream_t st) {
+  if (rows == 0) return;
+  if (is_f32)
+    launch_pdl(add_layernorm_kernel<float>, dim3(rows), dim3(256), W * sizeof(float), st, residual, delta, w1, b1, static_cast<float*>(y1), w2, b2,
+               static_cast<float*>(y2), W, y_pitch, eps);
+  else
+    launch_pdl(add_layernorm_kernel<__nv_bfloat16>, dim3(rows), dim3(256), W * sizeof(float), st, residual, delta, w1, b1, static_cast<__nv_bfloat16*>(y1), w2,
+               b2, static_cast<__nv_bfloat16*>(y2), W, y_pitch, eps);
+}
+void launch_gated_act(const void* in, long long ld_in, void* out, long long ld_out, int rows, int I, int act, bool is_f32, cudaStream_t st) {
+  const long long total = static_cast<long long>(rows) * (I / 8);
+  if (total == 0) return;
+  const dim3 grid(static_cast<unsigned>((total + 255) / 256));
+  if (is_f32) launch_pdl(gated_act_kernel<float>, grid, dim3(256), 0, st, static_cast<const float*>(in), ld_in, static_cast<float*>(out), ld_out, I, act, total);
+  else
+    launch_pdl(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(in), ld_in, static_cast<__nv_bfloat16*>(out), ld_out, I,
+               act, total);
 }
 int launch_rope_kv(void* qkv, const int* positions, const long long* slots, const void* qn, const void* kn, const float* cos_t,
                    const float* sin_t, void* k_cache, void* v_cache, int T, int H, int KV, int D, int block_size, int rot_half,

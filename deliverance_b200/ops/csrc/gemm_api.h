@@ -230,6 +230,55 @@ void launch_a2a_receive(const A2AParams* p, unsigned epoch, int* local_offsets, 
 void launch_a2a_return(const A2AParams* p, const int* local_offsets, const int* seg, const void* ys, int max_rows, int H, unsigned epoch, cudaStream_t st);
 void launch_a2a_wait(const A2AParams* p, unsigned epoch, cudaStream_t st);
 
+// latent.cu: latent attention (compressed key / value cache); see the file comment for the layouts. is_f32: every tensor is fp32
+struct LatentGeom {
+  int H, dk, dn, R, Rp, dr, drp;   // heads; padded q columns per head, its unrotated part; latent size, padded; rotated size, padded in the cache
+  int dv, Kp;                      // value size per head, latent columns of the value weights (32-padded)
+  int off_c, off_r, off_g;         // column offsets in the projection rows: latent, rotated key, gate (-1: no gate)
+};
+void launch_latent_prepare(void* p, long long ld, int rows, const int* positions, const long long* slots, const float* norm_w, const float* cos_t,
+                           const float* sin_t, int half, int max_pos, void* c_cache, void* r_cache, const LatentGeom& g, float eps, bool is_f32,
+                           cudaStream_t st);
+void launch_latent_gather(const void* c_cache, const void* r_cache, const int* bt, int bt_stride, int page, const int* seq, const int* key0,
+                          const int* n_keys, const int* row0, int num_seqs, int max_rows, void* c_out, int c_pitch, void* r_out, int r_pitch, int Rp, int drp,
+                          cudaStream_t st);
+void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int rows, const void* wuk, void* q_lat, const LatentGeom& g, cudaStream_t st);
+int launch_latent_decode(const void* q_lat, const void* c_cache, const void* r_cache, const int* bt, int bt_stride, const int* row_seq, const int* row_ctx,
+                         int rows, float* part_o, float* part_ml, const LatentGeom& g, int page, float scale, int window, int splits, cudaStream_t st);
+void launch_latent_expand(const float* part_o, const float* part_ml, int splits, const int* row_idx, int rows, const void* wuv, const void* p, long long ld,
+                          void* out, int out_pitch, const LatentGeom& g, cudaStream_t st);
+int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, const int* row_seq, const int* row_ctx, int rows, const float* wuk,
+                           const float* wuv, const float* c_cache, const float* r_cache, const int* bt, int bt_stride, float* out, int out_pitch,
+                           const LatentGeom& g, int page, float scale, int window, cudaStream_t st);
+void launch_linear_f32(const float* x, int ldx, const float* w, const float* bias, float* out, int ldo, int M, int N, int K, cudaStream_t st);
+
+// attention_tc.cu, latent layout: q [T, H * dk] (pitch q_pitch), k [kv_rows, H * kn] and v [kv_rows, H * DV] with one pitch, kr [kv_rows, dk - kn]
+struct LatentTcArgs {
+  const void *q, *k, *v, *kr;
+  long long T, kv_rows;
+  int q_pitch, kv_pitch, kr_pitch;
+  int H, dk, kn, dv;
+  const int *q_start, *q_len, *ctx, *kv_row0, *tile_seq, *tile_q0;  // ctx: keys of a sequence in k / v (its query rows are the last q_len)
+  int num_tiles;
+  void* out;
+  int out_pitch;
+  const void* gate;
+  int gate_pitch;
+  float scale;
+  int window;
+  int* status;
+};
+int prefill_latent_tc_dv(int dk, int dv);
+int prefill_latent_tc_tile_rows(int dv_padded);
+int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st);
+
+// elementwise.cu, fp32 residual stream
+void launch_bigram_embedding(const void* table, const void* bigram, const int* ids, const int* prev, float* out, int rows, int W, int vocab, int buckets,
+                             long long mul_prev, long long mul_cur, float scale, bool is_f32, cudaStream_t st);
+void launch_add_layernorm(float* residual, const float* delta, const float* w1, const float* b1, void* y1, const float* w2, const float* b2, void* y2,
+                          int rows, int W, int y_pitch, float eps, bool is_f32, cudaStream_t st);
+void launch_gated_act(const void* in, long long ld_in, void* out, long long ld_out, int rows, int I, int act, bool is_f32, cudaStream_t st);
+
 // aux.cu
 void launch_lora_delta(const void* x, int ldx, const void* A, const void* Bs, void* y, int ldy, int M, int K, int N, int r, cudaStream_t st);
 void launch_pool(const void* h, int H, const int* start, const int* len, int S, int mode, int normalize, float* out, cudaStream_t st);

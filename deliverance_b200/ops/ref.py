@@ -71,6 +71,25 @@ def rope_tables(head_dim: int, max_pos: int, theta: float, factor: float = 1.0, 
     return torch.cos(ang).float(), torch.sin(ang).float()
 
 
+def yarn_rope_tables(dims: int, max_pos: int, base: float, scaling: Optional[dict] = None):
+    """cos/sin tables ``[max_pos, dims/2]`` fp32 with YaRN frequency interpolation. ``scaling``: ``factor``, ``original`` (context
+    length the base frequencies were made for), ``fast`` / ``slow`` (full turns over that context at which a pair is kept as it is /
+    fully slowed down by ``factor``; a linear ramp over the pair index lies between). Both tables carry ``0.1 ln(factor) + 1``."""
+    if not scaling:
+        return rope_tables(dims, max_pos, base, 1.0)
+    i = torch.arange(0, dims // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / dims)
+    pair_of = lambda turns: dims * math.log(float(scaling["original"]) / (2.0 * math.pi * float(turns))) / (2.0 * math.log(base))  # noqa: E731
+    lo = max(math.floor(pair_of(scaling["fast"])), 0)
+    hi = min(math.ceil(pair_of(scaling["slow"])), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    factor = float(scaling["factor"])
+    inv = f / factor * ramp + f * (1.0 - ramp)
+    ang = torch.arange(max_pos, dtype=torch.float64).unsqueeze(1) * inv.unsqueeze(0)
+    mult = 0.1 * math.log(factor) + 1.0
+    return (torch.cos(ang) * mult).float(), (torch.sin(ang) * mult).float()
+
+
 def apply_rope(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
     """x ``[T, heads, d]``; rotates the first ``2 * cos.shape[1]`` dims with pairs (i, i + half)."""
     half = cos.shape[1]
@@ -157,6 +176,25 @@ def act_mul(gate_up: torch.Tensor, act: str) -> torch.Tensor:
 def embedding(table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     out = table[ids.long()].float() * scale
     return out.to(dtype or table.dtype)
+
+
+def bigram_embedding(table, bigram, ids, prev, mul_prev: int, mul_cur: int, scale: float) -> torch.Tensor:
+    out = table[ids.long()].float() * scale
+    if bigram is not None:
+        buckets = bigram.shape[0] - 1
+        row = torch.remainder(prev.long() * mul_prev + ids.long() * mul_cur, buckets)
+        out = out + bigram[torch.where(prev < 0, torch.full_like(row, buckets), row)].float()
+    return out
+
+
+def add_layernorm(residual, delta, norm1, norm2, eps, pitch, dtype):
+    if delta is not None:
+        residual.add_(delta.float())
+    mean = residual.mean(dim=-1, keepdim=True)
+    d = residual - mean
+    n = d * torch.rsqrt(d.pow(2).mean(dim=-1, keepdim=True) + eps)
+    pad = pitch - residual.shape[-1]
+    return tuple(None if nb is None else F.pad(n * nb[0] + nb[1], (0, pad)).to(dtype) for nb in (norm1, norm2))
 
 
 def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
