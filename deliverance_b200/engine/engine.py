@@ -437,7 +437,7 @@ class Engine:
     def replay_step(self, entries: list) -> Optional[torch.Tensor]:
         """One batch of ``(request, next tokens, wanted places among them)``: prompt portions and single tokens together, exactly the
         forward passes of a scheduled step (a batch of single tokens of started requests is a decode step, captured graph included).
-        Returns fp32 logits of the wanted places in order, or None when nothing is wanted."""
+        Returns fp32 logits of the wanted places in order (host memory), or None when nothing is wanted."""
         seqs, rows, base = [], [], 0
         for r, tokens, want in entries:
             if not tokens:
@@ -471,10 +471,12 @@ class Engine:
         for r, tokens, _ in entries:
             r.computed += len(tokens)
         if not rows:
+            if self.device.type == "cuda":  # the pinned staging buffers of a captured step are used again two steps later
+                torch.cuda.current_stream(self.device).synchronize()
             return None
         if decode:  # one row per entry; batches of portions return the wanted rows only
             logits = logits.index_select(0, torch.tensor(rows, dtype=torch.int64, device=logits.device))
-        return self._full(logits)
+        return self._full(logits).cpu()
 
     # ------------------------------------------------------------------------------------------------ decode
     def _decode_inputs(self, reqs: list[Request]):
