@@ -14,12 +14,15 @@ import torch
 from .loader import ShardSpec, shard_dense, shard_q4
 from .quantizer import DEFAULT_Q4_FILTER
 from .safetensors_io import Q4Tensor, TensorInfo
-from .tiny import build_tensors  # noqa: F401  (small models reuse the tiny builder)
+from ..config import config_model_type
+from .tiny import build_tensors, fatotar_is_norm, fatotar_shapes  # noqa: F401  (small models reuse the tiny builder)
 
 
 def _shapes(cfg: dict) -> dict[str, tuple]:
     """name -> shape for decoder families (llama, mistral, qwen2, qwen3, gemma2, gemma3, mixtral, qwen3_moe)."""
-    mt = cfg["model_type"]
+    mt = config_model_type(cfg)
+    if mt == "fatotar":
+        return fatotar_shapes(cfg)
     h, L, V = cfg["hidden_size"], cfg["num_hidden_layers"], cfg["vocab_size"]
     nh, nkv = cfg["num_attention_heads"], cfg.get("num_key_value_heads") or cfg["num_attention_heads"]
     hd = cfg.get("head_dim") or h // nh
@@ -89,6 +92,8 @@ class SyntheticLoader:
     def _gen(self, name):
         shape = self.shapes[name]
         g = torch.Generator(device=self.device).manual_seed((self.seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFF)
+        if config_model_type(self.cfg) == "fatotar" and fatotar_is_norm(name):
+            return (1.0 + torch.randn(shape, generator=g, device=self.device) * 0.02).to(self.dtype)
         if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
             base = 0.0 if self.cfg["model_type"] in ("gemma2", "gemma3_text") else 1.0
             return (base + torch.randn(shape, generator=g, device=self.device) * 0.02).to(self.dtype)

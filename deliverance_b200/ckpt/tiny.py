@@ -12,6 +12,7 @@ from typing import Optional
 
 import torch
 
+from ..config import config_model_type
 from .safetensors_io import write_safetensors, write_sharded
 
 
@@ -19,7 +20,70 @@ def _rand(gen, *shape, std=0.02, dtype=torch.float32):
     return (torch.randn(*shape, generator=gen, dtype=torch.float32) * std).to(dtype)
 
 
+def fatotar_config(width: int, vocab: int, layers: list, loop: Optional[dict] = None, eps: float = 1e-5, scale: float = 2.0,
+                   bigram: Optional[dict] = None, **extra) -> dict:
+    """``config.json`` of a Fatotar model. ``layers``: one dict of sizes per layer (``heads, dim, rot_dim, vdim, kv_rank, window, base,
+    scaling, ff``, score ``scale``; ``ff`` 0 = no feed-forward)."""
+    out = []
+    for L in layers:
+        rot = {"base": L.get("base", 10000.0), "dims": L["rot_dim"]}
+        if L.get("scaling"):
+            rot["scaling"] = L["scaling"]
+        out.append({"type": "latent_attention", "mlp": {"kind": "dense", "ff": L["ff"]} if L.get("ff") else None,
+                    "mixer": {"heads": L["heads"], "dim": L["dim"], "rot_dim": L["rot_dim"], "vdim": L["vdim"], "kv_rank": L["kv_rank"],
+                              "mask": {"size": L["window"]}, "rot": rot, "scale": L.get("scale", (L["dim"] + L["rot_dim"]) ** -0.5)}})
+    cfg = {"architecture": "Fatotar", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": out,
+           "embedding": {"scale": scale, "bigram": bigram or {"buckets": 211, "mul_prev": 31, "mul_cur": 7}}}
+    if loop:
+        cfg["loop"] = loop
+    cfg.update(extra)
+    return cfg
+
+
+def fatotar_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape of a Fatotar checkpoint."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "head": (V, W), "final.norm": (W,), "final.norm.b": (W,), "bigram": (cfg["embedding"]["bigram"]["buckets"] + 1, W)}
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        H, dn, dr, dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        s.update({p + "norm1": (W,), p + "norm1.b": (W,), p + "mix.q": (H * (dn + dr), W), p + "mix.dkv": (R + dr, W), p + "mix.dkv.norm": (R,),
+                  p + "mix.uk": (H * dn, R), p + "mix.uv": (H * dv, R), p + "mix.g": (H * dv, W), p + "mix.o": (W, H * dv)})
+        if L.get("mlp"):
+            F = L["mlp"]["ff"]
+            s.update({p + "norm2": (W,), p + "norm2.b": (W,), p + "mlp.gate": (F, W), p + "mlp.gate.b": (F,), p + "mlp.up": (F, W), p + "mlp.up.b": (F,),
+                      p + "mlp.down": (W, F), p + "mlp.down.b": (W,)})
+    return s
+
+
+def fatotar_is_norm(name: str) -> bool:
+    return name.rsplit(".", 1)[-1].startswith("norm")
+
+
+def _fatotar_tensors(cfg: dict, seed: int, dtype) -> dict:
+    """Random weights with projections scaled by their fan-in, so that every mechanism moves the output."""
+    g = torch.Generator().manual_seed(seed)
+    t = {}
+    for name, shape in fatotar_shapes(cfg).items():
+        r = torch.randn(*shape, generator=g, dtype=torch.float32)
+        if fatotar_is_norm(name):
+            r = 1.0 + 0.2 * r
+        elif len(shape) == 1:
+            r = 0.2 * r
+        elif name not in ("embed", "bigram"):
+            r = r * shape[1] ** -0.5
+        t[name] = r.to(dtype)
+    return t
+
+
 def tiny_config(model_type: str, **over) -> dict:
+    if model_type == "fatotar":
+        size = dict(heads=3, dim=20, rot_dim=6, vdim=12, kv_rank=40, window=24, ff=52)
+        yarn = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 2.0}
+        kw = dict(width=92, vocab=261, layers=[dict(size), dict(size, window=40, base=500.0, scaling=yarn), dict(size, heads=2, vdim=24, ff=0)],
+                  loop={"start": 0, "stop": 2, "times": 2})
+        kw.update(over)
+        return fatotar_config(**kw)
     base = dict(
         model_type=model_type, vocab_size=256, hidden_size=64, intermediate_size=128, num_hidden_layers=2,
         num_attention_heads=4, num_key_value_heads=2, max_position_embeddings=256, rms_norm_eps=1e-5, rope_theta=10000.0,
@@ -61,7 +125,9 @@ def tiny_config(model_type: str, **over) -> dict:
 
 def build_tensors(cfg: dict, seed: int = 0, dtype=torch.float32, std: float = 0.02) -> dict:
     g = torch.Generator().manual_seed(seed)
-    mt = cfg["model_type"]
+    mt = config_model_type(cfg)
+    if mt == "fatotar":
+        return _fatotar_tensors(cfg, seed, dtype)
     R = lambda *s: _rand(g, *s, std=std, dtype=dtype)  # noqa: E731
     ones = lambda n: (torch.ones(n) + torch.randn(n, generator=g) * 0.05).to(dtype)  # noqa: E731
     t: dict = {}
