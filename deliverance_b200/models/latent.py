@@ -76,14 +76,15 @@ class LatentAttention:
         c_cache, r_cache = kv_pair
         with stage("latentattention.input_projection"):
             p = ops.linear(x, self.w_in)
-        with stage("latentattention.rope_norm_cache"):
-            lop.prepare(s, p, batch.positions, batch.slots, self.norm, self.cos, self.sin, c_cache, r_cache, self.eps)
+        write = (batch.positions, batch.slots, self.norm, self.cos, self.sin, c_cache, r_cache, self.eps)
         args = (self.wuk, self.wuv, c_cache, r_cache, batch.block_tables, out, self.scale, self.window)
         if batch.is_decode:
             span = max(batch.ctx_len_host) if batch.ctx_len_host else self.cos.shape[0]
             with stage("latentattention.score_value"):
-                lop.rows_attention(s, p, None, None, batch.ctx_len, *args, splits=self._splits(p.shape[0], span))
+                lop.rows_attention(s, p, None, None, batch.ctx_len, *args, splits=self._splits(p.shape[0], span), write=write)
             return
+        with stage("latentattention.rope_norm_cache"):
+            lop.prepare(s, p, *write)
         plan = self._plan(batch)
         if plan["rows"] is not None:
             row_idx, row_seq, row_ctx, span = plan["rows"]

@@ -1529,7 +1529,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("add_layernorm", &add_layernorm);
   m.def("gated_act", &gated_act);
   m.def("latent_prepare", &latent_prepare);
-  m.def("latent_decode", &latent_decode);
+  m.def("latent_decode", &latent_decode, py::arg("p"), py::arg("row_idx"), py::arg("row_seq"), py::arg("row_ctx"), py::arg("wuk"), py::arg("wuv"),
+        py::arg("c_cache"), py::arg("r_cache"), py::arg("block_tables"), py::arg("out"), py::arg("geom"), py::arg("scale"), py::arg("window"),
+        py::arg("splits"), py::arg("positions") = py::none(), py::arg("slots") = py::none(), py::arg("norm_w") = py::none(), py::arg("cos") = py::none(),
+        py::arg("sin") = py::none(), py::arg("eps") = 0.0);
+  m.def("latent_head_groups", [](int64_t n) { dlv::g_latent_head_groups = static_cast<int>(n); });
   m.def("latent_gather", &latent_gather);
   m.def("latent_prefill", &latent_prefill);
   m.def("latent_rows_f32", &latent_rows_f32);

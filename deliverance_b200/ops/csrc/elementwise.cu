@@ -327,26 +327,58 @@ __global__ void __launch_bounds__(256) add_layernorm_kernel(float* __restrict__ 
                                                             const float* __restrict__ b2, TIO* __restrict__ y2, int W, int y_pitch, float eps) {
   pdl_wait();
   pdl_trigger();
-  extern __shared__ float row[];
+  extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   const size_t base = static_cast<size_t>(blockIdx.x) * W, yb = static_cast<size_t>(blockIdx.x) * y_pitch;
+  const bool vec = (W & 3) == 0;  // rows start on 16 bytes then
   float s = 0.f;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) {
-    float v = residual[base + i];
-    if (delta != nullptr) {
-      v += delta[base + i];
-      residual[base + i] = v;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(residual + base + i);
+      if (delta != nullptr) {
+        const float4 d = *reinterpret_cast<const float4*>(delta + base + i);
+        v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+        *reinterpret_cast<float4*>(residual + base + i) = v;
+      }
+      *reinterpret_cast<float4*>(row + i) = v;
+      s += (v.x + v.y) + (v.z + v.w);
     }
-    row[i] = v;
-    s += v;
+  } else {
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+      float v = residual[base + i];
+      if (delta != nullptr) {
+        v += delta[base + i];
+        residual[base + i] = v;
+      }
+      row[i] = v;
+      s += v;
+    }
   }
-  const float mean = block_sum(s, red) / W;
+  const float mean = block_sum(s, red) / W;  // (its barriers also publish the row)
   float ss = 0.f;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     const float d = row[i] - mean;
     ss += d * d;
   }
   const float inv = rsqrtf(block_sum(ss, red) / W + eps);
+  auto norm4 = [&](int i, const float* w, const float* b, TIO* y) {
+    const float4 v = *reinterpret_cast<const float4*>(row + i), wv = *reinterpret_cast<const float4*>(w + i), bv = *reinterpret_cast<const float4*>(b + i);
+    const float o0 = (v.x - mean) * inv * wv.x + bv.x, o1 = (v.y - mean) * inv * wv.y + bv.y, o2 = (v.z - mean) * inv * wv.z + bv.z,
+                o3 = (v.w - mean) * inv * wv.w + bv.w;
+    if constexpr (sizeof(TIO) == 2) *reinterpret_cast<uint2*>(y + yb + i) = make_uint2(pack_bf162(o0, o1), pack_bf162(o2, o3));
+    else *reinterpret_cast<float4*>(y + yb + i) = make_float4(o0, o1, o2, o3);
+  };
+  if (vec && (y_pitch & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      if (y1 != nullptr) norm4(i, w1, b1, y1);
+      if (y2 != nullptr) norm4(i, w2, b2, y2);
+    }
+    for (int i = W + threadIdx.x; i < y_pitch; i += blockDim.x) {
+      if (y1 != nullptr) io_st(y1 + yb + i, 0.f);
+      if (y2 != nullptr) io_st(y2 + yb + i, 0.f);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < y_pitch; i += blockDim.x) {
     const float n = i < W ? (row[i] - mean) * inv : 0.f;
     if (y1 != nullptr) io_st(y1 + yb + i, i < W ? n * w1[i] + b1[i] : 0.f);

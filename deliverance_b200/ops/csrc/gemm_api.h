@@ -236,17 +236,36 @@ struct LatentGeom {
   int dv, Kp;                      // value size per head, latent columns of the value weights (32-padded)
   int off_c, off_r, off_g;         // column offsets in the projection rows: latent, rotated key, gate (-1: no gate)
 };
-void launch_latent_prepare(void* p, long long ld, int rows, const int* positions, const long long* slots, const float* norm_w, const float* cos_t,
-                           const float* sin_t, int half, int max_pos, void* c_cache, void* r_cache, const LatentGeom& g, float eps, bool is_f32,
-                           cudaStream_t st);
+struct LatentPrep {
+  const int* positions;
+  const long long* slots;
+  const float *norm_w, *cos_t, *sin_t;
+  int half, max_pos;
+  void *c_cache, *r_cache;
+  float eps;
+};
+void launch_latent_prepare(void* p, long long ld, int rows, const LatentPrep& pr, const LatentGeom& g, bool is_f32, cudaStream_t st);
 void launch_latent_gather(const void* c_cache, const void* r_cache, const int* bt, int bt_stride, int page, const int* seq, const int* key0,
                           const int* n_keys, const int* row0, int num_seqs, int max_rows, void* c_out, int c_pitch, void* r_out, int r_pitch, int Rp, int drp,
                           cudaStream_t st);
-void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int rows, const void* wuk, void* q_lat, const LatentGeom& g, cudaStream_t st);
-int launch_latent_decode(const void* q_lat, const void* c_cache, const void* r_cache, const int* bt, int bt_stride, const int* row_seq, const int* row_ctx,
-                         int rows, float* part_o, float* part_ml, const LatentGeom& g, int page, float scale, int window, int splits, cudaStream_t st);
-void launch_latent_expand(const float* part_o, const float* part_ml, int splits, const int* row_idx, int rows, const void* wuv, const void* p, long long ld,
-                          void* out, int out_pitch, const LatentGeom& g, cudaStream_t st);
+void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int rows, const void* wuk, void* q_lat, const LatentGeom& g,
+                          const LatentPrep* prep, cudaStream_t st);
+struct LatentDecodeArgs {
+  const void *q_lat, *c_cache, *r_cache;
+  const int* bt;
+  int bt_stride;
+  const int *row_seq, *row_ctx;
+  int rows, page;
+  float scale;
+  int window, splits;      // splits: a power of two
+  void* o_lat;             // bf16 [rows, H, Rp]: result when the splits of a row are one cluster
+  float *part_o, *part_ml; // else fp32 [rows, H, clusters, Rp] and [rows, H, clusters, 2]
+};
+int latent_cluster_size(int splits);
+extern int g_latent_head_groups;
+int launch_latent_decode(const LatentDecodeArgs& a, const LatentGeom& g, cudaStream_t st);
+void launch_latent_expand(const LatentDecodeArgs& a, const int* row_idx, const void* wuv, const void* p, long long ld, void* out, int out_pitch,
+                          const LatentGeom& g, cudaStream_t st);
 int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, const int* row_seq, const int* row_ctx, int rows, const float* wuk,
                            const float* wuv, const float* c_cache, const float* r_cache, const int* bt, int bt_stride, float* out, int out_pitch,
                            const LatentGeom& g, int page, float scale, int window, cudaStream_t st);

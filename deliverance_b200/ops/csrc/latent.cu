@@ -12,6 +12,7 @@
 // Cache: c [pages, 1, page, Rp] and r [pages, 1, page, drp], Rp / drp = R / dr padded to 16 with zeros.
 #include <stdexcept>
 #include <string>
+#include <type_traits>
 
 #include "common.cuh"
 #include "gemm_api.h"
@@ -71,38 +72,16 @@ __device__ __forceinline__ void store8(float* p, const float* f) {
   *reinterpret_cast<float4*>(p + 4) = *reinterpret_cast<const float4*>(f + 4);
 }
 
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 }  // namespace
 
 // ------------------------------------------------------------------------------------------------ rotation, latent norm, cache write
-// One warp per (row, unit): unit h < H rotates the rotated query part of head h in place; unit H norms the latent, rotates the shared key
-// part and writes both to the cache rows (the projection row itself keeps its values).
+// One warp: norm of the latent and rotation of the shared key part of one projection row, both written to cache row `slot`.
 template <typename T>
-__global__ void __launch_bounds__(256) latent_prepare_kernel(T* __restrict__ p, long long ld, int rows, const int* __restrict__ positions,
-                                                             const long long* __restrict__ slots, const float* __restrict__ norm_w,
-                                                             const float* __restrict__ cos_t, const float* __restrict__ sin_t, int half, int max_pos,
-                                                             T* __restrict__ c_cache, T* __restrict__ r_cache, LatentGeom g, int dn_pad, float eps) {
-  pdl_wait();
-  pdl_trigger();
-  const int wg = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  const int units = g.H + 1;
-  if (wg >= rows * units) return;
-  const int t = wg / units, h = wg % units;
-  int pos = positions[t];
-  pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
-  const float* ct = cos_t + static_cast<size_t>(pos) * half;
-  const float* st = sin_t + static_cast<size_t>(pos) * half;
-  T* row = p + static_cast<long long>(t) * ld;
-  if (h < g.H) {
-    T* q = row + h * g.dk + dn_pad;
-    for (int i = lane; i < half; i += 32) {
-      const float u = ld1(q + i), v = ld1(q + i + half), c = ct[i], s = st[i];
-      st1(q + i, u * c - v * s);
-      st1(q + i + half, v * c + u * s);
-    }
-    return;
-  }
-  const long long slot = slots[t];
-  if (slot < 0) return;
+__device__ __forceinline__ void latent_cache_row(const T* __restrict__ row, long long slot, int pos, const LatentPrep& pr, const LatentGeom& g, int lane) {
+  const float* ct = pr.cos_t + static_cast<size_t>(pos) * pr.half;
+  const float* st = pr.sin_t + static_cast<size_t>(pos) * pr.half;
   const T* src = row + g.off_c;
   const int R8 = (g.R + 7) & ~7;
   float ss = 0.f;
@@ -113,39 +92,82 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(T* __restrict__ p, 
     for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
   }
   ss = warp_sum(ss);
-  const float inv = rsqrtf(ss / g.R + eps);
-  T* dst = c_cache + slot * g.Rp;
+  const float inv = rsqrtf(ss / g.R + pr.eps);
+  T* dst = static_cast<T*>(pr.c_cache) + slot * g.Rp;
   for (int i = lane * 8; i < g.Rp; i += 256) {
     float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
     if (i < R8) load8(src + i, f);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) f[e] *= inv * norm_w[i + e];  // (norm_w is zero-padded to Rp)
+    for (int e = 0; e < 8; ++e) f[e] *= inv * pr.norm_w[i + e];  // (norm_w is zero-padded to Rp)
     store8(dst + i, f);
   }
   const T* kr = row + g.off_r;
-  T* rd = r_cache + slot * g.drp;
+  T* rd = static_cast<T*>(pr.r_cache) + slot * g.drp;
   for (int i = lane; i < g.drp; i += 32) {
     float v = 0.f;
-    if (i < half) v = ld1(kr + i) * ct[i] - ld1(kr + i + half) * st[i];
-    else if (i < 2 * half) v = ld1(kr + i) * ct[i - half] + ld1(kr + i - half) * st[i - half];
+    if (i < pr.half) v = ld1(kr + i) * ct[i] - ld1(kr + i + pr.half) * st[i];
+    else if (i < 2 * pr.half) v = ld1(kr + i) * ct[i - pr.half] + ld1(kr + i - pr.half) * st[i - pr.half];
     else if (i < g.dr) v = ld1(kr + i);
     st1(rd + i, v);
   }
 }
+__device__ __forceinline__ int clamp_pos(int pos, int max_pos) { return pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos); }
 
-void launch_latent_prepare(void* p, long long ld, int rows, const int* positions, const long long* slots, const float* norm_w, const float* cos_t,
-                           const float* sin_t, int half, int max_pos, void* c_cache, void* r_cache, const LatentGeom& g, float eps, bool is_f32,
-                           cudaStream_t st) {
-  if (rows == 0) return;
+// grid.y 0: rotates the rotated query parts in place, one thread per VEC pairs (row, head, pairs i .. i + VEC - 1); grid.y 1: one warp per row
+// for the cache (the projection row itself keeps its latent and key).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) latent_prepare_kernel(T* __restrict__ p, long long ld, int rows, LatentPrep pr, LatentGeom g, int dn_pad) {
+  pdl_wait();
+  pdl_trigger();
+  if (blockIdx.y == 1) {
+    const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (t >= rows || pr.slots[t] < 0) return;
+    latent_cache_row<T>(p + t * ld, pr.slots[t], clamp_pos(pr.positions[t], pr.max_pos), pr, g, threadIdx.x & 31);
+    return;
+  }
+  const int per_head = pr.half / VEC, per_row = g.H * per_head;
+  const long long idx = static_cast<long long>(blockIdx.x) * 256 + threadIdx.x;
+  if (idx >= static_cast<long long>(rows) * per_row) return;
+  const int t = static_cast<int>(idx / per_row), k = static_cast<int>(idx % per_row), h = k / per_head, i = (k % per_head) * VEC;
+  const int pos = clamp_pos(pr.positions[t], pr.max_pos);
+  T* q = p + t * ld + h * g.dk + dn_pad + i;
+  const float* ct = pr.cos_t + static_cast<size_t>(pos) * pr.half + i;
+  const float* st = pr.sin_t + static_cast<size_t>(pos) * pr.half + i;
+  if constexpr (VEC == 8) {
+    float u[8], v[8], c[8], s[8];
+    load8(q, u);
+    load8(q + pr.half, v);
+    load8(ct, c);
+    load8(st, s);
+    float a[8], b[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      a[e] = u[e] * c[e] - v[e] * s[e];
+      b[e] = v[e] * c[e] + u[e] * s[e];
+    }
+    store8(q, a);
+    store8(q + pr.half, b);
+  } else {
+    const float u = ld1(q), v = ld1(q + pr.half), c = ct[0], s = st[0];
+    st1(q, u * c - v * s);
+    st1(q + pr.half, v * c + u * s);
+  }
+}
+
+template <typename T>
+static void launch_latent_prepare_t(void* p, long long ld, int rows, const LatentPrep& pr, const LatentGeom& g, cudaStream_t st) {
   const int dn_pad = (g.dn + 63) / 64 * 64;
-  const long long warps = static_cast<long long>(rows) * (g.H + 1);
-  const dim3 grid(static_cast<unsigned>((warps + 7) / 8));
-  if (is_f32)
-    launch_pdl(latent_prepare_kernel<float>, grid, dim3(256), 0, st, static_cast<float*>(p), ld, rows, positions, slots, norm_w, cos_t, sin_t, half, max_pos,
-               static_cast<float*>(c_cache), static_cast<float*>(r_cache), g, dn_pad, eps);
-  else
-    launch_pdl(latent_prepare_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<__nv_bfloat16*>(p), ld, rows, positions, slots, norm_w, cos_t, sin_t,
-               half, max_pos, static_cast<__nv_bfloat16*>(c_cache), static_cast<__nv_bfloat16*>(r_cache), g, dn_pad, eps);
+  const int vec = pr.half % 8 == 0 ? 8 : 1;
+  const long long rot = (static_cast<long long>(rows) * g.H * (pr.half / vec) + 255) / 256, cache = (rows + 7) / 8;
+  const dim3 grid(static_cast<unsigned>(rot > cache ? rot : cache), 2);
+  if (vec == 8) launch_pdl(latent_prepare_kernel<T, 8>, grid, dim3(256), 0, st, static_cast<T*>(p), ld, rows, pr, g, dn_pad);
+  else launch_pdl(latent_prepare_kernel<T, 1>, grid, dim3(256), 0, st, static_cast<T*>(p), ld, rows, pr, g, dn_pad);
+}
+
+void launch_latent_prepare(void* p, long long ld, int rows, const LatentPrep& pr, const LatentGeom& g, bool is_f32, cudaStream_t st) {
+  if (rows == 0) return;
+  if (is_f32) launch_latent_prepare_t<float>(p, ld, rows, pr, g, st);
+  else launch_latent_prepare_t<__nv_bfloat16>(p, ld, rows, pr, g, st);
 }
 
 // ------------------------------------------------------------------------------------------------ gather of cached rows for expansion
@@ -181,12 +203,25 @@ void launch_latent_gather(const void* c_cache, const void* r_cache, const int* b
 // q_lat[i][h] = [Wuk_h^T q_n (Rp) | q_r (drp)] for row i (row row_idx[i] of p). wuk [H][Rp][dn_pad]. mma.sync with 16 rows as the A operand;
 // A and B use the same assignment of k elements to the instruction's k positions (lane c of a group of four owns 8 consecutive elements of
 // every 32), so both operands are read with 16-byte loads. grid (H, row tiles of 16, blocks of 128 latent columns), 4 warps x 32 columns.
+// With `prep` (decode batches, row_idx == nullptr) the launch also does the work of latent_prepare_kernel: the query's rotated part is rotated
+// on its way to q_lat, and the CTAs of one more grid column write the cache rows.
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const __nv_bfloat16* __restrict__ p, long long ld, const int* __restrict__ row_idx, int rows,
                                                             const __nv_bfloat16* __restrict__ wuk, __nv_bfloat16* __restrict__ q_lat, LatentGeom g,
-                                                            int dn_pad) {
+                                                            int dn_pad, LatentPrep pr, int prep) {
+  const int h = blockIdx.x, i0 = blockIdx.y * 16, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, c = lane & 3;
+  if (h < g.H) {  // weights do not depend on the kernel in front: towards L2 while it finishes
+    const char* w0 = reinterpret_cast<const char*>(wuk + (static_cast<size_t>(h) * g.Rp + blockIdx.z * 128) * dn_pad);
+    const int bytes = min(128, g.Rp - static_cast<int>(blockIdx.z) * 128) * dn_pad * 2;
+    for (int o = threadIdx.x * 128; o < bytes; o += 128 * 128) prefetch_l2(w0 + o);
+  }
   pdl_wait();
   pdl_trigger();
-  const int h = blockIdx.x, i0 = blockIdx.y * 16, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, c = lane & 3;
+  if (h == g.H) {
+    for (int r = blockIdx.z * 4 + warp; r < 16; r += 4 * gridDim.z)
+      if (i0 + r < rows && pr.slots[i0 + r] >= 0)
+        latent_cache_row<__nv_bfloat16>(p + (i0 + r) * ld, pr.slots[i0 + r], clamp_pos(pr.positions[i0 + r], pr.max_pos), pr, g, lane);
+    return;
+  }
   const int CW = g.Rp + g.drp;
   const int n_base = blockIdx.z * 128 + warp * 32;
   if (n_base < g.Rp) {
@@ -219,93 +254,177 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const __nv_bfloat16*
       if (vb) *reinterpret_cast<uint32_t*>(q_lat + (static_cast<size_t>(i0 + gq + 8) * g.H + h) * CW + col) = pack_bf162(acc[n][2], acc[n][3]);
     }
   }
-  if (blockIdx.z == 0) {
-    for (int e = threadIdx.x; e < 16 * g.drp; e += 128) {
-      const int i = i0 + e / g.drp, d = e % g.drp;
-      if (i >= rows) continue;
-      const long long r = row_idx ? row_idx[i] : i;
-      q_lat[(static_cast<size_t>(i) * g.H + h) * CW + g.Rp + d] = p[r * ld + h * g.dk + dn_pad + d];  // (zero beyond dr: padding columns)
+  // rotated part: 8 threads per row, columns shared out over the blocks of the grid's z direction
+  const int i = i0 + (threadIdx.x >> 3);
+  if (i < rows) {
+    const long long r = row_idx ? row_idx[i] : i;
+    const __nv_bfloat16* q = p + r * ld + h * g.dk + dn_pad;
+    __nv_bfloat16* dst = q_lat + (static_cast<size_t>(i) * g.H + h) * CW + g.Rp;
+    const size_t at = prep ? static_cast<size_t>(clamp_pos(pr.positions[i], pr.max_pos)) * pr.half : 0;
+    for (int d = (threadIdx.x & 7) + 8 * blockIdx.z; d < g.drp; d += 8 * gridDim.z) {
+      __nv_bfloat16 v = q[d];  // (zero beyond dr: padding columns)
+      if (prep && d < 2 * pr.half) {
+        const int k = d < pr.half ? d : d - pr.half;
+        const float a = bf2f(q[k]), b = bf2f(q[k + pr.half]), cs = pr.cos_t[at + k], sn = pr.sin_t[at + k];
+        v = f2bf(d < pr.half ? a * cs - b * sn : b * cs + a * sn);
+      }
+      dst[d] = v;
     }
   }
 }
 
-void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int rows, const void* wuk, void* q_lat, const LatentGeom& g, cudaStream_t st) {
+void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int rows, const void* wuk, void* q_lat, const LatentGeom& g,
+                          const LatentPrep* prep, cudaStream_t st) {
   if (rows == 0) return;
-  launch_pdl(latent_absorb_kernel, dim3(g.H, (rows + 15) / 16, (g.Rp + 127) / 128), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(p), ld, row_idx, rows,
-             static_cast<const __nv_bfloat16*>(wuk), static_cast<__nv_bfloat16*>(q_lat), g, (g.dn + 63) / 64 * 64);
+  const LatentPrep none = {};
+  launch_pdl(latent_absorb_kernel, dim3(g.H + (prep ? 1 : 0), (rows + 15) / 16, (g.Rp + 127) / 128), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(p),
+             ld, row_idx, rows, static_cast<const __nv_bfloat16*>(wuk), static_cast<__nv_bfloat16*>(q_lat), g, (g.dn + 63) / 64 * 64, prep ? *prep : none,
+             prep ? 1 : 0);
 }
 
+// CTAs per cluster for a number of splits that is a power of two
+int latent_cluster_size(int splits) { return splits >= 8 ? 8 : (splits >= 4 ? 4 : (splits >= 2 ? 2 : 1)); }
+int g_latent_head_groups = 0;  // 1: groups of 16 heads only (tests, comparisons)
+
 // ------------------------------------------------------------------------------------------------ decode attention over the latent cache
-// grid (rows, groups of 16 * MH heads, splits), 8 warps. All heads of the group share every cached key row: tiles of BK keys ([c | r], padded
-// pitch so that ldmatrix is free of bank conflicts) arrive by cp.async in two stages; the score tile [16 MH heads x BK keys] is computed with
-// the keys split over the warps, goes through shared memory for the online softmax (fp32), and the probabilities come back as bf16 A
-// operand of the weighted sum, for which the warps split the latent columns (the K rows double as V). Partial sums leave in fp32, with the
-// running maximum and sum of every (row, head, split); latent_expand_kernel merges them.
-template <int MH, int BK>
+// grid (splits, rows, groups of 16 * MH heads), 8 * MH warps. All heads of the group share every cached key row: tiles of 32 keys ([c | r],
+// padded pitch so that ldmatrix is free of bank conflicts) arrive by cp.async, NST - 1 tiles ahead (one bulk copy per row and part instead
+// was slower, 77 against 64 us at 64 sequences of 2048 keys of 512 + 64: the copy engine starts one in about 40 ns). Per tile: the
+// scores [16 MH heads x 32 keys] (a warp owns 16 heads, 8 keys and half of the k range; most of its part of the query stays in registers,
+// because shared-memory bandwidth is what the tile loop runs out of first), through shared memory to the online softmax (fp32), and back as
+// the bf16 A operand of the weighted sum, for which the warps split the latent columns (the K rows double as V). For MH = 1 two CTAs share
+// an SM, so that the barriers of one hide under the other. The splits of a row form thread-block clusters of up to eight CTAs, which merge
+// their sums through distributed shared memory: with one cluster per row the normalised bf16 result leaves (o_lat), else one fp32 partial
+// (sum, maximum, denominator) per cluster.
+constexpr int kLdBK = 32;
+template <int MH>
 struct LatentDecodeSmem {
-  int pitch, pitch_p, pitch_s;
-  int off_q, off_p, off_s, off_st, bytes;
+  static constexpr int kRows = 16 * MH, kStages = MH == 1 ? 2 : 3;
+  static constexpr int kPitchP = (kLdBK + 8) * 2, kPitchS = kLdBK + 4;  // bytes, floats
+  int pitch, off_q, off_p, off_s, off_st, bytes;
   __host__ __device__ explicit LatentDecodeSmem(int CW) {
-    pitch = (CW + 8) * 2;         // CW is a multiple of 16: an odd number of 16-byte units
-    pitch_p = (BK + 8) * 2;
-    pitch_s = BK + 4;             // floats
-    off_q = 2 * BK * pitch;
-    off_p = off_q + 16 * MH * pitch;
-    off_s = off_p + 16 * MH * pitch_p;
-    off_st = off_s + 16 * MH * pitch_s * 4;
-    bytes = off_st + 3 * 16 * MH * 4;
+    pitch = (CW + 8) * 2;  // CW is a multiple of 16: an odd number of 16-byte units
+    off_q = kStages * kLdBK * pitch;
+    off_p = off_q + kRows * pitch;
+    off_s = off_p + kRows * kPitchP;
+    off_st = off_s + 2 * kRows * kPitchS * 4;
+    bytes = off_st + (3 + 8) * kRows * 4;
   }
 };
 
-template <int NPW, int MH, int BK>  // NPW: 16-column blocks of the latent per warp
-__global__ void __launch_bounds__(256) latent_decode_kernel(const __nv_bfloat16* __restrict__ q_lat, const __nv_bfloat16* __restrict__ c_cache,
-                                                            const __nv_bfloat16* __restrict__ r_cache, const int* __restrict__ bt, int bt_stride,
-                                                            const int* __restrict__ row_seq, const int* __restrict__ row_ctx, float* __restrict__ part_o,
-                                                            float* __restrict__ part_ml, LatentGeom g, int page, float scale, int window, int splits) {
+__device__ __forceinline__ uint32_t map_cluster(const void* p, uint32_t rank) {
+  uint32_t r;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(smem_u32(p)), "r"(rank));
+  return r;
+}
+__device__ __forceinline__ float ld_cluster_f1(const void* p, uint32_t rank) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(map_cluster(p, rank)) : "memory");
+  return v;
+}
+__device__ __forceinline__ float4 ld_cluster_f4(const void* p, uint32_t rank) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(map_cluster(p, rank)) : "memory");
+  return v;
+}
+__device__ __forceinline__ void cluster_barrier() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+// NPW: 16-column blocks of the latent per warp; NQ: k16 steps of the query a warp keeps in registers
+template <int NPW, int MH, int NQ>
+__global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) latent_decode_kernel(
+    const __nv_bfloat16* __restrict__ q_lat, const __nv_bfloat16* __restrict__ c_cache, const __nv_bfloat16* __restrict__ r_cache, const int* __restrict__ bt,
+    int bt_stride, const int* __restrict__ row_seq, const int* __restrict__ row_ctx, __nv_bfloat16* __restrict__ o_lat, float* __restrict__ part_o,
+    float* __restrict__ part_ml, LatentGeom g, int page, float scale, int window, int cs) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(128) uint8_t lsm[];
+  using L = LatentDecodeSmem<MH>;
+  constexpr int BK = kLdBK, ROWS = L::kRows, NST = L::kStages, NT = 256 * MH, NW = 8 * MH;
   const int CW = g.Rp + g.drp;
-  const LatentDecodeSmem<MH, BK> L(CW);
+  const L lay(CW);
   const uint32_t base_u = smem_u32(lsm);
-  float* sS = reinterpret_cast<float*>(lsm + L.off_s);
-  float* sM = reinterpret_cast<float*>(lsm + L.off_st);
-  float* sL = sM + 16 * MH;
-  float* sA = sL + 16 * MH;
-  const int i = blockIdx.x, h0 = blockIdx.y * 16 * MH, sp = blockIdx.z;
+  float* sS = reinterpret_cast<float*>(lsm + lay.off_s);
+  float* sM = reinterpret_cast<float*>(lsm + lay.off_st);
+  float* sL = sM + ROWS;
+  float* sA = sL + ROWS;
+  float* sW = sA + ROWS;  // [8][ROWS] merge weights
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, t4 = lane & 3;
-  const int nh = min(16 * MH, g.H - h0);
+  const int splits = gridDim.x, sp = blockIdx.x, i = blockIdx.y, h0 = blockIdx.z * ROWS;
+  const int nh = min(ROWS, g.H - h0);
   const int ctx = row_ctx[i];
-  const long long bt_row = static_cast<long long>(row_seq ? row_seq[i] : i) * bt_stride;
+  const int* bt_row = bt + static_cast<long long>(row_seq ? row_seq[i] : i) * bt_stride;
   const int first_key = (window > 0 && ctx > window) ? ctx - window : 0;
   const int tl = first_key / BK, th = (ctx + BK - 1) / BK;
   const int per = (th - tl + splits - 1) / splits;
-  const int t0 = tl + sp * per, t1 = min(th, t0 + per);
+  const int t0 = tl + sp * per, nt = max(0, min(th, t0 + per) - t0);
 
+  // NT / 32 threads per key row. A tile of 32 keys lies inside one page (page sizes are multiples of 32), so rows behind the context are
+  // rows of the same page: finite values that the mask gives weight zero.
   const int cq = CW / 8, cc = g.Rp / 8;  // 16-byte chunks per row: whole, latent part
-  for (int r = warp; r < 16 * MH; r += 8) {
+  const int lrow = tid / (NT / 32), lcol = tid % (NT / 32);
+  // place of the next tile to load: page index, its id (fetched one tile ahead of use) and the tile's first row in it
+  int pidx = t0 * BK / page, poff = t0 * BK - pidx * page, pg = nt > 0 ? bt_row[pidx] : 0;
+  const uint32_t ldst = base_u + lrow * lay.pitch + lcol * 16, stage_bytes = BK * lay.pitch;
+  const char* cbase = reinterpret_cast<const char*>(c_cache) + lcol * 16;
+  const char* rbase = reinterpret_cast<const char*>(r_cache) + lcol * 16;
+  const bool full_c = cc == 2 * NPW * (NT / 32);
+  auto load_tile = [&](int j) {
+    const uint32_t slot = static_cast<uint32_t>(pg * page + poff + lrow);  // (cache rows fit 31 bits: checked on the host)
+    const uint32_t dst = ldst + (j % NST) * stage_bytes;
+    const char* c = cbase + static_cast<unsigned long long>(slot) * static_cast<uint32_t>(g.Rp * 2);
+    const char* r = rbase + static_cast<unsigned long long>(slot) * static_cast<uint32_t>(g.drp * 2);
+    if (full_c) {
+#pragma unroll
+      for (int k = 0; k < 2 * NPW; ++k) cp_async16(dst + k * (NT / 2), c + k * (NT / 2), true);
+    } else {
+#pragma unroll
+      for (int k = 0; k < 2 * NPW; ++k)
+        if (lcol + k * (NT / 32) < cc) cp_async16(dst + k * (NT / 2), c + k * (NT / 2), true);
+    }
+    if (lcol < cq - cc) cp_async16(dst + cc * 16, r, true);
+    if (cq - cc > NT / 32)
+      for (int k = lcol + NT / 32; k < cq - cc; k += NT / 32) cp_async16(dst + (cc + k - lcol) * 16, r + (k - lcol) * 16, true);
+    poff += BK;
+    if (poff == page) {
+      poff = 0;
+      ++pidx;
+      if (j + 1 < nt) pg = bt_row[pidx];
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < NST - 1; ++j) {
+    if (j < nt) load_tile(j);
+    cp_async_commit();
+  }
+  for (int r = warp; r < ROWS; r += NW) {
     const __nv_bfloat16* src = q_lat + (static_cast<size_t>(i) * g.H + h0 + r) * CW;
     for (int k = lane; k < cq; k += 32)
-      *reinterpret_cast<uint4*>(lsm + L.off_q + r * L.pitch + k * 16) = r < nh ? *reinterpret_cast<const uint4*>(src + k * 8) : make_uint4(0u, 0u, 0u, 0u);
+      *reinterpret_cast<uint4*>(lsm + lay.off_q + r * lay.pitch + k * 16) = r < nh ? *reinterpret_cast<const uint4*>(src + k * 8) : make_uint4(0u, 0u, 0u, 0u);
   }
-  if (tid < 16 * MH) {
+  if (tid < ROWS) {
     sM[tid] = -INFINITY;
     sL[tid] = 0.f;
   }
-  auto load_tile = [&](int tile, int buf) {
+  __syncthreads();
+  const int np = g.Rp / 16, nks = CW / 16;
+  // score product of this warp: head group sm, keys skey .. + 7, k16 steps [ks0, ks0 + nk)
+  const int sm = warp >> 3, skey = (warp & 3) * 8, skh = (warp >> 2) & 1;
+  const int ks0 = skh * (nks / 2), nk = skh ? nks - nks / 2 : nks / 2;
+  const uint32_t qa = base_u + lay.off_q + (sm * 16 + (lane & 15)) * lay.pitch + (lane >> 4) * 16 + ks0 * 32;
+  // shared-memory addresses that only move with the stage
+  const uint32_t ka0 = base_u + (skey + (lane & 7)) * lay.pitch + (lane >> 3) * 16 + ks0 * 32;  // two k16 steps per ldmatrix.x4
+  const uint32_t va0 = base_u + ((lane & 7) + ((lane >> 3) & 1) * 8) * lay.pitch + (lane >> 4) * 16 + warp * 32;
+  const uint32_t pa0 = base_u + lay.off_p + (lane & 15) * L::kPitchP + (lane >> 4) * 16;
+  float* const sdst = sS + (skh * ROWS + sm * 16 + gq) * L::kPitchS + skey + 2 * t4;
+  const bool all_blocks = np == NPW * NW;
+  uint32_t soff = 0;  // byte offset of the current stage
+  uint32_t qr[NQ > 0 ? NQ : 1][4];
 #pragma unroll
-    for (int e = 0; e < BK / 8; ++e) {
-      const int r = warp * (BK / 8) + e, key = tile * BK + r;
-      const bool valid = key < ctx;
-      const long long slot = valid ? static_cast<long long>(bt[bt_row + key / page]) * page + key % page : 0;
-      const uint32_t dst = base_u + (buf * BK + r) * L.pitch;
-      for (int k = lane; k < cq; k += 32) {
-        const __nv_bfloat16* src = k < cc ? c_cache + slot * g.Rp + k * 8 : r_cache + slot * g.drp + (k - cc) * 8;
-        cp_async16(dst + k * 16, src, valid);
-      }
-    }
-    cp_async_commit();
-  };
+  for (int k = 0; k < NQ; ++k)
+    if (k < nk) ldmatrix_x4(qa + k * 32, qr[k]);
+    else qr[k][0] = qr[k][1] = qr[k][2] = qr[k][3] = 0u;
   float o[MH][NPW][2][4];
 #pragma unroll
   for (int m = 0; m < MH; ++m)
@@ -313,77 +432,80 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const __nv_bfloat16*
     for (int j = 0; j < NPW; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[m][j][0][e] = o[m][j][1][e] = 0.f;
-  const int np = g.Rp / 16;
-  if (t0 < t1) load_tile(t0, 0);
-  for (int tile = t0; tile < t1; ++tile) {
-    const int buf = (tile - t0) & 1;
-    if (tile + 1 < t1) {
-      load_tile(tile + 1, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
-    const uint32_t kb = base_u + buf * BK * L.pitch;
-    // ---- scores: MH == 1: warp w takes 8 keys; MH == 2: warps split as 2 head groups x 4 groups of 16 keys
-    if (MH == 2 || warp * 8 < BK) {
-      constexpr int NT = MH == 2 ? BK / 32 : 1;
-      const int m = MH == 2 ? (warp & 1) : 0, key_w = MH == 2 ? (warp >> 1) * (BK / 4) : warp * 8;
-      float s[NT][4];
+  for (int it = 0; it < nt; ++it) {
+    const int tile = t0 + it;
+    cp_async_wait<NST - 2>();
+    __syncthreads();  // the tile is here, and every warp is done with the stage of the previous one
+    if (it + NST - 1 < nt) load_tile(it + NST - 1);
+    cp_async_commit();
+    {
+      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};  // two accumulators: half the dependent chain
+      const uint32_t ka = ka0 + soff;
+      const uint32_t ka2 = ka - ((lane >> 4) << 5);  // one step: ldmatrix.x2 (lanes 16.. repeat the addresses of lanes 0..)
+      if (NQ > 0 && nk >= NQ) {
 #pragma unroll
-      for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-      const uint32_t qa = base_u + L.off_q + (m * 16 + (lane & 15)) * L.pitch + (lane >> 4) * 16;
-      const uint32_t ka = kb + (key_w + (NT == 2 ? (lane & 7) + (lane >> 4) * 8 : (lane & 7))) * L.pitch + ((lane >> 3) & 1) * 16;
-#pragma unroll 4
-      for (int ks = 0; ks < CW / 16; ++ks) {
-        uint32_t a[4];
-        ldmatrix_x4(qa + ks * 32, a);
-        if constexpr (NT == 2) {
+        for (int k = 0; k + 1 < NQ; k += 2) {
           uint32_t b[4];
-          ldmatrix_x4(ka + ks * 32, b);
-          mma_16816(s[0], a, b[0], b[1]);
-          mma_16816(s[1], a, b[2], b[3]);
-        } else {
+          ldmatrix_x4(ka + k * 32, b);
+          mma_16816(s0, qr[k], b[0], b[1]);
+          mma_16816(s1, qr[k + 1], b[2], b[3]);
+        }
+        if constexpr (NQ % 2 == 1) {
           uint32_t b[2];
-          ldmatrix_x2(ka + ks * 32, b);
-          mma_16816(s[0], a, b[0], b[1]);
+          ldmatrix_x2(ka2 + (NQ - 1) * 32, b);
+          mma_16816(s0, qr[NQ - 1], b[0], b[1]);
+        }
+      } else {
+#pragma unroll
+        for (int k = 0; k < NQ; k += 2) {
+          if (k + 1 < NQ && k + 1 < nk) {
+            uint32_t b[4];
+            ldmatrix_x4(ka + k * 32, b);
+            mma_16816(s0, qr[k], b[0], b[1]);
+            mma_16816(s1, qr[k + 1 < NQ ? k + 1 : k], b[2], b[3]);
+          } else if (k < nk) {
+            uint32_t b[2];
+            ldmatrix_x2(ka2 + k * 32, b);
+            mma_16816(s0, qr[k], b[0], b[1]);
+          }
         }
       }
-#pragma unroll
-      for (int n = 0; n < NT; ++n) {
-        const int col = key_w + n * 8 + 2 * t4;
-        float* d = sS + (m * 16 + gq) * L.pitch_s + col;
-        *reinterpret_cast<float2*>(d) = make_float2(s[n][0], s[n][1]);
-        *reinterpret_cast<float2*>(d + 8 * L.pitch_s) = make_float2(s[n][2], s[n][3]);
+      int k = NQ;
+      for (; k + 1 < nk; k += 2) {
+        uint32_t a0[4], a1[4], b[4];
+        ldmatrix_x4(ka + k * 32, b);
+        ldmatrix_x4(qa + k * 32, a0);
+        ldmatrix_x4(qa + k * 32 + 32, a1);
+        mma_16816(s0, a0, b[0], b[1]);
+        mma_16816(s1, a1, b[2], b[3]);
       }
+      if (k < nk) {
+        uint32_t a[4], b[2];
+        ldmatrix_x4(qa + k * 32, a);
+        ldmatrix_x2(ka2 + k * 32, b);
+        mma_16816(s0, a, b[0], b[1]);
+      }
+      *reinterpret_cast<float2*>(sdst) = make_float2(s0[0] + s1[0], s0[1] + s1[1]);
+      *reinterpret_cast<float2*>(sdst + 8 * L::kPitchS) = make_float2(s0[2] + s1[2], s0[3] + s1[3]);
     }
     __syncthreads();
-    // ---- online softmax: 256 / (16 MH) threads per head row
+    // ---- online softmax: 16 threads per head row, two neighbouring keys each
     {
-      constexpr int TPR = 16 / MH, KPT = BK / TPR;
-      const int r = tid / TPR, c0 = tid % TPR;
-      float v[KPT], mx = -INFINITY;
+      const int r = tid >> 4, c0 = (tid & 15) * 2, key = tile * BK + c0;
+      const float2 a = *reinterpret_cast<const float2*>(sS + r * L::kPitchS + c0), b = *reinterpret_cast<const float2*>(sS + (ROWS + r) * L::kPitchS + c0);
+      const float v0 = (key < ctx && key >= first_key) ? (a.x + b.x) * scale : -INFINITY;
+      const float v1 = (key + 1 < ctx && key + 1 >= first_key) ? (a.y + b.y) * scale : -INFINITY;
+      float mx = fmaxf(v0, v1);
 #pragma unroll
-      for (int e = 0; e < KPT; ++e) {
-        const int col = e * TPR + c0, key = tile * BK + col;
-        v[e] = (key < ctx && key >= first_key) ? sS[r * L.pitch_s + col] * scale : -INFINITY;
-        mx = fmaxf(mx, v[e]);
-      }
-#pragma unroll
-      for (int off = 1; off < TPR; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      for (int off = 1; off < 16; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
       const float m_old = sM[r], m_new = fmaxf(m_old, mx);
-      float sum = 0.f;
-      __nv_bfloat16* pr = reinterpret_cast<__nv_bfloat16*>(lsm + L.off_p + r * L.pitch_p);
+      const float w0 = v0 == -INFINITY ? 0.f : __expf(v0 - m_new), w1 = v1 == -INFINITY ? 0.f : __expf(v1 - m_new);
+      *reinterpret_cast<uint32_t*>(lsm + lay.off_p + r * L::kPitchP + c0 * 2) = pack_bf162(w0, w1);
+      float sum = w0 + w1;
 #pragma unroll
-      for (int e = 0; e < KPT; ++e) {
-        const float w = v[e] == -INFINITY ? 0.f : __expf(v[e] - m_new);
-        sum += w;
-        pr[e * TPR + c0] = f2bf(w);
-      }
-#pragma unroll
-      for (int off = 1; off < TPR; off <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      for (int off = 1; off < 16; off <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
       __syncwarp();
-      if (c0 == 0) {
+      if ((tid & 15) == 0) {
         const float alpha = m_old == -INFINITY ? 0.f : __expf(m_old - m_new);
         sA[r] = alpha;
         sM[r] = m_new;
@@ -391,190 +513,273 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const __nv_bfloat16*
       }
     }
     __syncthreads();
-    // ---- weighted sum: warp w owns the 16-column blocks w, w + 8, ...
+    // ---- weighted sum: warp w owns the 16-column blocks w, w + NW, ...
 #pragma unroll
     for (int m = 0; m < MH; ++m) {
       const float a0 = sA[m * 16 + gq], a1 = sA[m * 16 + gq + 8];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-      for (int j = 0; j < NPW; ++j)
+        for (int j = 0; j < NPW; ++j)
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          o[m][j][n][0] *= a0;
-          o[m][j][n][1] *= a0;
-          o[m][j][n][2] *= a1;
-          o[m][j][n][3] *= a1;
-        }
+          for (int n = 0; n < 2; ++n) {
+            o[m][j][n][0] *= a0;
+            o[m][j][n][1] *= a0;
+            o[m][j][n][2] *= a1;
+            o[m][j][n][3] *= a1;
+          }
+      }
     }
+    auto weighted = [&](auto whole) {
 #pragma unroll
-    for (int ks = 0; ks < BK / 16; ++ks) {
-      uint32_t a[MH][4];
+      for (int ks = 0; ks < BK / 16; ++ks) {
+        uint32_t a[MH][4];
 #pragma unroll
-      for (int m = 0; m < MH; ++m) ldmatrix_x4(base_u + L.off_p + (m * 16 + (lane & 15)) * L.pitch_p + (lane >> 4) * 16 + ks * 32, a[m]);
+        for (int m = 0; m < MH; ++m) ldmatrix_x4(pa0 + m * 16 * L::kPitchP + ks * 32, a[m]);
+        const uint32_t va = va0 + soff + ks * 16 * lay.pitch;
 #pragma unroll
-      for (int j = 0; j < NPW; ++j) {
-        const int blk = warp + 8 * j;
-        if (blk < np) {  // warp-uniform
-          uint32_t b[4];
-          ldmatrix_x4_trans(kb + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + blk * 32 + (lane >> 4) * 16, b);
+        for (int j = 0; j < NPW; ++j) {
+          if (decltype(whole)::value || warp + NW * j < np) {  // warp-uniform
+            uint32_t b[4];
+            ldmatrix_x4_trans(va + j * NW * 32, b);
 #pragma unroll
-          for (int m = 0; m < MH; ++m) {
-            mma_16816(o[m][j][0], a[m], b[0], b[1]);
-            mma_16816(o[m][j][1], a[m], b[2], b[3]);
+            for (int m = 0; m < MH; ++m) {
+              mma_16816(o[m][j][0], a[m], b[0], b[1]);
+              mma_16816(o[m][j][1], a[m], b[2], b[3]);
+            }
           }
         }
       }
-    }
-    __syncthreads();  // the stage, the scores and the probabilities are overwritten by the next tile
+    };
+    if (all_blocks) weighted(std::true_type());
+    else weighted(std::false_type());
+    soff = soff == (NST - 1) * stage_bytes ? 0 : soff + stage_bytes;
   }
-  // ---- partial results
+  cp_async_wait<0>();
+  __syncthreads();
+  // ---- merge of the cluster's sums
+  const int outer = splits / cs, op = sp / cs, PO = g.Rp + 4;
+  float* sO = reinterpret_cast<float*>(lsm);  // [ROWS][PO] (aliases the stages)
 #pragma unroll
   for (int m = 0; m < MH; ++m)
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = m * 16 + gq + half * 8;
-      if (r >= nh) continue;
-      float* dst = part_o + ((static_cast<size_t>(i) * g.H + h0 + r) * splits + sp) * g.Rp;
+    for (int j = 0; j < NPW; ++j) {
+      const int blk = warp + NW * j;
+      if (blk >= np) continue;
 #pragma unroll
-      for (int j = 0; j < NPW; ++j) {
-        const int blk = warp + 8 * j;
-        if (blk >= np) continue;
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-          *reinterpret_cast<float2*>(dst + blk * 16 + n * 8 + 2 * t4) = make_float2(o[m][j][n][2 * half], o[m][j][n][2 * half + 1]);
+      for (int n = 0; n < 2; ++n) {
+        float* d = sO + (m * 16 + gq) * PO + blk * 16 + n * 8 + 2 * t4;
+        *reinterpret_cast<float2*>(d) = make_float2(o[m][j][n][0], o[m][j][n][1]);
+        *reinterpret_cast<float2*>(d + 8 * PO) = make_float2(o[m][j][n][2], o[m][j][n][3]);
       }
     }
-  if (tid < nh) {
-    float* ml = part_ml + ((static_cast<size_t>(i) * g.H + h0 + tid) * splits + sp) * 2;
-    ml[0] = sM[tid];
-    ml[1] = sL[tid];
-  }
-}
-
-template <int NPW, int MH, int BK>
-static int launch_latent_decode_t(const void* q_lat, const void* c_cache, const void* r_cache, const int* bt, int bt_stride, const int* row_seq,
-                                  const int* row_ctx, int rows, float* part_o, float* part_ml, const LatentGeom& g, int page, float scale, int window,
-                                  int splits, cudaStream_t st) {
-  const LatentDecodeSmem<MH, BK> L(g.Rp + g.drp);
-  if (L.bytes > 227 * 1024) return 1;
-  static PerDeviceOnce attr_once;
-  if (attr_once.first()) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NPW, MH, BK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-    if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode attention: cudaFuncSetAttribute: ") + cudaGetErrorString(e));
-  }
-  launch_pdl(latent_decode_kernel<NPW, MH, BK>, dim3(rows, (g.H + 16 * MH - 1) / (16 * MH), splits), dim3(256), static_cast<size_t>(L.bytes), st,
-             static_cast<const __nv_bfloat16*>(q_lat), static_cast<const __nv_bfloat16*>(c_cache), static_cast<const __nv_bfloat16*>(r_cache), bt, bt_stride,
-             row_seq, row_ctx, part_o, part_ml, g, page, scale, window, splits);
-  return 0;
-}
-
-int launch_latent_decode(const void* q_lat, const void* c_cache, const void* r_cache, const int* bt, int bt_stride, const int* row_seq, const int* row_ctx,
-                         int rows, float* part_o, float* part_ml, const LatentGeom& g, int page, float scale, int window, int splits, cudaStream_t st) {
-  if (rows == 0) return 0;
-#define DLV_LD(N, M, B) \
-  return launch_latent_decode_t<N, M, B>(q_lat, c_cache, r_cache, bt, bt_stride, row_seq, row_ctx, rows, part_o, part_ml, g, page, scale, window, splits, st)
-  if (g.Rp <= 128) {
-    if (g.H > 16) { DLV_LD(1, 2, 64); }
-    DLV_LD(1, 1, 64);
-  }
-  if (g.Rp <= 256) {
-    if (g.H > 16) { DLV_LD(2, 2, 64); }
-    DLV_LD(2, 1, 64);
-  }
-  if (g.Rp <= 512) {
-    if (g.H > 16 && LatentDecodeSmem<2, 64>(g.Rp + g.drp).bytes <= 227 * 1024) { DLV_LD(4, 2, 64); }
-    if (LatentDecodeSmem<1, 64>(g.Rp + g.drp).bytes <= 227 * 1024) { DLV_LD(4, 1, 64); }
-  }
-  if (g.Rp <= 1024) { DLV_LD(8, 1, 32); }
-#undef DLV_LD
-  return 1;
-}
-
-// ------------------------------------------------------------------------------------------------ merge of the splits, value weights, gate
-// out[row][h * dv + v] = sigmoid(gate) * sum_r wuv[h][v][r] * o_lat[r], with o_lat = the normalised sum over the splits. wuv [H][dv8][Kp].
-// grid (H, row tiles of 16, blocks of 32 value columns), 4 warps x 8 columns; the merged rows are the A operand, staged in shared memory.
-constexpr int kLatentMaxSplits = 64;
-__global__ void __launch_bounds__(128) latent_expand_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
-                                                            const int* __restrict__ row_idx, int rows, const __nv_bfloat16* __restrict__ wuv,
-                                                            const __nv_bfloat16* __restrict__ p, long long ld, __nv_bfloat16* __restrict__ out, int out_pitch,
-                                                            LatentGeom g) {
-  pdl_wait();
-  pdl_trigger();
-  extern __shared__ __align__(16) uint8_t esm[];
-  const int pitch = g.Kp + 8;
-  __nv_bfloat16* sO = reinterpret_cast<__nv_bfloat16*>(esm);                 // [16][pitch]
-  float* sW = reinterpret_cast<float*>(esm + 16 * pitch * 2);                // [16][splits] weights, already divided by the row's sum
-  const int h = blockIdx.x, i0 = blockIdx.y * 16, n0 = blockIdx.z * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, c = lane & 3;
-  const int nr = min(16, rows - i0);
-  if (tid < 16) {
-    if (tid < nr) {
-      const float* ml = part_ml + (static_cast<size_t>(i0 + tid) * g.H + h) * splits * 2;
-      float m = -INFINITY;
-      for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
-      float den = 0.f;
-      for (int s = 0; s < splits; ++s) {
-        const float w = ml[2 * s] == -INFINITY ? 0.f : __expf(ml[2 * s] - m);
-        sW[tid * splits + s] = w;
-        den += w * ml[2 * s + 1];
+  const int rank = sp % cs;
+  if (cs > 1) cluster_barrier();
+  else __syncthreads();
+  if (tid < ROWS) {
+    float m = -INFINITY, ms[8], l = 0.f;
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (s < cs) {
+        ms[s] = cs > 1 ? ld_cluster_f1(sM + tid, s) : sM[tid];
+        m = fmaxf(m, ms[s]);
       }
-      const float inv = den > 0.f ? 1.f / den : 0.f;
-      for (int s = 0; s < splits; ++s) sW[tid * splits + s] *= inv;
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (s < cs) {
+        ms[s] = ms[s] == -INFINITY ? 0.f : __expf(ms[s] - m);
+        l += ms[s] * (cs > 1 ? ld_cluster_f1(sL + tid, s) : sL[tid]);
+      }
+    const float inv = outer > 1 ? 1.f : (l > 0.f ? 1.f / l : 0.f);
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (s < cs) sW[s * ROWS + tid] = ms[s] * inv;
+    if (outer > 1 && rank == 0 && tid < nh) {
+      float* ml = part_ml + ((static_cast<size_t>(i) * g.H + h0 + tid) * outer + op) * 2;
+      ml[0] = m;
+      ml[1] = l;
     }
   }
   __syncthreads();
-  const int quads = g.Kp / 4;
-  for (int e = tid; e < 16 * quads; e += 128) {
+  const int quads = g.Rp / 4;
+  for (int e = rank * NT + tid; e < nh * quads; e += cs * NT) {
     const int r = e / quads, k = (e % quads) * 4;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < nr && k < g.Rp) {
-      const float* src = part_o + (static_cast<size_t>(i0 + r) * g.H + h) * splits * g.Rp + k;
-      for (int s = 0; s < splits; ++s) {
-        const float w = sW[r * splits + s];
-        const float4 a = *reinterpret_cast<const float4*>(src + static_cast<size_t>(s) * g.Rp);
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (s < cs) {
+        const float w = sW[s * ROWS + r];
+        const float4 a = cs > 1 ? ld_cluster_f4(sO + r * PO + k, s) : *reinterpret_cast<const float4*>(sO + r * PO + k);
         v.x += w * a.x;
         v.y += w * a.y;
         v.z += w * a.z;
         v.w += w * a.w;
       }
+    const size_t head = static_cast<size_t>(i) * g.H + h0 + r;
+    if (outer > 1) *reinterpret_cast<float4*>(part_o + (head * outer + op) * g.Rp + k) = v;
+    else *reinterpret_cast<uint2*>(o_lat + head * g.Rp + k) = make_uint2(pack_bf162(v.x, v.y), pack_bf162(v.z, v.w));
+  }
+  if (cs > 1) cluster_barrier();  // nobody leaves while a peer still reads its shared memory
+}
+
+template <int NPW, int MH, int NQ>
+static int launch_latent_decode_t(const LatentDecodeArgs& a, const LatentGeom& g, cudaStream_t st) {
+  const LatentDecodeSmem<MH> L(g.Rp + g.drp);
+  if (L.bytes > 227 * 1024) return 1;
+  static PerDeviceOnce attr_once;
+  if (attr_once.first()) {
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NPW, MH, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode attention: cudaFuncSetAttribute: ") + cudaGetErrorString(e));
+  }
+  const int cs = latent_cluster_size(a.splits);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(a.splits, a.rows, (g.H + 16 * MH - 1) / (16 * MH));
+  cfg.blockDim = dim3(256 * MH);
+  cfg.dynamicSmemBytes = static_cast<size_t>(L.bytes);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = g_pdl_enabled ? 1 : 0;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = cs;
+  attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = cs > 1 ? 2 : 1;
+  cudaError_t e = cudaLaunchKernelEx(&cfg, latent_decode_kernel<NPW, MH, NQ>, static_cast<const __nv_bfloat16*>(a.q_lat),
+                                     static_cast<const __nv_bfloat16*>(a.c_cache), static_cast<const __nv_bfloat16*>(a.r_cache), a.bt, a.bt_stride, a.row_seq,
+                                     a.row_ctx, static_cast<__nv_bfloat16*>(a.o_lat), a.part_o, a.part_ml, g, a.page, a.scale, a.window, cs);
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode attention launch: ") + cudaGetErrorString(e));
+  return 0;
+}
+
+int launch_latent_decode(const LatentDecodeArgs& a, const LatentGeom& g, cudaStream_t st) {
+  if (a.rows == 0) return 0;
+  if (a.page % kLdBK != 0 || a.splits % latent_cluster_size(a.splits) != 0) return 2;
+  const bool two = g.H > 16 && LatentDecodeSmem<2>(g.Rp + g.drp).bytes <= 227 * 1024 && g_latent_head_groups != 1;
+  if (g.Rp <= 128) return two ? launch_latent_decode_t<1, 2, 6>(a, g, st) : launch_latent_decode_t<1, 1, 6>(a, g, st);
+  if (g.Rp <= 256) return two ? launch_latent_decode_t<1, 2, 9>(a, g, st) : launch_latent_decode_t<2, 1, 9>(a, g, st);
+  if (g.Rp <= 512) return two ? launch_latent_decode_t<2, 2, 12>(a, g, st) : launch_latent_decode_t<4, 1, 12>(a, g, st);
+  if (g.Rp <= 1024) return launch_latent_decode_t<8, 1, 0>(a, g, st);
+  return 1;
+}
+
+// ------------------------------------------------------------------------------------------------ value weights, gate (and merge)
+// out[row][h * dv + v] = sigmoid(gate) * sum_r wuv[h][v][r] * o_lat[r]. wuv [H][dv8][Kp]. grid (H, row tiles of 16, blocks of 32 value
+// columns), 4 warps x 8 columns, operands read as in latent_absorb_kernel. MERGE: o_lat is first summed from `outer` partials per row and head
+// into shared memory (few rows: a batch that needs more splits than one cluster).
+template <bool MERGE>
+__global__ void __launch_bounds__(128) latent_expand_kernel(const __nv_bfloat16* __restrict__ o_lat, const float* __restrict__ part_o,
+                                                            const float* __restrict__ part_ml, int outer, const int* __restrict__ row_idx, int rows,
+                                                            const __nv_bfloat16* __restrict__ wuv, const __nv_bfloat16* __restrict__ p, long long ld,
+                                                            __nv_bfloat16* __restrict__ out, int out_pitch, LatentGeom g) {
+  const int h = blockIdx.x, i0 = blockIdx.y * 16, n0 = blockIdx.z * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, c = lane & 3;
+  const int dv8 = (g.dv + 7) & ~7;
+  {  // weights do not depend on the kernel in front: towards L2 while it finishes
+    const char* w0 = reinterpret_cast<const char*>(wuv + (static_cast<size_t>(h) * dv8 + n0) * g.Kp);
+    for (int o = tid * 128; o < min(32, dv8 - n0) * g.Kp * 2; o += 128 * 128) prefetch_l2(w0 + o);
+  }
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) uint8_t esm[];
+  const int pitch = g.Kp + 8;
+  __nv_bfloat16* sO = reinterpret_cast<__nv_bfloat16*>(esm);                 // [16][pitch]
+  float* sW = reinterpret_cast<float*>(esm + 16 * pitch * 2);                // [16][outer] weights, already divided by the row's sum
+  const int nr = min(16, rows - i0);
+  if (MERGE) {
+    if (tid < nr) {
+      const float* ml = part_ml + (static_cast<size_t>(i0 + tid) * g.H + h) * outer * 2;
+      float m = -INFINITY;
+      for (int s = 0; s < outer; ++s) m = fmaxf(m, ml[2 * s]);
+      float den = 0.f;
+      for (int s = 0; s < outer; ++s) {
+        const float w = ml[2 * s] == -INFINITY ? 0.f : __expf(ml[2 * s] - m);
+        sW[tid * outer + s] = w;
+        den += w * ml[2 * s + 1];
+      }
+      const float inv = den > 0.f ? 1.f / den : 0.f;
+      for (int s = 0; s < outer; ++s) sW[tid * outer + s] *= inv;
     }
-    *reinterpret_cast<uint2*>(sO + r * pitch + k) = make_uint2(pack_bf162(v.x, v.y), pack_bf162(v.z, v.w));
-  }
-  __syncthreads();
-  const int dv8 = (g.dv + 7) & ~7, nb = n0 + warp * 8;
-  if (nb >= dv8) return;
-  float acc[4] = {0.f, 0.f, 0.f, 0.f};
-  const __nv_bfloat16* w = wuv + (static_cast<size_t>(h) * dv8 + nb + gq) * g.Kp + c * 8;
-  const __nv_bfloat16* xa = sO + gq * pitch + c * 8;
+    __syncthreads();
+    const int quads = g.Kp / 4;
+    for (int e = tid; e < 16 * quads; e += 128) {
+      const int r = e / quads, k = (e % quads) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < nr && k < g.Rp) {
+        const float* src = part_o + (static_cast<size_t>(i0 + r) * g.H + h) * outer * g.Rp + k;
 #pragma unroll 4
-  for (int k0 = 0; k0 < g.Kp; k0 += 32) {
-    const uint4 b = __ldg(reinterpret_cast<const uint4*>(w + k0));
-    const uint4 x0 = *reinterpret_cast<const uint4*>(xa + k0), x1 = *reinterpret_cast<const uint4*>(xa + 8 * pitch + k0);
-    const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
-    mma_16816(acc, a0, b.x, b.y);
-    mma_16816(acc, a1, b.z, b.w);
+        for (int s = 0; s < outer; ++s) {
+          const float w = sW[r * outer + s];
+          const float4 a = *reinterpret_cast<const float4*>(src + static_cast<size_t>(s) * g.Rp);
+          v.x += w * a.x;
+          v.y += w * a.y;
+          v.z += w * a.z;
+          v.w += w * a.w;
+        }
+      }
+      *reinterpret_cast<uint2*>(sO + r * pitch + k) = make_uint2(pack_bf162(v.x, v.y), pack_bf162(v.z, v.w));
+    }
+    __syncthreads();
   }
+  const int nb = n0 + warp * 8;
+  if (nb >= dv8) return;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  const bool va = gq < nr, vb = gq + 8 < nr;
+  const __nv_bfloat16* ga = o_lat + (static_cast<size_t>(i0 + (va ? gq : 0)) * g.H + h) * g.Rp + c * 8;
+  const __nv_bfloat16* gb = o_lat + (static_cast<size_t>(i0 + (vb ? gq + 8 : 0)) * g.H + h) * g.Rp + c * 8;
+  const __nv_bfloat16* xa = sO + gq * pitch + c * 8;
+  const __nv_bfloat16* w = wuv + (static_cast<size_t>(h) * dv8 + nb + gq) * g.Kp + c * 8;
+  // the epilogue's gate values travel under the product
+  float gate[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+  long long orow[2];
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int i = gq + half * 8;
-    if (i >= nr) continue;
-    const long long row = row_idx ? row_idx[i0 + i] : i0 + i;
+    orow[half] = i < nr ? (row_idx ? row_idx[i0 + i] : i0 + i) : 0;
+#pragma unroll
+    for (int e = 0; e < 2; ++e)
+      if (g.off_g >= 0 && i < nr && nb + 2 * c + e < g.dv) gate[half][e] = bf2f(p[orow[half] * ld + g.off_g + h * g.dv + nb + 2 * c + e]);
+  }
+  float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+  for (int k0 = 0; k0 < g.Kp; k0 += 32) {
+    const uint4 b = __ldg(reinterpret_cast<const uint4*>(w + k0));
+    uint4 x0, x1;
+    if (MERGE) {
+      x0 = *reinterpret_cast<const uint4*>(xa + k0);
+      x1 = *reinterpret_cast<const uint4*>(xa + 8 * pitch + k0);
+    } else {
+      const bool in = k0 + c * 8 < g.Rp;
+      x0 = va && in ? *reinterpret_cast<const uint4*>(ga + k0) : zero;
+      x1 = vb && in ? *reinterpret_cast<const uint4*>(gb + k0) : zero;
+    }
+    const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
+    mma_16816(acc, a0, b.x, b.y);
+    mma_16816(acc2, a1, b.z, b.w);
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    if (gq + half * 8 >= nr) continue;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int v = nb + 2 * c + e;
       if (v >= g.dv) continue;
-      float y = acc[half * 2 + e];
-      if (g.off_g >= 0) y /= 1.f + __expf(-bf2f(p[row * ld + g.off_g + h * g.dv + v]));
-      out[row * out_pitch + h * g.dv + v] = f2bf(y);
+      float y = acc[half * 2 + e] + acc2[half * 2 + e];
+      if (g.off_g >= 0) y /= 1.f + __expf(-gate[half][e]);
+      out[orow[half] * out_pitch + h * g.dv + v] = f2bf(y);
     }
   }
 }
 
-void launch_latent_expand(const float* part_o, const float* part_ml, int splits, const int* row_idx, int rows, const void* wuv, const void* p, long long ld,
-                          void* out, int out_pitch, const LatentGeom& g, cudaStream_t st) {
-  if (rows == 0) return;
-  const size_t smem = static_cast<size_t>(16) * (g.Kp + 8) * 2 + static_cast<size_t>(16) * splits * 4;
-  if (splits > kLatentMaxSplits || smem > 48 * 1024) throw std::runtime_error("latent expand: too many splits or latent columns");
-  launch_pdl(latent_expand_kernel, dim3(g.H, (rows + 15) / 16, (g.dv + 31) / 32), dim3(128), smem, st, part_o, part_ml, splits, row_idx, rows,
-             static_cast<const __nv_bfloat16*>(wuv), static_cast<const __nv_bfloat16*>(p), ld, static_cast<__nv_bfloat16*>(out), out_pitch, g);
+void launch_latent_expand(const LatentDecodeArgs& a, const int* row_idx, const void* wuv, const void* p, long long ld, void* out, int out_pitch,
+                          const LatentGeom& g, cudaStream_t st) {
+  if (a.rows == 0) return;
+  const int outer = a.splits / latent_cluster_size(a.splits);
+  const size_t smem = outer > 1 ? static_cast<size_t>(16) * (g.Kp + 8) * 2 + static_cast<size_t>(16) * outer * 4 : 0;
+  if (smem > 48 * 1024) throw std::runtime_error("latent expand: too many splits or latent columns");
+  const dim3 grid(g.H, (a.rows + 15) / 16, (g.dv + 31) / 32);
+  const auto *ol = static_cast<const __nv_bfloat16*>(a.o_lat), *w = static_cast<const __nv_bfloat16*>(wuv), *pp = static_cast<const __nv_bfloat16*>(p);
+  auto* o = static_cast<__nv_bfloat16*>(out);
+  if (outer > 1) launch_pdl(latent_expand_kernel<true>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g);
+  else launch_pdl(latent_expand_kernel<false>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g);
 }
 
 // ------------------------------------------------------------------------------------------------ 32-bit form

@@ -106,17 +106,21 @@ def prepare(s: LatentShape, p, positions, slots, norm_w, cos, sin, c_cache, r_ca
 
 
 def rows_attention(s: LatentShape, p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, scale: float, window: int,
-                   splits: int = 1) -> None:
+                   splits: int = 1, write=None) -> None:
     """Rows of ``p`` one by one against the cache (decode, short portions), absorbed form. Row ``i`` is ``p[row_idx[i]]`` of block-table
     row ``row_seq[i]`` and sees the last ``window`` of its first ``row_ctx[i]`` keys; ``None`` index arrays mean ``i``. Writes the gated
-    heads to columns ``[0, H * vdim)`` of the rows of ``out``."""
+    heads to columns ``[0, H * vdim)`` of the rows of ``out``. ``write`` = the arguments of :func:`prepare` behind ``p``, for a decode batch
+    whose rows were not prepared yet (on CUDA in bf16 that work rides in the first launch)."""
+    if write is not None and (not _cuda(p) or p.dtype == torch.float32):
+        prepare(s, p, *write)
     if _cuda(p):
         if p.dtype == torch.float32:
             _count()
             require_ext().latent_rows_f32(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window)
         else:
             _count(3)
-            require_ext().latent_decode(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window, splits)
+            require_ext().latent_decode(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window, splits,
+                                        *(() if write is None else (*write[:5], write[7])))
         return
     n = row_ctx.shape[0]
     ps = c_cache.shape[2]
@@ -155,14 +159,19 @@ def prefill_tile_rows(dv: int) -> int:
 
 
 def pick_splits(rows: int, s: LatentShape, span: Optional[int]) -> int:
-    """Split-KV factor of :func:`rows_attention`: the smallest one that fills the resident CTA slots evenly, at least two 64-key tiles each."""
-    ctas = max(1, rows * ((s.heads + 31) // 32 if s.heads > 16 else 1))
-    slots = 148 * (2 if s.Rp <= 256 else 1)
-    most = 64 if span is None else max(1, min(64, (span + 127) // 128))
-    best, best_eff = 1, 0.0
-    for k in range(1, most + 1):
-        n = ctas * k
-        eff = n / (-(-n // slots) * slots)
-        if eff > best_eff + 0.03:
-            best, best_eff = k, eff
+    """Split-KV factor of :func:`rows_attention`, a power of two: the cheapest by waves of CTAs x (32-key tiles per CTA + a fixed cost), plus
+    the merge of what does not fit one cluster of eight. (Clusters leave some SMs of a GPC unused: fewer CTAs are resident then.)"""
+    two = s.heads > 16
+    ctas = max(1, rows * ((s.heads + 31) // 32 if two else 1))
+    slots = 148 * (1 if two or s.Rp > 512 else 2)
+    tiles = max(1, (span + 31) // 32) if span is not None else 4096
+    best, best_cost = 1, None
+    for k in (1, 2, 4, 8, 16, 32, 64):
+        if k > 1 and 2 * k > tiles:
+            break
+        resident = int(slots * (0.8 if k >= 8 else 0.9 if k > 1 else 1.0))
+        outer = max(1, k // 8)
+        cost = -(-ctas * k // resident) * (-(-tiles // k) + 6) + (outer * (0.5 + 0.08 * rows) if outer > 1 else 0.0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = k, cost
     return best
