@@ -5,7 +5,7 @@
 Per size: prefill tokens/s (4 prompts of 2048), decode tokens/s at 1, 8 and 64 sequences (captured step replayed on the device, context
 2048), and device times of the kernels of one layer with their roofline fractions (L2 flushed before every timed launch; medians).
 The GQA decoder (llama family) has the same width, feed-forward, layer runs, vocabulary and query heads; its head_dim is 128 (64 for the
-small size) with one KV head per four query heads. Fractions are of the measured copy bandwidth and cuBLAS bf16 burst rate.
+small size) with one KV head per four query heads; its attention kernels are timed with the same sliding window. Fractions are of the measured copy bandwidth and cuBLAS bf16 burst rate.
 """
 from __future__ import annotations
 
@@ -180,31 +180,32 @@ def kernel_times(fat, gqa, z: dict, t: Timer, peaks: dict) -> list:
         cf, rf = kf.layer(0)
         cg, vg = kg.layer(0)
         wbytes = s.heads * s.kv_rank * (s.dim + s.vdim) * 2
-        add(f"rotation, norm, cache write {tag}", lambda: lop.prepare(s, p, b.positions, b.slots, mx.norm, mx.cos, mx.sin, cf, rf, 1e-5),
-            (T * (s.kv_rank + s.rot_dim + H * s.rot_dim) * 4, 0),
-            lambda: ops.rope_kv(qkv, b.positions, b.slots, None, None, gqa.cos, gqa.sin, cg, vg, H, KV, D, 1e-5), (T * (H + 2 * KV) * D * 4, 0))
         q = qkv[:, : H * D]
         if n == 1:
             span = min(2048, z["window"])
             sp = mx._splits(B, 2048)
             gsp = _engine_splits(B, KV)
-            args = (mx.wuk, mx.wuv, cf, rf, b.block_tables, row, mx.scale, mx.window, sp)
+            args = (mx.wuk, mx.wuv, cf, rf, b.block_tables, row, mx.scale, mx.window, sp, (b.positions, b.slots, mx.norm, mx.cos, mx.sin, cf, rf, 1e-5))
             keyb = B * span * (s.kv_rank + s.rot_dim) * 2
+            # absorbed query + rotation, norm and cache write + attention + value expansion and gate (three launches) against attention + merge
             add(f"decode attention {tag}", lambda: lop.rows_attention(s, p, None, None, b.ctx_len, *args),
                 (keyb + wbytes + T * H * (s.dim + s.rot_dim + 2 * s.vdim) * 2, 2.0 * B * H * (span * (2 * s.kv_rank + s.rot_dim) + s.kv_rank * (s.dim + s.vdim))),
-                lambda: ops.decode_attention(q, cg, vg, b.block_tables, b.ctx_len, H, D ** -0.5, 0.0, 0, gsp), (B * 2048 * 2 * KV * D * 2 + T * H * D * 4, 0))
+                lambda: ops.decode_attention(q, cg, vg, b.block_tables, b.ctx_len, H, D ** -0.5, 0.0, z["window"], gsp),
+                (B * span * 2 * KV * D * 2 + T * H * D * 4, 0))
         else:
+            add(f"rotation, norm, cache write {tag}", lambda: lop.prepare(s, p, b.positions, b.slots, mx.norm, mx.cos, mx.sin, cf, rf, 1e-5),
+                (T * (s.kv_rank + s.rot_dim + H * s.rot_dim) * 4, 0),
+                lambda: ops.rope_kv(qkv, b.positions, b.slots, None, None, gqa.cos, gqa.sin, cg, vg, H, KV, D, 1e-5), (T * (H + 2 * KV) * D * 4, 0))
             a = mx._plan(b)["prompts"]
             win = z["window"]
             pairs = B * (n * (n + 1) / 2 if win >= n else win * (n - win) + win * (win + 1) / 2)
-            full = B * n * (n + 1) / 2
             c, kr = lop.gather(s, cf, rf, b.block_tables, a["seq"], a["key0"], a["n_keys"], a["row0"], a["max_rows"], a["total"])
             kvx = ops.linear(c, mx.w_expand)
             add(f"prompt attention {tag}", lambda: lop.prefill_attention(s, p, kvx, kr, a["q_start"], a["q_len"], a["n_keys"], a["row0"], a["tile_seq"],
                                                                          a["tile_q0"], row, mx.scale, mx.window),
                 (0, 2.0 * pairs * H * (s.dim + s.rot_dim + s.vdim)),
-                lambda: ops.prefill_attention(q, cg, vg, b.block_tables, b.q_start, b.q_len, b.ctx_len, H, D ** -0.5, 0.0, 0, True, b.tile_seq, b.tile_q0,
-                                              tiles_for=b.tiles), (0, 4.0 * full * H * D))
+                lambda: ops.prefill_attention(q, cg, vg, b.block_tables, b.q_start, b.q_len, b.ctx_len, H, D ** -0.5, 0.0, win, True, b.tile_seq, b.tile_q0,
+                                              tiles_for=b.tiles), (0, 4.0 * pairs * H * D))
             xg = torch.randn(T, W, device=dev).to(torch.bfloat16)
             add(f"key / value expansion {tag} (against the gate|up GEMM)", lambda: ops.linear(c, mx.w_expand),
                 (mx.w_expand.N * mx.w_expand.K * 2 + T * (mx.w_expand.N + mx.w_expand.K) * 2, 2.0 * T * s.kv_rank * s.heads * (s.dim + s.vdim)),

@@ -498,7 +498,9 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
       float mx = fmaxf(v0, v1);
 #pragma unroll
       for (int off = 1; off < 16; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float m_old = sM[r], m_new = fmaxf(m_old, mx);
+      // the running maximum follows only when the scores have outgrown it by more than 8: a stale one costs head-room (weights up to e^8), a
+      // new one a pass over the accumulators
+      const float m_old = sM[r], m_new = mx > m_old + 8.f ? mx : m_old;
       const float w0 = v0 == -INFINITY ? 0.f : __expf(v0 - m_new), w1 = v1 == -INFINITY ? 0.f : __expf(v1 - m_new);
       *reinterpret_cast<uint32_t*>(lsm + lay.off_p + r * L::kPitchP + c0 * 2) = pack_bf162(w0, w1);
       float sum = w0 + w1;
@@ -506,7 +508,7 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
       for (int off = 1; off < 16; off <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
       __syncwarp();
       if ((tid & 15) == 0) {
-        const float alpha = m_old == -INFINITY ? 0.f : __expf(m_old - m_new);
+        const float alpha = m_old == m_new ? 1.f : __expf(m_old - m_new);  // (exp of -infinity: 0)
         sA[r] = alpha;
         sM[r] = m_new;
         sL[r] = sL[r] * alpha + sum;
