@@ -403,10 +403,6 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
     for (int k = lane; k < cq; k += 32)
       *reinterpret_cast<uint4*>(lsm + lay.off_q + r * lay.pitch + k * 16) = r < nh ? *reinterpret_cast<const uint4*>(src + k * 8) : make_uint4(0u, 0u, 0u, 0u);
   }
-  if (tid < ROWS) {
-    sM[tid] = -INFINITY;
-    sL[tid] = 0.f;
-  }
   __syncthreads();
   const int np = g.Rp / 16, nks = CW / 16;
   // score product of this warp: head group sm, keys skey .. + 7, k16 steps [ks0, ks0 + nk)
@@ -432,6 +428,7 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
     for (int j = 0; j < NPW; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[m][j][0][e] = o[m][j][1][e] = 0.f;
+  float m_run = -INFINITY, l_run = 0.f;  // softmax state of head row tid / 16
   for (int it = 0; it < nt; ++it) {
     const int tile = t0 + it;
     cp_async_wait<NST - 2>();
@@ -489,37 +486,36 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
       *reinterpret_cast<float2*>(sdst + 8 * L::kPitchS) = make_float2(s0[2] + s1[2], s0[3] + s1[3]);
     }
     __syncthreads();
-    // ---- online softmax: 16 threads per head row, two neighbouring keys each
+    // ---- online softmax: 16 threads per head row, two neighbouring keys each. The running maximum (the same in a row's threads) follows only
+    // when a score has outgrown it by more than 8: a stale one costs head-room (weights up to e^8), a new one a reduction and a pass over the
+    // accumulators. The denominator stays a partial sum per thread until the end.
+    bool grown;
     {
       const int r = tid >> 4, c0 = (tid & 15) * 2, key = tile * BK + c0;
       const float2 a = *reinterpret_cast<const float2*>(sS + r * L::kPitchS + c0), b = *reinterpret_cast<const float2*>(sS + (ROWS + r) * L::kPitchS + c0);
       const float v0 = (key < ctx && key >= first_key) ? (a.x + b.x) * scale : -INFINITY;
       const float v1 = (key + 1 < ctx && key + 1 >= first_key) ? (a.y + b.y) * scale : -INFINITY;
-      float mx = fmaxf(v0, v1);
+      float mx = fmaxf(v0, v1), alpha = 1.f;
+      grown = __any_sync(0xffffffffu, mx > m_run + 8.f);
+      if (grown) {  // warp-uniform
 #pragma unroll
-      for (int off = 1; off < 16; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      // the running maximum follows only when the scores have outgrown it by more than 8: a stale one costs head-room (weights up to e^8), a
-      // new one a pass over the accumulators
-      const float m_old = sM[r], m_new = mx > m_old + 8.f ? mx : m_old;
-      const float w0 = v0 == -INFINITY ? 0.f : __expf(v0 - m_new), w1 = v1 == -INFINITY ? 0.f : __expf(v1 - m_new);
-      *reinterpret_cast<uint32_t*>(lsm + lay.off_p + r * L::kPitchP + c0 * 2) = pack_bf162(w0, w1);
-      float sum = w0 + w1;
-#pragma unroll
-      for (int off = 1; off < 16; off <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
-      __syncwarp();
-      if ((tid & 15) == 0) {
-        const float alpha = m_old == m_new ? 1.f : __expf(m_old - m_new);  // (exp of -infinity: 0)
-        sA[r] = alpha;
-        sM[r] = m_new;
-        sL[r] = sL[r] * alpha + sum;
+        for (int off = 1; off < 16; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+        if (mx > m_run + 8.f) {
+          alpha = __expf(m_run - mx);  // (exp of -infinity: 0)
+          l_run *= alpha;
+          m_run = mx;
+        }
       }
+      if ((tid & 15) == 0) sA[r] = alpha;
+      const float w0 = v0 == -INFINITY ? 0.f : __expf(v0 - m_run), w1 = v1 == -INFINITY ? 0.f : __expf(v1 - m_run);
+      *reinterpret_cast<uint32_t*>(lsm + lay.off_p + r * L::kPitchP + c0 * 2) = pack_bf162(w0, w1);
+      l_run += w0 + w1;
     }
-    __syncthreads();
     // ---- weighted sum: warp w owns the 16-column blocks w, w + NW, ...
+    if (__syncthreads_or(grown)) {
 #pragma unroll
-    for (int m = 0; m < MH; ++m) {
-      const float a0 = sA[m * 16 + gq], a1 = sA[m * 16 + gq + 8];
-      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+      for (int m = 0; m < MH; ++m) {
+        const float a0 = sA[m * 16 + gq], a1 = sA[m * 16 + gq + 8];
 #pragma unroll
         for (int j = 0; j < NPW; ++j)
 #pragma unroll
@@ -557,6 +553,12 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
     soff = soff == (NST - 1) * stage_bytes ? 0 : soff + stage_bytes;
   }
   cp_async_wait<0>();
+#pragma unroll
+  for (int off = 1; off < 16; off <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
+  if ((tid & 15) == 0) {
+    sM[tid >> 4] = m_run;
+    sL[tid >> 4] = l_run;
+  }
   __syncthreads();
   // ---- merge of the cluster's sums
   const int outer = splits / cs, op = sp / cs, PO = g.Rp + 4;

@@ -90,7 +90,7 @@ def replay(engine, plan, requests):
 
 # --------------------------------------------------------------------------------------------------- single mechanisms
 @pytest.mark.parametrize("run", RUNS)
-@pytest.mark.parametrize("W,mp,mc,buckets", [(40, 127, 17, 61), (33, 1, 1, 7), (64, 4093, 9001, 1000)])
+@pytest.mark.parametrize("W,mp,mc,buckets", [(40, 139, 23, 61), (33, 1, 1, 7), (64, 4093, 9001, 1000)])
 def test_bigram_embedding(run, W, mp, mc, buckets):
     device, dtype = run
     V, toks = 50000, [49999, 0, 0, 3, 49998, 49999, 49999, 1]
