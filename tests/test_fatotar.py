@@ -552,3 +552,28 @@ def test_the_row_form_and_the_expanded_form_agree_on_cuda():
             ops.check_status()
     finally:
         ops.set_bounds_check(False)
+
+
+@gpu
+def test_groups_of_16_heads_give_the_same_decode_result():
+    """More than 16 heads per CTA (the default) and groups of 16, with one cluster per row and with several."""
+    run = ("cuda", torch.bfloat16)
+    mixer, m, W, kv, pages = mixer_case(run, 24, 32, 16, 24, 320, 900)
+    h = torch.randn(700, 48, generator=torch.Generator().manual_seed(6)).to(torch.bfloat16)
+    want = plain.latent_attention(W, m, "", h.double(), 1e-5)[697:]
+    s, ext = mixer.shape, ops.require_ext()
+    run_mixer(mixer, kv, h[:697], [697], pages, run)
+    for groups in (0, 1):
+        ext.latent_head_groups(groups)
+        try:
+            for splits in (1, 2, 8, 32):
+                mixer._splits = lambda rows, span: splits  # noqa: B023
+                out = []
+                for t in range(697, 700):
+                    b = make_batch([{"tokens": [0], "start": t, "pages": pages}], kv.page_size, "cuda")
+                    y = torch.zeros(1, s.out_width, dtype=torch.bfloat16, device="cuda")
+                    mixer.forward(h[t : t + 1].cuda(), b, kv.layer(0), y, lambda _: _Stage())
+                    out.append(y.float().cpu())
+                assert rel(torch.cat(out), want) < tol(torch.bfloat16), (groups, splits)
+        finally:
+            ext.latent_head_groups(0)
