@@ -124,6 +124,10 @@ def build_model(cfg: ModelConfig, device, dtype, tp: TensorParallelContext):
         from .models.fatotar import FatotarModel
 
         return FatotarModel(cfg, device, dtype, tp)
+    if cfg.model_type == "fopivik":
+        from .models.fopivik import FopivikModel
+
+        return FopivikModel(cfg, device, dtype, tp)
     return DecoderModel(cfg, device, dtype, tp)
 
 

@@ -18,10 +18,10 @@ from dataclasses import dataclass, field
 from typing import Any, Optional
 
 SUPPORTED_MODEL_TYPES = (
-    "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert", "fatotar",
+    "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert", "fatotar", "fopivik",
 )
 # designs whose config.json names an architecture instead of a model_type
-_ARCHITECTURE_TYPES = {"fatotar": "fatotar"}
+_ARCHITECTURE_TYPES = {"fatotar": "fatotar", "fopivik": "fopivik"}
 
 # transformers' Gemma3TextConfig defaults: hub configs of the multimodal checkpoints leave most text fields out
 _GEMMA3_TEXT_DEFAULTS = dict(vocab_size=262208, hidden_size=2304, intermediate_size=9216, num_hidden_layers=26, num_attention_heads=8,
@@ -56,7 +56,7 @@ class ModelConfig:
     attn_softcap: float = 0.0
     final_softcap: float = 0.0
     sliding_window: int = 0
-    layer_types: tuple[str, ...] = ()  # per layer: "attention" | "sliding" | "mamba" | "latent"
+    layer_types: tuple[str, ...] = ()  # per layer: "attention" | "sliding" | "mamba" | "latent" | "gla"
     # norms
     norm_weight_offset: float = 0.0  # gemma: (1 + w)
     post_norms: bool = False  # gemma2: post-attention and post-feedforward norms
@@ -206,6 +206,15 @@ def layer_run_order(n_layers: int, loop: Optional[dict]) -> tuple[int, ...]:
     return tuple(range(start)) + tuple(range(start, stop)) * times + tuple(range(stop, n_layers))
 
 
+def loop_pass_starts(n_layers: int, loop: Optional[dict]) -> dict:
+    """Layer run (index into :func:`layer_run_order`) at which each pass of the loop begins -> number of the pass."""
+    if not loop:
+        return {}
+    layer_run_order(n_layers, loop)  # (validates)
+    start, span = int(loop["start"]), int(loop["stop"]) - int(loop["start"])
+    return {start + t * span: t for t in range(int(loop["times"]))}
+
+
 def _parse_fatotar(d: dict) -> ModelConfig:
     """Fatotar: latent attention and a dense gated feed-forward side by side on one residual stream, LayerNorms, a hashed-bigram
     embedding, a range of layers that runs several times. Every layer carries its own sizes; ``extra["layers"]`` keeps them as
@@ -229,6 +238,35 @@ def _parse_fatotar(d: dict) -> ModelConfig:
         pad_token_id=d.get("pad_token_id"), layer_types=tuple("latent" for _ in order), use_rope=False, add_bos=False, raw=d,
     )
     cfg.extra = {"layers": layers, "order": order, "bigram": d["embedding"].get("bigram")}
+    return cfg
+
+
+def _parse_fopivik(d: dict) -> ModelConfig:
+    """Fopivik: gated-linear-attention and sliding-window softmax-attention layers in any order, routed experts, LayerNorms before and
+    after every sublayer, a range of layers that runs several times on a mix of the stream and the embedding. Every layer carries its own
+    sizes; ``extra["layers"]`` keeps them as given, ``extra["order"]`` is the weight layer of every layer run (a run has its own cache or
+    state), ``extra["passes"]`` maps the runs that begin a pass to its number. The context length is not part of the design."""
+    layers = list(d["layers"])
+    for i, L in enumerate(layers):
+        if L["type"] not in ("attention", "gla"):
+            raise ValueError(f"layer {i}: unknown mixer '{L['type']}'")
+        if L.get("mlp") and L["mlp"]["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward '{L['mlp']['kind']}'")
+    order = layer_run_order(len(layers), d.get("loop"))
+    soft = [L["mixer"] for L in layers if L["type"] == "attention"]
+    ff = [L["mlp"] for L in layers if L.get("mlp")]
+    cfg = ModelConfig(
+        model_type="fopivik", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), num_layers=len(order),
+        num_heads=max([int(m["heads"]) for m in soft] or [1]), num_kv_heads=max([int(m["kv_heads"]) for m in soft] or [1]),
+        head_dim=max([int(m["dim"]) for m in soft] or [8]), intermediate_size=max([int(m["expert"]["ff"]) for m in ff] or [0]),
+        max_position_embeddings=int(d.get("max_position_embeddings") or 131072), norm_eps=float(d["norm"]["eps"]), hidden_act="silu",
+        residual_multiplier=float(d["residual_mult"]), final_softcap=float(d.get("logit_softcap") or 0.0),
+        num_experts=max([int(m["router"]["experts"]) for m in ff] or [0]), experts_per_token=max([int(m["router"]["top"]) for m in ff] or [0]),
+        moe_intermediate_size=max([int(m["expert"]["ff"]) for m in ff] or [0]), norm_topk_prob=False, bos_token_id=d.get("bos_token_id"),
+        eos_token_ids=_eos(d.get("eos_token_id")), pad_token_id=d.get("pad_token_id"),
+        layer_types=tuple("gla" if layers[i]["type"] == "gla" else "sliding" for i in order), use_rope=False, add_bos=False, raw=d,
+    )
+    cfg.extra = {"layers": layers, "order": order, "passes": loop_pass_starts(len(layers), d.get("loop"))}
     return cfg
 
 
@@ -256,6 +294,8 @@ def parse_config(d: dict) -> ModelConfig:
         raise ValueError(f"unsupported model_type '{mt}' (supported: {', '.join(SUPPORTED_MODEL_TYPES)})")
     if mt == "fatotar":
         return _parse_fatotar(d)
+    if mt == "fopivik":
+        return _parse_fopivik(d)
     if mt in ("gemma4", "gemma4_text"):
         return _parse_gemma4(d)
     if mt in ("gemma3", "gemma3_text"):

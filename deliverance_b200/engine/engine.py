@@ -118,13 +118,8 @@ class Engine:
             # (a rank with a smaller pool would run a different batch and the collectives would no longer match): take the minimum
             mine = torch.tensor([float(pages)], dtype=torch.float32, device=self.device)
             pages = int(min(float(t.item()) for t in tp.collectives.all_gather(mine)))
-        mamba_shapes = None
-        slots = self.config.max_state_slots
-        if any(k == "mamba" for k in layout["layer_kinds"]):
-            c = self.cfg
-            mamba_shapes = {"conv": (c.mamba_conv_dim, c.mamba_d_conv - 1), "ssm": (c.mamba_n_heads, c.mamba_d_head, c.mamba_d_state)}
-            slots = slots or self.config.max_seqs
-        self.kv = PagedKVCache(layout, pages, self.device, model.dtype, self.config.kv, slots, mamba_shapes)
+        self.hybrid = any(layout.get("state_shapes") or [])  # recurrent layers: every sequence holds a state slot
+        self.kv = PagedKVCache(layout, pages, self.device, model.dtype, self.config.kv, self._state_slots(layout))
         self.page_size = self.kv.page_size
         self.max_pages_per_seq = (self.cfg.max_position_embeddings + self.page_size - 1) // self.page_size
         self.waiting: list[Request] = []
@@ -137,7 +132,6 @@ class Engine:
                         "graph_replays": 0, "kernel_launches": 0}
         # (a family that runs on the PyTorch operator set reads lengths on the host inside its forward: not capturable)
         self.use_graphs = bool(self.config.cuda_graphs and self.device.type == "cuda" and getattr(model, "supports_cuda_graphs", True))
-        self.hybrid = mamba_shapes is not None
         self.needs_prev = bool(getattr(model, "reads_previous_token", False))  # batches carry the token in front of every token
         # one-step lookahead of greedy graph decode: the step in flight whose sampled tokens the host has not read yet
         self._inflight: Optional[dict] = None
@@ -147,11 +141,15 @@ class Engine:
             e = ops.require_ext()
             e.init_scratch(self.device.index if self.device.index is not None else torch.cuda.current_device())
 
+    def _state_slots(self, layout) -> int:
+        return (self.config.max_state_slots or self.config.max_seqs) if any(layout.get("state_shapes") or []) else 0
+
     def _auto_pages(self, layout) -> int:
         per = max(1, PagedKVCache.bytes_per_page(layout, self.config.kv.block_size, self.model.dtype))
         if self.device.type == "cuda":
             free, _ = torch.cuda.mem_get_info(self.device)
-            budget = int(free * self.config.kv_memory_fraction)
+            free -= (1 + self._state_slots(layout)) * PagedKVCache.bytes_per_state_slot(layout)
+            budget = int(max(0, free) * self.config.kv_memory_fraction)
             # enough for max_seqs full contexts, never more than the budget
             want = self.config.max_seqs * ((self.cfg.max_position_embeddings + self.config.kv.block_size - 1) // self.config.kv.block_size) + 1
             return max(2, min(want, budget // per))
@@ -437,7 +435,8 @@ class Engine:
     def replay_step(self, entries: list) -> Optional[torch.Tensor]:
         """One batch of ``(request, next tokens, wanted places among them)``: prompt portions and single tokens together, exactly the
         forward passes of a scheduled step (a batch of single tokens of started requests is a decode step, captured graph included).
-        Returns fp32 logits of the wanted places in order (host memory), or None when nothing is wanted."""
+        Returns fp32 logits of the wanted places in order (host memory; scaled and soft-capped as the sampler sees them), or None when
+        nothing is wanted."""
         seqs, rows, base = [], [], 0
         for r, tokens, want in entries:
             if not tokens:
@@ -476,7 +475,11 @@ class Engine:
             return None
         if decode:  # one row per entry; batches of portions return the wanted rows only
             logits = logits.index_select(0, torch.tensor(rows, dtype=torch.int64, device=logits.device))
-        return self._full(logits).cpu()
+        logits = self._full(logits)
+        cap, inv_scale = self.cfg.final_softcap, self._inv_logit_scale()
+        if cap > 0 or inv_scale != 1.0:  # (a captured step's logits buffer stays as it is)
+            logits = ops.logits_post(logits.clone(), None, cap, inv_scale)
+        return logits.cpu()
 
     # ------------------------------------------------------------------------------------------------ decode
     def _decode_inputs(self, reqs: list[Request]):
@@ -660,6 +663,7 @@ class Engine:
             h["ctx"][n:] = 1
             h["slots"][n:] = torch.arange(n, bucket, dtype=torch.int64) % ps  # padded rows write into the scratch page
             bt[n:, :1] = 0
+            h["st"][n:] = 0  # ... and update the scratch state slot, not the slot an earlier batch had in this row
         b: ForwardBatch = g["batch"]
         b.token_ids.copy_(h["tok"], non_blocking=True)
         if dev_tokens is not None:  # lookahead: the previous step's samples never left the device
@@ -745,7 +749,7 @@ class Engine:
                     if r.guide is not None:
                         m[i] = r.guide.allowed_mask()
                 mask = m
-        inv_scale = 1.0 / cfg.logits_scaling if cfg.logits_scaling not in (0.0, 1.0) else 1.0
+        inv_scale = self._inv_logit_scale()
         all_greedy_plain = mask is None and all(r.sampling.greedy and not r.params.logprobs for r in reqs)
         if all_greedy_plain:
             tokens = self._greedy(logits).tolist()  # softcap and positive scaling keep the argmax
@@ -756,6 +760,9 @@ class Engine:
                 logits = ops.logits_post(logits if not self.use_graphs else logits.clone(), mask, cfg.final_softcap, inv_scale)
             tokens, lps = self.sampler.sample(logits, [r.sampling for r in reqs])
         return self._advance(reqs, tokens, lps)
+
+    def _inv_logit_scale(self) -> float:
+        return 1.0 / self.cfg.logits_scaling if self.cfg.logits_scaling not in (0.0, 1.0) else 1.0
 
     def _greedy(self, logits: torch.Tensor) -> torch.Tensor:
         fn = getattr(self.model, "greedy_tokens", None)

@@ -14,11 +14,14 @@ whose reference counts are bumped, so a hit costs no copy and no extra memory, a
 
 Layout per attention layer: ``k[pages, KV, page_size, D]`` and ``v[...]`` in the working dtype; page 0 is a scratch page
 that padded batch rows write to. Latent-attention layers use the same pair with one "head": ``k`` holds the compressed vectors, ``v``
-the rotated key parts shared by all heads (a width of its own, ``v_dim_per_layer``). Recurrent (mamba) layers get per-sequence state slots instead of pages.
+the rotated key parts shared by all heads (a width of its own, ``v_dim_per_layer``). Recurrent layers (Mamba2, gated linear
+attention) have no pages: a sequence holds one state slot, an index into the fp32 tensors named by the layout's ``state_shapes`` (one
+entry per layer: None, or name -> shape of one sequence's state). Slot 0 is a scratch slot that padded batch rows update.
 """
 from __future__ import annotations
 
 import hashlib
+import math
 from collections import OrderedDict
 from dataclasses import dataclass
 from typing import Optional
@@ -226,7 +229,7 @@ class PagedKVCache:
     """Device storage + allocator + prefix cache for one model replica (one tensor-parallel rank)."""
 
     def __init__(self, layout: dict, num_pages: int, device, dtype, settings: Optional[KvCacheSettings] = None,
-                 max_state_slots: int = 0, mamba_shapes: Optional[dict] = None):
+                 max_state_slots: int = 0):
         self.settings = settings or KvCacheSettings()
         self.page_size = self.settings.block_size
         if self.page_size % 32:
@@ -243,8 +246,9 @@ class PagedKVCache:
         dims = layout.get("head_dim_per_layer") or [layout["head_dim"]] * len(kinds)
         v_dims = layout.get("v_dim_per_layer") or dims
         shared = layout.get("shared_from") or [-1] * len(kinds)
-        for i, kind in enumerate(kinds):
-            if kind == "mamba":
+        states = layout.get("state_shapes") or [None] * len(kinds)
+        for i in range(len(kinds)):
+            if states[i]:
                 self.k.append(None)
                 self.v.append(None)
             elif shared[i] >= 0:
@@ -257,18 +261,21 @@ class PagedKVCache:
         self.allocator = PageAllocator(num_pages)
         self.prefix = PrefixCache(self.settings, self.allocator)
         self.prefix.kv = self
-        # recurrent state (hybrid models): per layer conv_state [slots, convDim, K-1] and ssm_state [slots, H, d_head, S]
-        self.conv_state: dict[int, torch.Tensor] = {}
-        self.ssm_state: dict[int, torch.Tensor] = {}
-        self.free_slots = list(range(max_state_slots - 1, -1, -1))
-        if mamba_shapes and max_state_slots > 0:
-            for i, kind in enumerate(kinds):
-                if kind == "mamba":
-                    self.conv_state[i] = torch.zeros((max_state_slots,) + tuple(mamba_shapes["conv"]), dtype=torch.float32, device=self.device)
-                    self.ssm_state[i] = torch.zeros((max_state_slots,) + tuple(mamba_shapes["ssm"]), dtype=torch.float32, device=self.device)
+        # recurrent state: name -> layer -> [1 + slots, ...] fp32 (slot 0 is scratch)
+        self.state: dict[str, dict[int, torch.Tensor]] = {}
+        self.free_slots = list(range(max_state_slots, 0, -1))
+        if max_state_slots > 0:
+            for i, shapes in enumerate(states):
+                for name, shape in (shapes or {}).items():
+                    t = torch.zeros((1 + max_state_slots,) + tuple(shape), dtype=torch.float32, device=self.device)
+                    self.state.setdefault(name, {})[i] = t
 
     def layer(self, i: int):
         return self.k[i], self.v[i]
+
+    @staticmethod
+    def bytes_per_state_slot(layout: dict) -> int:
+        return sum(4 * math.prod(shape) for shapes in layout.get("state_shapes") or [] if shapes for shape in shapes.values())
 
     @staticmethod
     def bytes_per_page(layout: dict, page_size: int, dtype) -> int:
@@ -277,7 +284,8 @@ class PagedKVCache:
         dims = layout.get("head_dim_per_layer") or [layout["head_dim"]] * len(kinds)
         shared = layout.get("shared_from") or [-1] * len(kinds)
         v_dims = layout.get("v_dim_per_layer") or dims
-        rows = sum(heads[i] * (dims[i] + v_dims[i]) for i, k in enumerate(kinds) if k != "mamba" and shared[i] < 0)
+        states = layout.get("state_shapes") or [None] * len(kinds)
+        rows = sum(heads[i] * (dims[i] + v_dims[i]) for i in range(len(kinds)) if not states[i] and shared[i] < 0)
         return rows * page_size * torch.empty((), dtype=dtype).element_size()
 
     # -- per-sequence page management ---------------------------------------------------------------------------
@@ -327,22 +335,23 @@ class PagedKVCache:
         if not self.free_slots:
             raise MemoryError("no free recurrent-state slot")
         s = self.free_slots.pop()
-        for t in list(self.conv_state.values()) + list(self.ssm_state.values()):
-            t[s].zero_()
+        for layers in self.state.values():
+            for t in layers.values():
+                t[s].zero_()
         return s
 
     def free_state_slot(self, s: int) -> None:
+        if s <= 0 or s in self.free_slots:
+            raise RuntimeError(f"state slot {s} is not in use")
         self.free_slots.append(s)
 
     def snapshot_state(self, slot: int) -> dict:
-        return {"conv": {i: t[slot].clone() for i, t in self.conv_state.items()},
-                "ssm": {i: t[slot].clone() for i, t in self.ssm_state.items()}}
+        return {name: {i: t[slot].clone() for i, t in layers.items()} for name, layers in self.state.items()}
 
     def restore_state(self, slot: int, snap: dict) -> None:
-        for i, t in snap["conv"].items():
-            self.conv_state[i][slot].copy_(t)
-        for i, t in snap["ssm"].items():
-            self.ssm_state[i][slot].copy_(t)
+        for name, layers in snap.items():
+            for i, t in layers.items():
+                self.state[name][i][slot].copy_(t)
 
     def attach_disk(self, directory: str, compression: str = "LZ4", bits: int = 4, max_bytes: int = 8 << 30, max_age_s: float = 0.0):
         """Spill evicted prefixes to ``directory`` and pull them back on later hits (attention-only models)."""

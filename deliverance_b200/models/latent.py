@@ -20,16 +20,16 @@ ROW_BY_ROW = 8
 
 
 class RotaryTables:
-    """cos / sin tables on one device, shared by the layers with the same rotation."""
+    """cos / sin tables on one device, shared by the layers with the same rotation. ``make``: table builder (frequency scaling rule)."""
 
-    def __init__(self, max_pos: int, device):
-        self.max_pos, self.device = max_pos, device
+    def __init__(self, max_pos: int, device, make=ref.yarn_rope_tables):
+        self.max_pos, self.device, self.make = max_pos, device, make
         self._tables: dict = {}
 
     def get(self, dims: int, base: float, scaling: Optional[dict]):
         key = (dims, base, tuple(sorted(scaling.items())) if scaling else None)
         if key not in self._tables:
-            cos, sin = ref.yarn_rope_tables(dims, self.max_pos, base, scaling)
+            cos, sin = self.make(dims, self.max_pos, base, scaling)
             self._tables[key] = (cos.to(self.device).contiguous(), sin.to(self.device).contiguous())
         return self._tables[key]
 

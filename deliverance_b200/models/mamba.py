@@ -19,7 +19,7 @@ def mamba_forward(model, i: int, lw, x: torch.Tensor, batch, kv) -> torch.Tensor
     cfg = model.cfg
     m = lw.mamba
     zx = ops.linear(x, m["in_proj"], out_f32=False)
-    conv_state, ssm_state = kv.conv_state[i], kv.ssm_state[i]
+    conv_state, ssm_state = kv.state["conv"][i], kv.state["ssm"][i]
     I = cfg.mamba_intermediate
     if x.device.type == "cuda":
         e = ops.require_ext()

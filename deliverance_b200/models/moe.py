@@ -1,4 +1,5 @@
-"""Mixture-of-experts feed-forward for mixtral, qwen3_moe and granitemoehybrid.
+"""Mixture-of-experts feed-forward for mixtral, qwen3_moe and granitemoehybrid, and :class:`RoutedExperts`, the same block with sizes
+and routing as parameters, for designs whose layers differ in them.
 
 Routing conventions (reference): Mixtral — softmax over all experts, top-k, renormalise
 (core/.../model/MixtureOfExpertsBlock.java:100-112); Qwen3-MoE — softmax over all, top-k, renormalise only with
@@ -16,7 +17,7 @@ import os
 import torch
 
 from .. import ops
-from ..ops import ref
+from ..ops import LinearWeight, ref
 
 
 _SM_COUNT = 148  # B200
@@ -90,12 +91,31 @@ def moe_forward_sharded(model, i: int, lw, x_own: torch.Tensor, a2a, total_rows:
 
 
 def _moe_cuda(model, lw, x, logits, E, k, mode, renorm, act, e0, ne):
-    e = ops.require_ext()
     st = model._stage
+    T = x.shape[0]
+    ys, pos, w, offsets = _experts_cuda(st, lw, x, logits, E, k, mode, renorm, act, e0, ne)
+    ep = ne != E
+    with st("moe.combine"):
+        fused = getattr(model.tp, "fused", None)
+        if ep and fused is not None:
+            y = fused.moe_combine_all_reduce(ys, pos, w, T, k, offsets, e0, ne)  # combine + sum over ranks in one kernel
+            if y is not None:
+                return y, True
+        ops._count()
+        rng = (offsets, e0, ne) if ep else (None, 0, 0)
+        return ops.require_ext().moe_combine(ys, pos, w, T, k, *rng), False
+
+
+def _experts_cuda(st, lw, x, logits, E, k, mode, renorm, act, e0, ne):
+    """Routing, expert-grouped gate|up, activation and down projection: ``(ys, pos, w, offsets)`` with the expert outputs ``ys [T * k, H]``
+    in grouped order, ``pos [T, k]`` the grouped row of every (token, slot) and its route weight ``w``."""
+    e = ops.require_ext()
     T, H = x.shape
     rows = T * k
     ep = ne != E
-    bn = ops.moe_token_tile(rows if not ep else max(1, rows * ne // E), ne, lw.experts_gate_up_grouped.q4)
+    gu_w, down_w = lw.experts_gate_up_grouped, lw.experts_down_grouped
+    f32 = x.dtype == torch.float32
+    bn = 64 if f32 else ops.moe_token_tile(rows if not ep else max(1, rows * ne // E), ne, gu_w.q4)
     if lw.fused_act_experts:
         bn = max(bn, 16)  # interleaved expert rows exist for the tensor-core grouped GEMM's epilogue only
     max_items = min((rows + bn - 1) // bn + ne, rows) if rows >= ne else rows
@@ -121,7 +141,11 @@ def _moe_cuda(model, lw, x, logits, E, k, mode, renorm, act, e0, ne):
         ops._count()
         return e.moe_gather(x, perm, k, *rng)
 
-    gu_w, down_w = lw.experts_gate_up_grouped, lw.experts_down_grouped
+    if f32:  # 32-bit models: plain FMA projections on the same work list
+        h = torch.empty(rows, gu_w.N // 2, dtype=x.dtype, device=x.device)
+        ops.gated_act_into(gu_w.run(gathered(), items, bn), act, h)
+        return down_w.run(h, items, bn), pos, w, offsets
+
     small = bn <= 64  # decode-sized groups: split K so that more CTAs stream weights
 
     def k_splits(wt) -> int:
@@ -153,11 +177,57 @@ def _moe_cuda(model, lw, x, logits, E, k, mode, renorm, act, e0, ne):
                 hmid = ops.act_mul(gu, act)
     with st("moe.down"):
         ys = down_w.run(hmid, items, bn, k_splits(down_w))
-    with st("moe.combine"):
-        fused = getattr(model.tp, "fused", None)
-        if ep and fused is not None:
-            y = fused.moe_combine_all_reduce(ys, pos, w, T, k, offsets, e0, ne)  # combine + sum over ranks in one kernel
-            if y is not None:
-                return y, True
-        ops._count()
-        return e.moe_combine(ys, pos, w, T, k, *rng), False
+    return ys, pos, w, offsets
+
+
+class RoutedExperts:
+    """Routed experts without biases: softmax (or top-k first) routing, ``top`` experts per token, gated activation. The result is left
+    in expert order (:class:`ops.Routed`) so that the norm behind it can do the weighted sum; ``ops.Routed.dense`` does it alone.
+
+    The expert width is padded to a multiple of 8 with zero rows, the input width to ``k_pad``."""
+
+    expert0, fused_act_experts = 0, False
+
+    def __init__(self, experts: int, top: int, act: str = "silu", mode: str = "softmax_topk", renorm: bool = False):
+        if not 0 < top <= experts:
+            raise ValueError(f"{top} of {experts} experts per token")
+        self.experts, self.top, self.act, self.mode, self.renorm = int(experts), int(top), act, mode, bool(renorm)
+        self.n_local_experts = self.experts
+        self.experts_gate_up: list = []
+        self.experts_down: list = []
+
+    def load(self, router, experts, ff: int, k_pad: int, device, dtype) -> "RoutedExperts":
+        """``experts``: (gate, up, down) per expert as stored."""
+        pad = torch.nn.functional.pad
+        ff8 = (ff + 7) // 8 * 8
+        put = lambda t: LinearWeight(t.to(device=device, dtype=dtype).contiguous())  # noqa: E731
+        if router.shape[0] != self.experts:
+            raise ValueError(f"router has {router.shape[0]} rows for {self.experts} experts")
+        self.router = put(pad(router, (0, k_pad - router.shape[1])))
+        for gate, up, down in experts:
+            if gate.shape[0] != ff or up.shape[0] != ff or down.shape[1] != ff:
+                raise ValueError(f"expert weights do not have the configured width {ff}")
+            wide = lambda t: pad(t, (0, k_pad - t.shape[1], 0, ff8 - ff))  # noqa: E731
+            self.experts_gate_up.append(put(torch.cat([wide(gate), wide(up)])))
+            self.experts_down.append(put(pad(down, (0, ff8 - ff, 0, k_pad - down.shape[0]))))
+        if torch.device(device).type == "cuda":
+            self.experts_gate_up_grouped = ops.GroupedLinearWeight(self.experts_gate_up)
+            self.experts_down_grouped = ops.GroupedLinearWeight(self.experts_down)
+            self.experts_gate_up, self.experts_down = [], []
+        return self
+
+    def nbytes(self) -> int:
+        if self.experts_gate_up:
+            return self.router.nbytes() + sum(w.nbytes() for w in self.experts_gate_up + self.experts_down)
+        return self.router.nbytes() + self.experts_gate_up_grouped.nbytes() + self.experts_down_grouped.nbytes()
+
+    def forward(self, x: torch.Tensor, stage) -> "ops.Routed":
+        with stage("moe.router"):
+            logits = ops.linear(x, self.router, out_f32=True)
+        if x.device.type == "cuda":
+            ys, pos, w, _ = _experts_cuda(stage, self, x, logits, self.experts, self.top, self.mode, self.renorm, self.act, 0, self.experts)
+            return ops.Routed(ys, pos.reshape(-1, self.top), w)
+        w, idx = ref.moe_route(logits, self.top, self.mode, self.renorm)
+        y = ref.moe_experts(x, w, idx, lambda e, rows: ops.linear(rows, self.experts_gate_up[e]), lambda e, h: ops.linear(h, self.experts_down[e]),
+                            self.experts, self.act)
+        return ops.Routed(y, None, None)

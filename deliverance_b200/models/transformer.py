@@ -589,8 +589,12 @@ class DecoderModel:
     # ------------------------------------------------------------------------------------------------ misc
     def kv_layout(self) -> dict:
         cfg = self.cfg
-        return {"layers": cfg.num_layers, "kv_heads": self.n_kv, "head_dim": cfg.head_dim,
-                "layer_kinds": [cfg.layer_type(i) for i in range(cfg.num_layers)]}
+        kinds = [cfg.layer_type(i) for i in range(cfg.num_layers)]
+        out = {"layers": cfg.num_layers, "kv_heads": self.n_kv, "head_dim": cfg.head_dim, "layer_kinds": kinds}
+        if "mamba" in kinds:
+            shapes = {"conv": (cfg.mamba_conv_dim, cfg.mamba_d_conv - 1), "ssm": (cfg.mamba_n_heads, cfg.mamba_d_head, cfg.mamba_d_state)}
+            out["state_shapes"] = [shapes if k == "mamba" else None for k in kinds]
+        return out
 
     def weight_bytes(self) -> int:
         n = self.embed.numel() * self.embed.element_size()

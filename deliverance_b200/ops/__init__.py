@@ -343,13 +343,17 @@ def embedding(table, ids, scale=1.0, pos_table=None, pos=None, type_table=None, 
     return out.to(dtype or table.dtype)
 
 
-def bigram_embedding(table, bigram, ids, prev, mul_prev: int, mul_cur: int, scale: float = 1.0) -> torch.Tensor:
+def bigram_embedding(table, bigram, ids, prev, mul_prev: int, mul_cur: int, scale: float = 1.0, copy_into=None) -> torch.Tensor:
     """fp32 ``table[ids] * scale + bigram[row]``; ``row = (prev * mul_prev + ids * mul_cur) mod buckets`` with ``buckets`` = rows of
-    ``bigram`` minus one, and the last row for tokens without a predecessor (``prev < 0``). ``bigram`` None: plain embedding."""
+    ``bigram`` minus one, and the last row for tokens without a predecessor (``prev < 0``). ``bigram`` None: plain embedding. ``copy_into``: a
+    column range ``[T, W]`` of wider rows that receives a copy in the table's type."""
     if _cuda(table):
         _count()
-        return require_ext().bigram_embedding(table, bigram, ids.to(torch.int32), prev, mul_prev, mul_cur, scale)
-    return ref.bigram_embedding(table, bigram, ids, prev, mul_prev, mul_cur, scale)
+        return require_ext().bigram_embedding(table, bigram, ids.to(torch.int32), prev, mul_prev, mul_cur, scale, copy_into)
+    out = ref.bigram_embedding(table, bigram, ids, prev, mul_prev, mul_cur, scale)
+    if copy_into is not None:
+        copy_into.copy_(out)
+    return out
 
 
 def add_layernorm(residual, delta, norm1, norm2, eps, pitch: int, dtype):
@@ -361,6 +365,36 @@ def add_layernorm(residual, delta, norm1, norm2, eps, pitch: int, dtype):
         _count()
         return tuple(require_ext().add_layernorm(residual, delta, w1, b1, w2, b2, eps, pitch, dtype == torch.float32))
     return ref.add_layernorm(residual, delta, norm1, norm2, eps, pitch, dtype)
+
+
+class Routed:
+    """Output of routed experts before the weighted sum: ``ys [T * k, W]`` in expert order, ``pos [T, k]`` rows of it per token, ``w [T, k]``
+    fp32 weights; or, with ``pos`` None, the finished ``[T, W]`` sum."""
+
+    def __init__(self, ys, pos, w):
+        self.ys, self.pos, self.w = ys, pos, w
+
+    def dense(self) -> torch.Tensor:
+        if self.pos is None:
+            return self.ys
+        return (self.ys[self.pos.long()].float() * self.w.unsqueeze(-1)).sum(dim=1)
+
+
+def sandwich_norm(residual, sub, w_sub, mult: float, w_next, eps: float, pitch: int, dtype, out=None):
+    """Norms behind and in front of a sublayer in one pass over an fp32 residual stream: ``residual += mult * LayerNorm(sub; w_sub)`` in place,
+    then ``LayerNorm(residual; w_next)``, or with ``w_next`` None the residual itself, in ``dtype``. LayerNorms have a weight and no bias.
+    ``sub``: ``[T, >= W]`` rows, a :class:`Routed` result (its weighted sum is formed here in fp32), or None (nothing is added). The result is
+    ``[T, pitch]`` (zeros behind the row width), or written to ``out``, a ``[T, W]`` column range of wider rows."""
+    if _cuda(residual):
+        _count()
+        ys, pos, w = (sub.ys, sub.pos, sub.w) if isinstance(sub, Routed) else (sub, None, None)
+        return require_ext().sandwich_norm(residual, ys, pos, w, w_sub, mult, w_next, eps, pitch, dtype == torch.float32, out)
+    W = residual.shape[1]
+    y = ref.sandwich_norm(residual, (sub.dense() if isinstance(sub, Routed) else sub[:, :W])[:, :W] if sub is not None else None, w_sub, mult, w_next, eps)
+    if out is None:
+        return torch.nn.functional.pad(y, (0, pitch - W)).to(dtype)
+    out.copy_(y)
+    return out
 
 
 def gated_act_into(gate_up, act: str, out) -> None:
@@ -566,7 +600,11 @@ class GroupedLinearWeight:
         if any(w.N != w0.N or w.K != w0.K or w.q4 != w0.q4 for w in weights):
             raise ValueError("experts of one layer must share shape and quantisation")
         self.E, self.N, self.K, self.q4 = len(weights), w0.N, w0.K, w0.q4
+        self.handle = None
         e = require_ext()
+        if not self.q4 and w0.w.dtype == torch.float32:  # 32-bit models: plain FMA projections (grouped_linear_f32)
+            self.data = torch.stack([w.w for w in weights]).contiguous()
+            return
         if self.q4:
             self.data = torch.cat([w.tiles for w in weights], 0).contiguous()
             self.handle = e.GemmWeight(self.data, True, self.E * ((self.N + 127) // 128) * 128, self.K)
@@ -579,6 +617,10 @@ class GroupedLinearWeight:
 
     def run(self, xs: torch.Tensor, items: torch.Tensor, bn: int, splits: int = 1, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         _count()
+        if self.handle is None:
+            if bn != 64 or splits != 1 or out is not None:
+                raise ValueError("fp32 grouped projections take 64-row work items")
+            return require_ext().grouped_linear_f32(xs, self.data, items)
         return self.handle.run_grouped(xs, items, self.N, bn, splits, out)
 
     def run_gemv_act(self, xs: torch.Tensor, items: torch.Tensor, act: str, perm: Optional[torch.Tensor] = None, k: int = 1) -> Optional[torch.Tensor]:
@@ -587,7 +629,7 @@ class GroupedLinearWeight:
         outside that kernel (the caller then runs projection and activation as two steps). With ``perm`` (the grouping permutation,
         ``[tokens * k]``) ``xs`` is the ungathered ``[tokens, K]`` activation: grouped row r reads token ``perm[r] // k``."""
         kind = fused_act_kind(act)
-        if kind == 0 or not self.q4:
+        if kind == 0 or not self.q4:  # (dense experts: two steps)
             return None
         out = self.handle.run_grouped_gemv_act(xs, items, self.N, kind, perm, k)
         if out is None:

@@ -90,6 +90,31 @@ def yarn_rope_tables(dims: int, max_pos: int, base: float, scaling: Optional[dic
     return (torch.cos(ang) * mult).float(), (torch.sin(ang) * mult).float()
 
 
+def banded_rope_tables(dims: int, max_pos: int, base: float, scaling: Optional[dict] = None):
+    """cos/sin tables ``[max_pos, dims/2]`` fp32 with Llama-3.1 frequency scaling. ``scaling``: pairs that turn more than ``high`` times
+    over ``original`` tokens keep their frequency, those that turn less than ``low`` times are slowed down by ``factor``, the turns in
+    between blend the two linearly."""
+    i = torch.arange(0, dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / dims)
+    if scaling:
+        factor, low, high = (float(scaling[k]) for k in ("factor", "low", "high"))
+        turns = float(scaling["original"]) * f / (2.0 * math.pi)
+        keep = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high != low else (turns > low).double()
+        f = f / factor * (1.0 - keep) + f * keep
+    ang = torch.arange(max_pos, dtype=torch.float64).unsqueeze(1) * f.unsqueeze(0)
+    return torch.cos(ang).float(), torch.sin(ang).float()
+
+
+def apply_rope_pairs(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """x ``[T, heads, d]``; rotates the first ``2 * cos.shape[1]`` dims with neighbouring pairs (2 i, 2 i + 1)."""
+    n = 2 * cos.shape[1]
+    c, s = cos[pos].unsqueeze(1), sin[pos].unsqueeze(1)
+    xf = x.float()
+    a, b = xf[..., 0:n:2], xf[..., 1:n:2]
+    out = torch.cat([torch.stack([a * c - b * s, b * c + a * s], dim=-1).flatten(-2), xf[..., n:]], dim=-1)
+    return out.to(x.dtype)
+
+
 def apply_rope(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
     """x ``[T, heads, d]``; rotates the first ``2 * cos.shape[1]`` dims with pairs (i, i + half)."""
     half = cos.shape[1]
@@ -128,17 +153,19 @@ def qk_prepare_and_cache(qkv, positions, slots, n_heads, n_kv, head_dim, q_norm_
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, scale, softcap=0.0, window=0,
-                    causal=True):
+                    causal=True, keep_first=0, sink=False):
     """Attention of ragged query rows against paged K/V.
 
     q ``[T, H, D]``; sequence ``i`` owns query rows ``[q_start[i], q_start[i] + q_len[i])`` which are the *last*
     ``q_len[i]`` positions of a context of ``ctx_len[i]`` cached tokens. Row at position ``p`` sees keys ``j <= p``
-    (and ``j > p - window`` when ``window > 0``). Score = ``softmax(softcap * tanh(scale * q.k / softcap))``.
+    (and ``j > p - window`` or ``j < keep_first`` when ``window > 0``). Score = ``softmax(softcap * tanh(scale * q.k / softcap))``;
+    ``sink``: a further score of 0 without a value takes part in the softmax. Values may be wider or narrower than keys.
     """
     T, H, D = q.shape
     nb, KV, bs, _ = k_cache.shape
+    DV = v_cache.shape[-1]
     group = H // KV
-    out = torch.zeros_like(q)
+    out = q.new_zeros(T, H, DV)
     for i in range(len(q_len)):
         ql, cl, qs = int(q_len[i]), int(ctx_len[i]), int(q_start[i])
         if ql == 0:
@@ -146,7 +173,7 @@ def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, 
         nblk = (cl + bs - 1) // bs
         blocks = block_tables[i, :nblk].long()
         k = k_cache[blocks].permute(1, 0, 2, 3).reshape(KV, nblk * bs, D)[:, :cl].float()
-        v = v_cache[blocks].permute(1, 0, 2, 3).reshape(KV, nblk * bs, D)[:, :cl].float()
+        v = v_cache[blocks].permute(1, 0, 2, 3).reshape(KV, nblk * bs, DV)[:, :cl].float()
         qi = q[qs : qs + ql].float().permute(1, 0, 2)  # H, ql, D
         k = k.repeat_interleave(group, dim=0)
         v = v.repeat_interleave(group, dim=0)
@@ -159,9 +186,9 @@ def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, 
         if causal:
             mask &= j <= pos
         if window and window > 0:
-            mask &= j > pos - window
+            mask &= (j > pos - window) | (j < keep_first)
         s = s.masked_fill(~mask.unsqueeze(0), float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        p = torch.softmax(F.pad(s, (0, 1)), dim=-1)[..., :-1] if sink else torch.softmax(s, dim=-1)
         out[qs : qs + ql] = torch.matmul(p, v).permute(1, 0, 2).to(q.dtype)
     return out
 
@@ -195,6 +222,17 @@ def add_layernorm(residual, delta, norm1, norm2, eps, pitch, dtype):
     n = d * torch.rsqrt(d.pow(2).mean(dim=-1, keepdim=True) + eps)
     pad = pitch - residual.shape[-1]
     return tuple(None if nb is None else F.pad(n * nb[0] + nb[1], (0, pad)).to(dtype) for nb in (norm1, norm2))
+
+
+def sandwich_norm(residual, sub, w_sub, mult, w_next, eps):
+    """fp32 ``residual += mult * LayerNorm(sub; w_sub)`` in place, then ``LayerNorm(residual; w_next)`` (the plain residual without it)."""
+    def norm(v, w):
+        d = v - v.mean(dim=-1, keepdim=True)
+        return d * torch.rsqrt(d.pow(2).mean(dim=-1, keepdim=True) + eps) * w
+
+    if sub is not None:
+        residual.add_(norm(sub.float(), w_sub), alpha=mult)
+    return residual if w_next is None else norm(residual, w_next)
 
 
 def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
@@ -281,6 +319,25 @@ def mamba2_sequential(zxbcdt, conv_w, conv_b, dt_bias, A_log, D, norm_w, eps, n_
         y = y * torch.rsqrt(y.pow(2).mean() + eps) * norm_w.float()
         out[t] = y
     return out
+
+
+# ---- gated linear attention ------------------------------------------------------------------------------------------
+def gla_sequential(q, k, v, z, q_scale: float, tau: float, state):
+    """Token-by-token gated linear attention of ONE sequence, fp32: ``S <- diag(sigmoid(z)^(1/tau)) S + k v^T``, ``o = S^T (q * q_scale)``.
+    q, k, z ``[T, H, dk]``, v ``[T, H, dv]``; ``state [H, dk, dv]`` is updated in place. Returns ``[T, H, dv]``."""
+    q, k, v = q.float() * q_scale, k.float(), v.float()
+    alpha = torch.exp(F.logsigmoid(z.float()) / tau)
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    for t in range(v.shape[0]):
+        state.mul_(alpha[t].unsqueeze(-1)).addcmul_(k[t].unsqueeze(-1), v[t].unsqueeze(-2))
+        out[t] = (state * q[t].unsqueeze(-1)).sum(dim=-2)
+    return out
+
+
+def gla_norm_gate(o, g, w, eps: float):
+    """``o [T, H, dv]`` RMS-normed over dv with the shared weight ``w [dv]``, times ``silu(g)``."""
+    o = o.float()
+    return o * torch.rsqrt(o.pow(2).mean(dim=-1, keepdim=True) + eps) * w * F.silu(g.float())
 
 
 # ---- sampling helpers --------------------------------------------------------------------------------------------------
