@@ -8,6 +8,7 @@
 // and (window == 0 or j > p - window)  (reference: core/.../generator/CausalSelfAttention.java:458-532,
 // tensor/.../operations/TensorOperations.java:225-271, tensor/.../VectorTensorMathUtils.java:34-78).
 #include "common.cuh"
+#include "gemm_api.h"
 
 namespace dlv {
 
@@ -240,11 +241,11 @@ __global__ void __launch_bounds__(128) decode_attn_kernel(
   }
 }
 
-// grid (num_seqs, H), D threads (D = 64 / 128 / 256). The split weights are computed once per CTA (thread s takes split s) and kept
+// grid (num_seqs, H), D threads rounded up to whole warps. The split weights are computed once per CTA (thread s takes split s) and kept
 // in shared memory; the weighted sum over the splits then runs with independent loads. (The first version had every thread walk
 // all splits twice with dependent loads: 12 us at 64 splits, more than the attention kernel it follows.)
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits) {
+                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits, int sink) {
   __shared__ float w_s[256];
   __shared__ float red[2][8];
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
@@ -272,6 +273,8 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   __syncthreads();
   den = 0.f;
   for (int i = 0; i < nw; ++i) den += red[1][i];
+  if (sink) den += __expf(-m);
+  if (d >= D) return;
   float num = 0.f;
   const int n_fast = splits < 256 ? splits : 256;
 #pragma unroll 8
@@ -307,7 +310,7 @@ static int launch_decode_t(const void* q, long long q_stride, const void* kc, co
                                                       scale, cap, window, splits);
   if (splits > 1) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits);
+    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits, 0);
   }
   return 0;
 }
@@ -389,25 +392,30 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     const __nv_bfloat16* __restrict__ q, long long q_stride, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables, int bt_stride,
     const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, float* part_o, float* part_ml, int* __restrict__ arrivals,
-    int H, int KV, int page_size, float scale, float softcap, int window, int splits) {
+    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk, int dv, int keep_first, int sink) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   using L = DecodeMma<D>;
   constexpr int CPR = D / 8;  // 16-byte chunks per row
   extern __shared__ __align__(128) uint8_t msm[];
-  const int b = blockIdx.x, kvh = blockIdx.y, sp = blockIdx.z;
+  // a CTA takes up to 16 of the query heads that share a KV head
+  const int heads_per_kv = H / KV, groups = (heads_per_kv + 15) / 16;
+  const int b = blockIdx.x, kvh = blockIdx.y / groups, sp = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t4 = lane & 3;
-  const int G = H / KV;
+  const int h0 = kvh * heads_per_kv + (blockIdx.y % groups) * 16;  // first query head of this CTA
+  const int G = min(16, (kvh + 1) * heads_per_kv - h0);
   const int ctx = ctx_lens[b];
   const int first_key = (window > 0 && ctx > window) ? ctx - window : 0;
-  // slices of 16 keys; the CTA's share of [first_key, ctx)
+  // slices of 16 keys: those that hold kept first tokens in front of the window, then [first_key, ctx); the CTA's share of that list
+  const int kept = min(keep_first, first_key);  // keys [0, kept) are visible beside the window
   const int sl_lo = first_key / 16, sl_hi = (ctx + 15) / 16;
-  const int per = (sl_hi - sl_lo + splits - 1) / splits;
-  const int s0 = sl_lo + sp * per, s1 = min(sl_hi, s0 + per);
+  const int sl_kept = min((kept + 15) / 16, sl_lo), sl_skip = sl_lo - sl_kept;  // list position i is slice i or, behind the kept ones, i + sl_skip
+  const int per = (sl_hi - sl_skip + splits - 1) / splits;
+  const int s0 = sp * per, s1 = min(sl_hi - sl_skip, s0 + per);
   uint8_t* ring = msm + warp * L::kWarpBytes;
   const uint32_t ring_u = smem_u32(ring);
-  const __nv_bfloat16* qrow = q + static_cast<long long>(b) * q_stride + static_cast<long long>(kvh) * G * D;
+  const __nv_bfloat16* qrow = q + static_cast<long long>(b) * q_stride + static_cast<long long>(h0) * dk;
 
   // ---- query A-fragments: registers (D <= 128) or a swizzled shared tile read with ldmatrix (D = 256)
   uint32_t qa[D <= 128 ? D / 16 : 1][4];
@@ -416,35 +424,35 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks) {
       const int d0 = ks * 16 + 2 * t4;
-      qa[ks][0] = g < G ? *reinterpret_cast<const uint32_t*>(qrow + g * D + d0) : 0u;
-      qa[ks][1] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qrow + (g + 8) * D + d0) : 0u;
-      qa[ks][2] = g < G ? *reinterpret_cast<const uint32_t*>(qrow + g * D + d0 + 8) : 0u;
-      qa[ks][3] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qrow + (g + 8) * D + d0 + 8) : 0u;
+      qa[ks][0] = g < G && d0 < dk ? *reinterpret_cast<const uint32_t*>(qrow + g * dk + d0) : 0u;
+      qa[ks][1] = g + 8 < G && d0 < dk ? *reinterpret_cast<const uint32_t*>(qrow + (g + 8) * dk + d0) : 0u;
+      qa[ks][2] = g < G && d0 + 8 < dk ? *reinterpret_cast<const uint32_t*>(qrow + g * dk + d0 + 8) : 0u;
+      qa[ks][3] = g + 8 < G && d0 + 8 < dk ? *reinterpret_cast<const uint32_t*>(qrow + (g + 8) * dk + d0 + 8) : 0u;
     }
   } else {
     for (int c = tid; c < 16 * CPR; c += 128) {
       const int r = c / CPR, cc = c % CPR;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < G) v = *reinterpret_cast<const uint4*>(qrow + r * D + cc * 8);
+      if (r < G && cc * 8 < dk) v = *reinterpret_cast<const uint4*>(qrow + r * dk + cc * 8);
       *reinterpret_cast<uint4*>(sQ + swz<D>(r, cc)) = v;
     }
     __syncthreads();
   }
 
-  auto load_slice = [&](int sl, int stage) {
-    // 16 keys x D of K and V: 2 * 16 * CPR chunks over 32 lanes
-    const int key0 = sl * 16;
+  auto slice_at = [&](int i) { return i < sl_kept ? i : i + sl_skip; };
+  auto load_slice = [&](int i, int stage) {
+    // 16 keys x D of K and V: 2 * 16 * CPR chunks over 32 lanes (zeros behind the real widths)
+    const int key0 = slice_at(i) * 16;
     const int page = block_tables[static_cast<long long>(b) * bt_stride + key0 / page_size];
-    const long long base = ((static_cast<long long>(page) * KV + kvh) * page_size + key0 % page_size) * D;
+    const long long row0 = (static_cast<long long>(page) * KV + kvh) * page_size + key0 % page_size;
     const uint32_t kdst = ring_u + stage * 2 * L::kSliceBytes, vdst = kdst + L::kSliceBytes;
 #pragma unroll
     for (int i = 0; i < 16 * CPR / 32; ++i) {
       const int c = i * 32 + lane;
       const int r = c / CPR, cc = c % CPR;
-      const bool valid = key0 + r < ctx;
-      const long long off = base + static_cast<long long>(valid ? r : 0) * D + cc * 8;
-      cp_async16(kdst + swz<D>(r, cc), k_cache + off, valid);
-      cp_async16(vdst + swz<D>(r, cc), v_cache + off, valid);
+      const bool in_ctx = key0 + r < ctx, vk = in_ctx && cc * 8 < dk, vv = in_ctx && cc * 8 < dv;
+      cp_async16(kdst + swz<D>(r, cc), k_cache + (vk ? (row0 + r) * dk + cc * 8 : row0 * dk), vk);
+      cp_async16(vdst + swz<D>(r, cc), v_cache + (vv ? (row0 + r) * dv + cc * 8 : row0 * dv), vv);
     }
   };
   // ---- per-warp pipeline over its slices
@@ -465,7 +473,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     cp_async_commit();
     cp_async_wait<L::kStages - 1>();
     __syncwarp();
-    const int key0 = (first + 4 * j) * 16;
+    const int key0 = slice_at(first + 4 * j) * 16;
     const uint32_t kbase = ring_u + stage * 2 * L::kSliceBytes, vbase = kbase + L::kSliceBytes;
     // S (16 heads x 16 keys) = Q K^T
     float sc[2][4];
@@ -493,7 +501,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + 2 * t4 + (e & 1);
         float v = softcap_apply(sc[nt][e] * scale, softcap);
-        v = (key < ctx && key >= first_key) ? v : -INFINITY;
+        v = (key < ctx && (key >= first_key || key < kept)) ? v : -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -572,8 +580,9 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     }
   }
   __syncthreads();
-  for (int idx = tid; idx < G * (D / 2); idx += 128) {
-    const int r = idx / (D / 2), d = (idx % (D / 2)) * 2;
+  const int dv2 = dv / 2;
+  for (int idx = tid; idx < G * dv2; idx += 128) {
+    const int r = idx / dv2, d = (idx % dv2) * 2;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, mg[(w * 16 + r) * (D + 2) + D]);
@@ -586,13 +595,14 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
       n1 += wt * row[d + 1];
       den += wt * row[D + 1];
     }
-    const int h = kvh * G + r;
+    const int h = h0 + r;
     if (splits == 1) {
+      if (sink) den += __expf(-m);  // the sink's score of 0, relative to the maximum
       const float inv = den > 0.f ? 1.f / den : 0.f;
-      *reinterpret_cast<uint32_t*>(out + (static_cast<long long>(b) * H + h) * D + d) = pack_bf162(n0 * inv, n1 * inv);
+      *reinterpret_cast<uint32_t*>(out + (static_cast<long long>(b) * H + h) * dv + d) = pack_bf162(n0 * inv, n1 * inv);
     } else {
       const long long base = (static_cast<long long>(b) * H + h) * splits + sp;
-      *reinterpret_cast<float2*>(part_o + base * D + d) = make_float2(n0, n1);
+      *reinterpret_cast<float2*>(part_o + base * dv + d) = make_float2(n0, n1);
       if (d == 0) {
         part_ml[base * 2] = m;
         part_ml[base * 2 + 1] = den;
@@ -658,7 +668,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
 template <int D>
 static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                                const int* ctx, void* out, float* po, float* pml, int* arrivals, int B, int H, int KV, int page,
-                               float scale, float cap, int window, int splits, cudaStream_t st) {
+                               float scale, float cap, int window, int splits, cudaStream_t st, int dk = D, int dv = D, AttnExtra x = {}) {
   using L = DecodeMma<D>;
   // the in-kernel merge keeps its weights in the warp-merge area of shared memory
   if (splits > 1 && (H / KV) * (splits + 1) > L::kMerge / 4) arrivals = nullptr;
@@ -666,14 +676,14 @@ static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc
   if (attr_once.first()) {
     cudaFuncSetAttribute(decode_attn_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
   }
-  dim3 grid(B, KV, splits);
+  dim3 grid(B, KV * ((H / KV + 15) / 16), splits);
   launch_pdl(decode_attn_mma_kernel<D>, dim3(grid), dim3(128), L::kBytes, st, static_cast<const __nv_bfloat16*>(q), q_stride,
                                                           static_cast<const __nv_bfloat16*>(kc), static_cast<const __nv_bfloat16*>(vc), bt,
                                                           bt_stride, ctx, static_cast<__nv_bfloat16*>(out), po, pml, arrivals, H, KV, page, scale,
-                                                          cap, window, splits);
+                                                          cap, window, splits, dk, dv, x.keep_first, x.sink);
   if (splits > 1 && arrivals == nullptr) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits);
+    launch_pdl(decode_merge_kernel, dim3(g2), dim3((dv + 31) / 32 * 32), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x.sink);
   }
   return 0;
 }
@@ -696,6 +706,97 @@ int launch_decode_attention_impl(const void* q, long long q_stride, const void* 
     }
   }
   return launch_decode_attention(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, B, H, KV, D, page, scale, cap, window, splits, st);
+}
+
+int launch_decode_attention_mma(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* ctx, void* out,
+                                float* po, float* pml, int B, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
+                                int splits, cudaStream_t st) {
+  if (B == 0) return 0;
+  const int D = dk > dv ? dk : dv;
+  if (dk % 8 != 0 || dv % 8 != 0 || D > 256 || page % 16 != 0 || q_stride % 8 != 0) return 1;
+#define DLV_DEC_MMA(DD) \
+  return launch_decode_mma_t<DD>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap, window, splits, st, dk, dv, x)
+  if (D <= 64) DLV_DEC_MMA(64);
+  if (D <= 128) DLV_DEC_MMA(128);
+  DLV_DEC_MMA(256);
+#undef DLV_DEC_MMA
+}
+
+// =====================================================================================================================
+// Any width, fp32 or bf16: one CTA per (row, query head) on CUDA cores
+// =====================================================================================================================
+// The warps take the visible keys (kept first tokens in front of the window, then the window) in turn, each with its own running maximum,
+// sum and value accumulators (shared memory), which are merged at the end. The 32-bit form of the attention layers, and the fallback for
+// heads the tensor-core kernels do not take.
+__device__ __forceinline__ float rows_ld(const float* p) { return *p; }
+__device__ __forceinline__ float rows_ld(const __nv_bfloat16* p) { return bf2f(*p); }
+__device__ __forceinline__ void rows_st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void rows_st(__nv_bfloat16* p, float v) { *p = f2bf(v); }
+
+template <typename TIO>
+__global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ q, long long q_stride, const TIO* __restrict__ k_cache,
+                                                        const TIO* __restrict__ v_cache, const int* __restrict__ bt, int bt_stride,
+                                                        const int* __restrict__ row_seq, const int* __restrict__ positions, TIO* __restrict__ out, int H, int KV,
+                                                        int dk, int dv, int page, float scale, float softcap, int window, int keep_first, int sink) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ float rsm[];  // q [dk] | accumulators [4][dv]
+  __shared__ float ml[4][2];
+  const int t = blockIdx.x, h = blockIdx.y, kvh = h / (H / KV);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float* acc = rsm + dk + warp * dv;
+  for (int d = tid; d < dk; d += 128) rsm[d] = rows_ld(q + t * q_stride + static_cast<long long>(h) * dk + d);
+  for (int d = lane; d < dv; d += 32) acc[d] = 0.f;
+  __syncthreads();
+  const int* table = bt + static_cast<long long>(row_seq != nullptr ? row_seq[t] : t) * bt_stride;
+  const int ctx = positions[t] + 1;
+  const int first = window > 0 && ctx > window ? ctx - window : 0, kept = min(keep_first, first);
+  float m = -INFINITY, l = 0.f;
+  for (int i = warp; i < kept + ctx - first; i += 4) {
+    const int key = i < kept ? i : first + i - kept;
+    const long long row = (static_cast<long long>(table[key / page]) * KV + kvh) * page + key % page;
+    float s = 0.f;
+    for (int d = lane; d < dk; d += 32) s += rsm[d] * rows_ld(k_cache + row * dk + d);
+    s = softcap_apply(warp_sum(s) * scale, softcap);
+    const float m_new = fmaxf(m, s), alpha = expf(m - m_new), pr = expf(s - m_new);
+    m = m_new;
+    l = l * alpha + pr;
+    for (int d = lane; d < dv; d += 32) acc[d] = acc[d] * alpha + pr * rows_ld(v_cache + row * dv + d);
+  }
+  if (lane == 0) {
+    ml[warp][0] = m;
+    ml[warp][1] = l;
+  }
+  __syncthreads();
+  m = fmaxf(fmaxf(ml[0][0], ml[1][0]), fmaxf(ml[2][0], ml[3][0]));
+  if (sink) m = fmaxf(m, 0.f);
+  float w[4], den = sink ? expf(-m) : 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    w[i] = ml[i][0] == -INFINITY ? 0.f : expf(ml[i][0] - m);
+    den += w[i] * ml[i][1];
+  }
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  for (int d = tid; d < dv; d += 128) {
+    const float* a = rsm + dk + d;
+    rows_st(out + (static_cast<long long>(t) * H + h) * dv + d, (w[0] * a[0] + w[1] * a[dv] + w[2] * a[2 * dv] + w[3] * a[3 * dv]) * inv);
+  }
+}
+
+int launch_attention_rows(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* row_seq,
+                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
+                          bool is_f32, cudaStream_t st) {
+  if (T == 0) return 0;
+  const size_t smem = static_cast<size_t>(dk + 4 * dv) * sizeof(float);
+  if (smem > 48 * 1024 - 256) return 1;
+#define DLV_ROWS(TT)                                                                                                                                     \
+  launch_pdl(attn_rows_kernel<TT>, dim3(T, H), dim3(128), smem, st, static_cast<const TT*>(q), q_stride, static_cast<const TT*>(kc),                      \
+             static_cast<const TT*>(vc), bt, bt_stride, row_seq, positions, static_cast<TT*>(out), H, KV, dk, dv, page, scale, cap, window, x.keep_first, \
+             x.sink)
+  if (is_f32) DLV_ROWS(float);
+  else DLV_ROWS(__nv_bfloat16);
+#undef DLV_ROWS
+  return 0;
 }
 
 // grid (num_q_tiles, H), 128 threads; tile i covers query rows [tile_q0[i], tile_q0[i] + 64) of sequence tile_seq[i]

@@ -23,7 +23,10 @@
 // (bounded), frees tensor memory and returns; CTAs that start after a recorded failure leave at once.
 //
 // Two layouts share the kernel (template parameter LATENT):
-//   paged   q [T, H * D], K and V rows in the paged cache, one head_dim for both, GQA groups;
+//   paged   q [T, H * dk], K and V rows in the paged cache, GQA groups; the real widths dk and dv may be smaller than DK and DV (multiples
+//           of 8): tensor-map bounds fill the columns behind a cache row with zeros, and query columns that reach into the next head meet
+//           zeros. The first `keep_first` keys stay visible beside a sliding window (their key tiles are listed in front of the window's),
+//           and `sink` adds a score of 0 without a value to the softmax;
 //   latent  keys and values expanded from the latent cache into flat rows (latent.cu): per head kn columns of an unrotated key part, one
 //           rotated key part shared by all heads (its own tensor map: it is copied behind the head's columns of every K tile, never
 //           materialised per head), DV columns of value. Key 0 of a sequence is its row kv_row0 of those buffers. The epilogue multiplies
@@ -55,11 +58,13 @@ struct AttnTcParams {
   int H, KV, page_size;
   float scale, softcap;
   int window, causal;
+  int keep_first, sink;
+  int dk;                      // query columns per head in q (paged layout: also the width of a K row)
   int* status;
+  int dv, out_pitch;           // real value columns per head, row pitch of out
   // latent layout only
   const int* kv_row0;          // [sequences] row of key 0 in the expanded buffers
   int kn_blocks;               // 64-column blocks of the per-head key part (the blocks behind it come from the shared part)
-  int dv, out_pitch;           // real value columns per head, row pitch of out
   const __nv_bfloat16* gate;   // gate logits [T, gate_pitch], head h at column h * dv (nullptr: no gate)
   int gate_pitch;
 };
@@ -130,6 +135,32 @@ __device__ __forceinline__ float fmax3(float a, float b, float c) {
   return y;
 }
 
+// f <- cap * tanh(f * a) for a thread's row of scores. Where all of a warp's arguments are small (scores far below the cap, the usual case)
+// the series of the hyperbolic tangent around 0 up to x^11 is exact to fp32 rounding and needs no special-function unit, which is what
+// limits the loop around it; otherwise tanh(x) = 1 - 2 / (e^(2 x) + 1), with an absolute error of a few units in the last place of 1.
+__device__ __forceinline__ void softcap_tile(float (&f)[kAtBN], float a, float cap) {
+  float mx = 0.f;
+#pragma unroll
+  for (int i = 0; i < kAtBN; ++i) mx = fmaxf(mx, fabsf(f[i]));
+  if (__all_sync(0xffffffffu, mx * a < 0.35f)) {
+    const float ac = a * cap, a2 = a * a;
+#pragma unroll
+    for (int i = 0; i < kAtBN; ++i) {
+      const float x2 = f[i] * f[i] * a2;
+      float s = fmaf(x2, -1382.f / 155925.f, 62.f / 2835.f);
+      s = fmaf(x2, s, -17.f / 315.f);
+      s = fmaf(x2, s, 2.f / 15.f);
+      s = fmaf(x2, s, -1.f / 3.f);
+      s = fmaf(x2, s, 1.f);
+      f[i] = f[i] * ac * s;
+    }
+  } else {
+    const float k = 2.f * 1.4426950408889634f * a;
+#pragma unroll
+    for (int i = 0; i < kAtBN; ++i) f[i] = cap - __fdividef(2.f * cap, ex2_approx(f[i] * k) + 1.f);
+  }
+}
+
 template <int DK, int DV, int QT, bool LATENT>
 __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,  // [T, H * DK], box 128 x 64
@@ -180,8 +211,12 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     b_q[q] = rows_q[q] > 0 ? (key_hi + kAtBN - 1) / kAtBN : a_q[q];
   }
   const int a0 = a_q[0], b0 = b_q[0], a1 = a_q[1], b1 = two ? b_q[1] : a_q[1];
-  const int lo = a0, hi = two ? max(b0, b1) : b0;  // key tiles this CTA loads
-  const int n_tiles = hi - lo;
+  // key tiles this CTA loads, in this order: those that hold kept first tokens in front of the window, then [lo, hi)
+  const int kept_tiles = (min(p.keep_first, ctx) + kAtBN - 1) / kAtBN;
+  const int lo = a0, hi = two ? max(b0, b1) : b0;
+  const int n_kept = min(kept_tiles, lo);
+  const int n_tiles = n_kept + hi - lo;
+  auto tile_at = [&](int u) { return u < n_kept ? u : lo + u - n_kept; };
 
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(bar_q), 1);
@@ -222,14 +257,14 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
       mbar_expect_tx(smem_u32(bar_q), (two ? 2 : 1) * L::kTileQ);
       for (int q = 0; q < (two ? 2 : 1); ++q)
         for (int c = 0; c < SUBK; ++c)
-          tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * DK + c * 64, qs + q0 + q * kAtBM);
+          tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0 + q * kAtBM);
     }
     const int box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;  // page_size is 32, 64 or 128
     int issued = 0;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t, ++issued) {
       const int s = t % NS;
-      const int kt = lo + t;
+      const int kt = tile_at(t);
       for (int kv = 0; kv < 2; ++kv) {
         uint64_t* full = kv == 0 ? &bar_k_full[s] : &bar_v_full[s];
         uint64_t* empty = kv == 0 ? &bar_k_empty[s] : &bar_v_empty[s];
@@ -285,30 +320,38 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     // feeds the pipe. Everything the two depend on travels through mbarriers; tcgen05.commit covers the MMAs of its own thread.
     constexpr uint32_t idesc_s = umma_idesc_bf16(kAtBM, kAtBN);
     constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(kAtBM, DV);
-    auto valid = [&](int j, int q) { return q == 0 ? (j >= a0 && j < b0) : (j >= a1 && j < b1); };
-    auto advance = [&](int& j, int& q) {  // next valid item; j == hi when there is none
+    auto valid = [&](int u, int q) {
+      const int j = tile_at(u);
+      return q == 0 ? ((j >= a0 || j < kept_tiles) && j < b0) : ((j >= a1 || j < kept_tiles) && j < b1);
+    };
+    auto advance = [&](int& u, int& q) {  // next valid item (u: place in the CTA's tile list); u == n_tiles when there is none
       do {
         if (two && q == 0) q = 1;
-        else { q = 0; ++j; }
-      } while (j < hi && !valid(j, q));
+        else { q = 0; ++u; }
+      } while (u < n_tiles && !valid(u, q));
     };
-    auto last_of_tile = [&](int j, int q) { return !two || q == 1 || !(j >= a1 && j < b1); };
+    auto last_of_tile = [&](int u, int q) { return !two || q == 1 || !valid(u, 1); };
+    // key tiles of query tile q before tile j (the same count its softmax warps keep)
+    auto count_at = [&](int u, int q) {
+      const int j = tile_at(u), a = q == 0 ? a0 : a1;
+      return j < kept_tiles ? j : j - max(a, kept_tiles) + kept_tiles;
+    };
     if (lane == 0) {
       bool ok = true;
-      int j = lo, q = 0;
-      if (n_tiles > 0 && !valid(j, q)) advance(j, q);
+      int u = 0, q = 0;
+      if (n_tiles > 0 && !valid(u, q)) advance(u, q);
       if (warp == kIssuer) {
         ok = mbar_wait(smem_u32(bar_q), 0, abort_flag, p.status);
         const uint64_t desc_q0 = umma_desc_k_sw128(smem_u32(smem)), desc_k0 = umma_desc_k_sw128(smem_u32(smem + L::kOffK));
-        int k_seen = lo - 1;  // key tiles whose K has been waited for
-        while (ok && j < hi) {
-          const int t = j - (q == 0 ? a0 : a1);
-          const int s = (j - lo) % NS;
+        int k_seen = -1;  // key tiles whose K has been waited for
+        while (ok && u < n_tiles) {
+          const int t = count_at(u, q);
+          const int s = u % NS;
           const uint32_t slot = q * 2 + (t & 1);
           if (t >= 2) ok = mbar_wait(smem_u32(&bar_pv_done[slot]), ((t >> 1) - 1) & 1, abort_flag, p.status);
-          if (ok && j > k_seen) {
-            ok = mbar_wait(smem_u32(&bar_k_full[s]), ((j - lo) / NS) & 1, abort_flag, p.status);
-            k_seen = j;
+          if (ok && u > k_seen) {
+            ok = mbar_wait(smem_u32(&bar_k_full[s]), (u / NS) & 1, abort_flag, p.status);
+            k_seen = u;
           }
           if (!ok) break;
           tc_fence_after();
@@ -321,18 +364,18 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
             const uint64_t adv_k = static_cast<uint64_t>(((k16 >> 2) * (kAtBN * 128) + (k16 & 3) * 32) >> 4);
             umma_bf16(d_s, desc_q + adv_q, desc_k + adv_k, idesc_s, k16 > 0 ? 1u : 0u);
           }
-          if (last_of_tile(j, q)) umma_commit(smem_u32(&bar_k_empty[s]));
+          if (last_of_tile(u, q)) umma_commit(smem_u32(&bar_k_empty[s]));
           umma_commit(smem_u32(&bar_s_full[slot]));
-          advance(j, q);
+          advance(u, q);
         }
       } else {
         const uint32_t v_base = smem_u32(smem + L::kOffV);
-        while (ok && j < hi) {
-          const int t = j - (q == 0 ? a0 : a1);
-          const int s = (j - lo) % NS;
+        while (ok && u < n_tiles) {
+          const int t = count_at(u, q);
+          const int s = u % NS;
           const uint32_t slot = q * 2 + (t & 1);
           ok = mbar_wait(smem_u32(&bar_p_full[slot]), (t >> 1) & 1, abort_flag, p.status) &&
-               mbar_wait(smem_u32(&bar_v_full[s]), ((j - lo) / NS) & 1, abort_flag, p.status);
+               mbar_wait(smem_u32(&bar_v_full[s]), (u / NS) & 1, abort_flag, p.status);
           if (!ok) break;
           tc_fence_after();
           const uint32_t tmem_p = tmem_base + kColS + slot * kAtBN, d_o = tmem_base + kColO + q * DV;
@@ -342,10 +385,10 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
             // 16 keys = two 8-row swizzle atoms (2048 bytes) further down the V tile; the 64-column blocks of D are kAtBN * 128 bytes apart
             umma_bf16_ts(d_o, tmem_p + k16 * 8, desc_v0 + static_cast<uint64_t>((k16 * 2048) >> 4), idesc_o, (t == 0 && k16 == 0) ? 0u : 1u);
           }
-          if (last_of_tile(j, q)) umma_commit(smem_u32(&bar_v_empty[s]));
+          if (last_of_tile(u, q)) umma_commit(smem_u32(&bar_v_empty[s]));
           umma_commit(smem_u32(&bar_pv_done[slot]));
-          advance(j, q);
-          if (j >= hi) umma_commit(smem_u32(bar_o_final));
+          advance(u, q);
+          if (u >= n_tiles) umma_commit(smem_u32(bar_o_final));
         }
         if (n_tiles == 0) umma_commit(smem_u32(bar_o_final));
       }
@@ -366,14 +409,15 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const int my_rows = q == 0 ? rows_q[0] : rows_q[1], my_first = q == 0 ? first_q[0] : first_q[1];
     const int ja = q == 0 ? a0 : a1, jb = q == 0 ? b0 : b1;
+    const int my_kept = min(kept_tiles, ja), my_tiles = my_kept + jb - ja;  // this query tile's key tiles: [0, my_kept), then [ja, jb)
     const int my_pos = my_first + r;
     const float c_log2 = 1.4426950408889634f;
     // scores stay in the units the tensor core delivers; kf turns a difference of scores into a base-2 exponent
     const float kf = p.softcap > 0.f ? c_log2 : p.scale * c_log2;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
-    for (int j = ja; j < jb && ok; ++j) {
-      const int t = j - ja;  // key tiles of this query tile so far
+    for (int t = 0; t < my_tiles && ok; ++t) {
+      const int j = t < my_kept ? t : ja + t - my_kept;
       const uint32_t slot = q * 2 + (t & 1);
       const uint32_t sb = lane_addr + kColS + slot * kAtBN;
       // warp-uniform: the loop holds warp-collective TMEM accesses
@@ -389,20 +433,18 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
         tmem_ld_wait();
       }
       if (p.softcap > 0.f) {
-        const float a = p.scale / p.softcap;
-#pragma unroll
-        for (int i = 0; i < kAtBN; ++i) f[i] = p.softcap * tanhf(f[i] * a);
+        softcap_tile(f, p.scale / p.softcap, p.softcap);
       }
       // is the whole tile visible to all 128 rows? (row 0 sees the fewest late keys, row 127 the fewest early ones)
-      const bool full = key_base + kAtBN <= min(ctx, p.causal ? my_first + 1 : ctx) && (p.window <= 0 || key_base >= my_first + kAtBM - p.window) &&
-                        my_rows == kAtBM;
+      const bool full = key_base + kAtBN <= min(ctx, p.causal ? my_first + 1 : ctx) && (p.window <= 0 || key_base >= my_first + kAtBM - p.window || key_base + kAtBN <= p.keep_first) && my_rows == kAtBM;
       if (!full) {
         // visible keys of this row inside the tile: [vlo, vhi)
         int vhi = min(ctx, p.causal ? my_pos + 1 : ctx) - key_base;
         int vlo = (p.window > 0 ? max(0, my_pos - p.window + 1) : 0) - key_base;
         if (r >= my_rows) vhi = vlo = 0;
+        const int kept = p.keep_first - key_base;  // keys of the tile in front of this one stay visible
 #pragma unroll
-        for (int i = 0; i < kAtBN; ++i) f[i] = (i >= vlo && i < vhi) ? f[i] : -INFINITY;
+        for (int i = 0; i < kAtBN; ++i) f[i] = ((i >= vlo || i < kept) && i < vhi) ? f[i] : -INFINITY;
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -467,14 +509,15 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     ok = __all_sync(0xffffffffu, ok && *abort_flag == 0);
     if (ok) {
       tc_fence_after();
+      if (p.sink) l_run += ex2_approx(-m_run * kf);  // the sink's score of 0, relative to the running maximum
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       const size_t trow = static_cast<size_t>(qs + q0 + q * kAtBM + r);
-      __nv_bfloat16* orow = p.out + (LATENT ? trow * p.out_pitch + static_cast<size_t>(h) * p.dv : trow * (static_cast<size_t>(p.H) * DV) + static_cast<size_t>(h) * DV);
+      __nv_bfloat16* orow = p.out + trow * p.out_pitch + static_cast<size_t>(h) * p.dv;
       const __nv_bfloat16* grow = LATENT && p.gate != nullptr ? p.gate + trow * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
 #pragma unroll 1
       for (int c0 = 0; c0 < DV; c0 += 32) {
         uint32_t v[32];
-        if (jb > ja) {
+        if (my_tiles > 0) {
           tmem_ld_x32(lane_addr + kColO + q * DV + c0, v);
           tmem_ld_wait();
         } else {
@@ -513,6 +556,7 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
         } else if (r < my_rows) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if (c0 + i >= p.dv) break;
             uint4 o;
             o.x = pack_bf162(__uint_as_float(v[i]) * inv, __uint_as_float(v[i + 1]) * inv);
             o.y = pack_bf162(__uint_as_float(v[i + 2]) * inv, __uint_as_float(v[i + 3]) * inv);
@@ -560,10 +604,10 @@ template <int D, int QT>
 static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
                                int num_tiles, cudaStream_t st) {
   CUtensorMap mq, mk, mv;
-  encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * D, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
+  encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * p.dk, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
   const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
-  encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
-  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), D, static_cast<uint64_t>(D) * 2, box_rows, 64, 128);
+  encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), p.dk, static_cast<uint64_t>(p.dk) * 2, box_rows, 64, 128);
+  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), p.dv, static_cast<uint64_t>(p.dv) * 2, box_rows, 64, 128);
   return launch_prefill_tc_maps<D, D, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
 }
 
@@ -596,6 +640,7 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
   p.window = a.window;
   p.causal = 1;
   p.status = a.status;
+  p.dk = a.dk;
   p.kv_row0 = a.kv_row0;
   p.kn_blocks = a.kn / 64;
   p.dv = a.dv;
@@ -623,13 +668,15 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
 // tensor memory beside the two score slots.
 int prefill_attention_tc_tile_rows(int D) { return D <= 128 ? 256 : 128; }
 
-// tile arrays: prefill_attention_tc_tile_rows(D) query rows per tile. page_size must be 32, 64 or 128. Returns 1 for an unsupported head_dim / page size.
+// tile arrays: prefill_attention_tc_tile_rows(max(dk, dv)) query rows per tile. page_size must be 32, 64 or 128. Returns 1 for an unsupported
+// head size (multiples of 8 up to 256) or page size.
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
-                                int num_tiles, void* out, int H, int KV, int D, int page, float scale, float cap, int window, int causal, int* status,
-                                cudaStream_t st) {
+                                int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
+                                AttnExtra x, int* status, cudaStream_t st) {
   if (num_tiles == 0) return 0;
-  if (page != 32 && page != 64 && page != 128) return 1;
+  const int D = dk > dv ? dk : dv;
+  if ((page != 32 && page != 64 && page != 128) || dk % 8 != 0 || dv % 8 != 0 || dk <= 0 || dv <= 0 || D > 256) return 1;
   AttnTcParams p = {};
   p.block_tables = bt;
   p.bt_stride = bt_stride;
@@ -646,14 +693,16 @@ int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, 
   p.softcap = cap;
   p.window = window;
   p.causal = causal;
+  p.keep_first = window > 0 ? x.keep_first : 0;
+  p.sink = x.sink;
+  p.dk = dk;
+  p.dv = dv;
+  p.out_pitch = H * dv;
   p.status = status;
   const long long cache_rows = num_pages * KV * page;
-  switch (D) {
-    case 64: return launch_prefill_tc_t<64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-    case 128: return launch_prefill_tc_t<128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-    case 256: return launch_prefill_tc_t<256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-    default: return 1;
-  }
+  if (D <= 64) return launch_prefill_tc_t<64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (D <= 128) return launch_prefill_tc_t<128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  return launch_prefill_tc_t<256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
 }
 
 }  // namespace dlv

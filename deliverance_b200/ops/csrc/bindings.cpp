@@ -720,7 +720,7 @@ int* split_arrival_counters(int device, int64_t needed) {
 }
 
 Tensor decode_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& ctx_lens,
-                        int64_t H, double scale, double softcap, int64_t window, int64_t splits, int64_t impl) {
+                        int64_t H, double scale, double softcap, int64_t window, int64_t splits, int64_t impl, int64_t keep_first, bool sink) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [B, H*D]");
   check_bf16(k_cache, "k_cache");
   check_bf16(v_cache, "v_cache");
@@ -729,19 +729,33 @@ Tensor decode_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt, "tables must be int32");
   const int B = static_cast<int>(q.size(0));
   const int KV = static_cast<int>(k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
+  const int DV = static_cast<int>(v_cache.size(3));
   TORCH_CHECK(q.size(1) == H * D && H % KV == 0 && page % 32 == 0, "shape mismatch (page size must be a multiple of 32)");
+  TORCH_CHECK(v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == KV && v_cache.size(2) == page, "k/v cache shape mismatch");
+  TORCH_CHECK(keep_first >= 0, "keep_first must not be negative");
   TORCH_CHECK(block_tables.dim() == 2 && block_tables.size(0) >= B && ctx_lens.numel() >= B, "bad table shapes");
   TORCH_CHECK((reinterpret_cast<uintptr_t>(q.data_ptr()) & 3) == 0, "q misaligned");
   c10::cuda::CUDAGuard guard(q.device());
-  Tensor out = new_out({B, H * D}, q.options());
+  Tensor out = new_out({B, H * DV}, q.options());
   if (splits < 1) splits = 1;
   Tensor po, pml;
   float *pop = nullptr, *pmlp = nullptr;
   if (splits > 1) {
-    po = new_out({B, H, splits, D}, q.options().dtype(at::kFloat));
+    po = new_out({B, H, splits, DV}, q.options().dtype(at::kFloat));
     pml = new_out({B, H, splits, 2}, q.options().dtype(at::kFloat));
     pop = po.data_ptr<float>();
     pmlp = pml.data_ptr<float>();
+  }
+  if (keep_first > 0 || sink || DV != D || (impl == 0 && (H / KV > 16 || (D != 64 && D != 128 && D != 256)))) {
+    TORCH_CHECK(impl == 0, "kept first keys, a sink and unequal widths are available in the tensor-core kernel only");
+    const dlv::AttnExtra x = {static_cast<int>(keep_first), sink ? 1 : 0};
+    const int rc = dlv::launch_decode_attention_mma(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr<int>(),
+                                                    static_cast<int>(block_tables.stride(0)), ctx_lens.data_ptr<int>(), out.data_ptr(), pop, pmlp, B,
+                                                    static_cast<int>(H), KV, D, DV, page, static_cast<float>(scale), static_cast<float>(softcap),
+                                                    static_cast<int>(window), x, static_cast<int>(splits), cur_stream());
+    TORCH_CHECK(rc == 0, "decode attention: head widths must be multiples of 8 up to 256");
+    check_last_error("decode_attention");
+    return out;
   }
   int* arrivals = (splits > 1 && g_decode_merge_in_kernel) ? split_arrival_counters(q.device().index(), static_cast<int64_t>(B) * KV) : nullptr;
   int rc = dlv::launch_decode_attention_impl(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr<int>(),
@@ -784,7 +798,7 @@ Tensor prefill_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v
 // Same contract as prefill_attention, on the tcgen05 / TMA kernel; tile arrays cover prefill_tc_tile_rows(head_dim) query rows per tile.
 Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& q_start,
                             const Tensor& q_len, const Tensor& ctx_lens, const Tensor& tile_seq, const Tensor& tile_q0, int64_t H, double scale,
-                            double softcap, int64_t window, bool causal) {
+                            double softcap, int64_t window, bool causal, int64_t keep_first, bool sink) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [T, H*D]");
   TORCH_CHECK(q.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0, "q rows must be 16-byte aligned");
   check_bf16(k_cache, "k_cache");
@@ -795,23 +809,29 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
   }
   const int T = static_cast<int>(q.size(0));
   const int KV = static_cast<int>(k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
-  TORCH_CHECK(k_cache.dim() == 4 && v_cache.sizes() == k_cache.sizes() && q.size(1) == H * D && H % KV == 0, "shape mismatch");
-  TORCH_CHECK((page == 32 || page == 64 || page == 128) && (D == 64 || D == 128 || D == 256), "page size 32 / 64 / 128 and head_dim 64 / 128 / 256");
+  const int DV = static_cast<int>(v_cache.size(3));
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == KV && v_cache.size(2) == page &&
+                  q.size(1) == H * D && H % KV == 0, "shape mismatch");
+  TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && D <= 256 && DV % 8 == 0 && DV <= 256,
+              "page size 32 / 64 / 128 and head widths that are multiples of 8 up to 256");
+  TORCH_CHECK(keep_first >= 0, "keep_first must not be negative");
   TORCH_CHECK(tile_seq.numel() == tile_q0.numel(), "tile arrays differ in length");
   c10::cuda::CUDAGuard guard(q.device());
-  Tensor out = new_out({T, H * D}, q.options());
+  Tensor out = new_out({T, H * DV}, q.options());
   DeviceScratch& s = scratch_for(q.device().index());
+  const dlv::AttnExtra x = {static_cast<int>(keep_first), sink ? 1 : 0};
   int rc = dlv::launch_prefill_attention_tc(q.data_ptr(), q.stride(0), T, k_cache.data_ptr(), v_cache.data_ptr(), k_cache.size(0), block_tables.data_ptr<int>(),
                                             static_cast<int>(block_tables.stride(0)), q_start.data_ptr<int>(), q_len.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                             tile_seq.data_ptr<int>(), tile_q0.data_ptr<int>(), static_cast<int>(tile_seq.numel()), out.data_ptr(),
-                                            static_cast<int>(H), KV, D, page, static_cast<float>(scale), static_cast<float>(softcap),
-                                            static_cast<int>(window), causal ? 1 : 0, s.status.data_ptr<int>(), cur_stream());
+                                            static_cast<int>(H), KV, D, DV, page, static_cast<float>(scale), static_cast<float>(softcap),
+                                            static_cast<int>(window), causal ? 1 : 0, x, s.status.data_ptr<int>(), cur_stream());
   TORCH_CHECK(rc == 0, "prefill attention (tcgen05): unsupported shape");
   check_last_error("prefill_attention_tc");
   return out;
 }
 
 #include "bindings_latent.inc"
+#include "bindings_gla.inc"
 
 // ---- sampling ---------------------------------------------------------------------------------------------------------
 std::vector<Tensor> argmax(const Tensor& logits, c10::optional<Tensor> mask, double softcap, double inv_scale) {
@@ -1127,9 +1147,10 @@ Tensor moe_items(const Tensor& offsets, int64_t e0, int64_t ne, int64_t bn, int6
 }
 // offsets / e0 / ne (optional): only rows of the local experts [e0, e0 + ne) are touched
 Tensor moe_gather(const Tensor& x, const Tensor& perm, int64_t k, c10::optional<Tensor> offsets, int64_t e0, int64_t ne) {
-  check_bf16(x, "x");
+  check_cuda(x, "x");
   check_cuda(perm, "perm");
-  TORCH_CHECK(perm.scalar_type() == at::kInt && x.dim() == 2 && x.size(1) % 8 == 0 && perm.numel() == x.size(0) * k, "bad gather arguments");
+  const int64_t row_bytes = x.dim() == 2 ? x.size(1) * x.element_size() : 1;
+  TORCH_CHECK(perm.scalar_type() == at::kInt && x.dim() == 2 && row_bytes % 16 == 0 && (reinterpret_cast<uintptr_t>(x.data_ptr()) & 15) == 0 && perm.numel() == x.size(0) * k, "bad gather arguments");
   c10::cuda::CUDAGuard guard(x.device());
   Tensor xs = new_out({perm.numel(), x.size(1)}, x.options());
   const int* off = nullptr;
@@ -1137,7 +1158,7 @@ Tensor moe_gather(const Tensor& x, const Tensor& perm, int64_t k, c10::optional<
     TORCH_CHECK(offsets.value().is_cuda() && offsets.value().scalar_type() == at::kInt && e0 + ne < offsets.value().numel(), "bad expert range");
     off = offsets.value().data_ptr<int>();
   }
-  dlv::launch_moe_gather(x.data_ptr(), perm.data_ptr<int>(), static_cast<int>(perm.numel()), static_cast<int>(k), static_cast<int>(x.size(1)), xs.data_ptr(), off, static_cast<int>(e0), static_cast<int>(ne), cur_stream());
+  dlv::launch_moe_gather(x.data_ptr(), perm.data_ptr<int>(), static_cast<int>(perm.numel()), static_cast<int>(k), static_cast<int>(row_bytes), xs.data_ptr(), off, static_cast<int>(e0), static_cast<int>(ne), cur_stream());
   check_last_error("moe_gather");
   return xs;
 }
@@ -1520,12 +1541,22 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("pos") = py::none(), py::arg("type_table") = py::none(), py::arg("types") = py::none());
   m.def("rope_kv", &rope_kv);
   m.def("decode_attention", &decode_attention, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("ctx_lens"),
-        py::arg("H"), py::arg("scale"), py::arg("softcap") = 0.0, py::arg("window") = 0, py::arg("splits") = 1, py::arg("impl") = 0);
+        py::arg("H"), py::arg("scale"), py::arg("softcap") = 0.0, py::arg("window") = 0, py::arg("splits") = 1, py::arg("impl") = 0,
+        py::arg("keep_first") = 0, py::arg("sink") = false);
   m.def("prefill_attention", &prefill_attention);
-  m.def("prefill_attention_tc", &prefill_attention_tc);
+  m.def("prefill_attention_tc", &prefill_attention_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("q_start"),
+        py::arg("q_len"), py::arg("ctx_lens"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"),
+        py::arg("causal"), py::arg("keep_first") = 0, py::arg("sink") = false);
+  m.def("attention_rows", &attention_rows);
+  m.def("rope_pairs_kv", &rope_pairs_kv);
+  m.def("sandwich_norm", &sandwich_norm);
+  m.def("grouped_linear_f32", &grouped_linear_f32);
+  m.def("gla_recurrent", &gla_recurrent);
+  m.def("gla_chunked", &gla_chunked);
   m.def("prefill_tc_tile_rows", &dlv::prefill_attention_tc_tile_rows);
   m.def("linear_f32", &linear_f32);
-  m.def("bigram_embedding", &bigram_embedding);
+  m.def("bigram_embedding", &bigram_embedding, py::arg("table"), py::arg("bigram"), py::arg("ids"), py::arg("prev"), py::arg("mul_prev"), py::arg("mul_cur"),
+        py::arg("scale"), py::arg("copy_into") = py::none());
   m.def("add_layernorm", &add_layernorm);
   m.def("gated_act", &gated_act);
   m.def("latent_prepare", &latent_prepare);

@@ -297,11 +297,12 @@ __device__ __forceinline__ void io_st(__nv_bfloat16* p, float v) { *p = f2bf(v);
 __device__ __forceinline__ void io_st(float* p, float v) { *p = v; }
 
 // out[t] = table[ids[t]] * scale + bigram[row]; row = (prev * mul_prev + id * mul_cur) mod buckets, or `buckets` (the extra last row) when the
-// token has no predecessor (prev < 0)
+// token has no predecessor (prev < 0); out2 (optional, pitch ld2): the same row in the table's type
 template <typename TIO>
 __global__ void __launch_bounds__(128) bigram_embedding_kernel(const TIO* __restrict__ table, const TIO* __restrict__ bigram, const int* __restrict__ ids,
                                                                const int* __restrict__ prev, float* __restrict__ out, int W, int vocab, int buckets,
-                                                               long long mul_prev, long long mul_cur, float scale) {
+                                                               long long mul_prev, long long mul_cur, float scale, TIO* __restrict__ out2,
+                                                               long long ld2) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
@@ -315,8 +316,11 @@ __global__ void __launch_bounds__(128) bigram_embedding_kernel(const TIO* __rest
     if (row < 0) row += buckets;
     bg = bigram + row * W;
   }
-  for (int i = threadIdx.x; i < W; i += blockDim.x)
-    out[static_cast<size_t>(t) * W + i] = io_ld(src + i) * scale + (bg != nullptr ? io_ld(bg + i) : 0.f);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = io_ld(src + i) * scale + (bg != nullptr ? io_ld(bg + i) : 0.f);
+    out[static_cast<size_t>(t) * W + i] = v;
+    if (out2 != nullptr) io_st(out2 + t * ld2 + i, v);
+  }
 }
 
 // residual += delta (when given; written back), then y1 = LayerNorm(residual; w1, b1) and, when w2 is given, y2 = LayerNorm(residual; w2, b2)
@@ -416,6 +420,216 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const TIO* __restrict__ 
   }
 }
 
+// ------------------------------------------------------------------------------------------------ sandwich norm
+// Norm behind a sublayer, scaled residual add and norm in front of the next sublayer in one pass over a row of the fp32 residual stream:
+//   residual += mult * LayerNorm(sub; w_sub)   (skipped without sub)
+//   y = LayerNorm(residual; w_next)            (the residual itself without w_next), columns W .. y_width zeroed
+// sub is one row [T, ld_sub] or, with pos, the weighted sum of k rows of an expert-ordered buffer: sum_j wts[t, j] * sub[pos[t, j]], formed
+// in fp32 in slot order. One CTA per row; the row lives in registers (NV groups of four columns per thread), both variances are means of
+// squared deviations.
+template <typename TIO>
+__device__ __forceinline__ void io_ld4(const TIO* p, float* v) {
+  if constexpr (sizeof(TIO) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf162(u.x), b = unpack_bf162(u.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  } else {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  }
+}
+template <typename TIO>
+__device__ __forceinline__ void io_st4(TIO* p, const float* v) {
+  if constexpr (sizeof(TIO) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf162(v[0], v[1]), pack_bf162(v[2], v[3]));
+  else *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+
+struct SandwichArgs {
+  float* residual;
+  const void* sub;
+  long long ld_sub;
+  const int* pos;
+  const float* wts;
+  int k;
+  const float* w_sub;
+  float mult;
+  const float* w_next;
+  void* y;
+  long long ld_y;
+  int W, y_width;
+  float eps;
+  int vec;  // rows, pitches and pointers allow four-column accesses
+};
+
+template <typename TSUB, typename TIO, int NV, int NT>
+__global__ void __launch_bounds__(NT) sandwich_norm_kernel(const SandwichArgs a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, W = a.W;
+  float* res = a.residual + static_cast<size_t>(t) * W;
+  TIO* y = static_cast<TIO*>(a.y) + t * a.ld_y;
+  const TSUB* sub = static_cast<const TSUB*>(a.sub);
+  float v[NV][4];
+  auto col = [&](int n) { return (n * NT + static_cast<int>(threadIdx.x)) * 4; };
+  pdl_wait();
+  pdl_trigger();
+  auto load = [&](auto* p, int c, float* o) {
+    if (a.vec) {
+      if (c < W) io_ld4(p + c, o);
+      else o[0] = o[1] = o[2] = o[3] = 0.f;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] = c + e < W ? io_ld(p + c + e) : 0.f;
+    }
+  };
+  auto deviation = [&](float mean) {  // sum of squared deviations of the real columns
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float d = v[n][e] - mean;
+        ss += col(n) + e < W ? d * d : 0.f;
+      }
+    return ss;
+  };
+  if (sub != nullptr) {
+    float r[NV][4];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) load(res, col(n), r[n]);
+    if (a.pos == nullptr) {
+#pragma unroll
+      for (int n = 0; n < NV; ++n) load(sub + t * a.ld_sub, col(n), v[n]);
+    } else {
+#pragma unroll
+      for (int n = 0; n < NV; ++n) v[n][0] = v[n][1] = v[n][2] = v[n][3] = 0.f;
+      for (int j = 0; j < a.k; ++j) {
+        const float wt = a.wts[static_cast<size_t>(t) * a.k + j];
+        const TSUB* row = sub + a.pos[static_cast<size_t>(t) * a.k + j] * a.ld_sub;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+          float o[4];
+          load(row, col(n), o);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[n][e] += wt * o[e];
+        }
+      }
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
+    const float mean = block_sum(s, red) / W;
+    const float inv = rsqrtf(block_sum(deviation(mean), red) / W + a.eps) * a.mult;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      float w[4];
+      load(a.w_sub, col(n), w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[n][e] = r[n][e] + (v[n][e] - mean) * inv * w[e];
+      if (a.vec) {
+        if (col(n) < W) io_st4(res + col(n), v[n]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (col(n) + e < W) res[col(n) + e] = v[n][e];
+          else v[n][e] = 0.f;
+        }
+      }
+      if (a.vec && col(n) >= W) v[n][0] = v[n][1] = v[n][2] = v[n][3] = 0.f;
+    }
+  } else {
+#pragma unroll
+    for (int n = 0; n < NV; ++n) load(res, col(n), v[n]);
+  }
+  float mean = 0.f, inv = 1.f;
+  if (a.w_next != nullptr) {
+    float s = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
+    mean = block_sum(s, red) / W;
+    inv = rsqrtf(block_sum(deviation(mean), red) / W + a.eps);
+  }
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    float o[4] = {v[n][0], v[n][1], v[n][2], v[n][3]};
+    if (a.w_next != nullptr) {
+      float w[4];
+      load(a.w_next, col(n), w);  // (zeros behind the row: so are the outputs there)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] = (v[n][e] - mean) * inv * w[e];
+    }
+    if (a.vec) {
+      if (col(n) < a.y_width) io_st4(y + col(n), o);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (col(n) + e < a.y_width) io_st(y + col(n) + e, o[e]);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ pair rotation + KV write
+// qkv rows [q (H * dk) | k (KV * dk) | v (KV * dv)], dk and dv multiples of 8. The first 2 * half columns of every query and key head are
+// rotated in neighbouring pairs (2 i, 2 i + 1); queries in place, keys on their way into the cache, values are copied. A thread takes
+// eight columns; query columns that are not rotated are not touched.
+template <typename TIO>
+__global__ void __launch_bounds__(256) rope_pairs_kv_kernel(TIO* __restrict__ qkv, long long ld, const int* __restrict__ positions,
+                                                            const long long* __restrict__ slots, const float* __restrict__ cos_t,
+                                                            const float* __restrict__ sin_t, TIO* __restrict__ k_cache, TIO* __restrict__ v_cache, int T, int H,
+                                                            int KV, int dk, int dv, int page, int half, int max_pos) {
+  pdl_wait();
+  pdl_trigger();
+  const int rot = (2 * half + 7) / 8, ck = dk / 8, cv = dv / 8;
+  const int nq = H * rot, nk = KV * ck, per = nq + nk + KV * cv;
+  const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= static_cast<long long>(T) * per) return;
+  const int t = static_cast<int>(idx / per);
+  int c = static_cast<int>(idx % per);
+  const TIO* src;
+  TIO* dst;
+  int d0 = 0;  // first column inside the head (rotated parts only)
+  bool rotate = false;
+  if (c < nq) {
+    d0 = (c % rot) * 8;
+    dst = qkv + t * ld + static_cast<long long>(c / rot) * dk + d0;
+    src = dst;
+    rotate = true;
+  } else {
+    const long long slot = slots[t];
+    if (slot < 0) return;
+    const long long blk = slot / page, off = slot % page;
+    c -= nq;
+    if (c < nk) {
+      d0 = (c % ck) * 8;
+      src = qkv + t * ld + static_cast<long long>(H) * dk + static_cast<long long>(c) * 8;
+      dst = k_cache + ((blk * KV + c / ck) * page + off) * dk + d0;
+      rotate = d0 < 2 * half;
+    } else {
+      c -= nk;
+      src = qkv + t * ld + static_cast<long long>(H + KV) * dk + static_cast<long long>(c) * 8;
+      dst = v_cache + ((blk * KV + c / cv) * page + off) * dv + (c % cv) * 8;
+    }
+  }
+  float x[8];
+  io_ld4(src, x);
+  io_ld4(src + 4, x + 4);
+  if (rotate) {
+    int pos = positions[t];
+    pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = d0 / 2 + e;
+      if (i < half) {
+        const float cs = cos_t[static_cast<size_t>(pos) * half + i], sn = sin_t[static_cast<size_t>(pos) * half + i];
+        const float u = x[2 * e], w = x[2 * e + 1];
+        x[2 * e] = u * cs - w * sn;
+        x[2 * e + 1] = w * cs + u * sn;
+      }
+    }
+  }
+  io_st4(dst, x);
+  io_st4(dst + 4, x + 4);
+}
+
 // ------------------------------------------------------------------------------------------------ launchers
 void launch_rmsnorm(const void* x, void* residual, const void* w, void* y, int T, int H, float eps, float offset,
                     float res_mult, cudaStream_t st) {
@@ -448,14 +662,15 @@ void launch_embedding(const void* table, const int* ids, const void* pos_table, 
                                       scale);
 }
 void launch_bigram_embedding(const void* table, const void* bigram, const int* ids, const int* prev, float* out, int rows, int W, int vocab, int buckets,
-                             long long mul_prev, long long mul_cur, float scale, bool is_f32, cudaStream_t st) {
+                             long long mul_prev, long long mul_cur, float scale, void* out2, long long ld2, bool is_f32, cudaStream_t st) {
   if (rows == 0) return;
   if (is_f32)
     launch_pdl(bigram_embedding_kernel<float>, dim3(rows), dim3(128), 0, st, static_cast<const float*>(table), static_cast<const float*>(bigram), ids, prev,
-               out, W, vocab, buckets, mul_prev, mul_cur, scale);
+               out, W, vocab, buckets, mul_prev, mul_cur, scale, static_cast<float*>(out2), ld2);
   else
     launch_pdl(bigram_embedding_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(table),
-               static_cast<const __nv_bfloat16*>(bigram), ids, prev, out, W, vocab, buckets, mul_prev, mul_cur, scale);
+               static_cast<const __nv_bfloat16*>(bigram), ids, prev, out, W, vocab, buckets, mul_prev, mul_cur, scale,
+               static_cast<__nv_bfloat16*>(out2), ld2);
 }
 void launch_add_layernorm(float* residual, const float* delta, const float* w1, const float* b1, void* y1, const float* w2, const float* b2, void* y2,
                           int rows, int W, int y_pitch, float eps, bool is_f32, cudaStream_t st) {
@@ -475,6 +690,36 @@ void launch_gated_act(const void* in, long long ld_in, void* out, long long ld_o
   else
     launch_pdl(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(in), ld_in, static_cast<__nv_bfloat16*>(out), ld_out, I,
                act, total);
+}
+template <typename TSUB, typename TIO>
+static void sandwich_dispatch(const SandwichArgs& a, int rows, cudaStream_t st) {
+  const int width = a.W > a.y_width ? a.W : a.y_width;
+  if (width <= 512) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 128>, dim3(rows), dim3(128), 0, st, a);
+  else if (width <= 1024) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 256>, dim3(rows), dim3(256), 0, st, a);
+  else if (width <= 2048) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 2, 256>, dim3(rows), dim3(256), 0, st, a);
+  else if (width <= 4096) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 256>, dim3(rows), dim3(256), 0, st, a);
+  else launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 1024>, dim3(rows), dim3(1024), 0, st, a);  // up to 16384 columns
+}
+void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bool sub_f32, const int* pos, const float* wts, int k, const float* w_sub,
+                          float mult, const float* w_next, void* y, long long ld_y, int rows, int W, int y_width, float eps, bool vec, bool is_f32,
+                          cudaStream_t st) {
+  if (rows == 0) return;
+  const SandwichArgs a = {residual, sub, ld_sub, pos, wts, k, w_sub, mult, w_next, y, ld_y, W, y_width, eps, vec ? 1 : 0};
+  if (is_f32) sandwich_dispatch<float, float>(a, rows, st);
+  else if (sub_f32) sandwich_dispatch<float, __nv_bfloat16>(a, rows, st);
+  else sandwich_dispatch<__nv_bfloat16, __nv_bfloat16>(a, rows, st);
+}
+void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const long long* slots, const float* cos_t, const float* sin_t, void* k_cache,
+                          void* v_cache, int T, int H, int KV, int dk, int dv, int page, int half, int max_pos, bool is_f32, cudaStream_t st) {
+  const long long n = static_cast<long long>(T) * (H * ((2 * half + 7) / 8) + KV * (dk / 8 + dv / 8));
+  if (n == 0) return;
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256));
+  if (is_f32)
+    launch_pdl(rope_pairs_kv_kernel<float>, grid, dim3(256), 0, st, static_cast<float*>(qkv), ld, positions, slots, cos_t, sin_t, static_cast<float*>(k_cache),
+               static_cast<float*>(v_cache), T, H, KV, dk, dv, page, half, max_pos);
+  else
+    launch_pdl(rope_pairs_kv_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<__nv_bfloat16*>(qkv), ld, positions, slots, cos_t, sin_t,
+               static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), T, H, KV, dk, dv, page, half, max_pos);
 }
 int launch_rope_kv(void* qkv, const int* positions, const long long* slots, const void* qn, const void* kn, const float* cos_t,
                    const float* sin_t, void* k_cache, void* v_cache, int T, int H, int KV, int D, int block_size, int rot_half,

@@ -124,6 +124,12 @@ int launch_rope_kv(void* qkv, const int* positions, const long long* slots, cons
                    const float* sin_t, void* k_cache, void* v_cache, int T, int H, int KV, int D, int block_size, int rot_half,
                    float eps, float norm_offset, int max_pos, cudaStream_t st);
 
+// Which keys of the sliding window's past stay visible, and whether a score of 0 without a value takes part in the softmax
+struct AttnExtra {
+  int keep_first = 0;
+  int sink = 0;
+};
+
 // attention.cu
 int launch_decode_attention(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                             const int* ctx, void* out, float* po, float* pml, int B, int H, int KV, int D, int page, float scale,
@@ -131,6 +137,14 @@ int launch_decode_attention(const void* q, long long q_stride, const void* kc, c
 int launch_decode_attention_impl(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                                  const int* ctx, void* out, float* po, float* pml, int* arrivals, int B, int H, int KV, int D, int page,
                                  float scale, float cap, int window, int splits, int impl, cudaStream_t st);
+// tensor-core decode kernel with separate key and value widths (multiples of 8, at most 256) and any group size; 1: unsupported shape
+int launch_decode_attention_mma(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* ctx, void* out,
+                                float* po, float* pml, int B, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
+                                int splits, cudaStream_t st);
+// one CTA per (row, query head) on CUDA cores, fp32 or bf16, any width; row_seq: sequence of every row (nullptr: row number)
+int launch_attention_rows(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* row_seq,
+                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
+                          bool is_f32, cudaStream_t st);
 int launch_prefill_attention(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                              const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                              int num_tiles, void* out, int H, int KV, int D, int page, float scale, float cap, int window,
@@ -155,8 +169,8 @@ void gemv_dense_run(const GemmWeightDesc* w, const void* x, int M, int ldx, void
 extern bool g_gemv_simt_only;  // gemm.cu: grouped JQ4 GEMV on CUDA cores instead of mma.sync (comparisons)
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
-                                int num_tiles, void* out, int H, int KV, int D, int page, float scale, float cap, int window, int causal, int* status,
-                                cudaStream_t st);
+                                int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
+                                AttnExtra x, int* status, cudaStream_t st);
 
 // sampling.cu
 void launch_argmax(const float* logits, int ld, int B, int V, const uint32_t* mask, int mask_ld, float softcap, float inv_scale,
@@ -179,7 +193,7 @@ void launch_moe_route(const float* logits, int T, int E, int k, int mode, int re
                       int* perm, int* pos, int* ws, cudaStream_t st);
 // `range` (optional) = offsets + first local expert and the count of local experts: rows outside
 // [offsets[e0], offsets[e0 + ne]) are skipped (expert parallelism: other ranks own them)
-void launch_moe_gather(const void* x, const int* perm, int rows, int k, int H, void* xs, const int* offsets, int e0, int ne,
+void launch_moe_gather(const void* x, const int* perm, int rows, int k, int row_bytes, void* xs, const int* offsets, int e0, int ne,
                        cudaStream_t st);
 void launch_moe_combine(const void* ys, const int* pos, const float* w, int T, int k, int H, void* out, const int* offsets, int e0,
                         int ne, cudaStream_t st);
@@ -270,6 +284,8 @@ int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, con
                            const float* wuv, const float* c_cache, const float* r_cache, const int* bt, int bt_stride, float* out, int out_pitch,
                            const LatentGeom& g, int page, float scale, int window, cudaStream_t st);
 void launch_linear_f32(const float* x, int ldx, const float* w, const float* bias, float* out, int ldo, int M, int N, int K, cudaStream_t st);
+// w stacks experts [N, K]; items: work list of launch_moe_items with 64 rows per item
+void launch_grouped_linear_f32(const float* x, int ldx, const float* w, float* out, int ldo, const int* items, int n_items, int N, int K, cudaStream_t st);
 
 // attention_tc.cu, latent layout: q [T, H * dk] (pitch q_pitch), k [kv_rows, H * kn] and v [kv_rows, H * DV] with one pitch, kr [kv_rows, dk - kn]
 struct LatentTcArgs {
@@ -293,9 +309,39 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st);
 
 // elementwise.cu, fp32 residual stream
 void launch_bigram_embedding(const void* table, const void* bigram, const int* ids, const int* prev, float* out, int rows, int W, int vocab, int buckets,
-                             long long mul_prev, long long mul_cur, float scale, bool is_f32, cudaStream_t st);
+                             long long mul_prev, long long mul_cur, float scale, void* out2, long long ld2, bool is_f32, cudaStream_t st);
 void launch_add_layernorm(float* residual, const float* delta, const float* w1, const float* b1, void* y1, const float* w2, const float* b2, void* y2,
                           int rows, int W, int y_pitch, float eps, bool is_f32, cudaStream_t st);
+void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bool sub_f32, const int* pos, const float* wts, int k, const float* w_sub,
+                          float mult, const float* w_next, void* y, long long ld_y, int rows, int W, int y_width, float eps, bool vec, bool is_f32,
+                          cudaStream_t st);
+void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const long long* slots, const float* cos_t, const float* sin_t, void* k_cache,
+                          void* v_cache, int T, int H, int KV, int dk, int dv, int page, int half, int max_pos, bool is_f32, cudaStream_t st);
+
+// gla.cu: gated linear attention. Projection rows p [T, ld] = q (H dk) | k (H dk) | v (H dv) | g (H dv) | a (rank), widths multiples of 8
+struct GlaArgs {
+  const void* p;
+  long long ld;
+  int H, dk, dv, dv_real, rank, off_k, off_v, off_g, off_a;
+  const float *a2, *a2_bias, *norm_w;  // [H dk, rank], [H dk], [dv]
+  float* state;                        // [slots, H, dk, dv]
+  const long long* slots;              // per sequence
+  const int *q_start, *q_len, *positions;
+  int num_seqs, rows;
+  float q_scale, inv_tau, eps;
+  float* o;   // fp32 [T, H dv] (unused by the fused decode step)
+  void* out;  // [T, H dv]
+};
+struct GlaChunks {
+  const int *seq, *row0, *len;    // per chunk
+  const int *first, *count;       // per sequence
+  int n_chunks, chunk;
+  void* qk;      // bf16 [T, H, 4, dk]: scaled queries (high, low part), scaled keys (high, low part)
+  void* a;       // bf16 [n_chunks, H, 2, chunk, chunk]
+  float* decay;  // [n_chunks, H, dk]
+};
+int launch_gla_recurrent(const GlaArgs& a, bool fused, bool is_f32, cudaStream_t st);
+int launch_gla_chunked(const GlaArgs& a, const GlaChunks& c, cudaStream_t st);
 void launch_gated_act(const void* in, long long ld_in, void* out, long long ld_out, int rows, int I, int act, bool is_f32, cudaStream_t st);
 
 // aux.cu

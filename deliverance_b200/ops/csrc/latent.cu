@@ -876,11 +876,19 @@ int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, con
 // ------------------------------------------------------------------------------------------------ fp32 projection
 // out = x W^T (+ bias), true fp32 FMA. 64 x 64 tiles, 256 threads with 4 x 4 accumulators, K in steps of 16.
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias,
-                                                         float* __restrict__ out, int ldo, int M, int N, int K) {
+                                                         float* __restrict__ out, int ldo, int M, int N, int K, const int4* __restrict__ items) {
   pdl_wait();
   pdl_trigger();
   __shared__ float sx[16][68], sw[16][68];
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  int m0 = blockIdx.y * 64;
+  if (items != nullptr) {  // grouped: (expert, first row, end row) per 64-row item, w stacks the experts
+    const int4 it = items[blockIdx.y];
+    if (it.x < 0) return;
+    w += static_cast<size_t>(it.x) * N * K;
+    m0 = it.y;
+    M = min(it.z, it.y + 64);
+  }
+  const int n0 = blockIdx.x * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
     for (int e = tid; e < 64 * 16; e += 256) {
@@ -916,7 +924,12 @@ void launch_linear_f32(const float* x, int ldx, const float* w, const float* bia
   if (M == 0 || N == 0) return;
   const unsigned gy = static_cast<unsigned>((M + 63) / 64);
   if (gy > 65535) throw std::runtime_error("fp32 projection: too many rows");
-  launch_pdl(linear_f32_kernel, dim3((N + 63) / 64, gy), dim3(256), 0, st, x, ldx, w, bias, out, ldo, M, N, K);
+  launch_pdl(linear_f32_kernel, dim3((N + 63) / 64, gy), dim3(256), 0, st, x, ldx, w, bias, out, ldo, M, N, K, static_cast<const int4*>(nullptr));
+}
+void launch_grouped_linear_f32(const float* x, int ldx, const float* w, float* out, int ldo, const int* items, int n_items, int N, int K, cudaStream_t st) {
+  if (n_items == 0 || N == 0) return;
+  launch_pdl(linear_f32_kernel, dim3((N + 63) / 64, static_cast<unsigned>(n_items)), dim3(256), 0, st, x, ldx, w, static_cast<const float*>(nullptr), out, ldo, 0,
+             N, K, reinterpret_cast<const int4*>(items));
 }
 
 }  // namespace dlv

@@ -2,7 +2,7 @@
 //   moe_route:   router logits [T, E] fp32 -> top-k weights / expert ids per token (softmax-all -> top-k -> optional
 //                renormalise, or top-k -> softmax over the k), per-expert histogram, exclusive offsets and the permutation
 //                that groups (token, slot) pairs by expert — one kernel launch + one small scan kernel.
-//   moe_gather:  x [T, H] -> xs [T*k, H] rows in expert-grouped order.
+//   moe_gather:  x [T, H] -> xs [T*k, H] rows in expert-grouped order (any element type).
 //   moe_combine: ys [T*k, H] (expert outputs in grouped order) -> out [T, H] = sum_j w[t, j] * ys[pos(t, j)]  (fp32 sum in
 //                slot order: deterministic, no atomics).
 // Reference semantics: core/.../model/MixtureOfExpertsBlock.java:78-112, qwen3/Qwen3MoeFeedForward.java:107-301,
@@ -285,16 +285,16 @@ __global__ void __launch_bounds__(32) moe_chunk_rank_kernel(const int* __restric
   }
 }
 
-__global__ void __launch_bounds__(128) moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ perm, int k, int H,
-                                                         __nv_bfloat16* __restrict__ xs, const int* __restrict__ offsets, int e0, int ne) {
+__global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict__ x, const int* __restrict__ perm, int k, int row_vecs,
+                                                         uint4* __restrict__ xs, const int* __restrict__ offsets, int e0, int ne) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   const int row = blockIdx.x;
   if (offsets != nullptr && (row < offsets[e0] || row >= offsets[e0 + ne])) return;  // another rank's expert
   const int t = perm[row] / k;
-  const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<size_t>(t) * H);
-  uint4* dst = reinterpret_cast<uint4*>(xs + static_cast<size_t>(row) * H);
-  for (int i = threadIdx.x; i < H / 8; i += blockDim.x) dst[i] = src[i];
+  const uint4* src = x + static_cast<size_t>(t) * row_vecs;
+  uint4* dst = xs + static_cast<size_t>(row) * row_vecs;
+  for (int i = threadIdx.x; i < row_vecs; i += blockDim.x) dst[i] = src[i];
 }
 
 __global__ void __launch_bounds__(128) moe_combine_kernel(const __nv_bfloat16* __restrict__ ys, const int* __restrict__ pos,
@@ -360,10 +360,10 @@ bool launch_moe_route_small(const float* logits, int T, int E, int k, int mode, 
   return launch_pdl(moe_route_small_kernel, dim3(1), dim3(1024), smem, st, logits, T, E, k, mode, renorm, w, idx, counts, offsets, perm, pos, e0,
                     ne, bn, max_items, reinterpret_cast<int4*>(items)) == cudaSuccess;
 }
-void launch_moe_gather(const void* x, const int* perm, int rows, int k, int H, void* xs, const int* offsets, int e0, int ne,
+void launch_moe_gather(const void* x, const int* perm, int rows, int k, int row_bytes, void* xs, const int* offsets, int e0, int ne,
                        cudaStream_t st) {
   if (rows == 0) return;
-  moe_gather_kernel<<<rows, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(x), perm, k, H, static_cast<__nv_bfloat16*>(xs), offsets, e0, ne);
+  moe_gather_kernel<<<rows, 128, 0, st>>>(static_cast<const uint4*>(x), perm, k, row_bytes / 16, static_cast<uint4*>(xs), offsets, e0, ne);
 }
 void launch_moe_combine(const void* ys, const int* pos, const float* w, int T, int k, int H, void* out, const int* offsets, int e0,
                         int ne, cudaStream_t st) {

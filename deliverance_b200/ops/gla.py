@@ -23,6 +23,7 @@ from .grouped import up8
 
 MAX_DK = 512  # key channels per head the CUDA kernels take
 MAX_DK_CHUNKED = 256
+MAX_DV_FUSED = 512  # one cluster of eight CTAs per head norms and gates inside the decode launch
 
 
 @dataclass(frozen=True)
@@ -78,8 +79,9 @@ def gla(s: GlaShape, p, a2, a2_bias, norm_w, state, batch, q_scale: float, tau: 
         e = ops.require_ext()
         args = (a2, a2_bias, norm_w, state, batch.state_slots, batch.q_start, batch.q_len, batch.positions, s.geometry(), q_scale, 1.0 / tau, eps)
         if batch.is_decode or p.dtype == torch.float32 or s.dk > MAX_DK_CHUNKED:
-            ops._count(e.gla_recurrent_launches(s.dv, p.dtype == torch.float32, batch.is_decode))
-            return e.gla_recurrent(p, *args, batch.is_decode)
+            fused = batch.is_decode and s.dv <= MAX_DV_FUSED
+            ops._count(1 if fused else 2)
+            return e.gla_recurrent(p, *args, fused)
         ops._count(3)
         return e.gla_chunked(p, *args, s.chunk, *chunk_plan(batch, s.chunk))
     k0, v0, g0, a0, w = s.offsets
