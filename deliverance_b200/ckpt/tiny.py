@@ -76,7 +76,86 @@ def _fatotar_tensors(cfg: dict, seed: int, dtype) -> dict:
     return t
 
 
+def fopivik_config(width: int, vocab: int, layers: list, loop: Optional[dict] = None, eps: float = 1e-5, residual_mult: float = 0.5,
+                   logit_softcap: float = 12.0, **extra) -> dict:
+    """``config.json`` of a Fopivik model. ``layers``: one dict of sizes per layer; softmax attention has ``heads, kv_heads, dim, vdim, window,
+    keep_first`` (and ``rot_dims, base, scaling, softcap, scale``), gated linear attention ``heads, dim, vdim, tau`` (``rank`` columns of the
+    decay projection); ``experts, top, ff`` for the routed experts (``experts`` 0 = no feed-forward)."""
+    out, ranks = [], {}
+    for i, L in enumerate(layers):
+        mlp = {"kind": "moe", "expert": {"ff": L["ff"]}, "router": {"experts": L["experts"], "top": L["top"]}} if L.get("experts") else None
+        if "tau" in L:
+            mixer = {k: L[k] for k in ("heads", "dim", "vdim", "tau")}
+            ranks[i] = L.get("rank", 8)
+            out.append({"type": "gla", "mixer": mixer, "mlp": mlp})
+            continue
+        rot = {"base": L.get("base", 10000.0), "dims": L.get("rot_dims", L["dim"])}
+        if L.get("scaling"):
+            rot["scaling"] = L["scaling"]
+        mixer = {k: L[k] for k in ("heads", "kv_heads", "dim", "vdim")}
+        mixer.update(mask={"size": L["window"], "keep_first": L.get("keep_first", 0)}, rot=rot, scale=L.get("scale", L["dim"] ** -0.5),
+                     softcap=L.get("softcap", 30.0))
+        out.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+    cfg = {"architecture": "Fopivik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": residual_mult,
+           "logit_softcap": logit_softcap, "layers": out}
+    if loop:
+        cfg["loop"] = loop
+    cfg.update(extra)
+    cfg["_decay_ranks"] = ranks  # (shapes of random checkpoints only; a model reads the rank off its tensors)
+    return cfg
+
+
+def fopivik_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape of a Fopivik checkpoint."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    if cfg.get("loop"):
+        s.update({"loop.in": (W, 2 * W), "loop.step": (cfg["loop"]["times"], W)})
+    ranks = {int(k): v for k, v in (cfg.get("_decay_ranks") or {}).items()}
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        G = m.get("kv_heads", H)
+        s.update({p + "norm1": (W,), p + "norm1b": (W,), p + "mix.q": (H * dk, W), p + "mix.k": (G * dk, W), p + "mix.v": (G * dv, W), p + "mix.o": (W, H * dv)})
+        if L["type"] == "gla":
+            R = ranks.get(i, 8)
+            s.update({p + "mix.g": (H * dv, W), p + "mix.norm": (dv,), p + "mix.a1": (R, W), p + "mix.a2": (H * dk, R), p + "mix.a2.b": (H * dk,)})
+        if L.get("mlp"):
+            F, E = L["mlp"]["expert"]["ff"], L["mlp"]["router"]["experts"]
+            s.update({p + "norm2": (W,), p + "norm2b": (W,), p + "mlp.router": (E, W)})
+            for e in range(E):
+                s.update({f"{p}mlp.e{e}.gate": (F, W), f"{p}mlp.e{e}.up": (F, W), f"{p}mlp.e{e}.down": (W, F)})
+    return s
+
+
+def fopivik_is_norm(name: str) -> bool:
+    return name.rsplit(".", 1)[-1].startswith("norm")
+
+
+def _fopivik_tensors(cfg: dict, seed: int, dtype) -> dict:
+    """Random weights with projections scaled by their fan-in, wide router logits and decays spread over fast and slow channels."""
+    g = torch.Generator().manual_seed(seed)
+    t = {}
+    for name, shape in fopivik_shapes(cfg).items():
+        r = torch.randn(*shape, generator=g, dtype=torch.float32)
+        if fopivik_is_norm(name):
+            r = 1.0 + 0.2 * r
+        elif name.endswith(".a2.b"):
+            r = 2.0 * r + 1.0
+        elif len(shape) == 2 and name not in ("embed", "loop.step"):
+            r = r * shape[1] ** -0.5 * (2.0 if name.endswith("router") else 1.0)
+        t[name] = r.to(dtype)
+    return t
+
+
 def tiny_config(model_type: str, **over) -> dict:
+    if model_type == "fopivik":
+        soft = dict(heads=6, kv_heads=2, dim=20, vdim=28, rot_dims=12, window=24, keep_first=5, experts=5, top=2, ff=36)
+        lin = dict(heads=3, dim=12, vdim=20, tau=4.0, experts=4, top=1, ff=24)
+        kw = dict(width=76, vocab=261, layers=[dict(lin), dict(soft, scaling={"factor": 4.0, "low": 1.0, "high": 4.0, "original": 64}), dict(lin, vdim=8, experts=0)],
+                  loop={"start": 0, "stop": 2, "times": 2})
+        kw.update(over)
+        return fopivik_config(**kw)
     if model_type == "fatotar":
         size = dict(heads=3, dim=20, rot_dim=6, vdim=12, kv_rank=40, window=24, ff=52)
         yarn = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 2.0}
@@ -128,6 +207,8 @@ def build_tensors(cfg: dict, seed: int = 0, dtype=torch.float32, std: float = 0.
     mt = config_model_type(cfg)
     if mt == "fatotar":
         return _fatotar_tensors(cfg, seed, dtype)
+    if mt == "fopivik":
+        return _fopivik_tensors(cfg, seed, dtype)
     R = lambda *s: _rand(g, *s, std=std, dtype=dtype)  # noqa: E731
     ones = lambda n: (torch.ones(n) + torch.randn(n, generator=g) * 0.05).to(dtype)  # noqa: E731
     t: dict = {}

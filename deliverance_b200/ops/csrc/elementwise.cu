@@ -705,7 +705,8 @@ void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bo
                           cudaStream_t st) {
   if (rows == 0) return;
   const SandwichArgs a = {residual, sub, ld_sub, pos, wts, k, w_sub, mult, w_next, y, ld_y, W, y_width, eps, vec ? 1 : 0};
-  if (is_f32) sandwich_dispatch<float, float>(a, rows, st);
+  if (is_f32 && sub_f32) sandwich_dispatch<float, float>(a, rows, st);
+  else if (is_f32) sandwich_dispatch<__nv_bfloat16, float>(a, rows, st);
   else if (sub_f32) sandwich_dispatch<float, __nv_bfloat16>(a, rows, st);
   else sandwich_dispatch<__nv_bfloat16, __nv_bfloat16>(a, rows, st);
 }
