@@ -155,13 +155,16 @@ def main() -> int:
     ap.add_argument("--parallelism", default="auto", choices=["auto", "dp", "tp"],
                     help="N > 1: tp (default) = one engine over N GPUs (tensor parallel, --batch sequences in total, strong scaling); "
                          "dp = one engine replica per GPU, --batch sequences each (weak scaling, no communication)")
-    ap.add_argument("--design", default=None, choices=["fatotar"],
-                    help="instead of the headline workload: prefill / decode throughput and kernel times of this design beside a GQA decoder of equal size (1 GPU)")
+    ap.add_argument("--design", default=None, choices=["fatotar", "fopivik"],
+                    help="instead of the headline workload: prefill / decode throughput and kernel times of this design beside the closest decoder of equal size (1 GPU)")
     ap.add_argument("--sizes", default="small,1b,3b", help="--design: sizes to run")
     ap.add_argument("--no-kernels", action="store_true", help="--design: throughput only")
     args = ap.parse_args()
     if args.design:
-        from deliverance_b200.bench.design_bench import main as design_main
+        if args.design == "fopivik":
+            from deliverance_b200.bench.fopivik_bench import main as design_main
+        else:
+            from deliverance_b200.bench.design_bench import main as design_main
 
         args.warmup, args.steps = max(3, args.warmup), min(args.steps, 128)
         return design_main(args)
