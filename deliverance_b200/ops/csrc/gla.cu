@@ -11,7 +11,8 @@
 //                         q exp(b) and k exp(-b) unless a channel's decay over the chunk would leave the fp32 range (then term by term).
 //   gla_chunks_kernel     one CTA per (64 value columns, head, sequence) walks the chunks: O^T = S^T Q^T + V^T A^T, then
 //                         S^T = S^T diag(exp(b_end)) + V^T K. S^T is the accumulator of the second product and, converted in registers,
-//                         the left operand of the first; chunk tiles arrive by cp.async in two stages.
+//                         the left operand of the first; eight warps = 4 x 16 value columns x 2 halves of the key channels, whose shares
+//                         of O meet in shared memory; chunk tiles arrive by cp.async in two stages.
 //   gla_norm_gate_kernel  norm and gate of prompt rows.
 #include <cooperative_groups.h>
 
@@ -398,17 +399,21 @@ struct GlaStage {
   static constexpr int kA = kV + C * PV * 2;
   static constexpr int kDec = kA + 2 * C * PA * 2;
   static constexpr int kBytes = (kDec + NK * 16 * 4 + 127) / 128 * 128;
-  static_assert(2 * kBytes <= 227 * 1024, "two stages must fit shared memory");
+  static constexpr int PO = kGlaCols + 4;
+  static constexpr int kTotal = 2 * kBytes + 2 * C * PO * 4;  // two stages, both halves' shares of the outputs
+  static_assert(NK % 2 == 0 && kTotal <= 227 * 1024, "two stages must fit shared memory");
 };
 
 template <int C, int NK>
-__global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const GlaChunks c) {
+__global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const GlaArgs a, const GlaChunks c) {
   pdl_wait();
   pdl_trigger();
   using L = GlaStage<C, NK>;
+  constexpr int NH = NK / 2;  // 16-channel tiles per warp
   extern __shared__ __align__(128) uint8_t gsm[];
   const int h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int g = lane >> 2, t4 = lane & 3;
+  const int g = lane >> 2, t4 = lane & 3, wd = warp & 3, hk = warp >> 2;  // 16 value columns, half of the key channels
+  float* so = reinterpret_cast<float*>(gsm + 2 * L::kBytes);
   const int c0 = blockIdx.x * kGlaCols, n_chunks = c.count[s], first = c.first[s];
   if (n_chunks == 0) return;
   const int dk = a.dk, dv = a.dv;
@@ -422,35 +427,35 @@ __global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const 
     const int ck = first + i, row0 = c.row0[ck], len = c.len[ck];
     const uint32_t base = smem_u32(gsm + stage * L::kBytes);
     constexpr int CH = NK * 2;  // 16-byte chunks per row and plane
-    for (int e = tid; e < 4 * C * CH; e += 128) {
+    for (int e = tid; e < 4 * C * CH; e += 256) {
       const int x = e % CH, t = (e / CH) % C, plane = e / (CH * C);
       const bool ok = t < len && x * 8 < dk;
       const __nv_bfloat16* src = qk + ((static_cast<size_t>(row0 + (ok ? t : 0)) * a.H + h) * 4 + plane) * dk + (ok ? x * 8 : 0);
       cp16(base + ((plane * C + t) * L::P + x * 8) * 2, src, ok);
     }
-    for (int e = tid; e < C * 8; e += 128) {
+    for (int e = tid; e < C * 8; e += 256) {
       const int t = e >> 3, x = (e & 7) * 8;
       const bool ok = t < len && c0 + x < dv;
       cp16(base + L::kV + (t * L::PV + x) * 2, p + static_cast<size_t>(row0 + (ok ? t : 0)) * a.ld + a.off_v + h * dv + (ok ? c0 + x : 0), ok);
     }
     const __nv_bfloat16* ap = am + (static_cast<size_t>(ck) * a.H + h) * 2 * C * C;
-    for (int e = tid; e < 2 * C * (C / 8); e += 128) {
+    for (int e = tid; e < 2 * C * (C / 8); e += 256) {
       const int r = e / (C / 8), x = (e % (C / 8)) * 8;
       cp16(base + L::kA + (r * L::PA + x) * 2, ap + r * C + x, true);
     }
-    for (int e = tid; e < NK * 4; e += 128) cp16(base + L::kDec + e * 16, c.decay + (static_cast<size_t>(ck) * a.H + h) * dk + (e * 4 < dk ? e * 4 : 0), e * 4 < dk);
+    for (int e = tid; e < NK * 4; e += 256) cp16(base + L::kDec + e * 16, c.decay + (static_cast<size_t>(ck) * a.H + h) * dk + (e * 4 < dk ? e * 4 : 0), e * 4 < dk);
     cp_commit();
   };
 
   load(0, 0);
   // S^T: rows = value columns (16 per warp), columns = key channels
-  float st[2 * NK][4];
-  const int vr = c0 + warp * 16 + g;
+  float st[2 * NH][4];
+  const int vr = c0 + wd * 16 + g, d_at = hk * NH * 16 + 2 * t4;
 #pragma unroll
-  for (int j = 0; j < 2 * NK; ++j)
+  for (int j = 0; j < 2 * NH; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = j * 8 + 2 * t4 + (e & 1), col = vr + (e >> 1) * 8;
+      const int d = d_at + j * 8 + (e & 1), col = vr + (e >> 1) * 8;
       st[j][e] = (!fresh && d < dk && col < dv) ? state[static_cast<size_t>(d) * dv + col] : 0.f;
     }
   for (int i = 0; i < n_chunks; ++i) {
@@ -467,9 +472,9 @@ __global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const 
 #pragma unroll
     for (int j = 0; j < C / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     // O^T = S^T Q^T
-    const uint32_t q_at = base + (((lane & 7) + (lane >> 4) * 8) * L::P + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t q_at = base + (((lane & 7) + (lane >> 4) * 8) * L::P + hk * NH * 16 + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
-    for (int kt = 0; kt < NK; ++kt) {
+    for (int kt = 0; kt < NH; ++kt) {
       uint32_t sh[4], sl[4];
       split2(st[2 * kt][0], st[2 * kt][1], sh[0], sl[0]);
       split2(st[2 * kt][2], st[2 * kt][3], sh[1], sl[1]);
@@ -488,11 +493,12 @@ __global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const 
         mma16816(o[2 * np + 1], sh, b[2], b[3]);
       }
     }
-    // O^T += V^T A^T
+    // O^T += V^T A^T (the halves take every other block of tokens)
     uint32_t vf[C / 16][4];
 #pragma unroll
     for (int ks = 0; ks < C / 16; ++ks) {
-      ldm_x4_t(base + L::kV + ((ks * 16 + (lane & 7) + (lane >> 4) * 8) * L::PV + warp * 16 + ((lane >> 3) & 1) * 8) * 2, vf[ks]);
+      ldm_x4_t(base + L::kV + ((ks * 16 + (lane & 7) + (lane >> 4) * 8) * L::PV + wd * 16 + ((lane >> 3) & 1) * 8) * 2, vf[ks]);
+      if ((ks & 1) != hk) continue;
 #pragma unroll
       for (int np = ks; np < C / 16; ++np) {
         const uint32_t at = base + L::kA + ((np * 16 + (lane & 7) + (lane >> 4) * 8) * L::PA + ks * 16 + ((lane >> 3) & 1) * 8) * 2;
@@ -505,28 +511,24 @@ __global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const 
         mma16816(o[2 * np + 1], vf[ks], b[2], b[3]);
       }
     }
-    const int row0 = c.row0[first + i], len = c.len[first + i];
 #pragma unroll
     for (int j = 0; j < C / 8; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = j * 8 + 2 * t4 + (e & 1), col = vr + (e >> 1) * 8;
-        if (t < len && col < dv) a.o[static_cast<size_t>(row0 + t) * (a.H * dv) + h * dv + col] = o[j][e];
-      }
+      for (int e = 0; e < 4; ++e) so[(hk * C + j * 8 + 2 * t4 + (e & 1)) * L::PO + wd * 16 + g + (e >> 1) * 8] = o[j][e];
     // S^T = S^T diag(decay) + V^T K
 #pragma unroll
-    for (int j = 0; j < 2 * NK; ++j) {
-      const float2 e = *reinterpret_cast<const float2*>(dec + j * 8 + 2 * t4);
+    for (int j = 0; j < 2 * NH; ++j) {
+      const float2 e = *reinterpret_cast<const float2*>(dec + d_at + j * 8);
       st[j][0] *= e.x;
       st[j][1] *= e.y;
       st[j][2] *= e.x;
       st[j][3] *= e.y;
     }
-    const uint32_t k_at = base + ((2 * C + (lane & 7) + ((lane >> 3) & 1) * 8) * L::P + (lane >> 4) * 8) * 2;
+    const uint32_t k_at = base + ((2 * C + (lane & 7) + ((lane >> 3) & 1) * 8) * L::P + hk * NH * 16 + (lane >> 4) * 8) * 2;
 #pragma unroll
     for (int ks = 0; ks < C / 16; ++ks)
 #pragma unroll
-      for (int jp = 0; jp < NK; ++jp) {
+      for (int jp = 0; jp < NH; ++jp) {
         uint32_t b[4];
         ldm_x4_t(k_at + (ks * 16 * L::P + jp * 16) * 2, b);
         mma16816(st[2 * jp], vf[ks], b[0], b[1]);
@@ -535,13 +537,20 @@ __global__ void __launch_bounds__(128) gla_chunks_kernel(const GlaArgs a, const 
         mma16816(st[2 * jp], vf[ks], b[0], b[1]);
         mma16816(st[2 * jp + 1], vf[ks], b[2], b[3]);
       }
-    __syncthreads();  // the stage is refilled by the next iteration's load
+    __syncthreads();  // the stage is refilled by the next iteration's load; both shares of the outputs are complete
+    const int row0 = c.row0[first + i], len = c.len[first + i];
+    for (int e = tid; e < C * (kGlaCols / 4); e += 256) {
+      const int t = e / (kGlaCols / 4), x = (e % (kGlaCols / 4)) * 4;
+      if (t >= len || c0 + x >= dv) continue;
+      const float4 u = *reinterpret_cast<const float4*>(so + t * L::PO + x), w = *reinterpret_cast<const float4*>(so + (C + t) * L::PO + x);
+      *reinterpret_cast<float4*>(a.o + static_cast<size_t>(row0 + t) * (a.H * dv) + h * dv + c0 + x) = make_float4(u.x + w.x, u.y + w.y, u.z + w.z, u.w + w.w);
+    }
   }
 #pragma unroll
-  for (int j = 0; j < 2 * NK; ++j)
+  for (int j = 0; j < 2 * NH; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = j * 8 + 2 * t4 + (e & 1), col = vr + (e >> 1) * 8;
+      const int d = d_at + j * 8 + (e & 1), col = vr + (e >> 1) * 8;
       if (d < dk && col < dv) state[static_cast<size_t>(d) * dv + col] = st[j][e];
     }
 }
@@ -551,10 +560,10 @@ static cudaError_t launch_chunks_t(const GlaArgs& a, const GlaChunks& c, cudaStr
   using L = GlaStage<C, NK>;
   static PerDeviceOnce once;
   if (once.first()) {
-    const cudaError_t e = cudaFuncSetAttribute(gla_chunks_kernel<C, NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * L::kBytes);
+    const cudaError_t e = cudaFuncSetAttribute(gla_chunks_kernel<C, NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal);
     if (e != cudaSuccess) return e;
   }
-  return launch_pdl(gla_chunks_kernel<C, NK>, dim3((a.dv + kGlaCols - 1) / kGlaCols, a.H, a.num_seqs), dim3(128), 2 * L::kBytes, st, a, c);
+  return launch_pdl(gla_chunks_kernel<C, NK>, dim3((a.dv + kGlaCols - 1) / kGlaCols, a.H, a.num_seqs), dim3(256), L::kTotal, st, a, c);
 }
 
 template <int C>
