@@ -240,7 +240,27 @@ int launch_gla_recurrent(const GlaArgs& a, bool fused, bool is_f32, cudaStream_t
 // =====================================================================================================================
 // Chunked form
 // =====================================================================================================================
-constexpr float kGlaMaxLogDecay = 60.f;  // exp(+-60) and its products with projections stay inside fp32
+// The chunked form keeps decay logarithms in base 2 (their sums are the arguments of the special-function unit, without a further rounding).
+constexpr float kGlaMaxLogDecay = 86.f;  // 2^(+-86) and its products with projections stay inside fp32
+__device__ __forceinline__ float exp2_sfu(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// log2(sigmoid(z)) = min(z, 0) log2(e) - log2(1 + e^-|z|); log(1 + x) = 2 artanh(x / (2 + x)) by the series of the inverse hyperbolic tangent,
+// whose argument is at most 1 / 3 here (eight terms: a relative error of 1e-8)
+__device__ __forceinline__ float log2_sigmoid(float z) {
+  constexpr float log2e = 1.4426950408889634f;
+  const float x = exp2_sfu(-fabsf(z) * log2e), s = __fdividef(x, 2.f + x), s2 = s * s;
+  float p = fmaf(s2, 1.f / 15.f, 1.f / 13.f);
+  p = fmaf(s2, p, 1.f / 11.f);
+  p = fmaf(s2, p, 1.f / 9.f);
+  p = fmaf(s2, p, 1.f / 7.f);
+  p = fmaf(s2, p, 1.f / 5.f);
+  p = fmaf(s2, p, 1.f / 3.f);
+  p = fmaf(s2, p, 1.f);
+  return (fminf(z, 0.f) - 2.f * s * p) * log2e;
+}
 
 template <int C>
 __global__ void __launch_bounds__(256) gla_prepare_kernel(const GlaArgs a, const GlaChunks c) {
@@ -250,32 +270,39 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const GlaArgs a, const
   const int ck = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int dk = a.dk, dk16 = (dk + 15) / 16 * 16, P = dk16 + 8;
   float* sb = reinterpret_cast<float*>(gsm);                               // [C][dk] decay logarithms, then their running sums
-  float* sx = sb + C * dk;                                                 // [C][8] part of the low-rank decay input
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sx + C * 8);        // [2][C][P] q exp(b), high and low parts
+  float* sx = sb + C * dk;                                                 // [C][16] part of the low-rank decay input
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sx + C * 16);       // [2][C][P] q exp(b), high and low parts
   __nv_bfloat16* sK = sQ + 2 * C * P;                                      // [2][C][P] k exp(-b)
   const int row0 = c.row0[ck], len = c.len[ck];
   const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(a.p);
   // ---- decay logarithms: a thread keeps one channel and takes every ng-th token
   const int ng = 256 / dk, d_own = tid % dk, grp = tid / dk;
-  for (int r0 = 0; r0 < a.rank; r0 += 8) {
+  for (int r0 = 0; r0 < a.rank; r0 += 16) {
+    const int nr = min(16, a.rank - r0);  // 8 or 16 columns of the decay input per round
     __syncthreads();
-    for (int e = tid; e < C * 2; e += 256) {
-      const int t = e >> 1, half = (e & 1) * 4;
+    for (int e = tid; e < C * 4; e += 256) {
+      const int t = e >> 2, x = (e & 3) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (t < len) v = g_ld4(p + static_cast<size_t>(row0 + t) * a.ld + a.off_a + r0 + half);
-      *reinterpret_cast<float4*>(sx + t * 8 + half) = v;
+      if (t < len && x < nr) v = g_ld4(p + static_cast<size_t>(row0 + t) * a.ld + a.off_a + r0 + x);
+      *reinterpret_cast<float4*>(sx + t * 16 + x) = v;
     }
     __syncthreads();
     if (grp < ng) {
       const float* wp = a.a2 + static_cast<size_t>(h * dk + d_own) * a.rank + r0;
-      const float4 w0 = *reinterpret_cast<const float4*>(wp), w1 = *reinterpret_cast<const float4*>(wp + 4);
+      float4 w[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) w[i] = i * 4 < nr ? *reinterpret_cast<const float4*>(wp + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
       const float bias = r0 == 0 ? a.a2_bias[h * dk + d_own] : 0.f;
-      const bool last = r0 + 8 >= a.rank;
+      const bool last = r0 + 16 >= a.rank;
+#pragma unroll 4
       for (int t = grp; t < C; t += ng) {
-        const float4 x0 = *reinterpret_cast<const float4*>(sx + t * 8), x1 = *reinterpret_cast<const float4*>(sx + t * 8 + 4);
-        float z = (r0 == 0 ? bias : sb[t * dk + d_own]) + w0.x * x0.x + w0.y * x0.y + w0.z * x0.z + w0.w * x0.w + w1.x * x1.x + w1.y * x1.y + w1.z * x1.z +
-                  w1.w * x1.w;
-        if (last) z = t < len ? log_sigmoid(z) * a.inv_tau : 0.f;
+        float z = r0 == 0 ? bias : sb[t * dk + d_own];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 x = *reinterpret_cast<const float4*>(sx + t * 16 + i * 4);
+          z += (w[i].x * x.x + w[i].y * x.y) + (w[i].z * x.z + w[i].w * x.w);
+        }
+        if (last) z = t < len ? log2_sigmoid(z) * a.inv_tau : 0.f;
         sb[t * dk + d_own] = z;
       }
     }
@@ -296,32 +323,37 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const GlaArgs a, const
   const bool fast = __syncthreads_and(small);
   // ---- scaled queries and keys
   __nv_bfloat16* qk = static_cast<__nv_bfloat16*>(c.qk);
-  const int half = dk / 2;
-  for (int e = tid; e < C * half; e += 256) {
-    const int t = e / half, d = (e % half) * 2;
-    float2 q = make_float2(0.f, 0.f), k = q;
-    if (t < len) {
-      const __nv_bfloat16* row = p + static_cast<size_t>(row0 + t) * a.ld + h * dk + d;
-      q = unpack_bf162(*reinterpret_cast<const uint32_t*>(row));
-      k = unpack_bf162(*reinterpret_cast<const uint32_t*>(row + a.off_k));
-    }
-    const float b0 = sb[t * dk + d], b1 = sb[t * dk + d + 1];
-    uint32_t qh, ql, kh, kl;
-    split2(q.x * a.q_scale * expf(b0), q.y * a.q_scale * expf(b1), qh, ql);
-    split2(k.x * expf(b_end[d] - b0), k.y * expf(b_end[d + 1] - b1), kh, kl);
-    if (t < len) {
-      uint32_t* dst = reinterpret_cast<uint32_t*>(qk + (static_cast<size_t>(row0 + t) * a.H + h) * 4 * dk + d);
-      dst[0] = qh;
-      dst[half] = ql;
-      dst[2 * half] = kh;
-      dst[3 * half] = kl;
-    }
-    if (fast) {
-      *reinterpret_cast<uint32_t*>(sQ + t * P + d) = qh;
-      *reinterpret_cast<uint32_t*>(sQ + (C + t) * P + d) = ql;
-      split2(k.x * expf(-b0), k.y * expf(-b1), kh, kl);
-      *reinterpret_cast<uint32_t*>(sK + t * P + d) = kh;
-      *reinterpret_cast<uint32_t*>(sK + (C + t) * P + d) = kl;
+  const int half = dk / 2, ng2 = 256 / half, grp2 = tid / half, d2 = (tid % half) * 2;  // a thread keeps one pair of channels
+  if (grp2 < ng2) {
+    const float2 be = *reinterpret_cast<const float2*>(b_end + d2);
+    const __nv_bfloat16* col = p + static_cast<size_t>(row0) * a.ld + h * dk + d2;
+    uint32_t* dst = reinterpret_cast<uint32_t*>(qk + (static_cast<size_t>(row0) * a.H + h) * 4 * dk + d2);
+    const size_t step = static_cast<size_t>(a.H) * 2 * dk;  // (in pairs)
+#pragma unroll 4
+    for (int t = grp2; t < C; t += ng2) {
+      uint32_t qu = 0u, ku = 0u;
+      if (t < len) {
+        qu = *reinterpret_cast<const uint32_t*>(col + t * a.ld);
+        ku = *reinterpret_cast<const uint32_t*>(col + t * a.ld + a.off_k);
+      }
+      const float2 q = unpack_bf162(qu), k = unpack_bf162(ku), b = *reinterpret_cast<const float2*>(sb + t * dk + d2);
+      uint32_t qh, ql, kh, kl;
+      split2(q.x * a.q_scale * exp2_sfu(b.x), q.y * a.q_scale * exp2_sfu(b.y), qh, ql);
+      split2(k.x * exp2_sfu(be.x - b.x), k.y * exp2_sfu(be.y - b.y), kh, kl);
+      if (t < len) {
+        uint32_t* row = dst + t * step;
+        row[0] = qh;
+        row[half] = ql;
+        row[2 * half] = kh;
+        row[3 * half] = kl;
+      }
+      if (fast) {
+        *reinterpret_cast<uint32_t*>(sQ + t * P + d2) = qh;
+        *reinterpret_cast<uint32_t*>(sQ + (C + t) * P + d2) = ql;
+        split2(k.x * exp2_sfu(-b.x), k.y * exp2_sfu(-b.y), kh, kl);
+        *reinterpret_cast<uint32_t*>(sK + t * P + d2) = kh;
+        *reinterpret_cast<uint32_t*>(sK + (C + t) * P + d2) = kl;
+      }
     }
   }
   if (dk16 != dk)
@@ -329,7 +361,7 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const GlaArgs a, const
       reinterpret_cast<uint32_t*>(sQ + (e >> 2) * P + dk)[e & 3] = 0u;
       reinterpret_cast<uint32_t*>(sK + (e >> 2) * P + dk)[e & 3] = 0u;
     }
-  for (int d = tid; d < dk; d += 256) c.decay[(static_cast<size_t>(ck) * a.H + h) * dk + d] = expf(b_end[d]);
+  for (int d = tid; d < dk; d += 256) c.decay[(static_cast<size_t>(ck) * a.H + h) * dk + d] = exp2_sfu(b_end[d]);
   __syncthreads();
   // ---- causal matrix of the chunk: the 16 x 16 blocks on and below the diagonal
   __nv_bfloat16* am = static_cast<__nv_bfloat16*>(c.a) + (static_cast<size_t>(ck) * a.H + h) * 2 * C * C;
@@ -378,7 +410,7 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const GlaArgs a, const
           if (s + j > t) continue;
           const __nv_bfloat16* k = p + static_cast<size_t>(row0 + s + j) * a.ld + a.off_k + h * dk;
           float acc = 0.f;
-          for (int d = 0; d < dk; ++d) acc += bf2f(q[d]) * bf2f(k[d]) * expf(sb[t * dk + d] - sb[(s + j) * dk + d]);
+          for (int d = 0; d < dk; ++d) acc += bf2f(q[d]) * bf2f(k[d]) * exp2_sfu(sb[t * dk + d] - sb[(s + j) * dk + d]);
           v[j] = acc * a.q_scale;
         }
       }
@@ -569,7 +601,7 @@ static cudaError_t launch_chunks_t(const GlaArgs& a, const GlaChunks& c, cudaStr
 template <int C>
 static cudaError_t launch_prepare_t(const GlaArgs& a, const GlaChunks& c, cudaStream_t st) {
   const int P = (a.dk + 15) / 16 * 16 + 8;
-  const size_t smem = static_cast<size_t>(C * a.dk + C * 8) * 4 + static_cast<size_t>(4) * C * P * 2;
+  const size_t smem = static_cast<size_t>(C * a.dk + C * 16) * 4 + static_cast<size_t>(4) * C * P * 2;
   static PerDeviceOnce once;
   if (once.first()) {
     const cudaError_t e = cudaFuncSetAttribute(gla_prepare_kernel<C>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
