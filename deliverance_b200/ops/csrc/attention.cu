@@ -387,30 +387,34 @@ struct DecodeMma {
   static constexpr int kBytes = (kRing > kMerge ? kRing : kMerge) + (D > 128 ? kQBytes : 0);
 };
 
-template <int D>
+// EXT: head widths below the tile width D, groups of more than 16 heads, kept first keys, a sink. Without it those are compile-time constants
+// (as run-time values they cost the plain kernel a tenth of its speed: the loop is paced by its address arithmetic).
+template <int D, bool EXT>
 __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, long long q_stride, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables, int bt_stride,
     const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, float* part_o, float* part_ml, int* __restrict__ arrivals,
-    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk, int dv, int keep_first, int sink) {
+    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk_ext, int dv_ext, int keep_ext, int sink_ext) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   using L = DecodeMma<D>;
   constexpr int CPR = D / 8;  // 16-byte chunks per row
   extern __shared__ __align__(128) uint8_t msm[];
+  const int dk = EXT ? dk_ext : D, dv = EXT ? dv_ext : D, keep_first = EXT ? keep_ext : 0;
+  const bool sink = EXT && sink_ext != 0;
   // a CTA takes up to 16 of the query heads that share a KV head
-  const int heads_per_kv = H / KV, groups = (heads_per_kv + 15) / 16;
+  const int heads_per_kv = H / KV, groups = EXT ? (heads_per_kv + 15) / 16 : 1;
   const int b = blockIdx.x, kvh = blockIdx.y / groups, sp = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t4 = lane & 3;
-  const int h0 = kvh * heads_per_kv + (blockIdx.y % groups) * 16;  // first query head of this CTA
-  const int G = min(16, (kvh + 1) * heads_per_kv - h0);
+  const int h0 = kvh * heads_per_kv + (EXT ? (blockIdx.y % groups) * 16 : 0);  // first query head of this CTA
+  const int G = EXT ? min(16, (kvh + 1) * heads_per_kv - h0) : heads_per_kv;
   const int ctx = ctx_lens[b];
   const int first_key = (window > 0 && ctx > window) ? ctx - window : 0;
   // slices of 16 keys: those that hold kept first tokens in front of the window, then [first_key, ctx); the CTA's share of that list
   const int kept = min(keep_first, first_key);  // keys [0, kept) are visible beside the window
   const int sl_lo = first_key / 16, sl_hi = (ctx + 15) / 16;
-  const int sl_kept = min((kept + 15) / 16, sl_lo), sl_skip = sl_lo - sl_kept;  // list position i is slice i or, behind the kept ones, i + sl_skip
+  const int sl_kept = EXT ? min((kept + 15) / 16, sl_lo) : 0, sl_skip = sl_lo - sl_kept;  // list position i is slice i or, behind the kept ones, i + sl_skip
   const int per = (sl_hi - sl_skip + splits - 1) / splits;
   const int s0 = sp * per, s1 = min(sl_hi - sl_skip, s0 + per);
   uint8_t* ring = msm + warp * L::kWarpBytes;
@@ -439,20 +443,28 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     __syncthreads();
   }
 
-  auto slice_at = [&](int i) { return i < sl_kept ? i : i + sl_skip; };
+  auto slice_at = [&](int i) { return EXT && i < sl_kept ? i : i + sl_skip; };
   auto load_slice = [&](int i, int stage) {
     // 16 keys x D of K and V: 2 * 16 * CPR chunks over 32 lanes (zeros behind the real widths)
     const int key0 = slice_at(i) * 16;
     const int page = block_tables[static_cast<long long>(b) * bt_stride + key0 / page_size];
     const long long row0 = (static_cast<long long>(page) * KV + kvh) * page_size + key0 % page_size;
+    const __nv_bfloat16 *kb = k_cache + row0 * dk, *vb = v_cache + row0 * dv;
     const uint32_t kdst = ring_u + stage * 2 * L::kSliceBytes, vdst = kdst + L::kSliceBytes;
 #pragma unroll
     for (int i = 0; i < 16 * CPR / 32; ++i) {
       const int c = i * 32 + lane;
       const int r = c / CPR, cc = c % CPR;
-      const bool in_ctx = key0 + r < ctx, vk = in_ctx && cc * 8 < dk, vv = in_ctx && cc * 8 < dv;
-      cp_async16(kdst + swz<D>(r, cc), k_cache + (vk ? (row0 + r) * dk + cc * 8 : row0 * dk), vk);
-      cp_async16(vdst + swz<D>(r, cc), v_cache + (vv ? (row0 + r) * dv + cc * 8 : row0 * dv), vv);
+      const bool valid = key0 + r < ctx;
+      if constexpr (EXT) {
+        const bool vk = valid && cc * 8 < dk, vv = valid && cc * 8 < dv;
+        cp_async16(kdst + swz<D>(r, cc), kb + (vk ? r * dk + cc * 8 : 0), vk);
+        cp_async16(vdst + swz<D>(r, cc), vb + (vv ? r * dv + cc * 8 : 0), vv);
+      } else {
+        const int off = (valid ? r : 0) * D + cc * 8;
+        cp_async16(kdst + swz<D>(r, cc), kb + off, valid);
+        cp_async16(vdst + swz<D>(r, cc), vb + off, valid);
+      }
     }
   };
   // ---- per-warp pipeline over its slices
@@ -501,7 +513,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + 2 * t4 + (e & 1);
         float v = softcap_apply(sc[nt][e] * scale, softcap);
-        v = (key < ctx && (key >= first_key || key < kept)) ? v : -INFINITY;
+        v = (key < ctx && (key >= first_key || (EXT && key < kept))) ? v : -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -665,7 +677,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
   }
 }
 
-template <int D>
+template <int D, bool EXT>
 static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                                const int* ctx, void* out, float* po, float* pml, int* arrivals, int B, int H, int KV, int page,
                                float scale, float cap, int window, int splits, cudaStream_t st, int dk = D, int dv = D, AttnExtra x = {}) {
@@ -674,10 +686,10 @@ static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc
   if (splits > 1 && (H / KV) * (splits + 1) > L::kMerge / 4) arrivals = nullptr;
   static PerDeviceOnce attr_once;
   if (attr_once.first()) {
-    cudaFuncSetAttribute(decode_attn_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
+    cudaFuncSetAttribute(decode_attn_mma_kernel<D, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
   }
   dim3 grid(B, KV * ((H / KV + 15) / 16), splits);
-  launch_pdl(decode_attn_mma_kernel<D>, dim3(grid), dim3(128), L::kBytes, st, static_cast<const __nv_bfloat16*>(q), q_stride,
+  launch_pdl(decode_attn_mma_kernel<D, EXT>, dim3(grid), dim3(128), L::kBytes, st, static_cast<const __nv_bfloat16*>(q), q_stride,
                                                           static_cast<const __nv_bfloat16*>(kc), static_cast<const __nv_bfloat16*>(vc), bt,
                                                           bt_stride, ctx, static_cast<__nv_bfloat16*>(out), po, pml, arrivals, H, KV, page, scale,
                                                           cap, window, splits, dk, dv, x.keep_first, x.sink);
@@ -696,11 +708,11 @@ int launch_decode_attention_impl(const void* q, long long q_stride, const void* 
   const int G = H / KV;
   if (impl == 0 && G <= 16 && page % 16 == 0 && (q_stride % 2) == 0) {
     switch (D) {
-      case 64: return launch_decode_mma_t<64>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 64: return launch_decode_mma_t<64, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
-      case 128: return launch_decode_mma_t<128>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 128: return launch_decode_mma_t<128, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
-      case 256: return launch_decode_mma_t<256>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 256: return launch_decode_mma_t<256, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
       default: return 1;
     }
@@ -715,7 +727,7 @@ int launch_decode_attention_mma(const void* q, long long q_stride, const void* k
   const int D = dk > dv ? dk : dv;
   if (dk % 8 != 0 || dv % 8 != 0 || D > 256 || page % 16 != 0 || q_stride % 8 != 0) return 1;
 #define DLV_DEC_MMA(DD) \
-  return launch_decode_mma_t<DD>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap, window, splits, st, dk, dv, x)
+  return launch_decode_mma_t<DD, true>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap, window, splits, st, dk, dv, x)
   if (D <= 64) DLV_DEC_MMA(64);
   if (D <= 128) DLV_DEC_MMA(128);
   DLV_DEC_MMA(256);
