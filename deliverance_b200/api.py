@@ -128,6 +128,10 @@ def build_model(cfg: ModelConfig, device, dtype, tp: TensorParallelContext):
         from .models.fopivik import FopivikModel
 
         return FopivikModel(cfg, device, dtype, tp)
+    if cfg.model_type == "dubozen":
+        from .models.dubozen import DubozenModel
+
+        return DubozenModel(cfg, device, dtype, tp)
     return DecoderModel(cfg, device, dtype, tp)
 
 

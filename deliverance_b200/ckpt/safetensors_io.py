@@ -147,7 +147,7 @@ def _payload(t: torch.Tensor) -> bytes:
     t = t.detach().contiguous().cpu()
     if t.numel() == 0:
         return b""
-    return t.view(torch.uint8).numpy().tobytes() if t.dtype != torch.uint8 else t.numpy().tobytes()
+    return t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.dtype != torch.uint8 else t.numpy().tobytes()
 
 
 def canonical_shape(shape: Iterable[int]) -> list[int]:

@@ -148,7 +148,98 @@ def _fopivik_tensors(cfg: dict, seed: int, dtype) -> dict:
     return t
 
 
+def dubozen_config(width: int, vocab: int, layers: list, streams: int = 2, eps: float = 1e-5, **extra) -> dict:
+    """``config.json`` of a Dubozen model. ``layers``: one dict of sizes per layer: ``heads, kv_heads, dim`` of the softmax attention with ``vdim``
+    (and ``v_mix``), or with ``right`` = ``(heads, dim, vdim, decays)`` of the lightning attention beside it (and ``left_scale, right_scale``);
+    ``rot_dims, base, scale``; ``ff`` alone for a dense feed-forward, with ``experts, top`` (and ``groups, keep, route_scale``) for routed experts,
+    ``ff`` 0 = none."""
+    out = []
+    for L in layers:
+        mlp = None
+        if L.get("ff") and L.get("experts"):
+            mlp = {"kind": "moe", "expert": {"ff": L["ff"]}, "router": {"experts": L["experts"], "top": L["top"], "scale": L.get("route_scale", 1.5),
+                                                                        "groups": {"count": L.get("groups", 1), "keep": L.get("keep", 1)}}}
+        elif L.get("ff"):
+            mlp = {"kind": "dense", "ff": L["ff"]}
+        soft = {k: L[k] for k in ("heads", "kv_heads", "dim")}
+        soft.update(vdim=L.get("vdim", L["dim"]), rot={"base": L.get("base", 10000.0), "dims": L.get("rot_dims", L["dim"] // 2 * 2)},
+                    scale=L.get("scale", L["dim"] ** -0.5))
+        if L.get("right"):
+            h, dk, dv, decay = L["right"]
+            mixer = {"left": soft, "left_scale": L.get("left_scale", 0.7), "right": {"heads": h, "dim": dk, "vdim": dv, "decay": list(decay)},
+                     "right_scale": L.get("right_scale", 0.4)}
+            out.append({"type": "parallel", "mixer": mixer, "mlp": mlp})
+        else:
+            out.append({"type": "attention", "mixer": dict(soft, v_mix=L.get("v_mix", True)), "mlp": mlp})
+    cfg = {"architecture": "Dubozen", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "layers": out}
+    cfg.update(extra)
+    return cfg
+
+
+def dubozen_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape of a Dubozen checkpoint."""
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+    s = {"embed": (V, W), "embed.norm": (W,), "final.norm": (W,)}
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        for q in (1, 2) if L.get("mlp") else (1,):
+            s.update({f"{p}norm{q}": (W,), f"{p}hc{q}.in": (S,), f"{p}hc{q}.out": (S,), f"{p}hc{q}.mix": (S, S)})
+        soft = m["left"] if L["type"] == "parallel" else m
+        H, G, dk, dv = soft["heads"], soft["kv_heads"], soft["dim"], soft["vdim"]
+        if L["type"] == "parallel":
+            a, b, r = p + "mix.left.", p + "mix.right.", m["right"]
+            R, rk, rv = r["heads"], r["dim"], r["vdim"]
+            s.update({a + "q": (H * dk, W), a + "k": (G * dk, W), a + "q.norm": (dk,), a + "k.norm": (dk,), a + "g": (H, W), a + "o": (W, H * dk),
+                      b + "q": (R * rk, W), b + "k": (R * rk, W), b + "v": (R * rv, W), b + "g": (R * rv, W), b + "o": (W, R * rv), b + "norm": (R * rv,)})
+        else:
+            a = p + "mix."
+            s.update({a + "q": (H * dk, W), a + "k": (G * dk, W), a + "v": (G * dv, W), a + "g": (H * dv, W), a + "o": (W, H * dv), a + "sink": (H,)})
+            if m.get("v_mix"):
+                s[a + "vmix"] = ()
+        if L.get("mlp") and L["mlp"]["kind"] == "dense":
+            F = L["mlp"]["ff"]
+            s.update({p + "mlp.gate": (F, W), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+        elif L.get("mlp"):
+            F, E = L["mlp"]["expert"]["ff"], L["mlp"]["router"]["experts"]
+            s.update({p + "mlp.router": (E, W), p + "mlp.correction": (E,)})
+            for e in range(E):
+                s.update({f"{p}mlp.e{e}.gate": (F, W), f"{p}mlp.e{e}.up": (F, W), f"{p}mlp.e{e}.down": (W, F)})
+    return s
+
+
+def dubozen_value(name: str, r, cfg: dict):
+    """Weight ``name`` from standard normal numbers ``r`` of its shape: projections scaled by their fan-in, mixes near the identity, every
+    mechanism moving the output."""
+    last = name.rsplit(".", 1)[-1]
+    if "norm" in last:
+        return 1.0 + 0.2 * r
+    if last == "vmix":
+        return 0.4 + 0.1 * r
+    if last == "sink":
+        return 1.0 + r
+    if last == "correction":
+        return 0.3 * r - 1.0  # (negative choice scores)
+    if ".hc" in name:
+        if last == "mix":
+            return 0.9 * torch.eye(r.shape[0], dtype=r.dtype, device=r.device) + 0.15 * r
+        return (0.7 + 0.3 * r) / (cfg["streams"] ** 0.5 if last == "in" else 1.0)
+    if len(r.shape) == 2 and name != "embed":
+        return r * r.shape[1] ** -0.5 * (2.0 if last == "router" else 1.0)
+    return r
+
+
+def _dubozen_tensors(cfg: dict, seed: int, dtype) -> dict:
+    g = torch.Generator().manual_seed(seed)
+    return {n: dubozen_value(n, torch.randn(shape, generator=g, dtype=torch.float32), cfg).to(dtype) for n, shape in dubozen_shapes(cfg).items()}
+
+
 def tiny_config(model_type: str, **over) -> dict:
+    if model_type == "dubozen":
+        soft = dict(heads=6, kv_heads=2, dim=20, vdim=28, rot_dims=12, ff=52)
+        both = dict(heads=4, kv_heads=1, dim=18, rot_dims=10, base=500.0, right=(3, 12, 20, (0.4, 0.97, 0.999)), ff=36, experts=6, top=2, groups=3, keep=2)
+        kw = dict(width=76, vocab=261, layers=[dict(soft), dict(both), dict(soft, heads=2, scale=0.4, ff=24, experts=5, top=2), dict(both, ff=0)], streams=3)
+        kw.update(over)
+        return dubozen_config(**kw)
     if model_type == "fopivik":
         soft = dict(heads=6, kv_heads=2, dim=20, vdim=28, rot_dims=12, window=24, keep_first=5, experts=5, top=2, ff=36)
         lin = dict(heads=3, dim=12, vdim=20, tau=4.0, experts=4, top=1, ff=24)
@@ -209,6 +300,8 @@ def build_tensors(cfg: dict, seed: int = 0, dtype=torch.float32, std: float = 0.
         return _fatotar_tensors(cfg, seed, dtype)
     if mt == "fopivik":
         return _fopivik_tensors(cfg, seed, dtype)
+    if mt == "dubozen":
+        return _dubozen_tensors(cfg, seed, dtype)
     R = lambda *s: _rand(g, *s, std=std, dtype=dtype)  # noqa: E731
     ones = lambda n: (torch.ones(n) + torch.randn(n, generator=g) * 0.05).to(dtype)  # noqa: E731
     t: dict = {}

@@ -19,9 +19,10 @@ from typing import Any, Optional
 
 SUPPORTED_MODEL_TYPES = (
     "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert", "fatotar", "fopivik",
+    "dubozen",
 )
 # designs whose config.json names an architecture instead of a model_type
-_ARCHITECTURE_TYPES = {"fatotar": "fatotar", "fopivik": "fopivik"}
+_ARCHITECTURE_TYPES = {"fatotar": "fatotar", "fopivik": "fopivik", "dubozen": "dubozen"}
 
 # transformers' Gemma3TextConfig defaults: hub configs of the multimodal checkpoints leave most text fields out
 _GEMMA3_TEXT_DEFAULTS = dict(vocab_size=262208, hidden_size=2304, intermediate_size=9216, num_hidden_layers=26, num_attention_heads=8,
@@ -71,7 +72,7 @@ class ModelConfig:
     experts_per_token: int = 0
     moe_intermediate_size: int = 0
     norm_topk_prob: bool = True
-    router_mode: str = "softmax_topk"  # "softmax_topk" (mixtral/qwen3) | "topk_softmax" (granite)
+    router_mode: str = "softmax_topk"  # "softmax_topk" (mixtral/qwen3) | "topk_softmax" (granite) | "sigmoid_topk" (dubozen)
     decoder_sparse_step: int = 1
     mlp_only_layers: tuple[int, ...] = ()
     shared_intermediate_size: int = 0
@@ -270,6 +271,39 @@ def _parse_fopivik(d: dict) -> ModelConfig:
     return cfg
 
 
+MAX_STREAMS = 16  # residual streams the CUDA kernel keeps in registers
+
+
+def _parse_dubozen(d: dict) -> ModelConfig:
+    """Dubozen: several residual streams with learned reads and writes per sublayer, grouped attention (sink, output gate, values mixed with the
+    first layer's) and grouped attention beside lightning attention in any order, dense or routed feed-forwards, tied embeddings. Every layer
+    carries its own sizes; ``extra["layers"]`` keeps them as given. The context length is not part of the design."""
+    layers, streams = list(d["layers"]), int(d["streams"])
+    if not layers:
+        raise ValueError("no layers")
+    if not 1 <= streams <= MAX_STREAMS:
+        raise ValueError(f"{streams} residual streams (between 1 and {MAX_STREAMS})")
+    for i, L in enumerate(layers):
+        if L["type"] not in ("attention", "parallel"):
+            raise ValueError(f"layer {i}: unknown mixer '{L['type']}'")
+        if L.get("mlp") and L["mlp"]["kind"] not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward '{L['mlp']['kind']}'")
+    soft = [L["mixer"]["left"] if L["type"] == "parallel" else L["mixer"] for L in layers]
+    dense = [int(L["mlp"]["ff"]) for L in layers if L.get("mlp") and L["mlp"]["kind"] == "dense"]
+    moe = [L["mlp"] for L in layers if L.get("mlp") and L["mlp"]["kind"] == "moe"]
+    cfg = ModelConfig(
+        model_type="dubozen", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), num_layers=len(layers),
+        num_heads=max(int(m["heads"]) for m in soft), num_kv_heads=max(int(m["kv_heads"]) for m in soft), head_dim=max(int(m["dim"]) for m in soft),
+        intermediate_size=max(dense or [0]), max_position_embeddings=int(d.get("max_position_embeddings") or 131072), norm_eps=float(d["norm"]["eps"]),
+        hidden_act="gelu_pytorch_tanh", tie_word_embeddings=True, num_experts=max([int(m["router"]["experts"]) for m in moe] or [0]),
+        experts_per_token=max([int(m["router"]["top"]) for m in moe] or [0]), moe_intermediate_size=max([int(m["expert"]["ff"]) for m in moe] or [0]),
+        router_mode="sigmoid_topk", bos_token_id=d.get("bos_token_id"), eos_token_ids=_eos(d.get("eos_token_id")), pad_token_id=d.get("pad_token_id"),
+        use_rope=False, add_bos=False, raw=d,
+    )
+    cfg.extra = {"layers": layers, "streams": streams}
+    return cfg
+
+
 def _eos(v: Any) -> tuple[int, ...]:
     if v is None:
         return ()
@@ -296,6 +330,8 @@ def parse_config(d: dict) -> ModelConfig:
         return _parse_fatotar(d)
     if mt == "fopivik":
         return _parse_fopivik(d)
+    if mt == "dubozen":
+        return _parse_dubozen(d)
     if mt in ("gemma4", "gemma4_text"):
         return _parse_gemma4(d)
     if mt in ("gemma3", "gemma3_text"):

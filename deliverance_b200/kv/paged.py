@@ -16,7 +16,8 @@ Layout per attention layer: ``k[pages, KV, page_size, D]`` and ``v[...]`` in the
 that padded batch rows write to. Latent-attention layers use the same pair with one "head": ``k`` holds the compressed vectors, ``v``
 the rotated key parts shared by all heads (a width of its own, ``v_dim_per_layer``). Recurrent layers (Mamba2, gated linear
 attention) have no pages: a sequence holds one state slot, an index into the fp32 tensors named by the layout's ``state_shapes`` (one
-entry per layer: None, or name -> shape of one sequence's state). Slot 0 is a scratch slot that padded batch rows update.
+entry per layer: None, or name -> shape of one sequence's state). Slot 0 is a scratch slot that padded batch rows update. A layer that has
+both (attention beside a recurrence) says so in the layout's ``paged`` (one flag per layer; default: the layers without a state).
 """
 from __future__ import annotations
 
@@ -247,8 +248,9 @@ class PagedKVCache:
         v_dims = layout.get("v_dim_per_layer") or dims
         shared = layout.get("shared_from") or [-1] * len(kinds)
         states = layout.get("state_shapes") or [None] * len(kinds)
+        paged = self.paged_layers(layout)
         for i in range(len(kinds)):
-            if states[i]:
+            if not paged[i]:
                 self.k.append(None)
                 self.v.append(None)
             elif shared[i] >= 0:
@@ -274,6 +276,11 @@ class PagedKVCache:
         return self.k[i], self.v[i]
 
     @staticmethod
+    def paged_layers(layout: dict) -> list:
+        states = layout.get("state_shapes") or [None] * len(layout["layer_kinds"])
+        return list(layout.get("paged") or [not s for s in states])
+
+    @staticmethod
     def bytes_per_state_slot(layout: dict) -> int:
         return sum(4 * math.prod(shape) for shapes in layout.get("state_shapes") or [] if shapes for shape in shapes.values())
 
@@ -284,8 +291,8 @@ class PagedKVCache:
         dims = layout.get("head_dim_per_layer") or [layout["head_dim"]] * len(kinds)
         shared = layout.get("shared_from") or [-1] * len(kinds)
         v_dims = layout.get("v_dim_per_layer") or dims
-        states = layout.get("state_shapes") or [None] * len(kinds)
-        rows = sum(heads[i] * (dims[i] + v_dims[i]) for i in range(len(kinds)) if not states[i] and shared[i] < 0)
+        paged = PagedKVCache.paged_layers(layout)
+        rows = sum(heads[i] * (dims[i] + v_dims[i]) for i in range(len(kinds)) if paged[i] and shared[i] < 0)
         return rows * page_size * torch.empty((), dtype=dtype).element_size()
 
     # -- per-sequence page management ---------------------------------------------------------------------------

@@ -1,7 +1,10 @@
 """Grouped-query attention mixer with per-layer sizes (``ops/grouped.py``): any decoder can use it. Score scale, soft-cap, window, kept
-first tokens, sink and rotation tables are parameters; it reads its input rows, keeps its cache in the pair ``kv.layer(i)`` and returns
-the output projection."""
+first tokens, sink, rotation tables and layout, head norms, value mixing and output gate are parameters; it reads its input rows, keeps its
+cache in the pair ``kv.layer(i)`` and returns the output projection (:meth:`forward`), or works between projections that it shares with
+another mixer (:meth:`pack`, :meth:`heads`)."""
 from __future__ import annotations
+
+from typing import Optional
 
 import torch
 
@@ -12,44 +15,95 @@ from .batch import ForwardBatch
 
 
 class GroupedAttention:
-    kind = "sliding"
-
-    def __init__(self, shape: GroupedShape, scale: float, softcap: float, window: int, keep_first: int, sink: bool, cos, sin, device, dtype):
+    def __init__(self, shape: GroupedShape, scale: float, softcap: float, window: int, keep_first: int, sink: bool, cos, sin, device, dtype,
+                 rotate: str = "pairs", eps: float = 0.0, mult: float = 1.0, v_mix: bool = False):
+        """``sink``: the softmax has a sink, of score 0 unless :meth:`pack` gets learned ones. ``rotate``: ``pairs`` (2 i, 2 i + 1) or ``halves``
+        (i, i + half) of the rotated columns. ``mult``: constant factor of the heads. ``v_mix``: the values are blended with those of the
+        first such layer of the forward pass."""
         self.shape, self.scale, self.softcap = shape, float(scale), float(softcap)
-        self.window, self.keep_first, self.sink = int(window), int(keep_first), bool(sink)
-        self.cos, self.sin = cos, sin
+        self.window, self.keep_first = int(window), int(keep_first)
+        self.kind = "sliding" if self.window > 0 else "attention"
+        self.sink = torch.zeros(shape.heads, dtype=torch.float32, device=device) if sink else None
+        self.cos, self.sin, self.rotate = cos, sin, rotate
+        self.eps, self.mult, self.v_mix = float(eps), float(mult), bool(v_mix)
+        self.lam = 0.0
+        self.q_norm = self.k_norm = None
         self.device, self.dtype = device, dtype
         if cos.shape[1] * 2 > shape.dim:
             raise ValueError(f"rotation covers {cos.shape[1] * 2} of {shape.dim} query / key columns")
+        if rotate not in ("pairs", "halves") or (rotate == "pairs" and (shape.tied or v_mix)):
+            raise ValueError("tied and mixed values need the 'halves' rotation")
 
-    def load(self, q, k, v, o, k_pad: int) -> "GroupedAttention":
-        """Weights as stored (``[out, in]``); ``k_pad``: padded input width of the rows :meth:`forward` gets."""
+    def pack(self, q, k, v, o, g=None, sink=None, q_norm=None, k_norm=None, vmix: Optional[float] = None) -> tuple:
+        """Weights as stored (``[out, in]``) -> (rows of the input projection, columns of the output projection) in the padded layout."""
         s = self.shape
-        for n, t, rows in (("q", q, s.heads * s.dim), ("k", k, s.kv_heads * s.dim), ("v", v, s.kv_heads * s.vdim)):
+        want = [("q", q, s.heads * s.dim), ("k", k, s.kv_heads * s.dim)]
+        if not s.tied:
+            want.append(("v", v, s.kv_heads * s.vdim))
+        if s.gate:
+            want.append(("g", g, s.heads * (s.vdim if s.gate == "columns" else 1)))
+        for n, t, rows in want:
             if t.shape[0] != rows:
                 raise ValueError(f"grouped attention: '{n}' has {t.shape[0]} rows, the configured sizes need {rows}")
         if o.shape[1] != s.heads * s.vdim:
             raise ValueError(f"grouped attention: 'o' has {o.shape[1]} columns, the configured sizes need {s.heads * s.vdim}")
-        w = torch.cat([pad_head_rows(q, s.heads, s.dim, s.dk), pad_head_rows(k, s.kv_heads, s.dim, s.dk), pad_head_rows(v, s.kv_heads, s.vdim, s.dv)])
-        w = torch.nn.functional.pad(w, (0, k_pad - w.shape[1]))
+        rows = [pad_head_rows(q, s.heads, s.dim, s.dk), pad_head_rows(k, s.kv_heads, s.dim, s.dk)]
+        if not s.tied:
+            rows.append(pad_head_rows(v, s.kv_heads, s.vdim, s.dv))
+        if s.gate:
+            rows.append(pad_head_rows(g, s.heads, s.vdim, s.dv) if s.gate == "columns" else g)
+        w = torch.cat(rows)
+        w = torch.nn.functional.pad(w, (0, 0, 0, s.width - w.shape[0]))
+        if sink is not None:
+            if sink.numel() != s.heads:
+                raise ValueError(f"grouped attention: {sink.numel()} sinks for {s.heads} heads")
+            self.sink = sink.reshape(-1).to(device=self.device, dtype=torch.float32).contiguous()
+        if q_norm is not None:
+            if q_norm.numel() != s.dim or k_norm.numel() != s.dim:
+                raise ValueError(f"grouped attention: head norms need {s.dim} weights")
+            norm = lambda t: torch.nn.functional.pad(t.reshape(-1).float(), (0, s.dk - s.dim)).to(self.device).contiguous()  # noqa: E731
+            self.q_norm, self.k_norm = norm(q_norm), norm(k_norm)
+        if vmix is not None:
+            self.lam = float(vmix)
+        return w, pad_head_columns(o, s.heads, s.vdim, s.dv)
+
+    def load(self, q, k, v, o, k_pad: int, **extra) -> "GroupedAttention":
+        """:meth:`pack` with projections of its own; ``k_pad``: padded input width of the rows :meth:`forward` gets."""
+        w, o = self.pack(q, k, v, o, **extra)
         put = lambda t: LinearWeight(t.to(device=self.device, dtype=self.dtype).contiguous())  # noqa: E731
-        self.w_in, self.w_out = put(w), put(pad_head_columns(o, s.heads, s.vdim, s.dv))
+        self.w_in, self.w_out = put(torch.nn.functional.pad(w, (0, k_pad - w.shape[1]))), put(o)
         return self
 
     def nbytes(self) -> int:
         return self.w_in.nbytes() + self.w_out.nbytes()
 
-    def forward(self, x, batch: ForwardBatch, kv, run: int, stage) -> torch.Tensor:
-        s = self.shape
-        k_cache, v_cache = kv.layer(run)
+    def forward(self, x, batch: ForwardBatch, kv, run: int, stage, shared: Optional[dict] = None) -> torch.Tensor:
+        """``shared``: what the layers of one forward pass hand on (the first mixing layer's values)."""
         with stage("groupedattention.qkv_projection"):
-            qkv = ops.linear(x, self.w_in)
-        with stage("groupedattention.rope"):
-            gop.rope_pairs_kv(s, qkv, batch.positions, batch.slots, self.cos, self.sin, k_cache, v_cache)
-        with stage("groupedattention.score_value"):
-            a = gop.attention(s, qkv, batch, k_cache, v_cache, self.scale, self.softcap, self.window, self.keep_first, self.sink, self._splits(batch))
+            p = ops.linear(x, self.w_in)
+        a = self.heads(p, batch, kv, run, stage, shared=shared)
         with stage("groupedattention.output_projection"):
             return ops.linear(a, self.w_out)
+
+    def heads(self, p, batch: ForwardBatch, kv, run: int, stage, out=None, shared: Optional[dict] = None) -> torch.Tensor:
+        """``p [T, shape.width]``: this mixer's columns of the projection rows -> gated heads ``[T, H * dv]`` (in ``out`` when given)."""
+        s = self.shape
+        k_cache, v_cache = kv.layer(run)
+        with stage("groupedattention.rope"):
+            if self.rotate == "pairs":
+                gop.rope_pairs_kv(s, p[:, : s.gate_at], batch.positions, batch.slots, self.cos, self.sin, k_cache, v_cache)
+            else:
+                first = None
+                if self.v_mix:
+                    v = p[:, s.v_at : s.v_at + s.v_width]
+                    first = shared.get("values")
+                    if first is None:
+                        shared["values"] = v
+                    elif first.shape != v.shape:
+                        raise ValueError(f"values of {v.shape[1]} columns cannot be mixed with {first.shape[1]}")
+                gop.rope_heads_kv(s, p, batch.positions, batch.slots, self.cos, self.sin, k_cache, v_cache, self.q_norm, self.k_norm, self.eps, first, self.lam)
+        with stage("groupedattention.score_value"):
+            return gop.attention(s, p, batch, k_cache, v_cache, self.scale, self.softcap, self.window, self.keep_first, self.sink, self._splits(batch), self.mult, out)
 
     def _splits(self, batch: ForwardBatch) -> int:
         """Split-KV factor of a decode step: a captured step knows the window but not the contexts it will see."""

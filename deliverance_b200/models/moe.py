@@ -21,6 +21,7 @@ from ..ops import LinearWeight, ref
 
 
 _SM_COUNT = 148  # B200
+_MODES = {"softmax_topk": 0, "topk_softmax": 1, "sigmoid_topk": 2}
 _ROUTE_ONE_LAUNCH = [os.environ.get("DLV_MOE_ROUTE", "fused") != "split"]  # decode-size routing in one launch ("split": the separate kernels)
 
 
@@ -125,13 +126,14 @@ def _experts_cuda(st, lw, x, logits, E, k, mode, renorm, act, e0, ne):
     with st("moe.route"):
         # weights [T, k] fp32, expert ids [T, k], counts [E], offsets [E + 1], perm: grouped row -> (token * k + slot), pos: inverse,
         # items: the grouped GEMM's work list. Decode-size batches get all of it from one launch.
-        mode_i = 0 if mode == "softmax_topk" else 1
-        routed = e.moe_route_items(logits.contiguous(), k, mode_i, bool(renorm), e0, ne, bn, max_items) if _ROUTE_ONE_LAUNCH[0] else []
+        mode_i = _MODES[mode]
+        rules = lw.routing_rules() if hasattr(lw, "routing_rules") else {}
+        routed = e.moe_route_items(logits.contiguous(), k, mode_i, bool(renorm), e0, ne, bn, max_items, **rules) if _ROUTE_ONE_LAUNCH[0] else []
         if routed:
             w, idx, counts, offsets, perm, pos, items = routed
             ops._count()
         else:
-            w, idx, counts, offsets, perm, pos = e.moe_route(logits.contiguous(), k, mode_i, bool(renorm))
+            w, idx, counts, offsets, perm, pos = e.moe_route(logits.contiguous(), k, mode_i, bool(renorm), **rules)
             items = e.moe_items(offsets, e0, ne, bn, max_items)
             ops._count(3)
         rng = (offsets, e0, ne) if ep else (None, 0, 0)
@@ -181,28 +183,41 @@ def _experts_cuda(st, lw, x, logits, E, k, mode, renorm, act, e0, ne):
 
 
 class RoutedExperts:
-    """Routed experts without biases: softmax (or top-k first) routing, ``top`` experts per token, gated activation. The result is left
-    in expert order (:class:`ops.Routed`) so that the norm behind it can do the weighted sum; ``ops.Routed.dense`` does it alone.
+    """Routed experts without biases: softmax, top-k first or sigmoid routing (``ref.moe_route``; the last with a correction of the choice,
+    ``groups`` of which ``keep`` take part, and a weight ``scale``), ``top`` experts per token, gated activation. The result is left in expert
+    order (:class:`ops.Routed`) so that the step behind it can do the weighted sum; ``ops.Routed.dense`` does it alone.
 
     The expert width is padded to a multiple of 8 with zero rows, the input width to ``k_pad``."""
 
     expert0, fused_act_experts = 0, False
 
-    def __init__(self, experts: int, top: int, act: str = "silu", mode: str = "softmax_topk", renorm: bool = False):
+    def __init__(self, experts: int, top: int, act: str = "silu", mode: str = "softmax_topk", renorm: bool = False, groups: int = 1, keep: int = 1,
+                 scale: float = 1.0):
         if not 0 < top <= experts:
             raise ValueError(f"{top} of {experts} experts per token")
+        if groups < 1 or experts % groups or not 1 <= keep <= groups or keep * (experts // groups) < top:
+            raise ValueError(f"{keep} of {groups} groups of {experts} experts, {top} experts per token")
+        self.groups, self.keep, self.scale = int(groups), int(keep), float(scale)
+        self.correction = None
         self.experts, self.top, self.act, self.mode, self.renorm = int(experts), int(top), act, mode, bool(renorm)
         self.n_local_experts = self.experts
         self.experts_gate_up: list = []
         self.experts_down: list = []
 
-    def load(self, router, experts, ff: int, k_pad: int, device, dtype) -> "RoutedExperts":
-        """``experts``: (gate, up, down) per expert as stored."""
+    def routing_rules(self) -> dict:
+        return {"correction": self.correction, "groups": self.groups, "keep": self.keep, "scale": self.scale}
+
+    def load(self, router, experts, ff: int, k_pad: int, device, dtype, correction=None) -> "RoutedExperts":
+        """``experts``: (gate, up, down) per expert as stored; ``correction [experts]``: added to the scores where experts are chosen."""
         pad = torch.nn.functional.pad
         ff8 = (ff + 7) // 8 * 8
         put = lambda t: LinearWeight(t.to(device=device, dtype=dtype).contiguous())  # noqa: E731
         if router.shape[0] != self.experts:
             raise ValueError(f"router has {router.shape[0]} rows for {self.experts} experts")
+        if correction is not None:
+            if correction.numel() != self.experts:
+                raise ValueError(f"{correction.numel()} corrections for {self.experts} experts")
+            self.correction = correction.reshape(-1).to(device=device, dtype=torch.float32).contiguous()
         self.router = put(pad(router, (0, k_pad - router.shape[1])))
         for gate, up, down in experts:
             if gate.shape[0] != ff or up.shape[0] != ff or down.shape[1] != ff:
@@ -227,7 +242,7 @@ class RoutedExperts:
         if x.device.type == "cuda":
             ys, pos, w, _ = _experts_cuda(stage, self, x, logits, self.experts, self.top, self.mode, self.renorm, self.act, 0, self.experts)
             return ops.Routed(ys, pos.reshape(-1, self.top), w)
-        w, idx = ref.moe_route(logits, self.top, self.mode, self.renorm)
+        w, idx = ref.moe_route(logits, self.top, self.mode, self.renorm, **self.routing_rules())
         y = ref.moe_experts(x, w, idx, lambda e, rows: ops.linear(rows, self.experts_gate_up[e]), lambda e, h: ops.linear(h, self.experts_down[e]),
                             self.experts, self.act)
         return ops.Routed(y, None, None)

@@ -397,6 +397,37 @@ def sandwich_norm(residual, sub, w_sub, mult: float, w_next, eps: float, pitch: 
     return out
 
 
+def stream_open(table, ids, w_open, streams: int, read, w_next, eps: float, pitch: int, dtype):
+    """Start of a decoder with several residual streams: every one is ``LayerNorm(table[ids]; w_open)`` in fp32. Returns the streams ``[T, S, W]`` and
+    ``LayerNorm(sum_s read[s] x_s; w_next)``, ``[T, pitch]`` in ``dtype``."""
+    T, W = ids.shape[0], table.shape[1]
+    X = torch.empty(T, streams, W, dtype=torch.float32, device=table.device)
+    if _cuda(table):
+        _count()
+        y = require_ext().stream_step(X, ids.to(torch.int32), w_open, table, None, None, None, None, True, read, w_next, eps, pitch, dtype == torch.float32)
+        return X, y
+    X.copy_(ref.layernorm_rows(table[ids.long()].float(), w_open, eps).unsqueeze(1))
+    return X, stream_step(X, None, None, None, read, w_next, eps, pitch, dtype)
+
+
+def stream_step(streams, sub, mix, write, read, w_next, eps: float, pitch: int, dtype, keep: bool = True):
+    """End of one sublayer and start of the next over fp32 streams ``[T, S, W]``: ``x_t = sum_s mix[s, t] x_s + write[t] sub`` in place, then
+    ``LayerNorm(sum_s read[s] x_s; w_next)`` as ``[T, pitch]`` rows (zeros behind the row width). ``sub``: ``[T, >= W]`` rows, a :class:`Routed`
+    result (its weighted sum is formed here in fp32), or None (the streams stay); ``read`` None: ones; ``w_next`` None: no norm; ``keep`` False:
+    nothing reads the streams again, they need not be written. LayerNorms have a weight and no bias."""
+    if _cuda(streams):
+        _count()
+        ys, pos, w = (sub.ys, sub.pos, sub.w) if isinstance(sub, Routed) else (sub, None, None)
+        return require_ext().stream_step(streams, None, None, ys, pos, w, mix, write, keep, read, w_next, eps, pitch, dtype == torch.float32)
+    W = streams.shape[2]
+    if sub is not None:
+        ref.stream_write(streams, (sub.dense() if isinstance(sub, Routed) else sub)[:, :W], mix, write)
+    y = ref.stream_read(streams, read)
+    if w_next is not None:
+        y = ref.layernorm_rows(y, w_next, eps)
+    return torch.nn.functional.pad(y, (0, pitch - W)).to(dtype)
+
+
 def gated_act_into(gate_up, act: str, out) -> None:
     """``out = act(gate) * up`` for ``gate_up [T, 2 I]``; ``out`` is an ``[T, I]`` column range of a wider row."""
     if _cuda(gate_up):

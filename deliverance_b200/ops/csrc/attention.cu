@@ -9,6 +9,7 @@
 // tensor/.../operations/TensorOperations.java:225-271, tensor/.../VectorTensorMathUtils.java:34-78).
 #include "common.cuh"
 #include "gemm_api.h"
+#include "io.cuh"
 
 namespace dlv {
 
@@ -241,11 +242,19 @@ __global__ void __launch_bounds__(128) decode_attn_kernel(
   }
 }
 
+// factor of one output column: out_mult, times sigmoid of the row's gate logit for the head or the column
+template <typename TIO>
+__device__ __forceinline__ float attn_gate(const AttnExtra& x, const TIO* gate, long long row, int h, int col) {
+  if (gate == nullptr) return x.out_mult;
+  const float z = io_ld(gate + row * x.gate_pitch + (x.gate_heads ? h : col));
+  return x.out_mult / (1.f + expf(-z));
+}
+
 // grid (num_seqs, H), D threads rounded up to whole warps. The split weights are computed once per CTA (thread s takes split s) and kept
 // in shared memory; the weighted sum over the splits then runs with independent loads. (The first version had every thread walk
 // all splits twice with dependent loads: 12 us at 64 splits, more than the attention kernel it follows.)
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits, int sink) {
+                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits, const AttnExtra x) {
   __shared__ float w_s[256];
   __shared__ float red[2][8];
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
@@ -273,7 +282,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   __syncthreads();
   den = 0.f;
   for (int i = 0; i < nw; ++i) den += red[1][i];
-  if (sink) den += __expf(-m);
+  if (x.sink != nullptr) den += __expf(x.sink[h] - m);
   if (d >= D) return;
   float num = 0.f;
   const int n_fast = splits < 256 ? splits : 256;
@@ -283,7 +292,8 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
     const float ms = part_ml[(base + s) * 2];
     num += ((ms == -INFINITY) ? 0.f : __expf(ms - m)) * part_o[(base + s) * D + d];
   }
-  out[(static_cast<long long>(b) * H + h) * D + d] = f2bf(den > 0.f ? num / den : 0.f);
+  const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * D;
+  out[b * pitch + h * D + d] = f2bf(den > 0.f ? num / den * attn_gate(x, static_cast<const __nv_bfloat16*>(x.gate), b, h, h * D + d) : 0.f);
 }
 
 template <int D, int GP>
@@ -310,7 +320,7 @@ static int launch_decode_t(const void* q, long long q_stride, const void* kc, co
                                                       scale, cap, window, splits);
   if (splits > 1) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits, 0);
+    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits, AttnExtra{});
   }
   return 0;
 }
@@ -387,34 +397,34 @@ struct DecodeMma {
   static constexpr int kBytes = (kRing > kMerge ? kRing : kMerge) + (D > 128 ? kQBytes : 0);
 };
 
-// EXT: head widths below the tile width D, groups of more than 16 heads, kept first keys, a sink. Without it those are compile-time constants
-// (as run-time values they cost the plain kernel a tenth of its speed: the loop is paced by its address arithmetic).
-template <int D, bool EXT>
+// EXT 1: head widths below the tile width D, groups of more than 16 heads, kept first keys. Without it those are compile-time constants (as
+// run-time values they cost the plain kernel a tenth of its speed: the loop is paced by its address arithmetic). EXT 1 and 2: the options
+// of AttnExtra that only the epilogue sees (sink, output gate, output pitch).
+template <int D, int EXT>
 __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, long long q_stride, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables, int bt_stride,
     const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, float* part_o, float* part_ml, int* __restrict__ arrivals,
-    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk_ext, int dv_ext, int keep_ext, int sink_ext) {
+    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk_ext, int dv_ext, const AttnExtra x) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   using L = DecodeMma<D>;
   constexpr int CPR = D / 8;  // 16-byte chunks per row
   extern __shared__ __align__(128) uint8_t msm[];
-  const int dk = EXT ? dk_ext : D, dv = EXT ? dv_ext : D, keep_first = EXT ? keep_ext : 0;
-  const bool sink = EXT && sink_ext != 0;
+  const int dk = EXT == 1 ? dk_ext : D, dv = EXT == 1 ? dv_ext : D, keep_first = EXT == 1 ? x.keep_first : 0;
   // a CTA takes up to 16 of the query heads that share a KV head
-  const int heads_per_kv = H / KV, groups = EXT ? (heads_per_kv + 15) / 16 : 1;
+  const int heads_per_kv = H / KV, groups = EXT == 1 ? (heads_per_kv + 15) / 16 : 1;
   const int b = blockIdx.x, kvh = blockIdx.y / groups, sp = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t4 = lane & 3;
-  const int h0 = kvh * heads_per_kv + (EXT ? (blockIdx.y % groups) * 16 : 0);  // first query head of this CTA
-  const int G = EXT ? min(16, (kvh + 1) * heads_per_kv - h0) : heads_per_kv;
+  const int h0 = kvh * heads_per_kv + (EXT == 1 ? (blockIdx.y % groups) * 16 : 0);  // first query head of this CTA
+  const int G = EXT == 1 ? min(16, (kvh + 1) * heads_per_kv - h0) : heads_per_kv;
   const int ctx = ctx_lens[b];
   const int first_key = (window > 0 && ctx > window) ? ctx - window : 0;
   // slices of 16 keys: those that hold kept first tokens in front of the window, then [first_key, ctx); the CTA's share of that list
   const int kept = min(keep_first, first_key);  // keys [0, kept) are visible beside the window
   const int sl_lo = first_key / 16, sl_hi = (ctx + 15) / 16;
-  const int sl_kept = EXT ? min((kept + 15) / 16, sl_lo) : 0, sl_skip = sl_lo - sl_kept;  // list position i is slice i or, behind the kept ones, i + sl_skip
+  const int sl_kept = EXT == 1 ? min((kept + 15) / 16, sl_lo) : 0, sl_skip = sl_lo - sl_kept;  // list position i is slice i or, behind the kept ones, i + sl_skip
   const int per = (sl_hi - sl_skip + splits - 1) / splits;
   const int s0 = sp * per, s1 = min(sl_hi - sl_skip, s0 + per);
   uint8_t* ring = msm + warp * L::kWarpBytes;
@@ -443,7 +453,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     __syncthreads();
   }
 
-  auto slice_at = [&](int i) { return EXT && i < sl_kept ? i : i + sl_skip; };
+  auto slice_at = [&](int i) { return EXT == 1 && i < sl_kept ? i : i + sl_skip; };
   auto load_slice = [&](int i, int stage) {
     // 16 keys x D of K and V: 2 * 16 * CPR chunks over 32 lanes (zeros behind the real widths)
     const int key0 = slice_at(i) * 16;
@@ -456,7 +466,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
       const int c = i * 32 + lane;
       const int r = c / CPR, cc = c % CPR;
       const bool valid = key0 + r < ctx;
-      if constexpr (EXT) {
+      if constexpr (EXT == 1) {
         const bool vk = valid && cc * 8 < dk, vv = valid && cc * 8 < dv;
         cp_async16(kdst + swz<D>(r, cc), kb + (vk ? r * dk + cc * 8 : 0), vk);
         cp_async16(vdst + swz<D>(r, cc), vb + (vv ? r * dv + cc * 8 : 0), vv);
@@ -513,7 +523,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + 2 * t4 + (e & 1);
         float v = softcap_apply(sc[nt][e] * scale, softcap);
-        v = (key < ctx && (key >= first_key || (EXT && key < kept))) ? v : -INFINITY;
+        v = (key < ctx && (key >= first_key || (EXT == 1 && key < kept))) ? v : -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -609,9 +619,17 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     }
     const int h = h0 + r;
     if (splits == 1) {
-      if (sink) den += __expf(-m);  // the sink's score of 0, relative to the maximum
+      if (EXT != 0 && x.sink != nullptr) den += __expf(x.sink[h] - m);  // relative to the maximum
       const float inv = den > 0.f ? 1.f / den : 0.f;
-      *reinterpret_cast<uint32_t*>(out + (static_cast<long long>(b) * H + h) * dv + d) = pack_bf162(n0 * inv, n1 * inv);
+      if constexpr (EXT != 0) {
+        const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(x.gate);
+        n0 *= attn_gate(x, gate, b, h, h * dv + d);
+        n1 *= attn_gate(x, gate, b, h, h * dv + d + 1);
+        const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * dv;
+        *reinterpret_cast<uint32_t*>(out + b * pitch + h * dv + d) = pack_bf162(n0 * inv, n1 * inv);
+      } else {
+        *reinterpret_cast<uint32_t*>(out + (static_cast<long long>(b) * H + h) * dv + d) = pack_bf162(n0 * inv, n1 * inv);
+      }
     } else {
       const long long base = (static_cast<long long>(b) * H + h) * splits + sp;
       *reinterpret_cast<float2*>(part_o + base * dv + d) = make_float2(n0, n1);
@@ -677,7 +695,7 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
   }
 }
 
-template <int D, bool EXT>
+template <int D, int EXT>
 static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                                const int* ctx, void* out, float* po, float* pml, int* arrivals, int B, int H, int KV, int page,
                                float scale, float cap, int window, int splits, cudaStream_t st, int dk = D, int dv = D, AttnExtra x = {}) {
@@ -692,10 +710,10 @@ static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc
   launch_pdl(decode_attn_mma_kernel<D, EXT>, dim3(grid), dim3(128), L::kBytes, st, static_cast<const __nv_bfloat16*>(q), q_stride,
                                                           static_cast<const __nv_bfloat16*>(kc), static_cast<const __nv_bfloat16*>(vc), bt,
                                                           bt_stride, ctx, static_cast<__nv_bfloat16*>(out), po, pml, arrivals, H, KV, page, scale,
-                                                          cap, window, splits, dk, dv, x.keep_first, x.sink);
+                                                          cap, window, splits, dk, dv, x);
   if (splits > 1 && arrivals == nullptr) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3((dv + 31) / 32 * 32), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x.sink);
+    launch_pdl(decode_merge_kernel, dim3(g2), dim3((dv + 31) / 32 * 32), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x);
   }
   return 0;
 }
@@ -708,11 +726,11 @@ int launch_decode_attention_impl(const void* q, long long q_stride, const void* 
   const int G = H / KV;
   if (impl == 0 && G <= 16 && page % 16 == 0 && (q_stride % 2) == 0) {
     switch (D) {
-      case 64: return launch_decode_mma_t<64, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 64: return launch_decode_mma_t<64, 0>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
-      case 128: return launch_decode_mma_t<128, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 128: return launch_decode_mma_t<128, 0>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
-      case 256: return launch_decode_mma_t<256, false>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
+      case 256: return launch_decode_mma_t<256, 0>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, arrivals, B, H, KV, page, scale, cap, window, splits,
                                                 st);
       default: return 1;
     }
@@ -726,8 +744,12 @@ int launch_decode_attention_mma(const void* q, long long q_stride, const void* k
   if (B == 0) return 0;
   const int D = dk > dv ? dk : dv;
   if (dk % 8 != 0 || dv % 8 != 0 || D > 256 || page % 16 != 0 || q_stride % 8 != 0) return 1;
-#define DLV_DEC_MMA(DD) \
-  return launch_decode_mma_t<DD, true>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap, window, splits, st, dk, dv, x)
+  const bool plain = dk == dv && H / KV <= 16 && x.keep_first == 0;  // only the epilogue differs from the plain kernel
+#define DLV_DEC_MMA(DD)                                                                                                                                  \
+  return plain && dk == DD ? launch_decode_mma_t<DD, 2>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap,      \
+                                                        window, splits, st, dk, dv, x)                                                                    \
+                           : launch_decode_mma_t<DD, 1>(q, q_stride, kc, vc, bt, bt_stride, ctx, out, po, pml, nullptr, B, H, KV, page, scale, cap,      \
+                                                        window, splits, st, dk, dv, x)
   if (D <= 64) DLV_DEC_MMA(64);
   if (D <= 128) DLV_DEC_MMA(128);
   DLV_DEC_MMA(256);
@@ -740,16 +762,11 @@ int launch_decode_attention_mma(const void* q, long long q_stride, const void* k
 // The warps take the visible keys (kept first tokens in front of the window, then the window) in turn, each with its own running maximum,
 // sum and value accumulators (shared memory), which are merged at the end. The 32-bit form of the attention layers, and the fallback for
 // heads the tensor-core kernels do not take.
-__device__ __forceinline__ float rows_ld(const float* p) { return *p; }
-__device__ __forceinline__ float rows_ld(const __nv_bfloat16* p) { return bf2f(*p); }
-__device__ __forceinline__ void rows_st(float* p, float v) { *p = v; }
-__device__ __forceinline__ void rows_st(__nv_bfloat16* p, float v) { *p = f2bf(v); }
-
 template <typename TIO>
 __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ q, long long q_stride, const TIO* __restrict__ k_cache,
                                                         const TIO* __restrict__ v_cache, const int* __restrict__ bt, int bt_stride,
                                                         const int* __restrict__ row_seq, const int* __restrict__ positions, TIO* __restrict__ out, int H, int KV,
-                                                        int dk, int dv, int page, float scale, float softcap, int window, int keep_first, int sink) {
+                                                        int dk, int dv, int page, float scale, float softcap, int window, const AttnExtra x) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float rsm[];  // q [dk] | accumulators [4][dv]
@@ -757,23 +774,23 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ 
   const int t = blockIdx.x, h = blockIdx.y, kvh = h / (H / KV);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   float* acc = rsm + dk + warp * dv;
-  for (int d = tid; d < dk; d += 128) rsm[d] = rows_ld(q + t * q_stride + static_cast<long long>(h) * dk + d);
+  for (int d = tid; d < dk; d += 128) rsm[d] = io_ld(q + t * q_stride + static_cast<long long>(h) * dk + d);
   for (int d = lane; d < dv; d += 32) acc[d] = 0.f;
   __syncthreads();
   const int* table = bt + static_cast<long long>(row_seq != nullptr ? row_seq[t] : t) * bt_stride;
   const int ctx = positions[t] + 1;
-  const int first = window > 0 && ctx > window ? ctx - window : 0, kept = min(keep_first, first);
+  const int first = window > 0 && ctx > window ? ctx - window : 0, kept = min(x.keep_first, first);
   float m = -INFINITY, l = 0.f;
   for (int i = warp; i < kept + ctx - first; i += 4) {
     const int key = i < kept ? i : first + i - kept;
     const long long row = (static_cast<long long>(table[key / page]) * KV + kvh) * page + key % page;
     float s = 0.f;
-    for (int d = lane; d < dk; d += 32) s += rsm[d] * rows_ld(k_cache + row * dk + d);
+    for (int d = lane; d < dk; d += 32) s += rsm[d] * io_ld(k_cache + row * dk + d);
     s = softcap_apply(warp_sum(s) * scale, softcap);
     const float m_new = fmaxf(m, s), alpha = expf(m - m_new), pr = expf(s - m_new);
     m = m_new;
     l = l * alpha + pr;
-    for (int d = lane; d < dv; d += 32) acc[d] = acc[d] * alpha + pr * rows_ld(v_cache + row * dv + d);
+    for (int d = lane; d < dv; d += 32) acc[d] = acc[d] * alpha + pr * io_ld(v_cache + row * dv + d);
   }
   if (lane == 0) {
     ml[warp][0] = m;
@@ -781,17 +798,19 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ 
   }
   __syncthreads();
   m = fmaxf(fmaxf(ml[0][0], ml[1][0]), fmaxf(ml[2][0], ml[3][0]));
-  if (sink) m = fmaxf(m, 0.f);
-  float w[4], den = sink ? expf(-m) : 0.f;
+  if (x.sink != nullptr) m = fmaxf(m, x.sink[h]);
+  float w[4], den = x.sink != nullptr ? expf(x.sink[h] - m) : 0.f;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     w[i] = ml[i][0] == -INFINITY ? 0.f : expf(ml[i][0] - m);
     den += w[i] * ml[i][1];
   }
   const float inv = den > 0.f ? 1.f / den : 0.f;
+  const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * dv;
   for (int d = tid; d < dv; d += 128) {
     const float* a = rsm + dk + d;
-    rows_st(out + (static_cast<long long>(t) * H + h) * dv + d, (w[0] * a[0] + w[1] * a[dv] + w[2] * a[2 * dv] + w[3] * a[3 * dv]) * inv);
+    const float v = (w[0] * a[0] + w[1] * a[dv] + w[2] * a[2 * dv] + w[3] * a[3 * dv]) * inv;
+    io_st(out + t * pitch + h * dv + d, v * attn_gate(x, static_cast<const TIO*>(x.gate), t, h, h * dv + d));
   }
 }
 
@@ -803,8 +822,7 @@ int launch_attention_rows(const void* q, long long q_stride, const void* kc, con
   if (smem > 48 * 1024 - 256) return 1;
 #define DLV_ROWS(TT)                                                                                                                                     \
   launch_pdl(attn_rows_kernel<TT>, dim3(T, H), dim3(128), smem, st, static_cast<const TT*>(q), q_stride, static_cast<const TT*>(kc),                      \
-             static_cast<const TT*>(vc), bt, bt_stride, row_seq, positions, static_cast<TT*>(out), H, KV, dk, dv, page, scale, cap, window, x.keep_first, \
-             x.sink)
+             static_cast<const TT*>(vc), bt, bt_stride, row_seq, positions, static_cast<TT*>(out), H, KV, dk, dv, page, scale, cap, window, x)
   if (is_f32) DLV_ROWS(float);
   else DLV_ROWS(__nv_bfloat16);
 #undef DLV_ROWS

@@ -26,7 +26,8 @@
 //   paged   q [T, H * dk], K and V rows in the paged cache, GQA groups; the real widths dk and dv may be smaller than DK and DV (multiples
 //           of 8): tensor-map bounds fill the columns behind a cache row with zeros, and query columns that reach into the next head meet
 //           zeros. The first `keep_first` keys stay visible beside a sliding window (their key tiles are listed in front of the window's),
-//           and `sink` adds a score of 0 without a value to the softmax;
+//           `sink` adds a score per head without a value to the softmax, the epilogue may multiply with a sigmoid output gate per column or
+//           per head and a constant;
 //   latent  keys and values expanded from the latent cache into flat rows (latent.cu): per head kn columns of an unrotated key part, one
 //           rotated key part shared by all heads (its own tensor map: it is copied behind the head's columns of every K tile, never
 //           materialised per head), DV columns of value. Key 0 of a sequence is its row kv_row0 of those buffers. The epilogue multiplies
@@ -58,15 +59,18 @@ struct AttnTcParams {
   int H, KV, page_size;
   float scale, softcap;
   int window, causal;
-  int keep_first, sink;
+  int keep_first;
+  const float* sink;           // [H] (nullptr: none)
   int dk;                      // query columns per head in q (paged layout: also the width of a K row)
   int* status;
-  int dv, out_pitch;           // real value columns per head, row pitch of out
-  // latent layout only
-  const int* kv_row0;          // [sequences] row of key 0 in the expanded buffers
-  int kn_blocks;               // 64-column blocks of the per-head key part (the blocks behind it come from the shared part)
-  const __nv_bfloat16* gate;   // gate logits [T, gate_pitch], head h at column h * dv (nullptr: no gate)
-  int gate_pitch;
+  int dv;                      // real value columns per head
+  long long out_pitch;         // row pitch of out
+  const int* kv_row0;          // latent layout: [sequences] row of key 0 in the expanded buffers
+  int kn_blocks;               // latent layout: 64-column blocks of the per-head key part (the blocks behind it come from the shared part)
+  const __nv_bfloat16* gate;   // gate logits [T, gate_pitch], head h at column h * dv, or one per head at column h (nullptr: no gate)
+  long long gate_pitch;
+  int gate_heads;
+  float out_mult;
 };
 
 // MN-major shared-memory descriptor (128-byte swizzle): the operand tile is stored as rows of the K dimension, each row 64 elements of
@@ -123,6 +127,18 @@ struct AttnTcSmem {
   static_assert(kStages >= 2 && DK % 64 == 0 && DV % 64 == 0, "attention tile does not fit");
   static_assert(256 + QT * DV <= 512, "score slots and accumulators exceed tensor memory");
 };
+
+// eight columns times the sigmoid of their gate logits
+__device__ __forceinline__ void gate8(float* w, const __nv_bfloat16* g) {
+  const uint4 gv = *reinterpret_cast<const uint4*>(g);
+  const uint32_t* gu = reinterpret_cast<const uint32_t*>(&gv);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 g2 = unpack_bf162(gu[e]);
+    w[2 * e] /= 1.f + __expf(-g2.x);
+    w[2 * e + 1] /= 1.f + __expf(-g2.y);
+  }
+}
 
 __device__ __forceinline__ float ex2_approx(float x) {
   float y;
@@ -509,11 +525,12 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     ok = __all_sync(0xffffffffu, ok && *abort_flag == 0);
     if (ok) {
       tc_fence_after();
-      if (p.sink) l_run += ex2_approx(-m_run * kf);  // the sink's score of 0, relative to the running maximum
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (p.sink != nullptr) l_run += ex2_approx(p.sink[h] * c_log2 - m_run * kf);  // relative to the running maximum
+      float inv = l_run > 0.f ? p.out_mult / l_run : 0.f;
       const size_t trow = static_cast<size_t>(qs + q0 + q * kAtBM + r);
       __nv_bfloat16* orow = p.out + trow * p.out_pitch + static_cast<size_t>(h) * p.dv;
-      const __nv_bfloat16* grow = LATENT && p.gate != nullptr ? p.gate + trow * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
+      const __nv_bfloat16* grow = p.gate != nullptr && !p.gate_heads ? p.gate + trow * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
+      if (!LATENT && p.gate_heads && r < my_rows) inv /= 1.f + __expf(-bf2f(p.gate[trow * p.gate_pitch + h]));
 #pragma unroll 1
       for (int c0 = 0; c0 < DV; c0 += 32) {
         uint32_t v[32];
@@ -534,16 +551,7 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
 #pragma unroll
               for (int e = 0; e < 8; ++e) w[e] = __uint_as_float(v[i + e]) * inv;
               if (vec) {
-                if (grow != nullptr) {
-                  const uint4 gv = *reinterpret_cast<const uint4*>(grow + c0 + i);
-                  const uint32_t* gu = reinterpret_cast<const uint32_t*>(&gv);
-#pragma unroll
-                  for (int e = 0; e < 4; ++e) {
-                    const float2 g2 = unpack_bf162(gu[e]);
-                    w[2 * e] /= 1.f + __expf(-g2.x);
-                    w[2 * e + 1] /= 1.f + __expf(-g2.y);
-                  }
-                }
+                if (grow != nullptr) gate8(w, grow + c0 + i);
                 *reinterpret_cast<uint4*>(orow + c0 + i) =
                     make_uint4(pack_bf162(w[0], w[1]), pack_bf162(w[2], w[3]), pack_bf162(w[4], w[5]), pack_bf162(w[6], w[7]));
               } else {
@@ -557,12 +565,11 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             if (c0 + i >= p.dv) break;
-            uint4 o;
-            o.x = pack_bf162(__uint_as_float(v[i]) * inv, __uint_as_float(v[i + 1]) * inv);
-            o.y = pack_bf162(__uint_as_float(v[i + 2]) * inv, __uint_as_float(v[i + 3]) * inv);
-            o.z = pack_bf162(__uint_as_float(v[i + 4]) * inv, __uint_as_float(v[i + 5]) * inv);
-            o.w = pack_bf162(__uint_as_float(v[i + 6]) * inv, __uint_as_float(v[i + 7]) * inv);
-            *reinterpret_cast<uint4*>(orow + c0 + i) = o;
+            float w[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) w[e] = __uint_as_float(v[i + e]) * inv;
+            if (grow != nullptr) gate8(w, grow + c0 + i);
+            *reinterpret_cast<uint4*>(orow + c0 + i) = make_uint4(pack_bf162(w[0], w[1]), pack_bf162(w[2], w[3]), pack_bf162(w[4], w[5]), pack_bf162(w[6], w[7]));
           }
         }
       }
@@ -600,7 +607,7 @@ static int launch_prefill_tc_maps(const CUtensorMap& mq, const CUtensorMap& mk, 
   return 0;
 }
 
-template <int D, int QT>
+template <int DK, int DV, int QT>
 static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
                                int num_tiles, cudaStream_t st) {
   CUtensorMap mq, mk, mv;
@@ -608,7 +615,7 @@ static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, c
   const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
   encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), p.dk, static_cast<uint64_t>(p.dk) * 2, box_rows, 64, 128);
   encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), p.dv, static_cast<uint64_t>(p.dv) * 2, box_rows, 64, 128);
-  return launch_prefill_tc_maps<D, D, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
+  return launch_prefill_tc_maps<DK, DV, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
 }
 
 // ---- latent layout -----------------------------------------------------------------------------------------------------
@@ -647,6 +654,7 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
   p.out_pitch = a.out_pitch;
   p.gate = static_cast<const __nv_bfloat16*>(a.gate);
   p.gate_pitch = a.gate_pitch;
+  p.out_mult = 1.f;
   CUtensorMap mq, mk, mv, mr;
   const uint64_t H = static_cast<uint64_t>(a.H), rows = static_cast<uint64_t>(a.kv_rows);
   encode_map_2d(&mq, 0, a.q, static_cast<uint64_t>(a.T), H * a.dk, static_cast<uint64_t>(a.q_pitch) * 2, kAtBM, 64, 128);
@@ -695,14 +703,19 @@ int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, 
   p.causal = causal;
   p.keep_first = window > 0 ? x.keep_first : 0;
   p.sink = x.sink;
+  p.gate = static_cast<const __nv_bfloat16*>(x.gate);
+  p.gate_pitch = x.gate_pitch;
+  p.gate_heads = x.gate_heads;
+  p.out_mult = x.out_mult;
   p.dk = dk;
   p.dv = dv;
-  p.out_pitch = H * dv;
+  p.out_pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * dv;
   p.status = status;
   const long long cache_rows = num_pages * KV * page;
-  if (D <= 64) return launch_prefill_tc_t<64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-  if (D <= 128) return launch_prefill_tc_t<128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-  return launch_prefill_tc_t<256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (D <= 64) return launch_prefill_tc_t<64, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (D <= 128 && dv <= 64) return launch_prefill_tc_t<128, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (D <= 128) return launch_prefill_tc_t<128, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  return launch_prefill_tc_t<256, 256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
 }
 
 }  // namespace dlv

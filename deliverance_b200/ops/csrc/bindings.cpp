@@ -719,8 +719,39 @@ int* split_arrival_counters(int device, int64_t needed) {
   return it->second.data_ptr<int>();
 }
 
+// Options of the attention kernels behind the mask: sink fp32 [H], gate logits [rows, H] (one per head) or [rows, H * dv] of q's type, a given output
+dlv::AttnExtra attn_extra(const Tensor& q, int64_t keep_first, const c10::optional<Tensor>& sink, const c10::optional<Tensor>& gate, double out_mult,
+                          const c10::optional<Tensor>& out, int64_t rows, int64_t H, int64_t dv) {
+  TORCH_CHECK(keep_first >= 0, "keep_first must not be negative");
+  dlv::AttnExtra x;
+  x.keep_first = static_cast<int>(keep_first);
+  x.out_mult = static_cast<float>(out_mult);
+  if (sink.has_value()) {
+    check_cuda(sink.value(), "sink");
+    TORCH_CHECK(sink.value().scalar_type() == at::kFloat && sink.value().numel() == H, "sink must be fp32 [heads]");
+    x.sink = sink.value().data_ptr<float>();
+  }
+  if (gate.has_value()) {
+    const Tensor& g = gate.value();
+    x.gate_heads = g.size(1) == H ? 1 : 0;
+    TORCH_CHECK(g.device() == q.device() && g.scalar_type() == q.scalar_type() && g.dim() == 2 && g.size(0) == rows && (g.size(1) == H || g.size(1) == H * dv) &&
+                    g.stride(1) == 1, "gate must be [rows, heads] or [rows, heads * value width] of the activations' type");
+    TORCH_CHECK(x.gate_heads || (g.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(g.data_ptr()) & 15) == 0), "gate rows must be 16-byte aligned");
+    x.gate = g.data_ptr();
+    x.gate_pitch = g.stride(0);
+  }
+  if (out.has_value()) {
+    const Tensor& o = out.value();
+    TORCH_CHECK(o.device() == q.device() && o.scalar_type() == q.scalar_type() && o.dim() == 2 && o.size(0) == rows && o.size(1) == H * dv && o.stride(1) == 1 &&
+                    o.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(o.data_ptr()) & 15) == 0, "out must be [rows, heads * value width] with 16-byte aligned rows");
+    x.out_pitch = o.stride(0);
+  }
+  return x;
+}
+
 Tensor decode_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& ctx_lens,
-                        int64_t H, double scale, double softcap, int64_t window, int64_t splits, int64_t impl, int64_t keep_first, bool sink) {
+                        int64_t H, double scale, double softcap, int64_t window, int64_t splits, int64_t impl, int64_t keep_first, c10::optional<Tensor> sink,
+                        c10::optional<Tensor> gate, double out_mult, c10::optional<Tensor> out_opt) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [B, H*D]");
   check_bf16(k_cache, "k_cache");
   check_bf16(v_cache, "v_cache");
@@ -732,11 +763,11 @@ Tensor decode_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_
   const int DV = static_cast<int>(v_cache.size(3));
   TORCH_CHECK(q.size(1) == H * D && H % KV == 0 && page % 32 == 0, "shape mismatch (page size must be a multiple of 32)");
   TORCH_CHECK(v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == KV && v_cache.size(2) == page, "k/v cache shape mismatch");
-  TORCH_CHECK(keep_first >= 0, "keep_first must not be negative");
   TORCH_CHECK(block_tables.dim() == 2 && block_tables.size(0) >= B && ctx_lens.numel() >= B, "bad table shapes");
   TORCH_CHECK((reinterpret_cast<uintptr_t>(q.data_ptr()) & 3) == 0, "q misaligned");
   c10::cuda::CUDAGuard guard(q.device());
-  Tensor out = new_out({B, H * DV}, q.options());
+  const dlv::AttnExtra x = attn_extra(q, keep_first, sink, gate, out_mult, out_opt, B, H, DV);
+  Tensor out = out_opt.has_value() ? out_opt.value() : new_out({B, H * DV}, q.options());
   if (splits < 1) splits = 1;
   Tensor po, pml;
   float *pop = nullptr, *pmlp = nullptr;
@@ -746,9 +777,8 @@ Tensor decode_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_
     pop = po.data_ptr<float>();
     pmlp = pml.data_ptr<float>();
   }
-  if (keep_first > 0 || sink || DV != D || (impl == 0 && (H / KV > 16 || (D != 64 && D != 128 && D != 256)))) {
-    TORCH_CHECK(impl == 0, "kept first keys, a sink and unequal widths are available in the tensor-core kernel only");
-    const dlv::AttnExtra x = {static_cast<int>(keep_first), sink ? 1 : 0};
+  if (keep_first > 0 || sink.has_value() || gate.has_value() || out_mult != 1.0 || out_opt.has_value() || DV != D || (impl == 0 && (H / KV > 16 || (D != 64 && D != 128 && D != 256)))) {
+    TORCH_CHECK(impl == 0, "kept first keys, a sink, an output gate and unequal widths are available in the tensor-core kernel only");
     const int rc = dlv::launch_decode_attention_mma(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr<int>(),
                                                     static_cast<int>(block_tables.stride(0)), ctx_lens.data_ptr<int>(), out.data_ptr(), pop, pmlp, B,
                                                     static_cast<int>(H), KV, D, DV, page, static_cast<float>(scale), static_cast<float>(softcap),
@@ -798,7 +828,8 @@ Tensor prefill_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v
 // Same contract as prefill_attention, on the tcgen05 / TMA kernel; tile arrays cover prefill_tc_tile_rows(head_dim) query rows per tile.
 Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& q_start,
                             const Tensor& q_len, const Tensor& ctx_lens, const Tensor& tile_seq, const Tensor& tile_q0, int64_t H, double scale,
-                            double softcap, int64_t window, bool causal, int64_t keep_first, bool sink) {
+                            double softcap, int64_t window, bool causal, int64_t keep_first, c10::optional<Tensor> sink, c10::optional<Tensor> gate,
+                            double out_mult, c10::optional<Tensor> out_opt) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [T, H*D]");
   TORCH_CHECK(q.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0, "q rows must be 16-byte aligned");
   check_bf16(k_cache, "k_cache");
@@ -814,12 +845,11 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
                   q.size(1) == H * D && H % KV == 0, "shape mismatch");
   TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && D <= 256 && DV % 8 == 0 && DV <= 256,
               "page size 32 / 64 / 128 and head widths that are multiples of 8 up to 256");
-  TORCH_CHECK(keep_first >= 0, "keep_first must not be negative");
   TORCH_CHECK(tile_seq.numel() == tile_q0.numel(), "tile arrays differ in length");
   c10::cuda::CUDAGuard guard(q.device());
-  Tensor out = new_out({T, H * DV}, q.options());
+  const dlv::AttnExtra x = attn_extra(q, keep_first, sink, gate, out_mult, out_opt, T, H, DV);
+  Tensor out = out_opt.has_value() ? out_opt.value() : new_out({T, H * DV}, q.options());
   DeviceScratch& s = scratch_for(q.device().index());
-  const dlv::AttnExtra x = {static_cast<int>(keep_first), sink ? 1 : 0};
   int rc = dlv::launch_prefill_attention_tc(q.data_ptr(), q.stride(0), T, k_cache.data_ptr(), v_cache.data_ptr(), k_cache.size(0), block_tables.data_ptr<int>(),
                                             static_cast<int>(block_tables.stride(0)), q_start.data_ptr<int>(), q_len.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                             tile_seq.data_ptr<int>(), tile_q0.data_ptr<int>(), static_cast<int>(tile_seq.numel()), out.data_ptr(),
@@ -832,6 +862,7 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
 
 #include "bindings_latent.inc"
 #include "bindings_gla.inc"
+#include "bindings_streams.inc"
 
 // ---- sampling ---------------------------------------------------------------------------------------------------------
 std::vector<Tensor> argmax(const Tensor& logits, c10::optional<Tensor> mask, double softcap, double inv_scale) {
@@ -1099,7 +1130,23 @@ py::bytes lz4_decompress_bytes(const std::string& comp, int64_t n_out) {
 // ---- MoE --------------------------------------------------------------------------------------------------------------
 // returns weights [T, k] f32, expert ids [T, k] i32, counts [E], offsets [E+1], perm [T*k], pos [T*k]
 bool g_moe_parallel_sort = true;  // (comparisons: false keeps the single-CTA grouping for every batch size)
-std::vector<Tensor> moe_route(const Tensor& logits, int64_t k, int64_t mode, bool renorm) {
+dlv::MoeRouting moe_routing(int64_t E, int64_t mode, bool renorm, const c10::optional<Tensor>& correction, int64_t groups, int64_t keep, double scale) {
+  dlv::MoeRouting r;
+  TORCH_CHECK(mode >= 0 && mode <= 2, "unknown routing mode");
+  TORCH_CHECK(groups >= 1 && groups <= dlv::kMoeMaxGroups && E % groups == 0 && keep >= 1 && keep <= groups, "bad expert groups (at most ", dlv::kMoeMaxGroups, ")");
+  r.mode = static_cast<int>(mode);
+  r.renorm = renorm ? 1 : 0;
+  r.groups = static_cast<int>(groups);
+  r.keep = static_cast<int>(keep);
+  r.scale = static_cast<float>(scale);
+  if (correction.has_value()) {
+    check_f32(correction.value(), E, "correction");
+    r.correction = correction.value().data_ptr<float>();
+  }
+  return r;
+}
+std::vector<Tensor> moe_route(const Tensor& logits, int64_t k, int64_t mode, bool renorm, c10::optional<Tensor> correction, int64_t groups, int64_t keep,
+                              double scale) {
   TORCH_CHECK(logits.is_cuda() && logits.scalar_type() == at::kFloat && logits.dim() == 2 && logits.is_contiguous(), "router logits must be fp32 [T, E]");
   const int T = static_cast<int>(logits.size(0)), E = static_cast<int>(logits.size(1));
   TORCH_CHECK(k >= 1 && k <= 16 && k <= E && E <= 1024, "unsupported top-k / expert count");
@@ -1110,7 +1157,7 @@ std::vector<Tensor> moe_route(const Tensor& logits, int64_t k, int64_t mode, boo
   Tensor ws;  // per-chunk expert histograms of the parallel grouping (prefill-size batches)
   const size_t ws_ints = g_moe_parallel_sort ? dlv::moe_route_workspace_ints(T, E, static_cast<int>(k)) : 0;
   if (ws_ints > 0) ws = new_out({static_cast<int64_t>(ws_ints)}, io);
-  dlv::launch_moe_route(logits.data_ptr<float>(), T, E, static_cast<int>(k), static_cast<int>(mode), renorm ? 1 : 0, w.data_ptr<float>(),
+  dlv::launch_moe_route(logits.data_ptr<float>(), T, E, static_cast<int>(k), moe_routing(E, mode, renorm, correction, groups, keep, scale), w.data_ptr<float>(),
                         idx.data_ptr<int>(), counts.data_ptr<int>(), offsets.data_ptr<int>(), perm.data_ptr<int>(), pos.data_ptr<int>(),
                         ws_ints > 0 ? ws.data_ptr<int>() : nullptr, cur_stream());
   check_last_error("moe_route");
@@ -1118,7 +1165,8 @@ std::vector<Tensor> moe_route(const Tensor& logits, int64_t k, int64_t mode, boo
 }
 // moe_route and moe_items of a decode-size batch in one launch: {w, idx, counts, offsets, perm, pos, items}; an empty vector when the
 // batch is too large for the single-CTA kernel (the caller then uses the two functions).
-std::vector<Tensor> moe_route_items(const Tensor& logits, int64_t k, int64_t mode, bool renorm, int64_t e0, int64_t ne, int64_t bn, int64_t max_items) {
+std::vector<Tensor> moe_route_items(const Tensor& logits, int64_t k, int64_t mode, bool renorm, int64_t e0, int64_t ne, int64_t bn, int64_t max_items,
+                                    c10::optional<Tensor> correction, int64_t groups, int64_t keep, double scale) {
   TORCH_CHECK(logits.is_cuda() && logits.scalar_type() == at::kFloat && logits.dim() == 2 && logits.is_contiguous(), "router logits must be fp32 [T, E]");
   const int T = static_cast<int>(logits.size(0)), E = static_cast<int>(logits.size(1));
   TORCH_CHECK(k >= 1 && k <= 16 && k <= E && E <= 1024, "unsupported top-k / expert count");
@@ -1128,7 +1176,7 @@ std::vector<Tensor> moe_route_items(const Tensor& logits, int64_t k, int64_t mod
   auto io = logits.options().dtype(at::kInt);
   Tensor w = new_out({T, k}, logits.options()), idx = new_out({T, k}, io), counts = new_out({E}, io);
   Tensor offsets = new_out({E + 1}, io), perm = new_out({T * k}, io), pos = new_out({T * k}, io), items = new_out({max_items, 4}, io);
-  const bool ok = dlv::launch_moe_route_small(logits.data_ptr<float>(), T, E, static_cast<int>(k), static_cast<int>(mode), renorm ? 1 : 0,
+  const bool ok = dlv::launch_moe_route_small(logits.data_ptr<float>(), T, E, static_cast<int>(k), moe_routing(E, mode, renorm, correction, groups, keep, scale),
                                               w.data_ptr<float>(), idx.data_ptr<int>(), counts.data_ptr<int>(), offsets.data_ptr<int>(),
                                               perm.data_ptr<int>(), pos.data_ptr<int>(), static_cast<int>(e0), static_cast<int>(ne),
                                               static_cast<int>(bn), static_cast<int>(max_items), items.data_ptr<int>(), cur_stream());
@@ -1542,12 +1590,18 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rope_kv", &rope_kv);
   m.def("decode_attention", &decode_attention, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("ctx_lens"),
         py::arg("H"), py::arg("scale"), py::arg("softcap") = 0.0, py::arg("window") = 0, py::arg("splits") = 1, py::arg("impl") = 0,
-        py::arg("keep_first") = 0, py::arg("sink") = false);
+        py::arg("keep_first") = 0, py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0, py::arg("out") = py::none());
   m.def("prefill_attention", &prefill_attention);
   m.def("prefill_attention_tc", &prefill_attention_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("q_start"),
         py::arg("q_len"), py::arg("ctx_lens"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"),
-        py::arg("causal"), py::arg("keep_first") = 0, py::arg("sink") = false);
-  m.def("attention_rows", &attention_rows);
+        py::arg("causal"), py::arg("keep_first") = 0, py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
+        py::arg("out") = py::none());
+  m.def("attention_rows", &attention_rows, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("row_seq"), py::arg("positions"),
+        py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"), py::arg("keep_first") = 0, py::arg("sink") = py::none(),
+        py::arg("gate") = py::none(), py::arg("out_mult") = 1.0, py::arg("out") = py::none());
+  m.def("rope_heads_kv", &rope_heads_kv);
+  m.def("stream_step", &stream_step);
+  m.def("lightning", &lightning);
   m.def("rope_pairs_kv", &rope_pairs_kv);
   m.def("sandwich_norm", &sandwich_norm);
   m.def("grouped_linear_f32", &grouped_linear_f32);
@@ -1601,10 +1655,12 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("lz4_decompress", &lz4_decompress_bytes);
   m.def("logprob_rows", &logprob_rows);
   m.def("logits_post", &logits_post, py::arg("logits"), py::arg("mask") = py::none(), py::arg("softcap") = 0.0, py::arg("inv_scale") = 1.0);
-  m.def("moe_route", &moe_route);
+  m.def("moe_route", &moe_route, py::arg("logits"), py::arg("k"), py::arg("mode"), py::arg("renorm"), py::arg("correction") = py::none(), py::arg("groups") = 1,
+        py::arg("keep") = 1, py::arg("scale") = 1.0);
   m.def("moe_parallel_sort", [](bool on) { g_moe_parallel_sort = on; });
   m.def("moe_items", &moe_items);
-  m.def("moe_route_items", &moe_route_items);
+  m.def("moe_route_items", &moe_route_items, py::arg("logits"), py::arg("k"), py::arg("mode"), py::arg("renorm"), py::arg("e0"), py::arg("ne"), py::arg("bn"),
+        py::arg("max_items"), py::arg("correction") = py::none(), py::arg("groups") = 1, py::arg("keep") = 1, py::arg("scale") = 1.0);
   m.def("moe_gather", &moe_gather, py::arg("x"), py::arg("perm"), py::arg("k"), py::arg("offsets") = py::none(), py::arg("e0") = 0, py::arg("ne") = 0);
   m.def("moe_combine", &moe_combine, py::arg("ys"), py::arg("pos"), py::arg("w"), py::arg("T"), py::arg("k"), py::arg("offsets") = py::none(),
         py::arg("e0") = 0, py::arg("ne") = 0);

@@ -5,7 +5,8 @@
 // Reference math: core/.../generator/RmsNorm.java:107-121, TransformerBlock.java:265-276, LayerNorm.java:20-151,
 // CausalSelfAttention.java:315-372,429-446, Qwen3CausalSelfAttention.java:74-92, EmbedInput.java:26-44,
 // native/src/main/c/simd/vector_simd.c:185-213 (the fused activation; here the product stays bf16, no int8 requant).
-#include "common.cuh"
+#include "gemm_api.h"
+#include "io.cuh"
 
 namespace dlv {
 
@@ -291,10 +292,6 @@ __global__ void __launch_bounds__(256) rope_kv_kernel(__nv_bfloat16* __restrict_
 // ------------------------------------------------------------------------------------------------ fp32 residual stream
 // Models that keep the residual stream in fp32: embedding with a hashed-bigram table, residual add + one or two LayerNorms of the same
 // row, gated activation with row pitches. TIO: bf16 or fp32 activations.
-__device__ __forceinline__ float io_ld(const __nv_bfloat16* p) { return bf2f(*p); }
-__device__ __forceinline__ float io_ld(const float* p) { return *p; }
-__device__ __forceinline__ void io_st(__nv_bfloat16* p, float v) { *p = f2bf(v); }
-__device__ __forceinline__ void io_st(float* p, float v) { *p = v; }
 
 // out[t] = table[ids[t]] * scale + bigram[row]; row = (prev * mul_prev + id * mul_cur) mod buckets, or `buckets` (the extra last row) when the
 // token has no predecessor (prev < 0); out2 (optional, pitch ld2): the same row in the table's type
@@ -427,23 +424,6 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const TIO* __restrict__ 
 // sub is one row [T, ld_sub] or, with pos, the weighted sum of k rows of an expert-ordered buffer: sum_j wts[t, j] * sub[pos[t, j]], formed
 // in fp32 in slot order. One CTA per row; the row lives in registers (NV groups of four columns per thread), both variances are means of
 // squared deviations.
-template <typename TIO>
-__device__ __forceinline__ void io_ld4(const TIO* p, float* v) {
-  if constexpr (sizeof(TIO) == 2) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    const float2 a = unpack_bf162(u.x), b = unpack_bf162(u.y);
-    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-  } else {
-    const float4 f = *reinterpret_cast<const float4*>(p);
-    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-  }
-}
-template <typename TIO>
-__device__ __forceinline__ void io_st4(TIO* p, const float* v) {
-  if constexpr (sizeof(TIO) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf162(v[0], v[1]), pack_bf162(v[2], v[3]));
-  else *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-
 struct SandwichArgs {
   float* residual;
   const void* sub;
@@ -630,6 +610,107 @@ __global__ void __launch_bounds__(256) rope_pairs_kv_kernel(TIO* __restrict__ qk
   io_st4(dst + 4, x + 4);
 }
 
+// ------------------------------------------------------------------------------------------------ per-head norm, half rotation, KV write
+// Projection rows p: queries at column 0 (H heads of dk columns), keys at off_k (KV heads of dk), values at off_v (KV heads of dv; off_v = off_k
+// when the values are the projected keys). Queries and keys: optional RMS norm over the head (dim real columns), then the pairs
+// (i, i + half), i < half, are rotated; queries in place, keys into the cache. Values go to the cache as projected or, with v_first,
+// blended with another row of the same token: (1 - lam) v + lam v_first.
+// LPH lanes of a warp own one (row, head): eight columns per lane and step, the head passes through shared memory so that the partner of
+// a rotated column is at hand whatever `half` is.
+template <typename TIO, int LPH>
+__global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) float hsm[];
+  const bool tied = a.off_v == a.off_k;
+  const int heads = a.H + a.KV + (tied ? 0 : a.KV);
+  const int sub = threadIdx.x % LPH, grp = threadIdx.x / LPH;
+  const long long idx = static_cast<long long>(blockIdx.x) * (256 / LPH) + grp;
+  const bool active = idx < static_cast<long long>(a.T) * heads;  // (all lanes reach the shuffles and warp barriers below)
+  const int t = active ? static_cast<int>(idx / heads) : 0, h = active ? static_cast<int>(idx % heads) : 0;
+  const bool is_q = h < a.H, is_v = h >= a.H + a.KV;
+  const int kvh = is_q ? 0 : (is_v ? h - a.H - a.KV : h - a.H);
+  TIO* row = static_cast<TIO*>(a.p) + t * a.ld;
+  long long at = 0;  // row of the caches
+  bool store = active;
+  if (!is_q) {
+    const long long slot = a.slots[t];
+    store = active && slot >= 0;
+    if (store) at = ((slot / a.page) * a.KV + kvh) * a.page + slot % a.page;
+  }
+  float* s = hsm + grp * a.dk;
+  const TIO* src = row + (is_q ? h * a.dk : (is_v ? a.off_v + kvh * a.dv : a.off_k + kvh * a.dk));
+  TIO* vdst = static_cast<TIO*>(a.v_cache) + at * a.dv;
+  const float* nw = is_v ? nullptr : (is_q ? a.q_norm : a.k_norm);
+  const int width = is_v ? a.dv : a.dk;
+  float ss = 0.f;
+  for (int c = sub * 8; c < width; c += LPH * 8) {
+    float x[8];
+    io_ld8(src + c, x);
+    if (is_v || (!is_q && tied)) {
+      if (a.v_first != nullptr) {
+        float f[8];
+        io_ld8(static_cast<const TIO*>(a.v_first) + t * a.ld_first + kvh * a.dv + c, f);
+        float y[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = (1.f - a.lam) * x[e] + a.lam * f[e];
+        if (store) io_st8(vdst + c, y);
+      } else if (store) {
+        io_st8(vdst + c, x);
+      }
+    }
+    if (!is_v) {
+      *reinterpret_cast<float4*>(s + c) = make_float4(x[0], x[1], x[2], x[3]);
+      *reinterpret_cast<float4*>(s + c + 4) = make_float4(x[4], x[5], x[6], x[7]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+    }
+  }
+#pragma unroll
+  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  __syncwarp();
+  if (is_v || !store) return;
+  const float inv = nw != nullptr ? rsqrtf(ss / a.dim + a.eps) : 1.f;
+  int pos = a.positions[t];
+  pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+  const float* cs = a.cos_t + static_cast<size_t>(pos) * a.half;
+  const float* sn = a.sin_t + static_cast<size_t>(pos) * a.half;
+  TIO* dst = is_q ? row + h * a.dk : static_cast<TIO*>(a.k_cache) + at * a.dk;
+  const int end = is_q && nw == nullptr ? min(a.dk, (2 * a.half + 7) / 8 * 8) : a.dk;  // queries that nothing changes stay where they are
+  for (int c = sub * 8; c < end; c += LPH * 8) {
+    float y[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int d = c + e;
+      float v = s[d] * inv;
+      if (nw != nullptr) v *= nw[d];
+      if (d < 2 * a.half) {
+        const bool low = d < a.half;
+        const int i = low ? d : d - a.half, o = low ? d + a.half : i;
+        float w = s[o] * inv;
+        if (nw != nullptr) w *= nw[o];
+        v = low ? v * cs[i] - w * sn[i] : v * cs[i] + w * sn[i];
+      }
+      y[e] = v;
+    }
+    io_st8(dst + c, y);
+  }
+}
+
+template <typename TIO>
+static int launch_rope_heads_t(const RopeHeadsArgs& a, cudaStream_t st) {
+  const int chunks = (a.dk > a.dv ? a.dk : a.dv) / 8;
+  const long long n = static_cast<long long>(a.T) * (a.H + (a.off_v == a.off_k ? 1 : 2) * a.KV);
+  auto go = [&](auto kernel, int lph) {
+    const int per = 256 / lph;
+    return launch_pdl(kernel, dim3(static_cast<unsigned>((n + per - 1) / per)), dim3(256), static_cast<size_t>(per) * a.dk * sizeof(float), st, a) == cudaSuccess ? 0 : 2;
+  };
+  if (chunks <= 4) return go(rope_heads_kv_kernel<TIO, 4>, 4);
+  if (chunks <= 8) return go(rope_heads_kv_kernel<TIO, 8>, 8);
+  if (chunks <= 16) return go(rope_heads_kv_kernel<TIO, 16>, 16);
+  return go(rope_heads_kv_kernel<TIO, 32>, 32);
+}
+
 // ------------------------------------------------------------------------------------------------ launchers
 void launch_rmsnorm(const void* x, void* residual, const void* w, void* y, int T, int H, float eps, float offset,
                     float res_mult, cudaStream_t st) {
@@ -721,6 +802,11 @@ void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const l
   else
     launch_pdl(rope_pairs_kv_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<__nv_bfloat16*>(qkv), ld, positions, slots, cos_t, sin_t,
                static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), T, H, KV, dk, dv, page, half, max_pos);
+}
+int launch_rope_heads_kv(const RopeHeadsArgs& a, bool is_f32, cudaStream_t st) {
+  if (a.T == 0) return 0;
+  if (a.dk > 1024 || a.dk % 8 != 0 || a.dv % 8 != 0) return 1;  // (the heads of a block share 48 KB)
+  return is_f32 ? launch_rope_heads_t<float>(a, st) : launch_rope_heads_t<__nv_bfloat16>(a, st);
 }
 int launch_rope_kv(void* qkv, const int* positions, const long long* slots, const void* qn, const void* kn, const float* cos_t,
                    const float* sin_t, void* k_cache, void* v_cache, int T, int H, int KV, int D, int block_size, int rot_half,

@@ -124,10 +124,17 @@ int launch_rope_kv(void* qkv, const int* positions, const long long* slots, cons
                    const float* sin_t, void* k_cache, void* v_cache, int T, int H, int KV, int D, int block_size, int rot_half,
                    float eps, float norm_offset, int max_pos, cudaStream_t st);
 
-// Which keys of the sliding window's past stay visible, and whether a score of 0 without a value takes part in the softmax
+// Options of the attention kernels beyond scale, soft-cap and window: first keys that stay visible beside the window; a score per head
+// that takes part in the softmax without a value; an output gate (out = head * out_mult * sigmoid(gate), one logit per column or one per
+// head, of the activations' type); the row pitch of the output (0: H * dv).
 struct AttnExtra {
   int keep_first = 0;
-  int sink = 0;
+  const float* sink = nullptr;  // [H]
+  const void* gate = nullptr;   // [T, gate_pitch]
+  long long gate_pitch = 0;
+  int gate_heads = 0;  // 1: one logit per head
+  float out_mult = 1.f;
+  long long out_pitch = 0;
 };
 
 // attention.cu
@@ -189,7 +196,17 @@ void launch_logprobs(const float* logits, int ld, int B, int V, const long long*
 
 // moe.cu
 size_t moe_route_workspace_ints(int T, int E, int k);  // ints of `ws` for the parallel grouping of large batches (0: not needed)
-void launch_moe_route(const float* logits, int T, int E, int k, int mode, int renorm, float* w, int* idx, int* counts, int* offsets,
+// How experts are chosen and weighted. mode 0: softmax over all, the largest (renorm: divided by their sum); 1: softmax over the k largest logits;
+// 2: sigmoid scores, the largest of score + correction among the `keep` best of `groups` equal groups of neighbours (a group counts the sum of
+// its two largest choice scores), weights = scores over their sum (+ 1e-20) times scale.
+struct MoeRouting {
+  int mode = 0, renorm = 0;
+  const float* correction = nullptr;  // [E]
+  int groups = 1, keep = 1;
+  float scale = 1.f;
+};
+constexpr int kMoeMaxGroups = 64;
+void launch_moe_route(const float* logits, int T, int E, int k, const MoeRouting& r, float* w, int* idx, int* counts, int* offsets,
                       int* perm, int* pos, int* ws, cudaStream_t st);
 // `range` (optional) = offsets + first local expert and the count of local experts: rows outside
 // [offsets[e0], offsets[e0 + ne]) are skipped (expert parallelism: other ranks own them)
@@ -198,7 +215,7 @@ void launch_moe_gather(const void* x, const int* perm, int rows, int k, int row_
 void launch_moe_combine(const void* ys, const int* pos, const float* w, int T, int k, int H, void* out, const int* offsets, int e0,
                         int ne, cudaStream_t st);
 void launch_moe_items(const int* offsets, int e0, int ne, int bn, int max_items, int* items, cudaStream_t st);
-bool launch_moe_route_small(const float* logits, int T, int E, int k, int mode, int renorm, float* w, int* idx, int* counts, int* offsets,
+bool launch_moe_route_small(const float* logits, int T, int E, int k, const MoeRouting& r, float* w, int* idx, int* counts, int* offsets,
                             int* perm, int* pos, int e0, int ne, int bn, int max_items, int* items, cudaStream_t st);
 
 // comm.cu: fused compute + collective kernels over peer memory (same protocol as the GEMM all-reduce epilogue)
@@ -317,6 +334,78 @@ void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bo
                           cudaStream_t st);
 void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const long long* slots, const float* cos_t, const float* sin_t, void* k_cache,
                           void* v_cache, int T, int H, int KV, int dk, int dv, int page, int half, int max_pos, bool is_f32, cudaStream_t st);
+
+// elementwise.cu: per-head norm, half rotation and cache write of projection rows p [T, ld] (columns: queries 0, keys off_k, values off_v)
+struct RopeHeadsArgs {
+  void* p;
+  long long ld;
+  int off_k, off_v;  // off_v == off_k: the values are the projected keys
+  const int* positions;
+  const long long* slots;
+  const float *cos_t, *sin_t;  // [max_pos, half]
+  void *k_cache, *v_cache;
+  int T, H, KV, dk, dv, dim, page, half, max_pos;  // dim: real columns of a head (the norm's divisor)
+  const float *q_norm, *k_norm;                    // [dk] or nullptr
+  float eps;
+  const void* v_first;  // values to blend with, row pitch ld_first (nullptr: none)
+  long long ld_first;
+  float lam;
+};
+int launch_rope_heads_kv(const RopeHeadsArgs& a, bool is_f32, cudaStream_t st);
+
+// streams.cu: several residual streams per token
+constexpr int kMaxStreams = 16;
+struct StreamArgs {
+  float* streams;  // [T, S, W]
+  int S, W;
+  const int* ids;  // given: the streams start from rows of sub = the embedding table [vocab, ld_sub], normed with w_open
+  int vocab;
+  const float* w_open;
+  const void* sub;  // output of the sublayer, rows of ld_sub (nullptr: nothing to write back)
+  long long ld_sub;
+  const int* pos;  // [T, k] rows of an expert-ordered sub, with weights wts [T, k]
+  const float* wts;
+  int k;
+  const float *mix, *write;  // [S, S] (from, to), [S]
+  int keep;                  // the streams are read again
+  const float* read;         // [S] (nullptr: ones)
+  const float* w_next;       // [W] (nullptr: no norm)
+  void* y;
+  long long ld_y;
+  int y_width;
+  float eps;
+  int vec;  // rows, pitches and pointers allow four-column accesses
+};
+int launch_stream_step(const StreamArgs& a, int rows, bool is_f32, cudaStream_t st);
+
+// lightning.cu: linear attention with one constant decay per head. Projection rows p [T, ld] = q (H dk) | k (H dk) | v (H dv) | g (H dv) at the given
+// first columns, widths multiples of 8
+struct LightningArgs {
+  const void* p;
+  long long ld;
+  int H, dk, dv, off_k, off_v, off_g;
+  const float* powers;  // [H, chunk + 2]: decay^0 .. decay^chunk, then what fp32 loses of decay^1
+  int chunk;
+  float* state;  // [slots, H, dk, dv]
+  const long long* slots;
+  const int *q_start, *q_len, *positions;
+  int num_seqs, rows;
+  float* o;  // fp32 [T, H dv]
+  // norm and gate
+  const float* norm_w;  // [H dv]
+  int real;             // real columns of all heads (the norm's divisor)
+  float eps, mult;
+  void* out;
+  long long ld_out;
+};
+struct LightningChunks {
+  const int *seq, *row0, *len;  // per chunk
+  const int *first, *count;     // per sequence
+  int n_chunks;
+  float* states;  // [n_chunks, H, dk, dv]: what each chunk adds, then the state in front of it
+};
+int launch_lightning_recurrent(const LightningArgs& a, bool is_f32, cudaStream_t st);
+int launch_lightning_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st);
 
 // gla.cu: gated linear attention. Projection rows p [T, ld] = q (H dk) | k (H dk) | v (H dv) | g (H dv) | a (rank), widths multiples of 8
 struct GlaArgs {

@@ -1,6 +1,6 @@
 // Mixture-of-experts routing and token shuffling.
 //   moe_route:   router logits [T, E] fp32 -> top-k weights / expert ids per token (softmax-all -> top-k -> optional
-//                renormalise, or top-k -> softmax over the k), per-expert histogram, exclusive offsets and the permutation
+//                renormalise, or top-k -> softmax over the k, or sigmoid scores with correction and group limits), per-expert histogram, exclusive offsets and the permutation
 //                that groups (token, slot) pairs by expert — one kernel launch + one small scan kernel.
 //   moe_gather:  x [T, H] -> xs [T*k, H] rows in expert-grouped order (any element type).
 //   moe_combine: ys [T*k, H] (expert outputs in grouped order) -> out [T, H] = sum_j w[t, j] * ys[pos(t, j)]  (fp32 sum in
@@ -8,6 +8,7 @@
 // Reference semantics: core/.../model/MixtureOfExpertsBlock.java:78-112, qwen3/Qwen3MoeFeedForward.java:107-301,
 // granitemoehybrid/GraniteMoeHybridMoeFeedForward.java:112-141.
 #include "common.cuh"
+#include "gemm_api.h"
 
 namespace dlv {
 
@@ -15,16 +16,76 @@ constexpr int kMaxTopK = 16;
 
 // Top-k of one token by one warp (E <= 1024): softmax statistics, k rounds of "every lane proposes its best remaining expert"
 // (ties -> lower index), weights by `mode` (0: softmax over all experts, then top-k, optional renormalisation; 1: softmax over
-// the k chosen). Lane 0 stores weights and expert ids, adds to the histogram `counts` (global or shared memory) and, when
+// the k chosen; 2: sigmoid scores with a correction and group limits, see MoeRouting). Lane 0 stores weights and expert ids, adds to the histogram `counts` (global or shared memory) and, when
 // `idx_copy` is given, keeps a second copy of the ids there.
-__device__ __forceinline__ void moe_topk_token(const float* __restrict__ row, int E, int k, int mode, int renorm, int lane,
+// best (value, index) of the warp, lower index on ties
+__device__ __forceinline__ void warp_best(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (ov > v || (ov == v && oi < i)) {
+      v = ov;
+      i = oi;
+    }
+  }
+}
+__device__ __forceinline__ float route_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Groups (bit g) whose experts may be chosen: the `keep` groups with the largest sums of their two best choice scores.
+__device__ __forceinline__ unsigned long long moe_kept_groups(const float* __restrict__ row, int E, const MoeRouting& r, int lane) {
+  if (r.groups <= 1 || r.keep >= r.groups) return ~0ull;
+  const int size = E / r.groups;
+  float score[kMoeMaxGroups / 32];
+#pragma unroll
+  for (int j = 0; j < kMoeMaxGroups / 32; ++j) {
+    const int g = lane + 32 * j;
+    score[j] = -INFINITY;
+    if (g >= r.groups) continue;
+    float a = -INFINITY, b = -INFINITY;  // the two best
+    for (int e = g * size; e < (g + 1) * size; ++e) {
+      const float v = route_sigmoid(row[e]) + (r.correction != nullptr ? r.correction[e] : 0.f);
+      if (v > a) {
+        b = a;
+        a = v;
+      } else if (v > b) {
+        b = v;
+      }
+    }
+    score[j] = size > 1 ? a + b : a;
+  }
+  unsigned long long kept = 0ull;
+  for (int n = 0; n < r.keep; ++n) {
+    float bv = -INFINITY;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int j = 0; j < kMoeMaxGroups / 32; ++j) {
+      const int g = lane + 32 * j;
+      if (g < r.groups && !((kept >> g) & 1ull) && (score[j] > bv || bi == 0x7fffffff)) {
+        bv = score[j];
+        bi = g;
+      }
+    }
+    warp_best(bv, bi);
+    kept |= 1ull << (bi & 63);
+  }
+  return kept;
+}
+
+__device__ __forceinline__ void moe_topk_token(const float* __restrict__ row, int E, int k, const MoeRouting& rt, int lane,
                                                float* __restrict__ w_out, int* __restrict__ idx_out, int* counts, int* idx_copy) {
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
-  mx = warp_max(mx);
-  float den = 0.f;
-  for (int e = lane; e < E; e += 32) den += __expf(row[e] - mx);
-  den = warp_sum(den);
+  const int mode = rt.mode;
+  float mx = -INFINITY, den = 0.f;
+  unsigned long long kept = ~0ull;
+  const int group = rt.groups > 1 ? E / rt.groups : E;
+  if (mode == 2) {
+    kept = moe_kept_groups(row, E, rt, lane);
+  } else {
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < E; e += 32) den += __expf(row[e] - mx);
+    den = warp_sum(den);
+  }
   float sel_v[kMaxTopK];
   int sel_i[kMaxTopK];
   unsigned long long taken_lo = 0ull;  // bitmask of this lane's taken slots (expert e = lane + 32 * j -> bit j)
@@ -33,21 +94,15 @@ __device__ __forceinline__ void moe_topk_token(const float* __restrict__ row, in
     int bi = 0x7fffffff;
     for (int e = lane, j = 0; e < E; e += 32, ++j) {
       if ((taken_lo >> j) & 1ull) continue;
-      const float v = row[e];
+      float v = row[e];
+      if (mode == 2) v = (kept >> (e / group)) & 1ull ? route_sigmoid(v) + (rt.correction != nullptr ? rt.correction[e] : 0.f) : -INFINITY;
       if (v > bv || (v == bv && e < bi)) {
         bv = v;
         bi = e;
       }
     }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > bv || (ov == bv && oi < bi)) {
-        bv = ov;
-        bi = oi;
-      }
-    }
+    warp_best(bv, bi);
+    if (bi >= E) bi = 0;  // (not a number among the logits: stay inside the tables)
     sel_v[r] = bv;
     sel_i[r] = bi;
     if ((bi & 31) == lane) taken_lo |= 1ull << (bi >> 5);
@@ -55,12 +110,18 @@ __device__ __forceinline__ void moe_topk_token(const float* __restrict__ row, in
   if (lane == 0) {
     float wts[kMaxTopK];
     float s = 0.f;
-    if (mode == 0) {
+    if (mode == 2) {
+      for (int r = 0; r < k; ++r) {
+        wts[r] = route_sigmoid(row[sel_i[r]]);
+        s += wts[r];
+      }
+      for (int r = 0; r < k; ++r) wts[r] = wts[r] / (s + 1e-20f) * rt.scale;
+    } else if (mode == 0) {
       for (int r = 0; r < k; ++r) {
         wts[r] = __expf(sel_v[r] - mx) / den;
         s += wts[r];
       }
-      if (renorm)
+      if (rt.renorm)
         for (int r = 0; r < k; ++r) wts[r] /= s;
     } else {
       for (int r = 0; r < k; ++r) {
@@ -79,14 +140,14 @@ __device__ __forceinline__ void moe_topk_token(const float* __restrict__ row, in
 }
 
 // one warp per token
-__global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__ logits, int T, int E, int k, int mode, int renorm,
+__global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__ logits, int T, int E, int k, const MoeRouting rt,
                                                        float* __restrict__ w_out, int* __restrict__ idx_out, int* __restrict__ counts) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
-  moe_topk_token(logits + static_cast<size_t>(t) * E, E, k, mode, renorm, lane, w_out + static_cast<size_t>(t) * k,
+  moe_topk_token(logits + static_cast<size_t>(t) * E, E, k, rt, lane, w_out + static_cast<size_t>(t) * k,
                  idx_out + static_cast<size_t>(t) * k, counts, nullptr);
 }
 
@@ -105,7 +166,7 @@ __device__ __forceinline__ int warp_incl_scan(int v, int lane) {
   }
   return v;
 }
-__global__ void __launch_bounds__(1024) moe_route_small_kernel(const float* __restrict__ logits, int T, int E, int k, int mode, int renorm,
+__global__ void __launch_bounds__(1024) moe_route_small_kernel(const float* __restrict__ logits, int T, int E, int k, const MoeRouting rt,
                                                                float* __restrict__ w_out, int* __restrict__ idx_out, int* __restrict__ counts,
                                                                int* __restrict__ offsets, int* __restrict__ perm, int* __restrict__ pos, int e0,
                                                                int ne, int bn, int max_items, int4* __restrict__ items) {
@@ -121,7 +182,7 @@ __global__ void __launch_bounds__(1024) moe_route_small_kernel(const float* __re
   for (int e = tid; e < E; e += 1024) cnt_s[e] = 0;
   __syncthreads();
   for (int t = warp; t < T; t += 32)
-    moe_topk_token(logits + static_cast<size_t>(t) * E, E, k, mode, renorm, lane, w_out + static_cast<size_t>(t) * k,
+    moe_topk_token(logits + static_cast<size_t>(t) * E, E, k, rt, lane, w_out + static_cast<size_t>(t) * k,
                    idx_out + static_cast<size_t>(t) * k, cnt_s, idx_s + t * k);
   __syncthreads();
   if (warp == 0) {  // exclusive scan of the histogram: lane l owns a contiguous chunk of experts
@@ -334,14 +395,14 @@ size_t moe_route_workspace_ints(int T, int E, int k) {
   const long long P = static_cast<long long>(T) * k;
   return P > kSortSerialMaxPairs ? static_cast<size_t>((P + kSortChunk - 1) / kSortChunk) * E : 0;
 }
-void launch_moe_route(const float* logits, int T, int E, int k, int mode, int renorm, float* w, int* idx, int* counts, int* offsets,
+void launch_moe_route(const float* logits, int T, int E, int k, const MoeRouting& r, float* w, int* idx, int* counts, int* offsets,
                       int* perm, int* pos, int* ws, cudaStream_t st) {
   cudaMemsetAsync(counts, 0, sizeof(int) * E, st);
   if (T == 0) {
     cudaMemsetAsync(offsets, 0, sizeof(int) * (E + 1), st);
     return;
   }
-  moe_topk_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, T, E, k, mode, renorm, w, idx, counts);
+  moe_topk_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, T, E, k, r, w, idx, counts);
   const int P = T * k;
   if (ws != nullptr && moe_route_workspace_ints(T, E, k) > 0) {
     const int C = (P + kSortChunk - 1) / kSortChunk;
@@ -353,11 +414,11 @@ void launch_moe_route(const float* logits, int T, int E, int k, int mode, int re
   moe_sort_kernel<<<1, 1024, sizeof(int) * (E + 1), st>>>(idx, counts, T, E, k, offsets, perm, pos);
 }
 // Decode-size batches: everything of launch_moe_route + launch_moe_items in one launch. False when the batch is too large for it.
-bool launch_moe_route_small(const float* logits, int T, int E, int k, int mode, int renorm, float* w, int* idx, int* counts, int* offsets,
+bool launch_moe_route_small(const float* logits, int T, int E, int k, const MoeRouting& r, float* w, int* idx, int* counts, int* offsets,
                             int* perm, int* pos, int e0, int ne, int bn, int max_items, int* items, cudaStream_t st) {
   if (T < 1 || T > kRouteSmallMaxTokens || T * k > kRouteSmallMaxPairs || E > 1024 || ne > 1024) return false;
   const size_t smem = sizeof(int) * (static_cast<size_t>(T) * k + 2 * E + ne + 3);
-  return launch_pdl(moe_route_small_kernel, dim3(1), dim3(1024), smem, st, logits, T, E, k, mode, renorm, w, idx, counts, offsets, perm, pos, e0,
+  return launch_pdl(moe_route_small_kernel, dim3(1), dim3(1024), smem, st, logits, T, E, k, r, w, idx, counts, offsets, perm, pos, e0,
                     ne, bn, max_items, reinterpret_cast<int4*>(items)) == cudaSuccess;
 }
 void launch_moe_gather(const void* x, const int* perm, int rows, int k, int row_bytes, void* xs, const int* offsets, int e0, int ne,

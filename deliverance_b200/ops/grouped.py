@@ -1,8 +1,11 @@
-"""Grouped-query softmax attention with per-layer sizes: unequal query / key and value widths, partial rotation of neighbouring pairs,
-sliding window with kept first tokens, score soft-cap and a sink in the denominator (a score of 0 that has no value).
+"""Grouped-query softmax attention with per-layer sizes: unequal query / key and value widths, partial rotation of neighbouring pairs or of
+the two halves of the rotated columns, per-head query / key norms, values that are the projected keys or a blend with another layer's,
+sliding window with kept first tokens, score soft-cap, a sink per head in the denominator (a score that has no value), an output gate per
+column or per head.
 
-One projection row is ``[q (H * dk) | k (G * dk) | v (G * dv)]`` with head widths rounded up to multiples of 8 (16-byte rows everywhere);
-the columns behind the real ones carry zero weights, so scores, cache rows and outputs are exact whatever the sizes. CUDA forms:
+One projection row is ``[q (H * dk) | k (G * dk) | v (G * dv) | g]`` with head widths rounded up to multiples of 8 (16-byte rows everywhere);
+the columns behind the real ones carry zero weights, so scores, cache rows and outputs are exact whatever the sizes. Tied values have no
+columns of their own; ``g`` is there for gated heads. CUDA forms:
 
 * prompts: the tcgen05 / TMA kernel (``attention_tc.cu``) over the paged cache, heads up to 256 wide;
 * decode: the split-KV tensor-core kernel (``attention.cu``), heads up to 256 wide;
@@ -28,10 +31,16 @@ class GroupedShape:
     kv_heads: int
     dim: int
     vdim: int
+    tied: bool = False  # the values are the projected keys
+    gate: str = ""  # output gate: "" | "columns" | "heads"
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads do not divide into {self.kv_heads} groups")
+        if self.tied and self.dim != self.vdim:
+            raise ValueError(f"keys of {self.dim} columns cannot be values of {self.vdim}")
+        if self.gate not in ("", "columns", "heads"):
+            raise ValueError(f"unknown output gate '{self.gate}'")
 
     @property
     def dk(self) -> int:
@@ -50,8 +59,25 @@ class GroupedShape:
         return self.kv_heads * self.dk
 
     @property
+    def v_at(self) -> int:
+        """First value column (tied values: the first key column)."""
+        return self.q_width if self.tied else self.q_width + self.k_width
+
+    @property
+    def v_width(self) -> int:
+        return self.kv_heads * self.dv
+
+    @property
+    def gate_at(self) -> int:
+        return self.q_width + self.k_width + (0 if self.tied else self.v_width)
+
+    @property
+    def gate_logits(self) -> int:
+        return {"": 0, "columns": self.out_width, "heads": self.heads}[self.gate]
+
+    @property
     def width(self) -> int:
-        return self.q_width + self.k_width + self.kv_heads * self.dv
+        return self.gate_at + up8(self.gate_logits)
 
     @property
     def out_width(self) -> int:
@@ -92,25 +118,61 @@ def rope_pairs_kv(s: GroupedShape, qkv, positions, slots, cos, sin, k_cache, v_c
     v_cache[blk, :, off, :] = v.reshape(T, s.kv_heads, s.dv).to(v_cache.dtype)
 
 
-def attention(s: GroupedShape, qkv, batch, k_cache, v_cache, scale: float, softcap: float, window: int, keep_first: int, sink: bool, splits: int):
-    """Heads of every row of the batch, ``[T, H * dv]``; the batch's keys and values are in the cache already."""
+def rope_heads_kv(s: GroupedShape, p, positions, slots, cos, sin, k_cache, v_cache, q_norm=None, k_norm=None, eps: float = 0.0, v_first=None,
+                  lam: float = 0.0) -> None:
+    """Optional per-head RMS norm of queries and keys (fp32 weights ``[dk]``, mean over the real columns), rotation of the pairs (i, i + half);
+    queries in place, keys into their cache rows. The values go to the cache as projected (tied: the keys as projected) or, with ``v_first
+    [T, G * dv]``, as ``(1 - lam) v + lam v_first``."""
+    if ops._cuda(p):
+        ops._count()
+        ops.require_ext().rope_heads_kv(p, s.q_width, s.v_at, positions, slots, cos, sin, k_cache, v_cache, s.heads, s.kv_heads, s.dk, s.dv, s.dim, q_norm, k_norm,
+                                        eps, v_first, lam)
+        return
+    T, pos = p.shape[0], positions.long()
+    q = p[:, : s.q_width].reshape(T, s.heads, s.dk)
+    k = p[:, s.q_width : s.q_width + s.k_width].reshape(T, s.kv_heads, s.dk)
+    v = p[:, s.v_at : s.v_at + s.v_width].reshape(T, s.kv_heads, s.dv)
+    if v_first is not None:
+        v = (1.0 - lam) * v.float() + lam * v_first.float().reshape(T, s.kv_heads, s.dv)
+    page = k_cache.shape[2]
+    blk, off = torch.div(slots, page, rounding_mode="floor"), slots % page
+    v_cache[blk, :, off, :] = v.to(v_cache.dtype)
+
+    def normed(x, w):
+        if w is None:
+            return x
+        x = x.float()
+        return x * torch.rsqrt(x.pow(2).sum(dim=-1, keepdim=True) / s.dim + eps) * w
+
+    k_cache[blk, :, off, :] = ref.apply_rope(normed(k, k_norm), pos, cos, sin).to(k_cache.dtype)
+    p[:, : s.q_width] = ref.apply_rope(normed(q, q_norm), pos, cos, sin).reshape(T, -1).to(p.dtype)
+
+
+def attention(s: GroupedShape, qkv, batch, k_cache, v_cache, scale: float, softcap: float, window: int, keep_first: int, sink, splits: int, mult: float = 1.0,
+              out=None):
+    """Heads of every row of the batch, ``[T, H * dv]`` (``out``: a column range of wider rows to write to); the batch's keys and values are
+    in the cache already. ``sink``: fp32 ``[H]`` or None. Gated shapes multiply with the sigmoid of their logits in ``qkv``, all with ``mult``."""
     q = qkv[:, : s.q_width]
-    mask = (float(scale), float(softcap), int(window), int(keep_first), bool(sink))
+    gate = qkv[:, s.gate_at : s.gate_at + s.gate_logits] if s.gate else None
     if not ops._cuda(qkv):
         o = ref.paged_attention(q.reshape(-1, s.heads, s.dk), k_cache, v_cache, batch.block_tables, batch.q_start.tolist(), batch.q_len.tolist(),
                                 batch.ctx_len.tolist(), scale, softcap, window, True, keep_first, sink)
-        return o.reshape(-1, s.out_width)
+        if gate is not None:
+            o = o.float() * torch.sigmoid(gate.float()).reshape(o.shape[0], s.heads, -1)
+        o = (o * mult).to(qkv.dtype).reshape(-1, s.out_width)
+        return o if out is None else out.copy_(o)
     e = ops.require_ext()
+    mask = (float(scale), float(softcap), int(window))
+    extra = {"keep_first": int(keep_first), "sink": sink, "gate": gate, "out_mult": float(mult), "out": out}
     if qkv.dtype == torch.float32 or not s.tensor_core:
         ops._count()
-        return e.attention_rows(q, k_cache, v_cache, batch.block_tables, None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask)
+        return e.attention_rows(q, k_cache, v_cache, batch.block_tables, None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask, **extra)
     if batch.is_decode:
         ops._count(1 if splits <= 1 else 2)
-        return e.decode_attention(q, k_cache, v_cache, batch.block_tables, batch.ctx_len, s.heads, mask[0], mask[1], mask[2], splits, 0, mask[3], mask[4])
+        return e.decode_attention(q, k_cache, v_cache, batch.block_tables, batch.ctx_len, s.heads, *mask, splits, 0, **extra)
     ts, t0 = batch.tiles(e.prefill_tc_tile_rows(max(s.dk, s.dv)))
     ops._count()
-    return e.prefill_attention_tc(q, k_cache, v_cache, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_len, ts, t0, s.heads, mask[0], mask[1],
-                                  mask[2], True, mask[3], mask[4])
+    return e.prefill_attention_tc(q, k_cache, v_cache, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_len, ts, t0, s.heads, *mask, True, **extra)
 
 
 def row_sequence(batch) -> torch.Tensor:

@@ -153,13 +153,14 @@ def qk_prepare_and_cache(qkv, positions, slots, n_heads, n_kv, head_dim, q_norm_
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, scale, softcap=0.0, window=0,
-                    causal=True, keep_first=0, sink=False):
+                    causal=True, keep_first=0, sink=None):
     """Attention of ragged query rows against paged K/V.
 
     q ``[T, H, D]``; sequence ``i`` owns query rows ``[q_start[i], q_start[i] + q_len[i])`` which are the *last*
     ``q_len[i]`` positions of a context of ``ctx_len[i]`` cached tokens. Row at position ``p`` sees keys ``j <= p``
     (and ``j > p - window`` or ``j < keep_first`` when ``window > 0``). Score = ``softmax(softcap * tanh(scale * q.k / softcap))``;
-    ``sink``: a further score of 0 without a value takes part in the softmax. Values may be wider or narrower than keys.
+    ``sink`` ``[H]``: a further score per head without a value takes part in the softmax (neither scaled nor capped). Values may be wider or
+    narrower than keys.
     """
     T, H, D = q.shape
     nb, KV, bs, _ = k_cache.shape
@@ -188,7 +189,10 @@ def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, 
         if window and window > 0:
             mask &= (j > pos - window) | (j < keep_first)
         s = s.masked_fill(~mask.unsqueeze(0), float("-inf"))
-        p = torch.softmax(F.pad(s, (0, 1)), dim=-1)[..., :-1] if sink else torch.softmax(s, dim=-1)
+        if sink is not None:
+            p = torch.softmax(torch.cat([s, sink.float().view(H, 1, 1).expand(H, ql, 1)], dim=-1), dim=-1)[..., :-1]
+        else:
+            p = torch.softmax(s, dim=-1)
         out[qs : qs + ql] = torch.matmul(p, v).permute(1, 0, 2).to(q.dtype)
     return out
 
@@ -240,12 +244,14 @@ def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 # ---- MoE -------------------------------------------------------------------------------------------------------------
-def moe_route(router_logits: torch.Tensor, k: int, mode: str, renorm: bool):
+def moe_route(router_logits: torch.Tensor, k: int, mode: str, renorm: bool, correction=None, groups: int = 1, keep: int = 1, scale: float = 1.0):
     """Return (weights ``[T, k]`` fp32, expert ids ``[T, k]``).
 
     ``softmax_topk``: softmax over all experts, take top-k, optionally renormalise (Mixtral always renormalises,
     MixtureOfExpertsBlock.java:100-112; Qwen3-MoE by ``norm_topk_prob``, Qwen3MoeFeedForward.java:276-301).
     ``topk_softmax``: take the top-k logits, softmax over those k (GraniteMoeHybridMoeFeedForward.java:112-141).
+    ``sigmoid_topk``: scores ``s = sigmoid(z)``; the largest ``s + correction`` among the experts of the ``keep`` best of ``groups`` equal groups
+    of neighbours (a group counts the sum of its two largest choice scores); weights ``scale * s / (sum + 1e-20)``.
     """
     lf = router_logits.float()
     if mode == "softmax_topk":
@@ -256,6 +262,17 @@ def moe_route(router_logits: torch.Tensor, k: int, mode: str, renorm: bool):
     elif mode == "topk_softmax":
         top, idx = torch.topk(lf, k, dim=-1)
         w = torch.softmax(top, dim=-1)
+    elif mode == "sigmoid_topk":
+        s = torch.sigmoid(lf)
+        choice = s if correction is None else s + correction.float()
+        if groups > 1 and keep < groups:
+            by_group = choice.view(choice.shape[0], groups, -1)
+            best = by_group.topk(min(2, by_group.shape[-1]), dim=-1).values.sum(dim=-1)
+            kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, best.topk(keep, dim=-1).indices, True)
+            choice = by_group.masked_fill(~kept.unsqueeze(-1), float("-inf")).flatten(1)
+        idx = choice.topk(k, dim=-1).indices
+        w = s.gather(1, idx)
+        w = w / (w.sum(dim=-1, keepdim=True) + 1e-20) * scale
     else:
         raise ValueError(mode)
     return w, idx
@@ -338,6 +355,34 @@ def gla_norm_gate(o, g, w, eps: float):
     """``o [T, H, dv]`` RMS-normed over dv with the shared weight ``w [dv]``, times ``silu(g)``."""
     o = o.float()
     return o * torch.rsqrt(o.pow(2).mean(dim=-1, keepdim=True) + eps) * w * F.silu(g.float())
+
+
+# ---- lightning attention ---------------------------------------------------------------------------------------------
+def lightning_sequential(q, k, v, decay, state):
+    """Token-by-token linear attention of ONE sequence with a constant decay per head, fp32: ``S <- decay S + k v^T``, ``o = S^T q``.
+    q, k ``[T, H, dk]``, v ``[T, H, dv]`` (activated), ``decay [H]``; ``state [H, dk, dv]`` is updated in place. Returns ``[T, H, dv]``."""
+    q, k, v = q.float(), k.float(), v.float()
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    d = decay.view(-1, 1, 1)
+    for t in range(v.shape[0]):
+        state.copy_(state.double() * d + k[t].unsqueeze(-1) * v[t].unsqueeze(-2))
+        out[t] = (state * q[t].unsqueeze(-1)).sum(dim=-2)
+    return out
+
+
+# ---- residual streams --------------------------------------------------------------------------------------------------
+def layernorm_rows(v, w, eps):
+    d = v - v.mean(dim=-1, keepdim=True)
+    return d * torch.rsqrt(d.pow(2).mean(dim=-1, keepdim=True) + eps) * w
+
+
+def stream_write(streams, y, mix, write):
+    """In place over ``[T, S, W]``: ``x_t = sum_s mix[s, t] x_s + write[t] y``."""
+    streams.copy_(torch.einsum("nsw,st->ntw", streams, mix) + write.view(1, -1, 1) * y.float().unsqueeze(1))
+
+
+def stream_read(streams, read):
+    return streams.sum(dim=1) if read is None else torch.einsum("nsw,s->nw", streams, read)
 
 
 # ---- sampling helpers --------------------------------------------------------------------------------------------------
