@@ -365,7 +365,7 @@ class Engine:
             if budget <= 0:
                 break
             n = min(len(r.fill) - r.computed, budget)
-            if self.hybrid:
+            if self.hybrid and self.kv.settings.enabled:
                 # recurrent state can only be snapshotted at chunk ends: stop chunks at the prefix-cache checkpoints
                 for L in self.kv.settings.checkpoint_lengths(len(r.fill)):
                     if r.computed < L < r.computed + n:
@@ -392,7 +392,7 @@ class Engine:
                 rate = (r.computed - r.prefix_hit) / max(now - r.t_submit, 1e-9)
                 _log.info("prefill progress request=%d tokens=%d/%d rate=%.0f tok/s eta=%.1f s", r.rid, r.computed, len(r.fill), rate,
                           (len(r.fill) - r.computed) / max(rate, 1e-9))
-            if self.hybrid and r.computed in self.kv.settings.checkpoint_lengths(len(r.fill)):
+            if self.hybrid and self.kv.settings.enabled and r.computed in self.kv.settings.checkpoint_lengths(len(r.fill)):
                 r.state_snapshots[r.computed] = self.kv.snapshot_state(r.state_slot)
             if r.computed >= len(r.fill):
                 self.kv.prefix.store(r.salt, r.fill, r.pages, r.state_snapshots if self.hybrid else None)

@@ -129,8 +129,7 @@ struct AttnTcSmem {
 };
 
 // eight columns times the sigmoid of their gate logits
-__device__ __forceinline__ void gate8(float* w, const __nv_bfloat16* g) {
-  const uint4 gv = *reinterpret_cast<const uint4*>(g);
+__device__ __forceinline__ void gate8(float* w, const uint4& gv) {
   const uint32_t* gu = reinterpret_cast<const uint32_t*>(&gv);
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
@@ -431,6 +430,12 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     // scores stay in the units the tensor core delivers; kf turns a difference of scores into a base-2 exponent
     const float kf = p.softcap > 0.f ? c_log2 : p.scale * c_log2;
     float m_run = -INFINITY, l_run = 0.f;
+    // gate logits of this row; threads behind the last row read that row's (every branch around tensor-memory accesses stays warp-uniform)
+    const size_t gate_row = static_cast<size_t>(qs + q0 + q * kAtBM + max(0, min(r, my_rows - 1)));
+    const __nv_bfloat16* grow = p.gate != nullptr && !p.gate_heads ? p.gate + gate_row * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
+    const bool gate_vec = grow != nullptr && (p.dv & 7) == 0;  // (then rows, heads and the gate are 16-byte aligned)
+    if (grow != nullptr)
+      for (int c = 0; c < p.dv; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + c));
     bool ok = true;
     for (int t = 0; t < my_tiles && ok; ++t) {
       const int j = t < my_kept ? t : ja + t - my_kept;
@@ -529,10 +534,15 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
       float inv = l_run > 0.f ? p.out_mult / l_run : 0.f;
       const size_t trow = static_cast<size_t>(qs + q0 + q * kAtBM + r);
       __nv_bfloat16* orow = p.out + trow * p.out_pitch + static_cast<size_t>(h) * p.dv;
-      const __nv_bfloat16* grow = p.gate != nullptr && !p.gate_heads ? p.gate + trow * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
-      if (!LATENT && p.gate_heads && r < my_rows) inv /= 1.f + __expf(-bf2f(p.gate[trow * p.gate_pitch + h]));
+      if (!LATENT && p.gate_heads) inv /= 1.f + __expf(-bf2f(p.gate[gate_row * p.gate_pitch + h]));
 #pragma unroll 1
       for (int c0 = 0; c0 < DV; c0 += 32) {
+        uint4 gv[4];  // the gate logits of this step, all on their way before the first is used
+        if (gate_vec) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (c0 + i * 8 < p.dv) gv[i] = *reinterpret_cast<const uint4*>(grow + c0 + i * 8);
+        }
         uint32_t v[32];
         if (my_tiles > 0) {
           tmem_ld_x32(lane_addr + kColO + q * DV + c0, v);
@@ -551,7 +561,7 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
 #pragma unroll
               for (int e = 0; e < 8; ++e) w[e] = __uint_as_float(v[i + e]) * inv;
               if (vec) {
-                if (grow != nullptr) gate8(w, grow + c0 + i);
+                if (grow != nullptr) gate8(w, gv[i / 8]);
                 *reinterpret_cast<uint4*>(orow + c0 + i) =
                     make_uint4(pack_bf162(w[0], w[1]), pack_bf162(w[2], w[3]), pack_bf162(w[4], w[5]), pack_bf162(w[6], w[7]));
               } else {
@@ -568,7 +578,7 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
             float w[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) w[e] = __uint_as_float(v[i + e]) * inv;
-            if (grow != nullptr) gate8(w, grow + c0 + i);
+            if (grow != nullptr) gate8(w, gv[i / 8]);
             *reinterpret_cast<uint4*>(orow + c0 + i) = make_uint4(pack_bf162(w[0], w[1]), pack_bf162(w[2], w[3]), pack_bf162(w[4], w[5]), pack_bf162(w[6], w[7]));
           }
         }

@@ -615,9 +615,9 @@ __global__ void __launch_bounds__(256) rope_pairs_kv_kernel(TIO* __restrict__ qk
 // when the values are the projected keys). Queries and keys: optional RMS norm over the head (dim real columns), then the pairs
 // (i, i + half), i < half, are rotated; queries in place, keys into the cache. Values go to the cache as projected or, with v_first,
 // blended with another row of the same token: (1 - lam) v + lam v_first.
-// LPH lanes of a warp own one (row, head): eight columns per lane and step, the head passes through shared memory so that the partner of
-// a rotated column is at hand whatever `half` is.
-template <typename TIO, int LPH>
+// LPH lanes of a warp own one (row, head), eight columns per lane and step. The partners of eight rotated columns lie in another lane's
+// registers when `half` is a multiple of eight and the head is one step wide (LANES); otherwise the head passes through shared memory.
+template <typename TIO, int LPH, bool LANES>
 __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs a) {
   pdl_wait();
   pdl_trigger();
@@ -625,8 +625,8 @@ __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs 
   const bool tied = a.off_v == a.off_k;
   const int heads = a.H + a.KV + (tied ? 0 : a.KV);
   const int sub = threadIdx.x % LPH, grp = threadIdx.x / LPH;
-  const long long idx = static_cast<long long>(blockIdx.x) * (256 / LPH) + grp;
-  const bool active = idx < static_cast<long long>(a.T) * heads;  // (all lanes reach the shuffles and warp barriers below)
+  const unsigned idx = blockIdx.x * (256u / LPH) + grp;
+  const bool active = idx < static_cast<unsigned>(a.T) * heads;  // (all lanes reach the shuffles and warp barriers below)
   const int t = active ? static_cast<int>(idx / heads) : 0, h = active ? static_cast<int>(idx % heads) : 0;
   const bool is_q = h < a.H, is_v = h >= a.H + a.KV;
   const int kvh = is_q ? 0 : (is_v ? h - a.H - a.KV : h - a.H);
@@ -636,16 +636,16 @@ __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs 
   if (!is_q) {
     const long long slot = a.slots[t];
     store = active && slot >= 0;
-    if (store) at = ((slot / a.page) * a.KV + kvh) * a.page + slot % a.page;
+    const unsigned su = static_cast<unsigned>(store ? slot : 0), page = static_cast<unsigned>(a.page);  // (the caches hold fewer than 2^32 rows)
+    at = (static_cast<long long>(su / page) * a.KV + kvh) * a.page + su % page;
   }
   float* s = hsm + grp * a.dk;
   const TIO* src = row + (is_q ? h * a.dk : (is_v ? a.off_v + kvh * a.dv : a.off_k + kvh * a.dk));
   TIO* vdst = static_cast<TIO*>(a.v_cache) + at * a.dv;
   const float* nw = is_v ? nullptr : (is_q ? a.q_norm : a.k_norm);
   const int width = is_v ? a.dv : a.dk;
-  float ss = 0.f;
+  float ss = 0.f, x[8] = {};
   for (int c = sub * 8; c < width; c += LPH * 8) {
-    float x[8];
     io_ld8(src + c, x);
     if (is_v || (!is_q && tied)) {
       if (a.v_first != nullptr) {
@@ -660,15 +660,24 @@ __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs 
       }
     }
     if (!is_v) {
-      *reinterpret_cast<float4*>(s + c) = make_float4(x[0], x[1], x[2], x[3]);
-      *reinterpret_cast<float4*>(s + c + 4) = make_float4(x[4], x[5], x[6], x[7]);
+      if constexpr (!LANES) {
+        *reinterpret_cast<float4*>(s + c) = make_float4(x[0], x[1], x[2], x[3]);
+        *reinterpret_cast<float4*>(s + c + 4) = make_float4(x[4], x[5], x[6], x[7]);
+      }
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
     }
   }
 #pragma unroll
   for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  __syncwarp();
+  float other[8];  // LANES: the partners of this lane's columns
+  if constexpr (LANES) {
+    const int hc = a.half / 8, from = sub < hc ? sub + hc : (sub < 2 * hc ? sub - hc : sub);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, x[e], from, LPH);
+  } else {
+    __syncwarp();
+  }
   if (is_v || !store) return;
   const float inv = nw != nullptr ? rsqrtf(ss / a.dim + a.eps) : 1.f;
   int pos = a.positions[t];
@@ -677,6 +686,32 @@ __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs 
   const float* sn = a.sin_t + static_cast<size_t>(pos) * a.half;
   TIO* dst = is_q ? row + h * a.dk : static_cast<TIO*>(a.k_cache) + at * a.dk;
   const int end = is_q && nw == nullptr ? min(a.dk, (2 * a.half + 7) / 8 * 8) : a.dk;  // queries that nothing changes stay where they are
+  if constexpr (LANES) {
+    const int c = sub * 8;
+    if (c >= end) return;
+    float w[8];
+    if (nw != nullptr) {
+      io_ld8(nw + c, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= inv * w[e];
+    }
+    if (c < 2 * a.half) {
+      const bool low = c < a.half;
+      const int i = low ? c : c - a.half;
+      if (nw != nullptr) {
+        io_ld8(nw + (low ? c + a.half : i), w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) other[e] *= inv * w[e];
+      }
+      float co[8], si[8];
+      io_ld8(cs + i, co);
+      io_ld8(sn + i, si);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = low ? x[e] * co[e] - other[e] * si[e] : x[e] * co[e] + other[e] * si[e];
+    }
+    io_st8(dst + c, x);
+    return;
+  }
   for (int c = sub * 8; c < end; c += LPH * 8) {
     float y[8];
 #pragma unroll
@@ -701,14 +736,18 @@ template <typename TIO>
 static int launch_rope_heads_t(const RopeHeadsArgs& a, cudaStream_t st) {
   const int chunks = (a.dk > a.dv ? a.dk : a.dv) / 8;
   const long long n = static_cast<long long>(a.T) * (a.H + (a.off_v == a.off_k ? 1 : 2) * a.KV);
-  auto go = [&](auto kernel, int lph) {
+  const bool lanes = a.half % 8 == 0 && a.dk <= 256;
+  auto go = [&](auto by_lanes, auto by_memory, int lph) {
     const int per = 256 / lph;
-    return launch_pdl(kernel, dim3(static_cast<unsigned>((n + per - 1) / per)), dim3(256), static_cast<size_t>(per) * a.dk * sizeof(float), st, a) == cudaSuccess ? 0 : 2;
+    const dim3 grid(static_cast<unsigned>((n + per - 1) / per));
+    const cudaError_t e = lanes ? launch_pdl(by_lanes, grid, dim3(256), 0, st, a)
+                                : launch_pdl(by_memory, grid, dim3(256), static_cast<size_t>(per) * a.dk * sizeof(float), st, a);
+    return e == cudaSuccess ? 0 : 2;
   };
-  if (chunks <= 4) return go(rope_heads_kv_kernel<TIO, 4>, 4);
-  if (chunks <= 8) return go(rope_heads_kv_kernel<TIO, 8>, 8);
-  if (chunks <= 16) return go(rope_heads_kv_kernel<TIO, 16>, 16);
-  return go(rope_heads_kv_kernel<TIO, 32>, 32);
+  if (chunks <= 4) return go(rope_heads_kv_kernel<TIO, 4, true>, rope_heads_kv_kernel<TIO, 4, false>, 4);
+  if (chunks <= 8) return go(rope_heads_kv_kernel<TIO, 8, true>, rope_heads_kv_kernel<TIO, 8, false>, 8);
+  if (chunks <= 16) return go(rope_heads_kv_kernel<TIO, 16, true>, rope_heads_kv_kernel<TIO, 16, false>, 16);
+  return go(rope_heads_kv_kernel<TIO, 32, true>, rope_heads_kv_kernel<TIO, 32, false>, 32);
 }
 
 // ------------------------------------------------------------------------------------------------ launchers
@@ -805,7 +844,7 @@ void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const l
 }
 int launch_rope_heads_kv(const RopeHeadsArgs& a, bool is_f32, cudaStream_t st) {
   if (a.T == 0) return 0;
-  if (a.dk > 1024 || a.dk % 8 != 0 || a.dv % 8 != 0) return 1;  // (the heads of a block share 48 KB)
+  if (a.dk > 1024 || a.dk % 8 != 0 || a.dv % 8 != 0 || static_cast<long long>(a.T) * (a.H + 2 * a.KV) > 0x7fffffffll) return 1;  // (the heads of a block share 48 KB)
   return is_f32 ? launch_rope_heads_t<float>(a, st) : launch_rope_heads_t<__nv_bfloat16>(a, st);
 }
 int launch_rope_kv(void* qkv, const int* positions, const long long* slots, const void* qn, const void* kn, const float* cos_t,

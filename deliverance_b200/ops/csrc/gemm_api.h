@@ -379,7 +379,7 @@ struct StreamArgs {
 int launch_stream_step(const StreamArgs& a, int rows, bool is_f32, cudaStream_t st);
 
 // lightning.cu: linear attention with one constant decay per head. Projection rows p [T, ld] = q (H dk) | k (H dk) | v (H dv) | g (H dv) at the given
-// first columns, widths multiples of 8
+// first columns, widths multiples of 8. The chunked form overwrites q, k and v with their activations.
 struct LightningArgs {
   const void* p;
   long long ld;
@@ -402,7 +402,8 @@ struct LightningChunks {
   const int *seq, *row0, *len;  // per chunk
   const int *first, *count;     // per sequence
   int n_chunks;
-  float* states;  // [n_chunks, H, dk, dv]: what each chunk adds, then the state in front of it
+  float* added;   // [n_chunks, H, dk, dv]: what each chunk adds to the state
+  void* states;   // bf16 [n_chunks, H, 2, dk, dv]: the state in front of each chunk, high and low parts
 };
 int launch_lightning_recurrent(const LightningArgs& a, bool is_f32, cudaStream_t st);
 int launch_lightning_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st);

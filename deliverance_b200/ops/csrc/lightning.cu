@@ -6,6 +6,7 @@
 //   lightning_recurrent_kernel  token by token, one CTA per (64 value columns, head, sequence), its part of the state in registers: decode
 //                               steps, the 32-bit form of prompts, and key widths the chunked form does not take.
 //   Prompts in chunks of 128 tokens. Nothing walks the chunks one by one but an elementwise kernel:
+//   lightning_act_kernel        the activations, in place (every CTA of the kernels below reads rows that others read too);
 //   lightning_chunk_kv_kernel   per (chunk, head, 64 value columns): what the chunk adds to the state, sum_s decay^(end - s) k_s v_s^T;
 //   lightning_scan_kernel       per (sequence, head, element): the state in front of every chunk, the slot's new state;
 //   lightning_chunk_out_kernel  per (chunk, head, 64 value columns): decay^(t + 1) S^T q_t plus the causal part inside the chunk, whose weights
@@ -25,10 +26,9 @@ namespace {
 constexpr int kLnCols = 64;    // value columns per CTA
 constexpr int kLnChunk = 128;  // tokens per chunk
 
-__device__ __forceinline__ float ln_silu(float z) { return z / (1.f + expf(-z)); }
-// the activation in the type the tensor cores read (both evaluation orders see the same numbers)
-__device__ __forceinline__ float ln_act(float z, const float*) { return ln_silu(z); }
-__device__ __forceinline__ float ln_act(float z, const __nv_bfloat16*) { return bf2f(f2bf(ln_silu(z))); }
+// silu; bf16 rows are activated into bf16, the type the tensor cores read (both evaluation orders see the same numbers)
+__device__ __forceinline__ float ln_act(float z, const float*) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float ln_act(float z, const __nv_bfloat16*) { return bf2f(f2bf(__fdividef(z, 1.f + __expf(-z)))); }
 
 }  // namespace
 
@@ -164,22 +164,28 @@ int launch_lightning_recurrent(const LightningArgs& a, bool is_f32, cudaStream_t
 // =====================================================================================================================
 // Chunked form. NK: 16-channel tiles of the key width (padded)
 // =====================================================================================================================
-__device__ __forceinline__ uint32_t act2(uint32_t u) {
-  const float2 f = unpack_bf162(u);
-  return pack_bf162(ln_silu(f.x), ln_silu(f.y));
+// q, k and v of every row are activated once, in place: columns [0, n) of the projection rows
+__global__ void __launch_bounds__(256) lightning_act_kernel(const LightningArgs a, __nv_bfloat16* p, int n) {
+  pdl_wait();
+  pdl_trigger();
+  const unsigned per = static_cast<unsigned>(n) / 8, i = blockIdx.x * 256u + threadIdx.x;
+  if (i >= per * static_cast<unsigned>(a.rows)) return;
+  __nv_bfloat16* at = p + static_cast<size_t>(i / per) * a.ld + (i % per) * 8;
+  float v[8];
+  io_ld8(at, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = ln_act(v[e], at);
+  io_st8(at, v);
 }
-// [kLnChunk][16 NK] tile of activated rows; columns behind dk and rows behind len are zero
+
+// copy of a [kLnChunk][16 NK] tile of rows, started here; columns behind dk and rows behind len become zero
 template <int NK>
-__device__ __forceinline__ void load_act_tile(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int len, int dk) {
+__device__ __forceinline__ void copy_tile(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int len, int dk) {
   constexpr int P = NK * 16 + 8, CH = NK * 2;
   for (int e = threadIdx.x; e < kLnChunk * CH; e += 256) {
     const int t = e / CH, x = (e % CH) * 8;
-    uint4 u = make_uint4(0u, 0u, 0u, 0u);
-    if (t < len && x < dk) {
-      u = *reinterpret_cast<const uint4*>(src + t * ld + x);
-      u = make_uint4(act2(u.x), act2(u.y), act2(u.z), act2(u.w));
-    }
-    *reinterpret_cast<uint4*>(dst + t * P + x) = u;
+    const bool ok = t < len && x < dk;
+    cp16(smem_u32(dst + t * P + x), src + (ok ? t * ld + x : 0), ok);
   }
 }
 
@@ -193,7 +199,7 @@ struct LnKv {
 template <int NK>
 struct LnOut {
   static constexpr int P = NK * 16 + 8;
-  static constexpr int kBytes = (2 * kLnChunk * P + kLnChunk * kLnPV + 2 * NK * 16 * kLnPV) * 2 + (kLnChunk + 4) * 4;
+  static constexpr int kBytes = (kLnChunk * P + kLnChunk * kLnPV + 2 * NK * 16 * kLnPV) * 2 + (kLnChunk + 4) * 4;
   static_assert(kBytes <= 227 * 1024, "tiles must fit shared memory");
 };
 
@@ -210,7 +216,8 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
   const int row0 = c.row0[ck], len = c.len[ck], dk = a.dk, dv = a.dv;
   const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(a.p) + static_cast<size_t>(row0) * a.ld;
   for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
-  load_act_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
+  copy_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
+  cp_commit();
   __syncthreads();
   for (int e = tid; e < kLnChunk * 8; e += 256) {
     const int t = e >> 3, x = (e & 7) * 8;
@@ -221,13 +228,14 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
       const float s = pw[len - 1 - t];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 f = unpack_bf162(act2(w[i]));
+        const float2 f = unpack_bf162(w[i]);
         split2(f.x * s, f.y * s, hi[i], lo[i]);
       }
     }
     *reinterpret_cast<uint4*>(sV + t * kLnPV + x) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
     *reinterpret_cast<uint4*>(sV + (kLnChunk + t) * kLnPV + x) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
+  cp_wait<0>();
   __syncthreads();
   // rows = key channels (16 per tile), columns = value columns: a warp takes MT row tiles x NT column tiles of 8
   constexpr int WM = NK < 8 ? NK : 8, WN = 8 / WM, MT = NK / WM, NT = 8 / WN;
@@ -258,7 +266,7 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
       }
     }
   }
-  float* u = c.states + (static_cast<size_t>(ck) * a.H + h) * dk * dv;
+  float* u = c.added + (static_cast<size_t>(ck) * a.H + h) * dk * dv;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -270,7 +278,8 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
     }
 }
 
-// a thread keeps four elements of a state and walks the sequence's chunks, four loads ahead
+// a thread keeps four elements of a state and walks the sequence's chunks, four loads ahead; the state in front of every chunk is left as
+// two bf16 planes (high and low parts), the operands of the next kernel
 __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs a, const LightningChunks c) {
   pdl_wait();
   pdl_trigger();
@@ -281,7 +290,8 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs
   float4 st = make_float4(0.f, 0.f, 0.f, 0.f);
   if (a.positions[a.q_start[s]] != 0) st = *slot;
   const float* pw = a.powers + static_cast<size_t>(h) * (kLnChunk + 2);
-  auto chunk = [&](int i) { return reinterpret_cast<float4*>(c.states + (static_cast<size_t>(first + i) * a.H + h) * per + at); };
+  auto chunk = [&](int i) { return reinterpret_cast<const float4*>(c.added + (static_cast<size_t>(first + i) * a.H + h) * per + at); };
+  __nv_bfloat16* planes = static_cast<__nv_bfloat16*>(c.states);
   constexpr int AHEAD = 4;
   float4 u[AHEAD];
 #pragma unroll
@@ -293,7 +303,12 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs
       if (i >= n) break;
       const float4 add = u[j];
       if (i + AHEAD < n) u[j] = *chunk(i + AHEAD);
-      *chunk(i) = st;
+      uint32_t h0, h1, l0, l1;
+      split2(st.x, st.y, h0, l0);
+      split2(st.z, st.w, h1, l1);
+      __nv_bfloat16* hi = planes + (static_cast<size_t>(first + i) * a.H + h) * 2 * per + at;
+      *reinterpret_cast<uint2*>(hi) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(hi + per) = make_uint2(l0, l1);
       const float d = pw[c.len[first + i]];
       st = make_float4(fmaf(st.x, d, add.x), fmaf(st.y, d, add.y), fmaf(st.z, d, add.z), fmaf(st.w, d, add.w));
     }
@@ -302,68 +317,74 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs
 }
 
 template <int NK>
-__global__ void __launch_bounds__(256) lightning_chunk_out_kernel(const LightningArgs a, const LightningChunks c) {
+__global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_kernel(const LightningArgs a, const LightningChunks c) {
   pdl_wait();
   pdl_trigger();
   using L = LnOut<NK>;
   constexpr int P = L::P;
   extern __shared__ __align__(16) uint8_t lsm[];
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(lsm);  // [128][P]
-  __nv_bfloat16* sK = sQ + kLnChunk * P;                      // [128][P]
+  __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(lsm);  // [128][P]
   __nv_bfloat16* sV = sK + kLnChunk * P;                      // [128][kLnPV]
   __nv_bfloat16* sS = sV + kLnChunk * kLnPV;                  // [2][16 NK][kLnPV] state in front of the chunk, high and low parts
   float* pw = reinterpret_cast<float*>(sS + 2 * NK * 16 * kLnPV);
   const int ck = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kLnCols, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int row0 = c.row0[ck], len = c.len[ck], dk = a.dk, dv = a.dv;
   const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(a.p) + static_cast<size_t>(row0) * a.ld;
-  for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
-  load_act_tile<NK>(sQ, p + h * dk, a.ld, len, dk);
-  load_act_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
+  const __nv_bfloat16* state = static_cast<const __nv_bfloat16*>(c.states) + (static_cast<size_t>(ck) * a.H + h) * 2 * dk * dv;
+  for (int e = tid; e < 2 * NK * 16 * 8; e += 256) {
+    const int d = (e >> 3) % (NK * 16), x = (e & 7) * 8, plane = e / (NK * 16 * 8);
+    const bool ok = d < dk && c0 + x < dv;
+    cp16(smem_u32(sS + (plane * NK * 16 + d) * kLnPV + x), state + (ok ? (static_cast<size_t>(plane) * dk + d) * dv + c0 + x : 0), ok);
+  }
+  cp_commit();
+  copy_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
   for (int e = tid; e < kLnChunk * 8; e += 256) {
     const int t = e >> 3, x = (e & 7) * 8;
-    uint4 u = make_uint4(0u, 0u, 0u, 0u);
-    if (t < len && c0 + x < dv) {
-      u = *reinterpret_cast<const uint4*>(p + t * a.ld + a.off_v + h * dv + c0 + x);
-      u = make_uint4(act2(u.x), act2(u.y), act2(u.z), act2(u.w));
-    }
-    *reinterpret_cast<uint4*>(sV + t * kLnPV + x) = u;
+    const bool ok = t < len && c0 + x < dv;
+    cp16(smem_u32(sV + t * kLnPV + x), p + (ok ? t * a.ld + a.off_v + h * dv + c0 + x : 0), ok);
   }
-  const float* state = c.states + (static_cast<size_t>(ck) * a.H + h) * dk * dv;
-  for (int e = tid; e < NK * 16 * 16; e += 256) {
-    const int d = e >> 4, x = (e & 15) * 4;
-    uint32_t h0 = 0u, h1 = 0u, l0 = 0u, l1 = 0u;
-    if (d < dk && c0 + x < dv) {
-      const float4 f = *reinterpret_cast<const float4*>(state + static_cast<size_t>(d) * dv + c0 + x);
-      split2(f.x, f.y, h0, l0);
-      split2(f.z, f.w, h1, l1);
-    }
-    *reinterpret_cast<uint2*>(sS + d * kLnPV + x) = make_uint2(h0, h1);
-    *reinterpret_cast<uint2*>(sS + (NK * 16 + d) * kLnPV + x) = make_uint2(l0, l1);
-  }
-  __syncthreads();
+  cp_commit();
+  for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
   const int r0 = warp * 16, g = lane >> 2, t4 = lane & 3;  // this warp's token rows
-  if (r0 >= len) return;
+  const bool mine = r0 < len;
+  uint32_t q[NK][4];  // query fragments, straight from the rows
+  {
+    const bool ok0 = r0 + g < len, ok1 = r0 + g + 8 < len;
+    const __nv_bfloat16* qa = p + h * dk + static_cast<long long>(ok0 ? r0 + g : 0) * a.ld + 2 * t4;
+    const __nv_bfloat16* qb = p + h * dk + static_cast<long long>(ok1 ? r0 + g + 8 : 0) * a.ld + 2 * t4;
+#pragma unroll
+    for (int kt = 0; kt < NK; ++kt) {
+      const bool lo = kt * 16 < dk, hi = kt * 16 + 8 < dk;  // (widths are multiples of 8)
+      q[kt][0] = ok0 && lo ? *reinterpret_cast<const uint32_t*>(qa + kt * 16) : 0u;
+      q[kt][1] = ok1 && lo ? *reinterpret_cast<const uint32_t*>(qb + kt * 16) : 0u;
+      q[kt][2] = ok0 && hi ? *reinterpret_cast<const uint32_t*>(qa + kt * 16 + 8) : 0u;
+      q[kt][3] = ok1 && hi ? *reinterpret_cast<const uint32_t*>(qb + kt * 16 + 8) : 0u;
+    }
+  }
+  cp_wait<1>();
+  __syncthreads();
   float o[8][4];
 #pragma unroll
   for (int n = 0; n < 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-  const uint32_t q_at = smem_u32(sQ + (r0 + (lane & 7) + ((lane >> 3) & 1) * 8) * P + (lane >> 4) * 8);
-  const uint32_t s_at = smem_u32(sS + ((lane & 7) + ((lane >> 3) & 1) * 8) * kLnPV + (lane >> 4) * 8);
   // ---- what the state contributes: decay^(t + 1) q_t S
+  if (mine) {
+    const uint32_t s_at = smem_u32(sS + ((lane & 7) + ((lane >> 3) & 1) * 8) * kLnPV + (lane >> 4) * 8);
 #pragma unroll
-  for (int kt = 0; kt < NK; ++kt) {
-    uint32_t q[4];
-    ldm_x4(q_at + kt * 32, q);
+    for (int kt = 0; kt < NK; ++kt)
 #pragma unroll
-    for (int np = 0; np < 4; ++np) {
-      uint32_t bh[4], bl[4];
-      ldm_x4_t(s_at + (kt * 16 * kLnPV + np * 16) * 2, bh);
-      ldm_x4_t(s_at + ((NK * 16 + kt * 16) * kLnPV + np * 16) * 2, bl);
-      mma16816(o[2 * np], q, bh[0], bh[1]);
-      mma16816(o[2 * np + 1], q, bh[2], bh[3]);
-      mma16816(o[2 * np], q, bl[0], bl[1]);
-      mma16816(o[2 * np + 1], q, bl[2], bl[3]);
-    }
+      for (int np = 0; np < 4; ++np) {
+        uint32_t bh[4], bl[4];
+        ldm_x4_t(s_at + (kt * 16 * kLnPV + np * 16) * 2, bh);
+        ldm_x4_t(s_at + ((NK * 16 + kt * 16) * kLnPV + np * 16) * 2, bl);
+        mma16816(o[2 * np], q[kt], bh[0], bh[1]);
+        mma16816(o[2 * np + 1], q[kt], bh[2], bh[3]);
+        mma16816(o[2 * np], q[kt], bl[0], bl[1]);
+        mma16816(o[2 * np + 1], q[kt], bl[2], bl[3]);
+      }
   }
+  cp_wait<0>();
+  __syncthreads();
+  if (!mine) return;
   const float d0 = pw[r0 + g + 1], d1 = pw[min(r0 + g + 9, kLnChunk)];
 #pragma unroll
   for (int n = 0; n < 8; ++n) {
@@ -379,11 +400,10 @@ __global__ void __launch_bounds__(256) lightning_chunk_out_kernel(const Lightnin
     float sc[2][4] = {};
 #pragma unroll
     for (int kt = 0; kt < NK; ++kt) {
-      uint32_t q[4], k[4];
-      ldm_x4(q_at + kt * 32, q);
+      uint32_t k[4];
       ldm_x4(k_at + (j * 16 * P + kt * 16) * 2, k);
-      mma16816(sc[0], q, k[0], k[1]);
-      mma16816(sc[1], q, k[2], k[3]);
+      mma16816(sc[0], q[kt], k[0], k[1]);
+      mma16816(sc[1], q[kt], k[2], k[3]);
     }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
@@ -426,6 +446,10 @@ static cudaError_t launch_chunked_t(const LightningArgs& a, const LightningChunk
     if (e == cudaSuccess) e = cudaFuncSetAttribute(lightning_chunk_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, LnOut<NK>::kBytes);
     if (e != cudaSuccess) return e;
   }
+  const int n = a.off_v + a.H * a.dv;
+  const unsigned vecs = static_cast<unsigned>(n) / 8 * static_cast<unsigned>(a.rows);
+  e = launch_pdl(lightning_act_kernel, dim3((vecs + 255) / 256), dim3(256), 0, st, a, static_cast<__nv_bfloat16*>(const_cast<void*>(a.p)), n);
+  if (e != cudaSuccess) return e;
   const dim3 grid(c.n_chunks, a.H, (a.dv + kLnCols - 1) / kLnCols);
   e = launch_pdl(lightning_chunk_kv_kernel<NK>, grid, dim3(256), LnKv<NK>::kBytes, st, a, c);
   if (e != cudaSuccess) return e;
@@ -437,6 +461,7 @@ static cudaError_t launch_chunked_t(const LightningArgs& a, const LightningChunk
 
 int launch_lightning_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st) {
   if (a.rows == 0 || c.n_chunks == 0) return 0;
+  if (a.off_k != a.H * a.dk || a.off_v != 2 * a.off_k || static_cast<long long>(a.rows) * (a.off_v + a.H * a.dv) / 8 > 0xffffff00ll) return 1;
   if (a.dk > 256 || a.chunk != kLnChunk || (a.dv + kLnCols - 1) / kLnCols > 65535) return 1;
   cudaError_t e;
   if (a.dk <= 32) e = launch_chunked_t<2>(a, c, st);

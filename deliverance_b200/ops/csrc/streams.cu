@@ -55,9 +55,22 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const StreamArgs a) {
       }
     inv = rsqrtf(block_sum(ss, red) / W + a.eps);
   };
-  float rd[SMAX];
+  // weights first: no kernel in front writes them, so their loads run under its tail
+  float rd[SMAX], wr[SMAX], mix[SMAX <= 4 ? SMAX : 1][SMAX <= 4 ? SMAX : 1], wn[NV <= 4 ? NV : 1][4];
+  const bool upd = !OPEN && sub != nullptr;
 #pragma unroll
-  for (int s = 0; s < SMAX; ++s) rd[s] = s < S && a.read != nullptr ? a.read[s] : 1.f;
+  for (int s = 0; s < SMAX; ++s) {
+    rd[s] = s < S && a.read != nullptr ? a.read[s] : 1.f;
+    wr[s] = upd && s < S ? a.write[s] : 0.f;
+    if constexpr (SMAX <= 4 && !OPEN)
+#pragma unroll
+      for (int q = 0; q < SMAX; ++q) mix[s][q] = upd && s < S && q < S ? a.mix[s * S + q] : 0.f;
+  }
+  if constexpr (NV <= 4) {
+    if (a.w_next != nullptr)
+#pragma unroll
+      for (int n = 0; n < NV; ++n) load(a.w_next, col(n), wn[n]);  // (zeros behind the row: so are the outputs there)
+  }
   pdl_wait();
   pdl_trigger();
   if constexpr (OPEN) {
@@ -81,15 +94,6 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const StreamArgs a) {
       for (int e = 0; e < 4; ++e) v[n][e] *= total;
     }
   } else {
-    float wr[SMAX], mix[SMAX][SMAX];
-    const bool upd = sub != nullptr;
-#pragma unroll
-    for (int s = 0; s < SMAX; ++s) {
-      wr[s] = upd && s < S ? a.write[s] : 0.f;
-      if constexpr (SMAX <= 4)
-#pragma unroll
-        for (int q = 0; q < SMAX; ++q) mix[s][q] = upd && s < S && q < S ? a.mix[s * S + q] : 0.f;
-    }
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
       const int c = col(n);
@@ -146,7 +150,12 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const StreamArgs a) {
     float o[4] = {v[n][0], v[n][1], v[n][2], v[n][3]};
     if (a.w_next != nullptr) {
       float w[4];
-      load(a.w_next, c, w);  // (zeros behind the row: so are the outputs there)
+      if constexpr (NV <= 4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[e] = wn[n][e];
+      } else {
+        load(a.w_next, c, w);
+      }
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[e] = (o[e] - mean) * inv * w[e];
     }
@@ -171,7 +180,7 @@ static cudaError_t stream_dispatch(const StreamArgs& a, int rows, cudaStream_t s
 }
 template <typename TIO>
 static cudaError_t stream_streams(const StreamArgs& a, int rows, cudaStream_t st) {
-  if (a.ids != nullptr) return stream_dispatch<TIO, kMaxStreams, true>(a, rows, st);
+  if (a.ids != nullptr) return a.S <= 2 ? stream_dispatch<TIO, 2, true>(a, rows, st) : stream_dispatch<TIO, kMaxStreams, true>(a, rows, st);
   if (a.S <= 2) return stream_dispatch<TIO, 2, false>(a, rows, st);
   if (a.S <= 4) return stream_dispatch<TIO, 4, false>(a, rows, st);
   return stream_dispatch<TIO, kMaxStreams, false>(a, rows, st);

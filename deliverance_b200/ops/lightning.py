@@ -6,7 +6,7 @@ real columns; ``silu(0) = 0``, so padded channels stay zero). The state is fp32,
 orders, the same numbers up to rounding:
 
 * recurrent (decode, fp32): every token updates the state in registers;
-* chunked (bf16 prompts): because the decay is a constant, what a chunk adds to the state does not depend on the state in front of it. All
+* chunked (bf16 prompts): the rows are activated in place. Because the decay is a constant, what a chunk adds to the state does not depend on the state in front of it. All
   chunks' contributions are computed at once, an elementwise pass turns them into the state in front of every chunk, and all chunks' outputs are
   computed at once. Weighted values, states and weights go through the tensor cores as pairs of bf16 numbers with fp32 accumulation.
 """
@@ -71,10 +71,10 @@ def decay_powers(decay) -> torch.Tensor:
 def lightning(s: LightningShape, p, decay, powers, norm_w, state, batch, eps: float, mult: float, out) -> None:
     """Rows of the projection -> normed, gated heads times ``mult`` in ``out [T, H * dv]`` (a column range of wider rows). ``decay``: fp64 ``[H]`` on
     the host; ``powers`` of :func:`decay_powers`, ``norm_w [H * dv]`` and ``state [slots, H, dk, dv]`` are fp32; the state slots of the batch's
-    sequences are advanced (a sequence at position 0 starts from zero)."""
+    sequences are advanced (a sequence at position 0 starts from zero). The q, k and v columns of ``p`` may be overwritten."""
     if ops._cuda(p):
         chunked = not (batch.is_decode or p.dtype == torch.float32 or s.dk > MAX_DK_CHUNKED)
-        ops._count(4 if chunked else 2)
+        ops._count(5 if chunked else 2)
         ops.require_ext().lightning(p, powers, CHUNK, norm_w, state, batch.state_slots, batch.q_start, batch.q_len, batch.positions, s.geometry(), eps, mult, out,
                                     list(chunk_plan(batch, CHUNK)) if chunked else [])
         return
