@@ -11,6 +11,8 @@
 #include "gemm_api.h"
 #include "io.cuh"
 
+#include <type_traits>
+
 namespace dlv {
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
@@ -253,14 +255,23 @@ __device__ __forceinline__ float attn_gate(const AttnExtra& x, const TIO* gate, 
 // grid (num_seqs, H), D threads rounded up to whole warps. The split weights are computed once per CTA (thread s takes split s) and kept
 // in shared memory; the weighted sum over the splits then runs with independent loads. (The first version had every thread walk
 // all splits twice with dependent loads: 12 us at 64 splits, more than the attention kernel it follows.)
+// EXT: with the options of AttnExtra.
+struct NoExtra {};
+template <bool EXT>
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits, const AttnExtra x) {
+                                    __nv_bfloat16* __restrict__ out, int H, int D, int splits,
+                                    const std::conditional_t<EXT, AttnExtra, NoExtra> x) {
   __shared__ float w_s[256];
   __shared__ float red[2][8];
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   const int b = blockIdx.x, h = blockIdx.y, d = threadIdx.x, lane = d & 31, wp = d >> 5, nw = (blockDim.x + 31) >> 5;
   const long long base = (static_cast<long long>(b) * H + h) * splits;
+  float factor = 1.f, sink = -INFINITY;  // (read here: their latency passes under the reductions)
+  if constexpr (EXT) {
+    if (d < D) factor = attn_gate(x, static_cast<const __nv_bfloat16*>(x.gate), b, h, h * D + d);
+    if (x.sink != nullptr) sink = x.sink[h];
+  }
   // maximum over the splits
   float m = -INFINITY;
   for (int s = d; s < splits; s += blockDim.x) m = fmaxf(m, part_ml[(base + s) * 2]);
@@ -282,7 +293,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   __syncthreads();
   den = 0.f;
   for (int i = 0; i < nw; ++i) den += red[1][i];
-  if (x.sink != nullptr) den += __expf(x.sink[h] - m);
+  if constexpr (EXT) den += __expf(sink - m);
   if (d >= D) return;
   float num = 0.f;
   const int n_fast = splits < 256 ? splits : 256;
@@ -292,8 +303,12 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
     const float ms = part_ml[(base + s) * 2];
     num += ((ms == -INFINITY) ? 0.f : __expf(ms - m)) * part_o[(base + s) * D + d];
   }
-  const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * D;
-  out[b * pitch + h * D + d] = f2bf(den > 0.f ? num / den * attn_gate(x, static_cast<const __nv_bfloat16*>(x.gate), b, h, h * D + d) : 0.f);
+  if constexpr (EXT) {
+    const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * D;
+    out[b * pitch + h * D + d] = f2bf(den > 0.f ? num / den * factor : 0.f);
+  } else {
+    out[(static_cast<long long>(b) * H + h) * D + d] = f2bf(den > 0.f ? num / den : 0.f);
+  }
 }
 
 template <int D, int GP>
@@ -320,7 +335,7 @@ static int launch_decode_t(const void* q, long long q_stride, const void* kc, co
                                                       scale, cap, window, splits);
   if (splits > 1) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits, AttnExtra{});
+    launch_pdl(decode_merge_kernel<false>, dim3(g2), dim3(D), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, D, splits, NoExtra{});
   }
   return 0;
 }
@@ -399,19 +414,31 @@ struct DecodeMma {
 
 // EXT 1: head widths below the tile width D, groups of more than 16 heads, kept first keys. Without it those are compile-time constants (as
 // run-time values they cost the plain kernel a tenth of its speed: the loop is paced by its address arithmetic). EXT 1 and 2: the options
-// of AttnExtra that only the epilogue sees (sink, output gate, output pitch).
+// of AttnExtra that only the epilogue sees (sink, output gate, output pitch); the plain kernel does not even carry them as parameters.
+template <int EXT>
+struct DecodeOptions {
+  int dk, dv;
+  AttnExtra x;
+};
+template <>
+struct DecodeOptions<0> {};
 template <int D, int EXT>
 __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, long long q_stride, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables, int bt_stride,
     const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, float* part_o, float* part_ml, int* __restrict__ arrivals,
-    int H, int KV, int page_size, float scale, float softcap, int window, int splits, int dk_ext, int dv_ext, const AttnExtra x) {
+    int H, int KV, int page_size, float scale, float softcap, int window, int splits, const DecodeOptions<EXT> opt) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   using L = DecodeMma<D>;
   constexpr int CPR = D / 8;  // 16-byte chunks per row
   extern __shared__ __align__(128) uint8_t msm[];
-  const int dk = EXT == 1 ? dk_ext : D, dv = EXT == 1 ? dv_ext : D, keep_first = EXT == 1 ? x.keep_first : 0;
+  int dk = D, dv = D, keep_first = 0;
+  if constexpr (EXT == 1) {
+    dk = opt.dk;
+    dv = opt.dv;
+    keep_first = opt.x.keep_first;
+  }
   // a CTA takes up to 16 of the query heads that share a KV head
   const int heads_per_kv = H / KV, groups = EXT == 1 ? (heads_per_kv + 15) / 16 : 1;
   const int b = blockIdx.x, kvh = blockIdx.y / groups, sp = blockIdx.z;
@@ -619,9 +646,12 @@ __global__ void __launch_bounds__(128, (D <= 128 ? 2 : 1)) decode_attn_mma_kerne
     }
     const int h = h0 + r;
     if (splits == 1) {
-      if (EXT != 0 && x.sink != nullptr) den += __expf(x.sink[h] - m);  // relative to the maximum
+      if constexpr (EXT != 0) {
+        if (opt.x.sink != nullptr) den += __expf(opt.x.sink[h] - m);  // relative to the maximum
+      }
       const float inv = den > 0.f ? 1.f / den : 0.f;
       if constexpr (EXT != 0) {
+        const AttnExtra& x = opt.x;
         const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(x.gate);
         n0 *= attn_gate(x, gate, b, h, h * dv + d);
         n1 *= attn_gate(x, gate, b, h, h * dv + d + 1);
@@ -707,13 +737,17 @@ static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc
     cudaFuncSetAttribute(decode_attn_mma_kernel<D, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
   }
   dim3 grid(B, KV * ((H / KV + 15) / 16), splits);
+  DecodeOptions<EXT> opt;
+  if constexpr (EXT != 0) opt = {dk, dv, x};
   launch_pdl(decode_attn_mma_kernel<D, EXT>, dim3(grid), dim3(128), L::kBytes, st, static_cast<const __nv_bfloat16*>(q), q_stride,
                                                           static_cast<const __nv_bfloat16*>(kc), static_cast<const __nv_bfloat16*>(vc), bt,
                                                           bt_stride, ctx, static_cast<__nv_bfloat16*>(out), po, pml, arrivals, H, KV, page, scale,
-                                                          cap, window, splits, dk, dv, x);
+                                                          cap, window, splits, opt);
   if (splits > 1 && arrivals == nullptr) {
     dim3 g2(B, H);
-    launch_pdl(decode_merge_kernel, dim3(g2), dim3((dv + 31) / 32 * 32), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x);
+    const dim3 block((dv + 31) / 32 * 32);
+    if constexpr (EXT != 0) launch_pdl(decode_merge_kernel<true>, g2, block, 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x);
+    else launch_pdl(decode_merge_kernel<false>, g2, block, 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, NoExtra{});
   }
   return 0;
 }
