@@ -267,11 +267,20 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
   const int b = blockIdx.x, h = blockIdx.y, d = threadIdx.x, lane = d & 31, wp = d >> 5, nw = (blockDim.x + 31) >> 5;
   const long long base = (static_cast<long long>(b) * H + h) * splits;
-  float factor = 1.f, sink = -INFINITY;  // (read here: their latency passes under the reductions)
+  float logit = 0.f, sink = -INFINITY;  // (read here: their latency passes under the reductions)
   if constexpr (EXT) {
-    if (d < D) factor = attn_gate(x, static_cast<const __nv_bfloat16*>(x.gate), b, h, h * D + d);
+    if (x.gate != nullptr && d < D) logit = bf2f(static_cast<const __nv_bfloat16*>(x.gate)[b * x.gate_pitch + (x.gate_heads ? h : h * D + d)]);
     if (x.sink != nullptr) sink = x.sink[h];
   }
+  // the first partials are on their way while the weights are worked out; the rest follows in batches of independent loads
+  constexpr int BATCH = 16;
+  const float* po = part_o + base * D + d;
+  float v[BATCH];
+  auto fetch = [&](int s0) {
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j) v[j] = d < D && s0 + j < splits ? po[static_cast<long long>(s0 + j) * D] : 0.f;
+  };
+  fetch(0);
   // maximum over the splits
   float m = -INFINITY;
   for (int s = d; s < splits; s += blockDim.x) m = fmaxf(m, part_ml[(base + s) * 2]);
@@ -297,14 +306,19 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   if (d >= D) return;
   float num = 0.f;
   const int n_fast = splits < 256 ? splits : 256;
-#pragma unroll 8
-  for (int s = 0; s < n_fast; ++s) num += w_s[s] * part_o[(base + s) * D + d];
+  for (int s0 = 0; s0 < n_fast; s0 += BATCH) {
+    if (s0 > 0) fetch(s0);
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j)
+      if (s0 + j < n_fast) num += w_s[s0 + j] * v[j];
+  }
   for (int s = n_fast; s < splits; ++s) {  // (more than 256 splits: weights recomputed)
     const float ms = part_ml[(base + s) * 2];
     num += ((ms == -INFINITY) ? 0.f : __expf(ms - m)) * part_o[(base + s) * D + d];
   }
   if constexpr (EXT) {
     const long long pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * D;
+    const float factor = x.gate != nullptr ? x.out_mult / (1.f + expf(-logit)) : x.out_mult;
     out[b * pitch + h * D + d] = f2bf(den > 0.f ? num / den * factor : 0.f);
   } else {
     out[(static_cast<long long>(b) * H + h) * D + d] = f2bf(den > 0.f ? num / den : 0.f);
