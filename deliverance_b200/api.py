@@ -132,6 +132,10 @@ def build_model(cfg: ModelConfig, device, dtype, tp: TensorParallelContext):
         from .models.dubozen import DubozenModel
 
         return DubozenModel(cfg, device, dtype, tp)
+    if cfg.model_type == "gevovik":
+        from .models.gevovik import GevovikModel
+
+        return GevovikModel(cfg, device, dtype, tp)
     return DecoderModel(cfg, device, dtype, tp)
 
 

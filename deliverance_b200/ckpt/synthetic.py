@@ -15,7 +15,7 @@ from .loader import ShardSpec, shard_dense, shard_q4
 from .quantizer import DEFAULT_Q4_FILTER
 from .safetensors_io import Q4Tensor, TensorInfo
 from ..config import config_model_type
-from .tiny import build_tensors, dubozen_shapes, dubozen_value, fatotar_is_norm, fatotar_shapes, fopivik_is_norm, fopivik_shapes  # noqa: F401  (small models reuse the tiny builder)
+from .tiny import build_tensors, dubozen_shapes, dubozen_value, fatotar_is_norm, fatotar_shapes, fopivik_is_norm, fopivik_shapes, gevovik_shapes, gevovik_value  # noqa: F401  (small models reuse the tiny builder)
 
 
 def _shapes(cfg: dict) -> dict[str, tuple]:
@@ -27,6 +27,8 @@ def _shapes(cfg: dict) -> dict[str, tuple]:
         return fopivik_shapes(cfg)
     if mt == "dubozen":
         return dubozen_shapes(cfg)
+    if mt == "gevovik":
+        return gevovik_shapes(cfg)
     h, L, V = cfg["hidden_size"], cfg["num_hidden_layers"], cfg["vocab_size"]
     nh, nkv = cfg["num_attention_heads"], cfg.get("num_key_value_heads") or cfg["num_attention_heads"]
     hd = cfg.get("head_dim") or h // nh
@@ -100,6 +102,8 @@ class SyntheticLoader:
             return (1.0 + torch.randn(shape, generator=g, device=self.device) * 0.02).to(self.dtype)
         if config_model_type(self.cfg) == "dubozen":
             return dubozen_value(name, torch.randn(shape, generator=g, device=self.device), self.cfg).to(self.dtype)
+        if config_model_type(self.cfg) == "gevovik":
+            return gevovik_value(name, torch.randn(shape, generator=g, device=self.device), self.cfg).to(self.dtype)
         if config_model_type(self.cfg) == "fopivik":
             r = torch.randn(shape, generator=g, device=self.device)
             if fopivik_is_norm(name):

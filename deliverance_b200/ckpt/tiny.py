@@ -233,7 +233,115 @@ def _dubozen_tensors(cfg: dict, seed: int, dtype) -> dict:
     return {n: dubozen_value(n, torch.randn(shape, generator=g, dtype=torch.float32), cfg).to(dtype) for n, shape in dubozen_shapes(cfg).items()}
 
 
+def gevovik_config(width: int, vocab: int, layers: list, eps: float = 1e-5, scale: float = 4.0, buckets: int = 61, mul: tuple = (13, 5), **extra) -> dict:
+    """``config.json`` of a Gevovik model. ``layers``: one dict of sizes per layer, told apart by their keys: ``state`` (Mamba-2: ``heads, vdim, state,
+    groups, conv, norm_groups``), ``right`` = ``(heads, kv_heads, dim, vdim, conv)`` of the gated delta rule beside attention (``heads, kv_heads, dim,
+    vdim, window, rot_dims, base, scaling, scale, left_scale, right_scale``; ``ranks`` = sizes of the two low-rank projections, kept in the weights
+    only), else latent attention (``heads, dim, rot_dim, vdim, kv_rank, base, scale, kv_from``). ``ff`` 0 = no feed-forward."""
+    out, ranks = [], {}
+    for i, L in enumerate(layers):
+        mlp = {"kind": "dense", "ff": L["ff"]} if L.get("ff") else None
+        if "state" in L:
+            kind, m = "mamba2", {k: L[k] for k in ("heads", "vdim", "state", "groups", "conv")}
+            m["norm_groups"] = L.get("norm_groups", 1)
+        elif "right" in L:
+            kind = "parallel"
+            left = {k: L[k] for k in ("heads", "kv_heads", "dim")}
+            rot = {"dims": L.get("rot_dims", L["dim"] // 2 * 2), "base": L.get("base", 10000.0)}
+            if L.get("scaling"):
+                rot["scaling"] = L["scaling"]
+            left.update(vdim=L.get("vdim", L["dim"]), rot=rot, scale=L.get("scale", L["dim"] ** -0.5), mask={"size": L["window"]})
+            m = {"left": left, "left_scale": L.get("left_scale", 0.7), "right": dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), L["right"])),
+                 "right_scale": L.get("right_scale", 0.8)}
+            ranks[str(i)] = list(L.get("ranks", (8, 8)))
+        else:
+            kind, m = "latent_attention", {k: L[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank")}
+            m.update(rot={"dims": L["rot_dim"], "base": L.get("base", 10000.0)}, scale=L.get("scale", (L["dim"] + L["rot_dim"]) ** -0.5))
+            if L.get("kv_from") is not None:
+                m["kv_from"] = L["kv_from"]
+        out.append({"type": kind, "mixer": m, "mlp": mlp})
+    cfg = {"architecture": "Gevovik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": out, "_ranks": ranks,
+           "embedding": {"scale": scale, "bigram": {"buckets": buckets, "mul_prev": mul[0], "mul_cur": mul[1]}}}
+    cfg.update(extra)
+    return cfg
+
+
+def gevovik_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape of a Gevovik checkpoint."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "final.norm": (), "head": (V, W)}
+    if cfg["embedding"].get("bigram"):
+        s["bigram"] = (cfg["embedding"]["bigram"]["buckets"] + 1, W)
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        a = p + "mix."
+        s[p + "norm1"] = ()
+        if L["type"] == "mamba2":
+            H, I, GN = m["heads"], m["heads"] * m["vdim"], m["groups"] * m["state"]
+            s.update({a + "in": (2 * I + 2 * GN + H, W), a + "conv": (I + 2 * GN, m["conv"]), a + "conv.b": (I + 2 * GN,), a + "dt_bias": (H,), a + "A_log": (H,),
+                      a + "D": (H,), a + "norm": (I,), a + "o": (W, I)})
+        elif L["type"] == "parallel":
+            l, r = m["left"], m["right"]
+            H, G, dk, dv, b = l["heads"], l["kv_heads"], l["dim"], l["vdim"], a + "left."
+            s.update({b + "q": (H * dk, W), b + "k": (G * dk, W), b + "v": (G * dv, W), b + "q.norm": (dk,), b + "k.norm": (dk,), b + "talk": (H, H), b + "temp": (H,),
+                      b + "g": (H, W), b + "o": (W, H * dv)})
+            H, G, dk, dv, b = r["heads"], r["kv_heads"], r["dim"], r["vdim"], a + "right."
+            ra, rg = cfg["_ranks"][str(i)]
+            for n, rows in (("q", G * dk), ("k", G * dk), ("v", H * dv)):
+                s.update({b + n: (rows, W), f"{b}{n}.conv": (rows, r["conv"])})
+            s.update({b + "b": (H, W), b + "A_log": (H,), b + "norm": (dv,), b + "a1": (ra, W), b + "a2": (H * dk, ra), b + "dt_bias": (H * dk,), b + "g1": (rg, W),
+                      b + "g2": (H * dv, rg), b + "o": (W, H * dv)})
+        else:
+            H, d, dr, dv, R = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+            s.update({a + "q": (H * (d + dr), W), a + "uk": (H * d, R), a + "uv": (H * dv, R), a + "sink": (H,), a + "o": (W, H * dv)})
+            if m.get("kv_from") is None:
+                s.update({a + "dkv": (R + dr, W), a + "dkv.norm": (R,)})
+        if L.get("mlp"):
+            F = L["mlp"]["ff"]
+            s.update({p + "norm2": (), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+    return s
+
+
+def gevovik_value(name: str, r, cfg: dict):
+    """Weight ``name`` from standard normal numbers ``r`` of its shape: projections scaled by their fan-in, decays from slow to fast, every mechanism
+    moving the output."""
+    last = name.rsplit(".", 1)[-1]
+    if "norm" in last or last == "D":
+        return 1.0 + 0.2 * r
+    if last == "A_log":
+        return 1.2 * r - 1.5
+    if last == "dt_bias":
+        return r - 2.0
+    if last == "sink":
+        return 1.5 + r
+    if last == "temp":
+        return 1.2 + 0.3 * r
+    if last == "talk":
+        return 0.7 * torch.eye(r.shape[0], dtype=r.dtype, device=r.device) + 0.3 * r
+    if last == "conv":
+        return 0.5 * r + 0.3
+    if name.endswith("conv.b"):
+        return 0.3 * r
+    if len(r.shape) == 2 and name not in ("embed", "bigram"):
+        return r * r.shape[1] ** -0.5 * (3.0 if name.endswith("left.q") or name.endswith("mix.q") else 1.0)
+    return r
+
+
+def _gevovik_tensors(cfg: dict, seed: int, dtype) -> dict:
+    g = torch.Generator().manual_seed(seed)
+    return {n: gevovik_value(n, torch.randn(shape, generator=g, dtype=torch.float32), cfg).to(dtype) for n, shape in gevovik_shapes(cfg).items()}
+
+
 def tiny_config(model_type: str, **over) -> dict:
+    if model_type == "gevovik":
+        ssd = dict(heads=6, vdim=12, state=20, groups=3, conv=4, norm_groups=2, ff=52)
+        both = dict(heads=6, kv_heads=2, dim=20, vdim=28, rot_dims=12, window=24, right=(4, 2, 12, 20, 3), ranks=(10, 6), ff=36)
+        lat = dict(heads=3, dim=20, rot_dim=6, vdim=12, kv_rank=40, ff=24)
+        yarn = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 2.0}
+        kw = dict(width=76, vocab=261, layers=[dict(lat), dict(ssd), dict(both, scaling=yarn, base=500.0), dict(lat, heads=2, vdim=20, kv_from=0, ff=0), dict(both, kv_heads=6),
+                                               dict(ssd, heads=4, groups=1, conv=2, norm_groups=1, ff=0)])
+        kw.update(over)
+        return gevovik_config(**kw)
     if model_type == "dubozen":
         soft = dict(heads=6, kv_heads=2, dim=20, vdim=28, rot_dims=12, ff=52)
         both = dict(heads=4, kv_heads=1, dim=18, rot_dims=10, base=500.0, right=(3, 12, 20, (0.4, 0.97, 0.999)), ff=36, experts=6, top=2, groups=3, keep=2)
@@ -302,6 +410,8 @@ def build_tensors(cfg: dict, seed: int = 0, dtype=torch.float32, std: float = 0.
         return _fopivik_tensors(cfg, seed, dtype)
     if mt == "dubozen":
         return _dubozen_tensors(cfg, seed, dtype)
+    if mt == "gevovik":
+        return _gevovik_tensors(cfg, seed, dtype)
     R = lambda *s: _rand(g, *s, std=std, dtype=dtype)  # noqa: E731
     ones = lambda n: (torch.ones(n) + torch.randn(n, generator=g) * 0.05).to(dtype)  # noqa: E731
     t: dict = {}

@@ -19,10 +19,10 @@ from typing import Any, Optional
 
 SUPPORTED_MODEL_TYPES = (
     "llama", "mistral", "mixtral", "gemma2", "gemma3_text", "gemma3", "gemma4_text", "gemma4", "qwen2", "qwen3", "qwen3_moe", "gpt2", "granitemoehybrid", "bert", "fatotar", "fopivik",
-    "dubozen",
+    "dubozen", "gevovik",
 )
 # designs whose config.json names an architecture instead of a model_type
-_ARCHITECTURE_TYPES = {"fatotar": "fatotar", "fopivik": "fopivik", "dubozen": "dubozen"}
+_ARCHITECTURE_TYPES = {"fatotar": "fatotar", "fopivik": "fopivik", "dubozen": "dubozen", "gevovik": "gevovik"}
 
 # transformers' Gemma3TextConfig defaults: hub configs of the multimodal checkpoints leave most text fields out
 _GEMMA3_TEXT_DEFAULTS = dict(vocab_size=262208, hidden_size=2304, intermediate_size=9216, num_hidden_layers=26, num_attention_heads=8,
@@ -304,6 +304,38 @@ def _parse_dubozen(d: dict) -> ModelConfig:
     return cfg
 
 
+def _parse_gevovik(d: dict) -> ModelConfig:
+    """Gevovik: Mamba-2, windowed grouped attention with mixed scores beside a gated delta rule, and latent attention with a sink in any order, plain
+    feed-forwards, a norm with one gain behind every sublayer, a hashed-bigram embedding. A latent layer may read the cache of an earlier one
+    (``kv_from``). Every layer carries its own sizes; ``extra["layers"]`` keeps them as given. The context length is not part of the design."""
+    layers = list(d["layers"])
+    if not layers:
+        raise ValueError("no layers")
+    for i, L in enumerate(layers):
+        if L["type"] not in ("mamba2", "parallel", "latent_attention"):
+            raise ValueError(f"layer {i}: unknown mixer '{L['type']}'")
+        if L.get("mlp") and L["mlp"]["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward '{L['mlp']['kind']}'")
+        m, src = L["mixer"], L["mixer"].get("kv_from") if L["type"] == "latent_attention" else None
+        if src is not None:
+            if not 0 <= src < i or layers[src]["type"] != "latent_attention" or layers[src]["mixer"].get("kv_from") is not None:
+                raise ValueError(f"layer {i}: kv_from {src} is not an earlier latent-attention layer with a cache of its own")
+            if any(layers[src]["mixer"][k] != m[k] for k in ("kv_rank", "rot_dim", "rot")):
+                raise ValueError(f"layer {i}: latent size or rotation differs from that of layer {src}, whose cache it reads")
+    soft = [L["mixer"]["left"] if L["type"] == "parallel" else L["mixer"] for L in layers if L["type"] != "mamba2"]
+    cfg = ModelConfig(
+        model_type="gevovik", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), num_layers=len(layers),
+        num_heads=max([int(m["heads"]) for m in soft] or [1]), num_kv_heads=1, head_dim=max([int(m["dim"]) for m in soft] or [8]),
+        intermediate_size=max([int(L["mlp"]["ff"]) for L in layers if L.get("mlp")] or [0]),
+        max_position_embeddings=int(d.get("max_position_embeddings") or 131072), norm_eps=float(d["norm"]["eps"]), hidden_act="relu2",
+        embedding_multiplier=float(d["embedding"].get("scale", 1.0)), bos_token_id=d.get("bos_token_id"), eos_token_ids=_eos(d.get("eos_token_id")),
+        pad_token_id=d.get("pad_token_id"), layer_types=tuple({"mamba2": "mamba", "parallel": "sliding"}.get(L["type"], "latent") for L in layers),
+        use_rope=False, add_bos=False, raw=d,
+    )
+    cfg.extra = {"layers": layers, "bigram": d["embedding"].get("bigram")}
+    return cfg
+
+
 def _eos(v: Any) -> tuple[int, ...]:
     if v is None:
         return ()
@@ -332,6 +364,8 @@ def parse_config(d: dict) -> ModelConfig:
         return _parse_fopivik(d)
     if mt == "dubozen":
         return _parse_dubozen(d)
+    if mt == "gevovik":
+        return _parse_gevovik(d)
     if mt in ("gemma4", "gemma4_text"):
         return _parse_gemma4(d)
     if mt in ("gemma3", "gemma3_text"):

@@ -20,7 +20,7 @@ import os
 import sys
 
 MAX_LIVE = 4
-FLOAT32_FAMILIES = ("fatotar", "fopivik", "dubozen")  # CUDA families with a true 32-bit path
+FLOAT32_FAMILIES = ("fatotar", "fopivik", "dubozen", "gevovik")  # CUDA families with a true 32-bit path
 
 
 def open_engine(model_dir: str, dtype: str, max_tokens: int, device: str = "auto", max_live: int = MAX_LIVE):

@@ -134,7 +134,7 @@ class FatotarModel(DecoderModel):
             with self._stage("layernorm"):
                 x1, x2 = ops.add_layernorm(residual, delta, lw.norm1, lw.norm2, eps, pitch, dt)
             row = (torch.zeros if lw.padded else torch.empty)(T, lw.row, dtype=dt, device=self.device)
-            lw.mixer.forward(x1, batch, kv.layer(run), row, self._stage)
+            lw.mixer.heads(x1, batch, kv.layer(run), row, self._stage)
             if lw.ff:
                 with self._stage("mlpblock.gate_up_projection"):
                     gu = ops.linear(x2, lw.gate_up)

@@ -1,5 +1,5 @@
 """Grouped-query attention mixer with per-layer sizes (``ops/grouped.py``): any decoder can use it. Score scale, soft-cap, window, kept
-first tokens, sink, rotation tables and layout, head norms, value mixing and output gate are parameters; it reads its input rows, keeps its
+first tokens, sink, rotation tables and layout, head norms, mixed scores, value mixing and output gate are parameters; it reads its input rows, keeps its
 cache in the pair ``kv.layer(i)`` and returns the output projection (:meth:`forward`), or works between projections that it shares with
 another mixer (:meth:`pack`, :meth:`heads`)."""
 from __future__ import annotations
@@ -27,15 +27,18 @@ class GroupedAttention:
         self.cos, self.sin, self.rotate = cos, sin, rotate
         self.eps, self.mult, self.v_mix = float(eps), float(mult), bool(v_mix)
         self.lam = 0.0
-        self.q_norm = self.k_norm = None
+        self.q_norm = self.k_norm = self.mix = None
         self.device, self.dtype = device, dtype
         if cos.shape[1] * 2 > shape.dim:
             raise ValueError(f"rotation covers {cos.shape[1] * 2} of {shape.dim} query / key columns")
-        if rotate not in ("pairs", "halves") or (rotate == "pairs" and (shape.tied or v_mix)):
-            raise ValueError("tied and mixed values need the 'halves' rotation")
+        if rotate not in ("pairs", "halves") or (rotate == "pairs" and (shape.tied or v_mix or shape.mixed)):
+            raise ValueError("tied values, mixed values and mixed scores need the 'halves' rotation")
+        if shape.mixed and (softcap or keep_first or sink):
+            raise ValueError("mixed scores go without soft-cap, kept tokens and sink")
 
-    def pack(self, q, k, v, o, g=None, sink=None, q_norm=None, k_norm=None, vmix: Optional[float] = None) -> tuple:
-        """Weights as stored (``[out, in]``) -> (rows of the input projection, columns of the output projection) in the padded layout."""
+    def pack(self, q, k, v, o, g=None, sink=None, q_norm=None, k_norm=None, vmix: Optional[float] = None, mix=None) -> tuple:
+        """Weights as stored (``[out, in]``) -> (rows of the input projection, columns of the output projection) in the padded layout. ``mix [H, H]`` (to,
+        from): head h's score becomes ``sum_g mix[h, g] score_g`` in front of the softmax."""
         s = self.shape
         want = [("q", q, s.heads * s.dim), ("k", k, s.kv_heads * s.dim)]
         if not s.tied:
@@ -65,6 +68,10 @@ class GroupedAttention:
             self.q_norm, self.k_norm = norm(q_norm), norm(k_norm)
         if vmix is not None:
             self.lam = float(vmix)
+        if s.mixed != (mix is not None) or (mix is not None and tuple(mix.shape) != (s.heads, s.heads)):
+            raise ValueError(f"grouped attention: mixed scores need a [{s.heads}, {s.heads}] matrix")
+        if mix is not None:
+            self.mix = mix.to(device=self.device, dtype=torch.float32).contiguous()
         return w, pad_head_columns(o, s.heads, s.vdim, s.dv)
 
     def load(self, q, k, v, o, k_pad: int, **extra) -> "GroupedAttention":
@@ -103,7 +110,7 @@ class GroupedAttention:
                         raise ValueError(f"values of {v.shape[1]} columns cannot be mixed with {first.shape[1]}")
                 gop.rope_heads_kv(s, p, batch.positions, batch.slots, self.cos, self.sin, k_cache, v_cache, self.q_norm, self.k_norm, self.eps, first, self.lam)
         with stage("groupedattention.score_value"):
-            return gop.attention(s, p, batch, k_cache, v_cache, self.scale, self.softcap, self.window, self.keep_first, self.sink, self._splits(batch), self.mult, out)
+            return gop.attention(s, p, batch, k_cache, v_cache, self.scale, self.softcap, self.window, self.keep_first, self.sink, self._splits(batch), self.mult, out, self.mix)
 
     def _splits(self, batch: ForwardBatch) -> int:
         """Split-KV factor of a decode step: a captured step knows the window but not the contexts it will see."""
@@ -112,7 +119,11 @@ class GroupedAttention:
         span = max(batch.ctx_len_host) if batch.ctx_len_host else self.cos.shape[0]
         if self.window > 0:
             span = min(span, self.window + self.keep_first)
+        if self.shape.mixed:  # (a CTA takes all heads)
+            return gop.mixed_splits(batch.num_seqs, span)
         return ops.decode_splits(batch.num_seqs, self.shape.kv_heads * ((self.shape.heads // self.shape.kv_heads + 15) // 16), span)
 
     def cache_layout(self) -> dict:
+        if self.shape.mixed:  # one wide row per token
+            return {"heads": 1, "k": self.shape.k_width, "v": self.shape.v_width, "state": None}
         return {"heads": self.shape.kv_heads, "k": self.shape.dk, "v": self.shape.dv, "state": None}

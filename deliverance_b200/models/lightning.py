@@ -34,10 +34,13 @@ class LightningAttention:
         self.norm = pad_head_rows(norm.float().reshape(-1, 1), H, s.vdim, s.dv).reshape(-1).to(self.device).contiguous()
         return w, pad_head_columns(o, H, s.vdim, s.dv)
 
-    def heads(self, p, batch: ForwardBatch, state, out, stage) -> None:
+    def nbytes(self) -> int:
+        return (self.norm.numel() + self.powers.numel()) * 4
+
+    def heads(self, p, batch: ForwardBatch, kv, run: int, out, stage) -> None:
         """``p [T, shape.width]``: this mixer's columns of the projection rows; the heads go to ``out [T, H * dv]``."""
         with stage("lightning.recurrence"):
-            lop.lightning(self.shape, p, self.decay, self.powers, self.norm, state, batch, self.eps, self.mult, out)
+            lop.lightning(self.shape, p, self.decay, self.powers, self.norm, kv.state["lightning"][run], batch, self.eps, self.mult, out)
 
-    def state_shape(self) -> tuple:
-        return self.shape.heads, self.shape.dk, self.shape.dv
+    def state_shapes(self) -> dict:
+        return {"lightning": (self.shape.heads, self.shape.dk, self.shape.dv)}

@@ -1,85 +1,67 @@
-"""Mamba2 mixer layer of granitemoehybrid.
+"""Mamba-2 mixer (``ops/mamba.py``): any decoder can use it. It reads its input rows, keeps a ring of convolution inputs and one fp32 state per
+sequence in the cache manager's state slots and returns the output projection.
 
-in_proj -> split ``[gate (I) | x (I) | B (G*S) | C (G*S) | dt (H)]`` -> ``dt = softplus(dt + dt_bias)`` -> causal depthwise
-conv1d with a rolling state + SiLU -> SSM recurrence ``h = h * exp(dt*A) + B * dt * x``, ``y = C.h + D*x`` -> ``y *= silu(gate)``
--> RMSNorm over the whole intermediate -> out_proj (reference: core/.../model/granitemoehybrid/GraniteMoeHybridMambaLayer.java:
-130-252; the reference walks tokens one by one). Per-sequence conv / SSM state lives in the KV manager's state slots and is
-reset when a sequence starts at position 0. On CUDA the scan runs chunked (csrc/mamba.cu): intra-chunk work is
-parallel over (head, d_head) with the state carried across chunks; decode is the single-token variant of the same kernel.
+granitemoehybrid's Mamba-2 layers run on the same operator (:func:`mamba_forward`; reference: core/.../model/granitemoehybrid/
+GraniteMoeHybridMambaLayer.java:130-252, which walks tokens one by one): ``[gate | x | B | C | dt]`` projection, causal depthwise convolution with a
+rolling state + SiLU, recurrence, ``silu(gate)``, RMS norm over the whole intermediate, output projection.
 """
 from __future__ import annotations
 
 import torch
 
 from .. import ops
-from ..ops import ref
+from ..ops import LinearWeight, mamba as mamba_op
+from ..ops.grouped import pad_head_columns, up8
+from ..ops.mamba import Mamba2Shape, Mamba2Weights
+from ..ops.short_conv import MAX_TAPS
+from .batch import ForwardBatch
+
+
+class Mamba2Mixer:
+    kind = "mamba"
+
+    def __init__(self, shape: Mamba2Shape, eps: float, device, dtype):
+        self.shape, self.eps = shape, float(eps)
+        self.device, self.dtype = device, dtype
+        if device.type == "cuda" and (shape.dn > mamba_op.MAX_STATE or shape.taps > MAX_TAPS):
+            raise ValueError(f"Mamba-2: state size {shape.state}, {shape.taps} taps (at most {mamba_op.MAX_STATE} and {MAX_TAPS} on CUDA)")
+
+    def load(self, w_in, conv, conv_b, dt_bias, A_log, D, norm, o, k_pad: int) -> "Mamba2Mixer":
+        """Weights as stored (``[out, in]``); ``k_pad``: padded input width of the rows :meth:`forward` gets."""
+        s = self.shape
+        rows = 2 * s.heads * s.vdim + 2 * s.groups * s.state + s.heads
+        if w_in.shape[0] != rows or o.shape[1] != s.heads * s.vdim:
+            raise ValueError(f"Mamba-2: projections of {w_in.shape[0]} rows and {o.shape[1]} columns, the configured sizes need {rows} and {s.heads * s.vdim}")
+        w = s.pad_input(w_in)
+        w = torch.nn.functional.pad(w, (0, k_pad - w.shape[1], 0, up8(w.shape[0]) - w.shape[0]))
+        put = lambda t: LinearWeight(t.to(device=self.device, dtype=self.dtype).contiguous())  # noqa: E731
+        self.w_in, self.w_out = put(w), put(pad_head_columns(o, s.heads, s.vdim, s.dv))
+        self.w = Mamba2Weights.pack(s, conv, conv_b, dt_bias, A_log, D, norm, self.device)
+        return self
+
+    def nbytes(self) -> int:
+        return self.w_in.nbytes() + self.w_out.nbytes() + self.w.conv.numel() * 4
+
+    def forward(self, x, batch: ForwardBatch, kv, run: int, stage) -> torch.Tensor:
+        with stage("mamba.input_projection"):
+            p = ops.linear(x, self.w_in)
+        with stage("mamba.recurrence"):
+            y = mamba_op.mamba2(self.shape, p, self.w, kv.state["conv"][run], kv.state["ssm"][run], batch, self.eps)
+        with stage("mamba.output_projection"):
+            return ops.linear(y, self.w_out)
+
+    def cache_layout(self) -> dict:
+        return {"heads": 1, "k": 8, "v": 8, "state": self.shape.state_shapes()}
 
 
 def mamba_forward(model, i: int, lw, x: torch.Tensor, batch, kv) -> torch.Tensor:
-    cfg = model.cfg
-    m = lw.mamba
-    zx = ops.linear(x, m["in_proj"], out_f32=False)
-    conv_state, ssm_state = kv.state["conv"][i], kv.state["ssm"][i]
-    I = cfg.mamba_intermediate
-    if x.device.type == "cuda":
-        e = ops.require_ext()
-        meta = _chunk_meta(batch, x.device)
-        ops._count(5 if not meta["multi"] else 7)
-        y = e.mamba2_forward(zx, m["conv_w"].reshape(-1), m["conv_b"], m["dt_bias"], m["A_log"], m["D"], m["norm_w"], conv_state, ssm_state,
-                             batch.state_slots, batch.q_start, batch.q_len, batch.positions, meta["row_seq"], meta["chunk_seq"],
-                             meta["chunk_row0"], meta["chunk_len"], meta["chunk_first"], meta["chunk_last"], meta["seq_chunk0"],
-                             meta["seq_nchunks"], meta["multi"], cfg.mamba_n_heads, cfg.mamba_d_head, cfg.mamba_n_groups, cfg.mamba_d_state,
-                             cfg.norm_eps)
-        return ops.linear(y, m["out_proj"])
-    out = torch.empty(x.shape[0], I, dtype=torch.float32)
-    qs, ql = batch.q_start.tolist(), batch.q_len.tolist()
-    slots = batch.state_slots.tolist()
-    starts = [int(batch.positions[s]) for s in qs]
-    for s, (a, n) in enumerate(zip(qs, ql)):
-        if n == 0:
-            continue
-        slot = slots[s]
-        if starts[s] == 0:
-            conv_state[slot].zero_()
-            ssm_state[slot].zero_()
-        out[a : a + n] = ref.mamba2_sequential(zx[a : a + n], m["conv_w"], m["conv_b"], m["dt_bias"], m["A_log"], m["D"], m["norm_w"],
-                                               cfg.norm_eps, cfg.mamba_n_heads, cfg.mamba_d_head, cfg.mamba_n_groups, cfg.mamba_d_state,
-                                               conv_state[slot], ssm_state[slot], "silu")
-    return ops.linear(out.to(x.dtype), m["out_proj"])
-
-
-CHUNK = 128
-
-
-def _chunk_meta(batch, device) -> dict:
-    """Index tensors of the chunked scan (cached on the batch). Decode batches build them with device ops only, so the
-    step stays capturable in a CUDA graph."""
-    cached = getattr(batch, "_mamba_meta", None)
-    if cached is not None:
-        return cached
-    i32 = dict(dtype=torch.int32, device=device)
-    if batch.is_decode:
-        n = batch.num_seqs
-        ar = torch.arange(n, **i32)
-        one = torch.ones(n, **i32)
-        meta = {"row_seq": ar, "chunk_seq": ar, "chunk_row0": ar, "chunk_len": one, "chunk_first": one, "chunk_last": one,
-                "seq_chunk0": ar, "seq_nchunks": one, "multi": False}
+    """One granitemoehybrid Mamba-2 layer: the projections are the model's (possibly JQ4) weights."""
+    m, s = lw.mamba, lw.mamba["shape"]
+    w = m["in_proj"]
+    if x.device.type == "cuda" and w.N % 8:  # the kernels read 16-byte pieces of the rows
+        p = torch.empty(x.shape[0], up8(w.N), dtype=x.dtype, device=x.device)
+        ops.linear(x, w, out=p[:, : w.N])
     else:
-        qs, ql = batch.q_start.tolist(), (batch.q_len_host or batch.q_len.tolist())
-        row_seq, cseq, crow, clen, cfirst, clast, s0, sn = [], [], [], [], [], [], [], []
-        for s, (a, n) in enumerate(zip(qs, ql)):
-            row_seq += [s] * n
-            s0.append(len(cseq))
-            nc = max(1, (n + CHUNK - 1) // CHUNK)
-            sn.append(nc)
-            for c in range(nc):
-                cseq.append(s)
-                crow.append(a + c * CHUNK)
-                clen.append(max(0, min(CHUNK, n - c * CHUNK)))
-                cfirst.append(1 if c == 0 else 0)
-                clast.append(1 if c == nc - 1 else 0)
-        t = lambda v: torch.tensor(v, dtype=torch.int32).to(device)  # noqa: E731
-        meta = {"row_seq": t(row_seq), "chunk_seq": t(cseq), "chunk_row0": t(crow), "chunk_len": t(clen), "chunk_first": t(cfirst),
-                "chunk_last": t(clast), "seq_chunk0": t(s0), "seq_nchunks": t(sn), "multi": any(v > 1 for v in sn)}
-    batch._mamba_meta = meta
-    return meta
+        p = ops.linear(x, w)
+    y = mamba_op.mamba2(s, p, m["weights"], kv.state["conv"][i], kv.state["ssm"][i], batch, model.cfg.norm_eps)
+    return ops.linear(y, m["out_proj"])

@@ -1,6 +1,6 @@
-"""Softmax attention and lightning attention side by side on the same input rows: ``a * attention(h) + b * lightning(h)``. All input projections of
-both are one GEMM; both write their gated heads, already times their constants, into one row buffer, so that the two output projections,
-whose results are summed anyway, are one GEMM too. A layer holds pages and a state slot."""
+"""Softmax attention and a recurrent mixer (lightning attention, gated delta rule) side by side on the same input rows: ``a * left(h) + b * right(h)``. All
+input projections of both are one GEMM; both write their gated heads, already times their constants, into one row buffer, so that the two output
+projections, whose results are summed anyway, are one GEMM too. A layer holds pages and a state slot."""
 from __future__ import annotations
 
 import torch
@@ -9,13 +9,12 @@ from .. import ops
 from ..ops import LinearWeight
 from .batch import ForwardBatch
 from .grouped import GroupedAttention
-from .lightning import LightningAttention
 
 
 class SideBySideMixer:
     kind = "attention"
 
-    def __init__(self, left: GroupedAttention, right: LightningAttention):
+    def __init__(self, left: GroupedAttention, right):
         self.left, self.right = left, right
 
     def load(self, left: tuple, right: tuple, k_pad: int) -> "SideBySideMixer":
@@ -27,7 +26,7 @@ class SideBySideMixer:
         return self
 
     def nbytes(self) -> int:
-        return self.w_in.nbytes() + self.w_out.nbytes()
+        return self.w_in.nbytes() + self.w_out.nbytes() + self.right.nbytes()
 
     def forward(self, x, batch: ForwardBatch, kv, run: int, stage, shared=None) -> torch.Tensor:
         ls, rs = self.left.shape, self.right.shape
@@ -35,9 +34,9 @@ class SideBySideMixer:
             p = ops.linear(x, self.w_in)
         row = torch.empty(x.shape[0], ls.out_width + rs.out_width, dtype=p.dtype, device=p.device)
         self.left.heads(p[:, : ls.width], batch, kv, run, stage, out=row[:, : ls.out_width])
-        self.right.heads(p[:, ls.width :], batch, kv.state["lightning"][run], row[:, ls.out_width :], stage)
+        self.right.heads(p[:, ls.width :], batch, kv, run, row[:, ls.out_width :], stage)
         with stage("sidebyside.output_projection"):
             return ops.linear(row, self.w_out)
 
     def cache_layout(self) -> dict:
-        return dict(self.left.cache_layout(), state={"lightning": self.right.state_shape()})
+        return dict(self.left.cache_layout(), state=self.right.state_shapes())

@@ -267,19 +267,22 @@ class DecoderModel:
             return ops.interleave_gate_up(gate, up)
         return _cat_weights([gate, up])
 
+    def _mamba_shape(self):
+        from ..ops.mamba import Mamba2Shape
+
+        cfg = self.cfg
+        return Mamba2Shape(cfg.mamba_n_heads, cfg.mamba_d_head, cfg.mamba_d_state, cfg.mamba_n_groups, cfg.mamba_d_conv)
+
     def _load_mamba(self, loader, p) -> dict:
-        f32 = lambda n: self._dev(loader.load_dense(p + n), torch.float32)  # noqa: E731
-        m = {
-            "in_proj": self._lin(loader.load(p + "in_proj.weight")),
-            "out_proj": self._lin(loader.load(p + "out_proj.weight")),
-            "conv_w": f32("conv1d.weight"),
-            "conv_b": f32("conv1d.bias") if loader.has(p + "conv1d.bias") else None,
-            "dt_bias": f32("dt_bias").reshape(-1),
-            "A_log": f32("A_log").reshape(-1),
-            "D": f32("D").reshape(-1),
-            "norm_w": f32("norm.weight").reshape(-1),
-        }
-        return m
+        from ..ops.mamba import Mamba2Weights
+
+        s = self._mamba_shape()
+        if s.dv != s.vdim or s.dn != s.state:
+            raise ValueError("Mamba-2 head and state sizes must be multiples of 8")
+        f32 = lambda n: loader.load_dense(p + n).float()  # noqa: E731
+        return {"shape": s, "in_proj": self._lin(loader.load(p + "in_proj.weight")), "out_proj": self._lin(loader.load(p + "out_proj.weight")),
+                "weights": Mamba2Weights.pack(s, f32("conv1d.weight"), f32("conv1d.bias") if loader.has(p + "conv1d.bias") else None, f32("dt_bias"), f32("A_log"),
+                                              f32("D"), f32("norm.weight"), self.device)}
 
     # ------------------------------------------------------------------------------------------------ LoRA hot swap
     def set_lora(self, adapter=None, prefix: str = "model.") -> None:
@@ -592,7 +595,7 @@ class DecoderModel:
         kinds = [cfg.layer_type(i) for i in range(cfg.num_layers)]
         out = {"layers": cfg.num_layers, "kv_heads": self.n_kv, "head_dim": cfg.head_dim, "layer_kinds": kinds}
         if "mamba" in kinds:
-            shapes = {"conv": (cfg.mamba_conv_dim, cfg.mamba_d_conv - 1), "ssm": (cfg.mamba_n_heads, cfg.mamba_d_head, cfg.mamba_d_state)}
+            shapes = self._mamba_shape().state_shapes()
             out["state_shapes"] = [shapes if k == "mamba" else None for k in kinds]
         return out
 

@@ -324,6 +324,7 @@ def act_mul(gate_up, act):
 
 
 def activation(x, act):
+    """Elementwise activation of bf16 or (CUDA) fp32 rows."""
     if _cuda(x):
         _count()
         return require_ext().activation(x.contiguous(), act)
@@ -380,17 +381,18 @@ class Routed:
         return (self.ys[self.pos.long()].float() * self.w.unsqueeze(-1)).sum(dim=1)
 
 
-def sandwich_norm(residual, sub, w_sub, mult: float, w_next, eps: float, pitch: int, dtype, out=None):
+def sandwich_norm(residual, sub, w_sub, mult: float, w_next, eps: float, pitch: int, dtype, out=None, rms: bool = False):
     """Norms behind and in front of a sublayer in one pass over an fp32 residual stream: ``residual += mult * LayerNorm(sub; w_sub)`` in place,
-    then ``LayerNorm(residual; w_next)``, or with ``w_next`` None the residual itself, in ``dtype``. LayerNorms have a weight and no bias.
+    then ``LayerNorm(residual; w_next)``, or with ``w_next`` None the residual itself, in ``dtype``. LayerNorms have a weight and no bias; ``rms``:
+    RMS norms instead. A weight of one element serves all columns.
     ``sub``: ``[T, >= W]`` rows, a :class:`Routed` result (its weighted sum is formed here in fp32), or None (nothing is added). The result is
     ``[T, pitch]`` (zeros behind the row width), or written to ``out``, a ``[T, W]`` column range of wider rows."""
     if _cuda(residual):
         _count()
         ys, pos, w = (sub.ys, sub.pos, sub.w) if isinstance(sub, Routed) else (sub, None, None)
-        return require_ext().sandwich_norm(residual, ys, pos, w, w_sub, mult, w_next, eps, pitch, dtype == torch.float32, out)
+        return require_ext().sandwich_norm(residual, ys, pos, w, w_sub, mult, w_next, eps, pitch, dtype == torch.float32, out, rms)
     W = residual.shape[1]
-    y = ref.sandwich_norm(residual, (sub.dense() if isinstance(sub, Routed) else sub[:, :W])[:, :W] if sub is not None else None, w_sub, mult, w_next, eps)
+    y = ref.sandwich_norm(residual, (sub.dense() if isinstance(sub, Routed) else sub[:, :W])[:, :W] if sub is not None else None, w_sub, mult, w_next, eps, rms)
     if out is None:
         return torch.nn.functional.pad(y, (0, pitch - W)).to(dtype)
     out.copy_(y)

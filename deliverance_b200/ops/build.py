@@ -14,8 +14,8 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(_HERE, "csrc")
 BUILD_DIR = os.path.join(_HERE, "_build")
 NAME = "_dlv_C"
-SOURCES = ["bindings.cpp", "gemm.cu", "gemm_persist.cu", "elementwise.cu", "attention.cu", "sampling.cu", "quant.cu", "moe.cu", "mamba.cu",
-           "latent.cu", "gla.cu", "lightning.cu", "streams.cu", "comm.cu", "noalloc.cu", "chain.cu", "aux.cu", "a2a.cu", "attention_tc.cu", "lz4_block.cpp"]
+SOURCES = ["bindings.cpp", "gemm.cu", "gemm_persist.cu", "elementwise.cu", "attention.cu", "sampling.cu", "quant.cu", "moe.cu", "short_conv.cu", "mamba.cu",
+           "latent.cu", "gla.cu", "delta.cu", "mixed.cu", "lightning.cu", "streams.cu", "comm.cu", "noalloc.cu", "chain.cu", "aux.cu", "a2a.cu", "attention_tc.cu", "lz4_block.cpp"]
 
 CUDA_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

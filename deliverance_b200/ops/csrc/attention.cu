@@ -766,6 +766,10 @@ static int launch_decode_mma_t(const void* q, long long q_stride, const void* kc
   return 0;
 }
 
+void launch_decode_merge(const float* po, const float* pml, void* out, int B, int H, int dv, int splits, AttnExtra x, cudaStream_t st) {
+  launch_pdl(decode_merge_kernel<true>, dim3(B, H), dim3((dv + 31) / 32 * 32), 0, st, po, pml, static_cast<__nv_bfloat16*>(out), H, dv, splits, x);
+}
+
 // impl: 0 = tensor-core kernel when it applies (group <= 16, page_size % 16 == 0), 1 = CUDA-core kernel
 int launch_decode_attention_impl(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                                  const int* ctx, void* out, float* po, float* pml, int* arrivals, int B, int H, int KV, int D, int page,
@@ -814,7 +818,7 @@ template <typename TIO>
 __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ q, long long q_stride, const TIO* __restrict__ k_cache,
                                                         const TIO* __restrict__ v_cache, const int* __restrict__ bt, int bt_stride,
                                                         const int* __restrict__ row_seq, const int* __restrict__ positions, TIO* __restrict__ out, int H, int KV,
-                                                        int dk, int dv, int page, float scale, float softcap, int window, const AttnExtra x) {
+                                                        int dk, int dv, int page, float scale, float softcap, int window, bool wide, const AttnExtra x) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float rsm[];  // q [dk] | accumulators [4][dv]
@@ -831,9 +835,13 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ 
   float m = -INFINITY, l = 0.f;
   for (int i = warp; i < kept + ctx - first; i += 4) {
     const int key = i < kept ? i : first + i - kept;
-    const long long row = (static_cast<long long>(table[key / page]) * KV + kvh) * page + key % page;
+    long long row = (static_cast<long long>(table[key / page]) * KV + kvh) * page + key % page, k_row = row;
+    if (wide) {
+      k_row = static_cast<long long>(table[key / page]) * page + key % page;
+      row = k_row * KV + kvh;
+    }
     float s = 0.f;
-    for (int d = lane; d < dk; d += 32) s += rsm[d] * io_ld(k_cache + row * dk + d);
+    for (int d = lane; d < dk; d += 32) s += rsm[d] * io_ld(k_cache + k_row * dk + d);
     s = softcap_apply(warp_sum(s) * scale, softcap);
     const float m_new = fmaxf(m, s), alpha = expf(m - m_new), pr = expf(s - m_new);
     m = m_new;
@@ -863,14 +871,14 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const TIO* __restrict__ 
 }
 
 int launch_attention_rows(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* row_seq,
-                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
-                          bool is_f32, cudaStream_t st) {
+                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, bool wide,
+                          AttnExtra x, bool is_f32, cudaStream_t st) {
   if (T == 0) return 0;
   const size_t smem = static_cast<size_t>(dk + 4 * dv) * sizeof(float);
   if (smem > 48 * 1024 - 256) return 1;
 #define DLV_ROWS(TT)                                                                                                                                     \
   launch_pdl(attn_rows_kernel<TT>, dim3(T, H), dim3(128), smem, st, static_cast<const TT*>(q), q_stride, static_cast<const TT*>(kc),                      \
-             static_cast<const TT*>(vc), bt, bt_stride, row_seq, positions, static_cast<TT*>(out), H, KV, dk, dv, page, scale, cap, window, x)
+             static_cast<const TT*>(vc), bt, bt_stride, row_seq, positions, static_cast<TT*>(out), H, KV, dk, dv, page, scale, cap, window, wide, x)
   if (is_f32) DLV_ROWS(float);
   else DLV_ROWS(__nv_bfloat16);
 #undef DLV_ROWS

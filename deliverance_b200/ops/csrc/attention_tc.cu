@@ -34,6 +34,11 @@
 //           with a sigmoid output gate and stores the dv real columns of every head.
 // Both take DK (query / key columns) and DV (value columns) as multiples of 64.
 //
+// Wide rows (paged layout, `wide`): a cache row holds the heads of all KV heads side by side, and a query head's keys are the WHOLE row (attention with
+// mixed scores: the mixing has moved to the query side, see ops/grouped.py), its values the dv columns of its own KV head. Rows of more than 256 key
+// columns go by in pieces of 128 columns (KM = 1: the query tile of up to 512 columns stays in shared memory; KM = 2: wider rows, the query's pieces
+// travel with the keys' pieces, from L2). KM = 0: whole key tiles.
+//
 // Replaces the reference's packed prefill attention (core/.../generator/CausalSelfAttention.java:458-502: per head QK^T GEMM over
 // the visible pages, causal scaled softmax with optional soft-cap, saxpy with V).
 #include <stdexcept>
@@ -71,6 +76,8 @@ struct AttnTcParams {
   long long gate_pitch;
   int gate_heads;
   float out_mult;
+  int wide;                    // cache rows hold all KV heads, keys are whole rows
+  int k_subs;                  // KM > 0: 64-column blocks of a key row
 };
 
 // MN-major shared-memory descriptor (128-byte swizzle): the operand tile is stored as rows of the K dimension, each row 64 elements of
@@ -107,6 +114,27 @@ __device__ __forceinline__ void tmem_st_x32(uint32_t taddr, const uint32_t* r) {
 }
 
 constexpr int kAtBM = 128, kAtBN = 64;  // query rows per score tile / keys per tile
+constexpr int kAtPiece = 2, kAtResident = 8;  // KM > 0: 64-column blocks per piece of a key row; most blocks of a query tile that stays in shared memory
+
+// KM > 0 (one query tile): a K stage is one piece of a key tile, with KM = 2 behind the query's piece
+template <int DV, int KM>
+struct AttnTcWideSmem {
+  static constexpr int kTileQ = kAtBM * 128 * kAtPiece;  // bytes of a query piece
+  static constexpr int kTileK = kAtBN * 128 * kAtPiece + (KM == 2 ? kTileQ : 0);
+  static constexpr int kOffKeys = KM == 2 ? kTileQ : 0;  // the keys inside a stage
+  static constexpr int kTileV = kAtBN * 128 * (DV / 64);
+  static constexpr int kStagesV = 2;
+  static constexpr int kOffK = KM == 1 ? kAtResident * kAtBM * 128 : 0;
+  static constexpr int kRoom = 227 * 1024 - 512 - 1024 - kOffK - kStagesV * kTileV;
+  static constexpr int kFit = kRoom / kTileK;
+  static constexpr int kStages = kFit >= 4 ? 4 : kFit;
+  static constexpr int kOffV = kOffK + kStages * kTileK;
+  static constexpr int kOffCtrl = kOffV + kStagesV * kTileV;
+  static constexpr int kBytes = kOffCtrl + 512 + 1024;
+  static constexpr int kThreads = 256;
+  static constexpr int kSubK = 0, kSubV = DV / 64;
+  static_assert(kStages >= 2 && DV % 64 == 0 && kBytes > 118 * 1024 && kBytes <= 227 * 1024 && 256 + DV <= 512, "attention tile does not fit");
+};
 
 template <int DK, int DV, int QT>
 struct AttnTcSmem {
@@ -116,7 +144,7 @@ struct AttnTcSmem {
   static constexpr int kTileV = kAtBN * 128 * kSubV;
   static constexpr int kRoom = 227 * 1024 - 512 - 1024 - QT * kTileQ;  // barriers + alignment slack
   static constexpr int kFit = kRoom / (kTileK + kTileV);
-  static constexpr int kStages = kFit >= 4 ? 4 : kFit;
+  static constexpr int kStages = kFit >= 4 ? 4 : kFit, kStagesV = kStages, kOffKeys = 0;
   static constexpr int kOffK = QT * kTileQ;
   static constexpr int kOffV = kOffK + kStages * kTileK;
   static constexpr int kOffCtrl = kOffV + kStages * kTileV;
@@ -176,15 +204,25 @@ __device__ __forceinline__ void softcap_tile(float (&f)[kAtBN], float a, float c
   }
 }
 
-template <int DK, int DV, int QT, bool LATENT>
-__global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
+template <int DK, int DV, int QT, int KM>
+struct AttnTcLayout {
+  using T = AttnTcSmem<DK, DV, QT>;
+};
+template <int DV, int KM>
+struct AttnTcLayout<0, DV, 1, KM> {
+  using T = AttnTcWideSmem<DV, KM>;
+};
+
+template <int DK, int DV, int QT, bool LATENT, int KM = 0>
+__global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,  // [T, H * DK], box 128 x 64
                            const __grid_constant__ CUtensorMap map_k,  // paged [pages * KV * page, DK], box min(page, 64) x 64; latent [rows, H * kn]
                            const __grid_constant__ CUtensorMap map_v,  // paged as K; latent [rows, H * DV], box 64 x 64
                            const __grid_constant__ CUtensorMap map_r,  // latent: shared key part [rows, DK - kn], box 64 x 64 (paged: unused)
                            const AttnTcParams p) {
-  using L = AttnTcSmem<DK, DV, QT>;
-  constexpr int NS = L::kStages, SUBK = L::kSubK, SUBV = L::kSubV;
+  using L = typename AttnTcLayout<DK, DV, QT, KM>::T;
+  constexpr int NS = L::kStages, NSV = L::kStagesV, SUBK = L::kSubK, SUBV = L::kSubV;
+  const int pieces = KM > 0 ? (p.k_subs + kAtPiece - 1) / kAtPiece : 1;  // K stages per key tile
   constexpr int kProducer = 1, kIssuer = 0, kIssuerPV = 2;
   extern __shared__ uint8_t at_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(at_raw) + 1023) & ~uintptr_t(1023));
@@ -268,18 +306,66 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
     // ---------------- TMA producer ----------------
     // One thread can start a tensor copy only every few hundred nanoseconds, whatever its size, and a key tile is several copies
     // (pages x D / 64 column blocks, for K and for V): the copies of a tile are spread over the lanes of the warp.
-    if (lane == 0) {
+    if (KM == 1) {
+      if (lane == 0) mbar_expect_tx(smem_u32(bar_q), p.k_subs * kAtBM * 128);
+      __syncwarp();
+      for (int c = lane; c < p.k_subs; c += 32)
+        tma_load_2d(smem_u32(smem + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0);
+    }
+    if (KM == 0 && lane == 0) {
       mbar_expect_tx(smem_u32(bar_q), (two ? 2 : 1) * L::kTileQ);
       for (int q = 0; q < (two ? 2 : 1); ++q)
         for (int c = 0; c < SUBK; ++c)
           tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0 + q * kAtBM);
     }
     const int box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;  // page_size is 32, 64 or 128
-    int issued = 0;
+    int issued = 0, issued_k = 0;  // key tiles; KM > 0: pieces of key tiles
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t, ++issued) {
       const int s = t % NS;
       const int kt = tile_at(t);
+      if constexpr (KM > 0) {
+        // the cache pages of the tile (64 keys: one or two of them), then the pieces of its key rows, then its values
+        const int n_pg = kAtBN / box_rows;
+        long long row_of[2] = {0, 0};
+        for (int pg = 0; pg < n_pg; ++pg) {
+          const int key0 = kt * kAtBN + pg * box_rows;
+          const int page = key0 < ctx ? p.block_tables[static_cast<long long>(seq) * p.bt_stride + key0 / p.page_size] : 0;
+          row_of[pg] = static_cast<long long>(page) * p.page_size + key0 % p.page_size;
+        }
+        for (int pc = 0; pc < pieces; ++pc, ++issued_k) {
+          const int st = issued_k % NS;
+          if (issued_k >= NS) ok = mbar_wait(smem_u32(&bar_k_empty[st]), ((issued_k / NS) - 1) & 1, abort_flag, p.status);
+          ok = __all_sync(0xffffffffu, ok);
+          if (!ok) break;
+          const int subs = min(kAtPiece, p.k_subs - pc * kAtPiece);
+          if (lane == 0) mbar_expect_tx(smem_u32(&bar_k_full[st]), subs * (kAtBN * 128 + (KM == 2 ? kAtBM * 128 : 0)));
+          __syncwarp();
+          uint8_t* dst = smem + L::kOffK + st * L::kTileK;
+          const int n_k = n_pg * subs;
+          if (lane < n_k) {
+            const int pg = lane / subs, c = lane - pg * subs;
+            tma_load_2d(smem_u32(dst + L::kOffKeys + c * (kAtBN * 128) + pg * box_rows * 128), &map_k, smem_u32(&bar_k_full[st]), (pc * kAtPiece + c) * 64,
+                        static_cast<int>(row_of[pg]));
+          } else if (KM == 2 && lane < n_k + subs) {
+            const int c = lane - n_k;
+            tma_load_2d(smem_u32(dst + c * (kAtBM * 128)), &map_q, smem_u32(&bar_k_full[st]), h * p.dk + (pc * kAtPiece + c) * 64, qs + q0);
+          }
+        }
+        if (!ok) break;
+        const int sv = t % NSV;
+        if (t >= NSV) ok = mbar_wait(smem_u32(&bar_v_empty[sv]), ((t / NSV) - 1) & 1, abort_flag, p.status);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(smem_u32(&bar_v_full[sv]), L::kTileV);
+        __syncwarp();
+        for (int i = lane; i < n_pg * SUBV; i += 32) {
+          const int pg = i / SUBV, c = i - pg * SUBV;
+          tma_load_2d(smem_u32(smem + L::kOffV + sv * L::kTileV + c * (kAtBN * 128) + pg * box_rows * 128), &map_v, smem_u32(&bar_v_full[sv]),
+                      kvh * p.dv + c * 64, static_cast<int>(row_of[pg]));
+        }
+        continue;
+      }
       for (int kv = 0; kv < 2; ++kv) {
         uint64_t* full = kv == 0 ? &bar_k_full[s] : &bar_v_full[s];
         uint64_t* empty = kv == 0 ? &bar_k_empty[s] : &bar_v_empty[s];
@@ -306,16 +392,26 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
           const int key0 = kt * kAtBN + pg * box_rows;
           // pages past the context are never read by an unmasked score; the scratch page 0 keeps the copy inside the cache
           const int page = key0 < ctx ? p.block_tables[static_cast<long long>(seq) * p.bt_stride + key0 / p.page_size] : 0;
-          const int row = (page * p.KV + kvh) * p.page_size + (key0 % p.page_size);
+          const int row = (p.wide ? page : page * p.KV + kvh) * p.page_size + (key0 % p.page_size);
           const uint32_t off = c * (kAtBN * 128) + pg * box_rows * 128;
-          tma_load_2d(smem_u32(dst + off), kv == 0 ? &map_k : &map_v, smem_u32(full), c * 64, row);
+          tma_load_2d(smem_u32(dst + off), kv == 0 ? &map_k : &map_v, smem_u32(full), (p.wide && kv == 1 ? kvh * p.dv : 0) + c * 64, row);
         }
       }
       if (!ok) break;
     }
     if (lane == 0 && *abort_flag) {
       // a wait ran out somewhere in the CTA: before shared memory goes away let the copies already issued land (bounded)
-      for (int t = issued > NS ? issued - NS : 0; t < issued; ++t) {
+      for (int t = issued_k > NS ? issued_k - NS : 0; KM > 0 && t < issued_k; ++t) {
+        const unsigned long long t0 = globaltimer_ns();
+        while (!mbar_try_wait(smem_u32(&bar_k_full[t % NS]), (t / NS) & 1) && globaltimer_ns() - t0 < 20000000ull) {
+        }
+      }
+      for (int t = issued > NSV ? issued - NSV : 0; KM > 0 && t < issued; ++t) {
+        const unsigned long long t0 = globaltimer_ns();
+        while (!mbar_try_wait(smem_u32(&bar_v_full[t % NSV]), (t / NSV) & 1) && globaltimer_ns() - t0 < 20000000ull) {
+        }
+      }
+      for (int t = issued > NS ? issued - NS : 0; KM == 0 && t < issued; ++t) {
         const unsigned long long t0 = globaltimer_ns();
         while (!(mbar_try_wait(smem_u32(&bar_k_full[t % NS]), (t / NS) & 1) && mbar_try_wait(smem_u32(&bar_v_full[t % NS]), (t / NS) & 1)) &&
                globaltimer_ns() - t0 < 20000000ull) {
@@ -356,7 +452,8 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
       int u = 0, q = 0;
       if (n_tiles > 0 && !valid(u, q)) advance(u, q);
       if (warp == kIssuer) {
-        ok = mbar_wait(smem_u32(bar_q), 0, abort_flag, p.status);
+        if (KM != 2) ok = mbar_wait(smem_u32(bar_q), 0, abort_flag, p.status);
+        int piece = 0;  // KM > 0: pieces of key tiles so far
         const uint64_t desc_q0 = umma_desc_k_sw128(smem_u32(smem)), desc_k0 = umma_desc_k_sw128(smem_u32(smem + L::kOffK));
         int k_seen = -1;  // key tiles whose K has been waited for
         while (ok && u < n_tiles) {
@@ -364,6 +461,28 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
           const int s = u % NS;
           const uint32_t slot = q * 2 + (t & 1);
           if (t >= 2) ok = mbar_wait(smem_u32(&bar_pv_done[slot]), ((t >> 1) - 1) & 1, abort_flag, p.status);
+          if constexpr (KM > 0) {
+            const uint32_t d_w = tmem_base + kColS + slot * kAtBN;
+            for (int pc = 0; ok && pc < pieces; ++pc, ++piece) {
+              const int st = piece % NS;
+              ok = mbar_wait(smem_u32(&bar_k_full[st]), (piece / NS) & 1, abort_flag, p.status);
+              if (!ok) break;
+              tc_fence_after();
+              const uint64_t desc_q = umma_desc_k_sw128(smem_u32(smem + (KM == 1 ? pc * L::kTileQ : L::kOffK + st * L::kTileK)));
+              const uint64_t desc_k = umma_desc_k_sw128(smem_u32(smem + L::kOffK + st * L::kTileK + L::kOffKeys));
+              const int subs = min(kAtPiece, p.k_subs - pc * kAtPiece);
+              for (int c = 0; c < subs; ++c)
+#pragma unroll
+                for (int k16 = 0; k16 < 4; ++k16)
+                  umma_bf16(d_w, desc_q + static_cast<uint64_t>((c * (kAtBM * 128) + k16 * 32) >> 4), desc_k + static_cast<uint64_t>((c * (kAtBN * 128) + k16 * 32) >> 4),
+                            idesc_s, (pc > 0 || c > 0 || k16 > 0) ? 1u : 0u);
+              umma_commit(smem_u32(&bar_k_empty[st]));
+            }
+            if (!ok) break;
+            umma_commit(smem_u32(&bar_s_full[slot]));
+            advance(u, q);
+            continue;
+          }
           if (ok && u > k_seen) {
             ok = mbar_wait(smem_u32(&bar_k_full[s]), (u / NS) & 1, abort_flag, p.status);
             k_seen = u;
@@ -387,10 +506,10 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
         const uint32_t v_base = smem_u32(smem + L::kOffV);
         while (ok && u < n_tiles) {
           const int t = count_at(u, q);
-          const int s = u % NS;
+          const int s = u % NSV;
           const uint32_t slot = q * 2 + (t & 1);
           ok = mbar_wait(smem_u32(&bar_p_full[slot]), (t >> 1) & 1, abort_flag, p.status) &&
-               mbar_wait(smem_u32(&bar_v_full[s]), (u / NS) & 1, abort_flag, p.status);
+               mbar_wait(smem_u32(&bar_v_full[s]), (u / NSV) & 1, abort_flag, p.status);
           if (!ok) break;
           tc_fence_after();
           const uint32_t tmem_p = tmem_base + kColS + slot * kAtBN, d_o = tmem_base + kColO + q * DV;
@@ -593,13 +712,13 @@ __global__ void __launch_bounds__(AttnTcSmem<DK, DV, QT>::kThreads, 1)
   }
 }
 
-template <int DK, int DV, int QT, bool LATENT>
+template <int DK, int DV, int QT, bool LATENT, int KM = 0>
 static int launch_prefill_tc_maps(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr, const AttnTcParams& p,
                                   int num_tiles, cudaStream_t st) {
-  using L = AttnTcSmem<DK, DV, QT>;
+  using L = typename AttnTcLayout<DK, DV, QT, KM>::T;
   static PerDeviceOnce attr_once;
   if (attr_once.first()) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel<DK, DV, QT, LATENT>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel<DK, DV, QT, LATENT, KM>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
     if (e != cudaSuccess) throw std::runtime_error(std::string("prefill attention (tcgen05): cudaFuncSetAttribute: ") + cudaGetErrorString(e));
   }
   cudaLaunchConfig_t cfg = {};
@@ -612,20 +731,21 @@ static int launch_prefill_tc_maps(const CUtensorMap& mq, const CUtensorMap& mk, 
   attr[0].val.programmaticStreamSerializationAllowed = g_pdl_enabled ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_attn_tc_kernel<DK, DV, QT, LATENT>, mq, mk, mv, mr, p);
+  cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_attn_tc_kernel<DK, DV, QT, LATENT, KM>, mq, mk, mv, mr, p);
   if (e != cudaSuccess) throw std::runtime_error(std::string("prefill attention (tcgen05) launch: ") + cudaGetErrorString(e));
   return 0;
 }
 
-template <int DK, int DV, int QT>
+template <int DK, int DV, int QT, int KM = 0>
 static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
                                int num_tiles, cudaStream_t st) {
   CUtensorMap mq, mk, mv;
   encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * p.dk, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
   const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
   encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), p.dk, static_cast<uint64_t>(p.dk) * 2, box_rows, 64, 128);
-  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), p.dv, static_cast<uint64_t>(p.dv) * 2, box_rows, 64, 128);
-  return launch_prefill_tc_maps<DK, DV, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
+  const uint64_t v_width = static_cast<uint64_t>(p.dv) * (p.wide ? p.KV : 1);
+  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), v_width, v_width * 2, box_rows, 64, 128);
+  return launch_prefill_tc_maps<DK, DV, QT, false, KM>(mq, mk, mv, mv, p, num_tiles, st);
 }
 
 // ---- latent layout -----------------------------------------------------------------------------------------------------
@@ -664,6 +784,7 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
   p.out_pitch = a.out_pitch;
   p.gate = static_cast<const __nv_bfloat16*>(a.gate);
   p.gate_pitch = a.gate_pitch;
+  p.sink = a.sink;
   p.out_mult = 1.f;
   CUtensorMap mq, mk, mv, mr;
   const uint64_t H = static_cast<uint64_t>(a.H), rows = static_cast<uint64_t>(a.kv_rows);
@@ -685,15 +806,21 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
 // Query rows one CTA of the tcgen05 prefill kernel covers: two 128-row tiles share the K / V tiles where their two accumulators fit
 // tensor memory beside the two score slots.
 int prefill_attention_tc_tile_rows(int D) { return D <= 128 ? 256 : 128; }
+int prefill_attention_wide_tile_rows(int k_width, int dv) {
+  if (k_width <= 0 || dv <= 0 || k_width % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
+  return k_width > 256 ? kAtBM : prefill_attention_tc_tile_rows(k_width > dv ? k_width : dv);
+}
 
 // tile arrays: prefill_attention_tc_tile_rows(max(dk, dv)) query rows per tile. page_size must be 32, 64 or 128. Returns 1 for an unsupported
 // head size (multiples of 8 up to 256) or page size.
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                                 int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
-                                AttnExtra x, int* status, cudaStream_t st) {
+                                bool wide, AttnExtra x, int* status, cudaStream_t st) {
   if (num_tiles == 0) return 0;
-  const int D = dk > dv ? dk : dv;
+  if (wide && (prefill_attention_wide_tile_rows(dk, dv) == 0 || x.keep_first != 0)) return 1;
+  const bool pieces = wide && dk > 256;
+  const int D = pieces ? dv : (dk > dv ? dk : dv);
   if ((page != 32 && page != 64 && page != 128) || dk % 8 != 0 || dv % 8 != 0 || dk <= 0 || dv <= 0 || D > 256) return 1;
   AttnTcParams p = {};
   p.block_tables = bt;
@@ -721,7 +848,18 @@ int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, 
   p.dv = dv;
   p.out_pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * dv;
   p.status = status;
-  const long long cache_rows = num_pages * KV * page;
+  p.wide = wide ? 1 : 0;
+  p.k_subs = (dk + 63) / 64;
+  const long long cache_rows = num_pages * (wide ? 1 : KV) * page;
+  if (pieces) {
+#define DLV_WIDE(DVV)                                                                                                               \
+  return p.k_subs <= kAtResident ? launch_prefill_tc_t<0, DVV, 1, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)          \
+                                 : launch_prefill_tc_t<0, DVV, 1, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
+    if (dv <= 64) DLV_WIDE(64);
+    if (dv <= 128) DLV_WIDE(128);
+    DLV_WIDE(256);
+#undef DLV_WIDE
+  }
   if (D <= 64) return launch_prefill_tc_t<64, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128 && dv <= 64) return launch_prefill_tc_t<128, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128) return launch_prefill_tc_t<128, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);

@@ -35,6 +35,7 @@ int act_code(const std::string& a) {
   if (a == "gelu") return 2;
   if (a == "relu") return 3;
   if (a == "tanh") return 4;
+  if (a == "relu2") return 5;
   TORCH_CHECK(false, "unknown activation ", a);
 }
 
@@ -601,10 +602,13 @@ Tensor act_mul(const Tensor& gate_up, const std::string& act) {
   return out;
 }
 Tensor activation(const Tensor& x, const std::string& act) {
-  check_bf16(x, "x");
+  check_cuda(x, "x");
+  const bool f32 = x.scalar_type() == at::kFloat;
+  TORCH_CHECK(f32 || x.scalar_type() == at::kBFloat16, "x must be bf16 or fp32");
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) & 15) == 0, "x misaligned");
   c10::cuda::CUDAGuard guard(x.device());
   Tensor out = new_out(x.sizes(), x.options());
-  dlv::launch_act(x.data_ptr(), out.data_ptr(), x.numel(), act_code(act), cur_stream());
+  dlv::launch_act(x.data_ptr(), out.data_ptr(), x.numel(), act_code(act), f32, cur_stream());
   check_last_error("activation");
   return out;
 }
@@ -829,7 +833,7 @@ Tensor prefill_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v
 Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& q_start,
                             const Tensor& q_len, const Tensor& ctx_lens, const Tensor& tile_seq, const Tensor& tile_q0, int64_t H, double scale,
                             double softcap, int64_t window, bool causal, int64_t keep_first, c10::optional<Tensor> sink, c10::optional<Tensor> gate,
-                            double out_mult, c10::optional<Tensor> out_opt) {
+                            double out_mult, c10::optional<Tensor> out_opt, int64_t kv_heads) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [T, H*D]");
   TORCH_CHECK(q.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0, "q rows must be 16-byte aligned");
   check_bf16(k_cache, "k_cache");
@@ -839,11 +843,15 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
     TORCH_CHECK(t->scalar_type() == at::kInt, "index tensors must be int32");
   }
   const int T = static_cast<int>(q.size(0));
-  const int KV = static_cast<int>(k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
-  const int DV = static_cast<int>(v_cache.size(3));
-  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == KV && v_cache.size(2) == page &&
-                  q.size(1) == H * D && H % KV == 0, "shape mismatch");
-  TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && D <= 256 && DV % 8 == 0 && DV <= 256,
+  // kv_heads > 0: wide rows, keys [pages, 1, page, D], values [pages, 1, page, kv_heads * DV]
+  const bool wide = kv_heads > 0;
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && v_cache.size(1) == k_cache.size(1) && (!wide || (k_cache.size(1) == 1 && v_cache.size(3) % kv_heads == 0)),
+              "shape mismatch");
+  const int KV = static_cast<int>(wide ? kv_heads : k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
+  const int DV = static_cast<int>(wide ? v_cache.size(3) / KV : v_cache.size(3));
+  TORCH_CHECK(v_cache.size(0) == k_cache.size(0) && v_cache.size(2) == page && q.size(1) == H * D && H % KV == 0 && k_cache.size(0) * KV * page < (int64_t(1) << 31),
+              "shape mismatch");
+  TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && (D <= 256 || wide) && DV % 8 == 0 && DV <= 256,
               "page size 32 / 64 / 128 and head widths that are multiples of 8 up to 256");
   TORCH_CHECK(tile_seq.numel() == tile_q0.numel(), "tile arrays differ in length");
   c10::cuda::CUDAGuard guard(q.device());
@@ -854,7 +862,7 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
                                             static_cast<int>(block_tables.stride(0)), q_start.data_ptr<int>(), q_len.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                             tile_seq.data_ptr<int>(), tile_q0.data_ptr<int>(), static_cast<int>(tile_seq.numel()), out.data_ptr(),
                                             static_cast<int>(H), KV, D, DV, page, static_cast<float>(scale), static_cast<float>(softcap),
-                                            static_cast<int>(window), causal ? 1 : 0, x, s.status.data_ptr<int>(), cur_stream());
+                                            static_cast<int>(window), causal ? 1 : 0, wide, x, s.status.data_ptr<int>(), cur_stream());
   TORCH_CHECK(rc == 0, "prefill attention (tcgen05): unsupported shape");
   check_last_error("prefill_attention_tc");
   return out;
@@ -863,6 +871,8 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
 #include "bindings_latent.inc"
 #include "bindings_gla.inc"
 #include "bindings_streams.inc"
+#include "bindings_recurrent.inc"
+#include "bindings_mixed.inc"
 
 // ---- sampling ---------------------------------------------------------------------------------------------------------
 std::vector<Tensor> argmax(const Tensor& logits, c10::optional<Tensor> mask, double softcap, double inv_scale) {
@@ -1454,50 +1464,6 @@ class DecodeChain {
   std::vector<Tensor> keep_;
 };
 
-// ---- Mamba2 -----------------------------------------------------------------------------------------------------------
-// meta: int32 tensors prepared on the host (row_seq [T], chunk_* [n_chunks], seq_chunk0 / seq_nchunks [S])
-Tensor mamba2_forward(const Tensor& zx, const Tensor& conv_w, c10::optional<Tensor> conv_b, const Tensor& dt_bias, const Tensor& A_log,
-                      const Tensor& D, const Tensor& norm_w, Tensor& conv_state, Tensor& ssm_state, const Tensor& slots, const Tensor& q_start,
-                      const Tensor& q_len, const Tensor& positions, const Tensor& row_seq, const Tensor& chunk_seq, const Tensor& chunk_row0,
-                      const Tensor& chunk_len, const Tensor& chunk_first, const Tensor& chunk_last, const Tensor& seq_chunk0,
-                      const Tensor& seq_nchunks, bool multi_chunk, int64_t H, int64_t d_head, int64_t G, int64_t S, double eps) {
-  check_bf16(zx, "zx");
-  const int T = static_cast<int>(zx.size(0));
-  const int I = static_cast<int>(H * d_head), conv_dim = static_cast<int>(I + 2 * G * S);
-  TORCH_CHECK(zx.dim() == 2 && zx.size(1) == I + conv_dim + H, "in_proj output has the wrong width");
-  for (const Tensor* t : std::initializer_list<const Tensor*>{&conv_w, &dt_bias, &A_log, &D, &norm_w, &conv_state, &ssm_state}) {
-    check_cuda(*t, "mamba parameter");
-    TORCH_CHECK(t->scalar_type() == at::kFloat, "mamba parameters and states are fp32");
-  }
-  const int K = static_cast<int>(conv_w.numel() / conv_dim);
-  TORCH_CHECK(conv_state.dim() == 3 && conv_state.size(1) == conv_dim && conv_state.size(2) == K - 1, "conv_state must be [slots, convDim, K-1]");
-  TORCH_CHECK(ssm_state.dim() == 4 && ssm_state.size(1) == H && ssm_state.size(2) == d_head && ssm_state.size(3) == S, "ssm_state must be [slots, H, d_head, S]");
-  check_cuda(slots, "slots");
-  TORCH_CHECK(slots.scalar_type() == at::kLong, "slots must be int64");
-  for (const Tensor* t : {&q_start, &q_len, &positions, &row_seq, &chunk_seq, &chunk_row0, &chunk_len, &chunk_first, &chunk_last, &seq_chunk0, &seq_nchunks}) {
-    check_cuda(*t, "index tensor");
-    TORCH_CHECK(t->scalar_type() == at::kInt, "index tensors must be int32");
-  }
-  const int num_seqs = static_cast<int>(q_len.numel()), n_chunks = static_cast<int>(chunk_seq.numel());
-  c10::cuda::CUDAGuard guard(zx.device());
-  auto fo = zx.options().dtype(at::kFloat);
-  Tensor xbc = new_out({T, conv_dim}, fo), ybuf = new_out({T, I}, fo);
-  Tensor cstate = new_out({std::max(1, n_chunks), H, d_head, S}, fo), cdecay = new_out({std::max(1, n_chunks), H}, fo);
-  Tensor out = new_out({T, I}, zx.options());
-  const float* cb = conv_b.has_value() ? conv_b.value().data_ptr<float>() : nullptr;
-  int rc = dlv::launch_mamba2(zx.data_ptr(), static_cast<int>(zx.stride(0)), T, num_seqs, I, conv_dim, K, static_cast<int>(H), static_cast<int>(d_head),
-                              static_cast<int>(G), static_cast<int>(S), conv_w.data_ptr<float>(), cb, dt_bias.data_ptr<float>(), A_log.data_ptr<float>(),
-                              D.data_ptr<float>(), norm_w.data_ptr<float>(), static_cast<float>(eps), conv_state.data_ptr<float>(), ssm_state.data_ptr<float>(),
-                              reinterpret_cast<const long long*>(slots.data_ptr<int64_t>()), row_seq.data_ptr<int>(), q_start.data_ptr<int>(),
-                              q_len.data_ptr<int>(), positions.data_ptr<int>(), n_chunks, chunk_seq.data_ptr<int>(), chunk_row0.data_ptr<int>(),
-                              chunk_len.data_ptr<int>(), chunk_first.data_ptr<int>(), chunk_last.data_ptr<int>(), seq_chunk0.data_ptr<int>(),
-                              seq_nchunks.data_ptr<int>(), multi_chunk ? 1 : 0, xbc.data_ptr<float>(), ybuf.data_ptr<float>(), cstate.data_ptr<float>(),
-                              cdecay.data_ptr<float>(), out.data_ptr(), cur_stream());
-  TORCH_CHECK(rc == 0, "mamba2: unsupported shape (code ", rc, ")");
-  check_last_error("mamba2_forward");
-  return out;
-}
-
 // ---- JQ4 ------------------------------------------------------------------------------------------------------------
 std::vector<Tensor> q4_quantize(const Tensor& w) {
   check_cuda(w, "w");
@@ -1595,10 +1561,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("prefill_attention_tc", &prefill_attention_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("q_start"),
         py::arg("q_len"), py::arg("ctx_lens"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"),
         py::arg("causal"), py::arg("keep_first") = 0, py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
-        py::arg("out") = py::none());
+        py::arg("out") = py::none(), py::arg("kv_heads") = 0);
   m.def("attention_rows", &attention_rows, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("row_seq"), py::arg("positions"),
         py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"), py::arg("keep_first") = 0, py::arg("sink") = py::none(),
-        py::arg("gate") = py::none(), py::arg("out_mult") = 1.0, py::arg("out") = py::none());
+        py::arg("gate") = py::none(), py::arg("out_mult") = 1.0, py::arg("out") = py::none(), py::arg("kv_heads") = 0);
   m.def("rope_heads_kv", &rope_heads_kv);
   m.def("stream_step", &stream_step);
   m.def("lightning", &lightning);
@@ -1616,7 +1582,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("latent_prepare", &latent_prepare);
   m.def("latent_decode", &latent_decode, py::arg("p"), py::arg("row_idx"), py::arg("row_seq"), py::arg("row_ctx"), py::arg("wuk"), py::arg("wuv"),
         py::arg("c_cache"), py::arg("r_cache"), py::arg("block_tables"), py::arg("out"), py::arg("geom"), py::arg("scale"), py::arg("window"),
-        py::arg("splits"), py::arg("positions") = py::none(), py::arg("slots") = py::none(), py::arg("norm_w") = py::none(), py::arg("cos") = py::none(),
+        py::arg("splits"), py::arg("sink") = py::none(), py::arg("positions") = py::none(), py::arg("slots") = py::none(), py::arg("norm_w") = py::none(), py::arg("cos") = py::none(),
         py::arg("sin") = py::none(), py::arg("eps") = 0.0);
   m.def("latent_head_groups", [](int64_t n) { dlv::g_latent_head_groups = static_cast<int>(n); });
   m.def("latent_gather", &latent_gather);
@@ -1669,7 +1635,19 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("tp_reduce_norm", &tp_reduce_norm, py::arg("comm"), py::arg("mode"), py::arg("ctas"), py::arg("M"), py::arg("N"), py::arg("kind"),
         py::arg("bias") = py::none(), py::arg("residual") = py::none(), py::arg("post_w") = py::none(), py::arg("norm_w") = py::none(), py::arg("out"),
         py::arg("eps") = 1e-6, py::arg("offset") = 0.0, py::arg("res_mult") = 1.0);
-  m.def("mamba2_forward", &mamba2_forward);
+  m.def("short_conv", &short_conv);
+  m.def("mamba2_decode", &mamba2_decode);
+  m.def("mamba2_prompt", &mamba2_prompt);
+  m.def("delta_decode", &delta_decode);
+  m.def("delta_prompt", &delta_prompt);
+  m.def("fold_heads", &fold_heads);
+  m.def("prefill_wide_tile_rows", [](int64_t k_width, int64_t dv) { return dlv::prefill_attention_wide_tile_rows(static_cast<int>(k_width), static_cast<int>(dv)); });
+  m.def("mixed_decode_ok", [](int64_t H, int64_t KV, int64_t dk, int64_t dv) {
+    return dlv::mixed_decode_supported(static_cast<int>(H), static_cast<int>(KV), static_cast<int>(dk), static_cast<int>(dv));
+  });
+  m.def("mixed_decode", &mixed_decode, py::arg("q"), py::arg("mix"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("ctx_lens"),
+        py::arg("H"), py::arg("KV"), py::arg("scale"), py::arg("window"), py::arg("splits"), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
+        py::arg("out") = py::none());
   m.def("q4_quantize", &q4_quantize);
   m.def("q4_dequantize", &q4_dequantize, py::arg("packed"), py::arg("scales"), py::arg("to_bf16") = false);
 }

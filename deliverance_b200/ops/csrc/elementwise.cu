@@ -105,6 +105,7 @@ __device__ __forceinline__ float act_apply(float g, int act) {
     case 1: return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));  // gelu tanh
     case 2: return 0.5f * g * (1.f + erff(g * 0.7071067811865475f));                            // gelu erf
     case 3: return fmaxf(g, 0.f);
+    case 5: return fmaxf(g, 0.f) * fmaxf(g, 0.f);  // squared relu
     default: return tanhf(g);
   }
 }
@@ -134,13 +135,21 @@ __global__ void __launch_bounds__(256) act_mul_kernel(const __nv_bfloat16* __res
   *reinterpret_cast<uint4*>(out + t * I + c) = ov;
 }
 
-// unary activation in place-capable form (gpt2 / bert MLP without an up projection)
-__global__ void __launch_bounds__(256) act_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, int act,
-                                                  long long n) {
+// unary activation (MLPs without an up projection): a thread takes eight elements
+template <typename TIO>
+__global__ void __launch_bounds__(256) act_kernel(const TIO* __restrict__ in, TIO* __restrict__ out, int act, long long n) {
   pdl_wait();     // no-op unless launched with programmatic stream serialization: the kernel in front has completed
   pdl_trigger();  // the next kernel may start its prologue (and a GEMM its weight prefetch) under this kernel's tail
-  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
-  if (i < n) out[i] = f2bf(act_apply(bf2f(in[i]), act));
+  const long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * 8;
+  if (i + 8 <= n) {
+    float v[8];
+    io_ld8(in + i, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = act_apply(v[e], act);
+    io_st8(out + i, v);
+  } else {
+    for (long long k = i; k < n; ++k) io_st(out + k, act_apply(io_ld(in + k), act));
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ embedding
@@ -421,6 +430,7 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const TIO* __restrict__ 
 // Norm behind a sublayer, scaled residual add and norm in front of the next sublayer in one pass over a row of the fp32 residual stream:
 //   residual += mult * LayerNorm(sub; w_sub)   (skipped without sub)
 //   y = LayerNorm(residual; w_next)            (the residual itself without w_next), columns W .. y_width zeroed
+// RMS: RMS norms instead of LayerNorms. A weight may be one number for all columns (sub_one, next_one).
 // sub is one row [T, ld_sub] or, with pos, the weighted sum of k rows of an expert-ordered buffer: sum_j wts[t, j] * sub[pos[t, j]], formed
 // in fp32 in slot order. One CTA per row; the row lives in registers (NV groups of four columns per thread), both variances are means of
 // squared deviations.
@@ -439,9 +449,10 @@ struct SandwichArgs {
   int W, y_width;
   float eps;
   int vec;  // rows, pitches and pointers allow four-column accesses
+  int sub_one, next_one;
 };
 
-template <typename TSUB, typename TIO, int NV, int NT>
+template <typename TSUB, typename TIO, int NV, int NT, bool RMS>
 __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const SandwichArgs a) {
   __shared__ float red[32];
   const int t = blockIdx.x, W = a.W;
@@ -494,15 +505,19 @@ __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const SandwichArgs a)
         }
       }
     }
-    float s = 0.f;
+    float mean = 0.f;
+    if constexpr (!RMS) {
+      float s = 0.f;
 #pragma unroll
-    for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
-    const float mean = block_sum(s, red) / W;
+      for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
+      mean = block_sum(s, red) / W;
+    }
     const float inv = rsqrtf(block_sum(deviation(mean), red) / W + a.eps) * a.mult;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
       float w[4];
-      load(a.w_sub, col(n), w);
+      if (a.sub_one) w[0] = w[1] = w[2] = w[3] = a.w_sub[0];
+      else load(a.w_sub, col(n), w);
 #pragma unroll
       for (int e = 0; e < 4; ++e) v[n][e] = r[n][e] + (v[n][e] - mean) * inv * w[e];
       if (a.vec) {
@@ -522,10 +537,12 @@ __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const SandwichArgs a)
   }
   float mean = 0.f, inv = 1.f;
   if (a.w_next != nullptr) {
-    float s = 0.f;
+    if constexpr (!RMS) {
+      float s = 0.f;
 #pragma unroll
-    for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
-    mean = block_sum(s, red) / W;
+      for (int n = 0; n < NV; ++n) s += (v[n][0] + v[n][1]) + (v[n][2] + v[n][3]);
+      mean = block_sum(s, red) / W;
+    }
     inv = rsqrtf(block_sum(deviation(mean), red) / W + a.eps);
   }
 #pragma unroll
@@ -533,9 +550,10 @@ __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const SandwichArgs a)
     float o[4] = {v[n][0], v[n][1], v[n][2], v[n][3]};
     if (a.w_next != nullptr) {
       float w[4];
-      load(a.w_next, col(n), w);  // (zeros behind the row: so are the outputs there)
+      if (a.next_one) w[0] = w[1] = w[2] = w[3] = a.w_next[0];
+      else load(a.w_next, col(n), w);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[e] = (v[n][e] - mean) * inv * w[e];
+      for (int e = 0; e < 4; ++e) o[e] = col(n) + e < W ? (v[n][e] - mean) * inv * w[e] : 0.f;
     }
     if (a.vec) {
       if (col(n) < a.y_width) io_st4(y + col(n), o);
@@ -637,7 +655,7 @@ __global__ void __launch_bounds__(256) rope_heads_kv_kernel(const RopeHeadsArgs 
     const long long slot = a.slots[t];
     store = active && slot >= 0;
     const unsigned su = static_cast<unsigned>(store ? slot : 0), page = static_cast<unsigned>(a.page);  // (the caches hold fewer than 2^32 rows)
-    at = (static_cast<long long>(su / page) * a.KV + kvh) * a.page + su % page;
+    at = a.wide ? static_cast<long long>(su) * a.KV + kvh : (static_cast<long long>(su / page) * a.KV + kvh) * a.page + su % page;
   }
   float* s = hsm + grp * a.dk;
   const TIO* src = row + (is_q ? h * a.dk : (is_v ? a.off_v + kvh * a.dv : a.off_k + kvh * a.dk));
@@ -769,10 +787,11 @@ void launch_act_mul(const void* in, void* out, long long T, int I, int act, cuda
   launch_pdl(act_mul_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, st, static_cast<const __nv_bfloat16*>(in),
                                                                              static_cast<__nv_bfloat16*>(out), I, act, total);
 }
-void launch_act(const void* in, void* out, long long n, int act, cudaStream_t st) {
+void launch_act(const void* in, void* out, long long n, int act, bool is_f32, cudaStream_t st) {
   if (n == 0) return;
-  act_kernel<<<static_cast<unsigned>((n + 255) / 256), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(in),
-                                                                     static_cast<__nv_bfloat16*>(out), act, n);
+  const dim3 grid(static_cast<unsigned>((n + 2047) / 2048));
+  if (is_f32) launch_pdl(act_kernel<float>, grid, dim3(256), 0, st, static_cast<const float*>(in), static_cast<float*>(out), act, n);
+  else launch_pdl(act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(in), static_cast<__nv_bfloat16*>(out), act, n);
 }
 void launch_embedding(const void* table, const int* ids, const void* pos_table, const int* pos, const void* type_table,
                       const int* types, void* out, int T, int H, int vocab, float scale, cudaStream_t st) {
@@ -811,24 +830,29 @@ void launch_gated_act(const void* in, long long ld_in, void* out, long long ld_o
     launch_pdl(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(in), ld_in, static_cast<__nv_bfloat16*>(out), ld_out, I,
                act, total);
 }
-template <typename TSUB, typename TIO>
-static void sandwich_dispatch(const SandwichArgs& a, int rows, cudaStream_t st) {
+template <typename TSUB, typename TIO, bool RMS>
+static void sandwich_dispatch_t(const SandwichArgs& a, int rows, cudaStream_t st) {
   const int width = a.W > a.y_width ? a.W : a.y_width;
-  if (width <= 512) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 128>, dim3(rows), dim3(128), 0, st, a);
-  else if (width <= 1024) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 256>, dim3(rows), dim3(256), 0, st, a);
-  else if (width <= 2048) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 2, 256>, dim3(rows), dim3(256), 0, st, a);
-  else if (width <= 4096) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 256>, dim3(rows), dim3(256), 0, st, a);
-  else launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 1024>, dim3(rows), dim3(1024), 0, st, a);  // up to 16384 columns
+  if (width <= 512) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 128, RMS>, dim3(rows), dim3(128), 0, st, a);
+  else if (width <= 1024) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 1, 256, RMS>, dim3(rows), dim3(256), 0, st, a);
+  else if (width <= 2048) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 2, 256, RMS>, dim3(rows), dim3(256), 0, st, a);
+  else if (width <= 4096) launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 256, RMS>, dim3(rows), dim3(256), 0, st, a);
+  else launch_pdl(sandwich_norm_kernel<TSUB, TIO, 4, 1024, RMS>, dim3(rows), dim3(1024), 0, st, a);  // up to 16384 columns
+}
+template <typename TSUB, typename TIO>
+static void sandwich_dispatch(const SandwichArgs& a, int rows, bool rms, cudaStream_t st) {
+  if (rms) sandwich_dispatch_t<TSUB, TIO, true>(a, rows, st);
+  else sandwich_dispatch_t<TSUB, TIO, false>(a, rows, st);
 }
 void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bool sub_f32, const int* pos, const float* wts, int k, const float* w_sub,
-                          float mult, const float* w_next, void* y, long long ld_y, int rows, int W, int y_width, float eps, bool vec, bool is_f32,
-                          cudaStream_t st) {
+                          bool sub_one, float mult, const float* w_next, bool next_one, bool rms, void* y, long long ld_y, int rows, int W, int y_width, float eps,
+                          bool vec, bool is_f32, cudaStream_t st) {
   if (rows == 0) return;
-  const SandwichArgs a = {residual, sub, ld_sub, pos, wts, k, w_sub, mult, w_next, y, ld_y, W, y_width, eps, vec ? 1 : 0};
-  if (is_f32 && sub_f32) sandwich_dispatch<float, float>(a, rows, st);
-  else if (is_f32) sandwich_dispatch<__nv_bfloat16, float>(a, rows, st);
-  else if (sub_f32) sandwich_dispatch<float, __nv_bfloat16>(a, rows, st);
-  else sandwich_dispatch<__nv_bfloat16, __nv_bfloat16>(a, rows, st);
+  const SandwichArgs a = {residual, sub, ld_sub, pos, wts, k, w_sub, mult, w_next, y, ld_y, W, y_width, eps, vec ? 1 : 0, sub_one ? 1 : 0, next_one ? 1 : 0};
+  if (is_f32 && sub_f32) sandwich_dispatch<float, float>(a, rows, rms, st);
+  else if (is_f32) sandwich_dispatch<__nv_bfloat16, float>(a, rows, rms, st);
+  else if (sub_f32) sandwich_dispatch<float, __nv_bfloat16>(a, rows, rms, st);
+  else sandwich_dispatch<__nv_bfloat16, __nv_bfloat16>(a, rows, rms, st);
 }
 void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const long long* slots, const float* cos_t, const float* sin_t, void* k_cache,
                           void* v_cache, int T, int H, int KV, int dk, int dv, int page, int half, int max_pos, bool is_f32, cudaStream_t st) {

@@ -117,7 +117,7 @@ void launch_rmsnorm(const void* x, void* residual, const void* w, void* y, int T
                     cudaStream_t st);
 void launch_layernorm(const void* x, const void* w, const void* b, void* y, int T, int H, float eps, cudaStream_t st);
 void launch_act_mul(const void* in, void* out, long long T, int I, int act, cudaStream_t st);
-void launch_act(const void* in, void* out, long long n, int act, cudaStream_t st);
+void launch_act(const void* in, void* out, long long n, int act, bool is_f32, cudaStream_t st);
 void launch_embedding(const void* table, const int* ids, const void* pos_table, const int* pos, const void* type_table,
                       const int* types, void* out, int T, int H, int vocab, float scale, cudaStream_t st);
 int launch_rope_kv(void* qkv, const int* positions, const long long* slots, const void* qn, const void* kn, const float* cos_t,
@@ -149,9 +149,10 @@ int launch_decode_attention_mma(const void* q, long long q_stride, const void* k
                                 float* po, float* pml, int B, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
                                 int splits, cudaStream_t st);
 // one CTA per (row, query head) on CUDA cores, fp32 or bf16, any width; row_seq: sequence of every row (nullptr: row number)
+// wide: queries of dk columns against whole cache rows k [pages, 1, page, dk], values v [pages, 1, page, KV * dv]
 int launch_attention_rows(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride, const int* row_seq,
-                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, AttnExtra x,
-                          bool is_f32, cudaStream_t st);
+                          const int* positions, void* out, int T, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, bool wide,
+                          AttnExtra x, bool is_f32, cudaStream_t st);
 int launch_prefill_attention(const void* q, long long q_stride, const void* kc, const void* vc, const int* bt, int bt_stride,
                              const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                              int num_tiles, void* out, int H, int KV, int D, int page, float scale, float cap, int window,
@@ -177,7 +178,9 @@ extern bool g_gemv_simt_only;  // gemm.cu: grouped JQ4 GEMV on CUDA cores instea
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                                 int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
-                                AttnExtra x, int* status, cudaStream_t st);
+                                bool wide, AttnExtra x, int* status, cudaStream_t st);
+// wide rows: query tile height for keys of k_width columns and values of dv columns per head, 0 when the kernel does not take them
+int prefill_attention_wide_tile_rows(int k_width, int dv);
 
 // sampling.cu
 void launch_argmax(const float* logits, int ld, int B, int V, const uint32_t* mask, int mask_ld, float softcap, float inv_scale,
@@ -237,13 +240,96 @@ void launch_scatter_reduce(const GemmScatterArgs* a, const GemmScatterPlan* plan
 void launch_scatter_finish(const GemmScatterArgs* a, const GemmScatterPlan* plan, int M, int N, void* out, const unsigned* group_targets,
                            int* status, cudaStream_t st);
 
-// mamba.cu
-int launch_mamba2(const void* zx, int ld, int T, int num_seqs, int I, int conv_dim, int K, int H, int d_head, int G, int S,
-                  const float* conv_w, const float* conv_b, const float* dt_bias, const float* A_log, const float* D, const float* norm_w,
-                  float eps, float* conv_state, float* ssm_state, const long long* slots, const int* row_seq, const int* q_start,
-                  const int* q_len, const int* positions, int n_chunks, const int* chunk_seq, const int* chunk_row0, const int* chunk_len,
-                  const int* chunk_first, const int* chunk_last, const int* seq_chunk0, const int* seq_nchunks, int multi_chunk,
-                  float* xbc, float* ybuf, float* chunk_state, float* chunk_decay, void* out, cudaStream_t st);
+struct LightningChunks;
+// short_conv.cu: causal convolution per channel + silu over columns p [T, C] (row pitch ld). w [taps, C], ring [slots, taps, C]: position p at p mod taps
+constexpr int kMaxTaps = 8;
+struct ConvArgs {
+  const void* p;
+  long long ld;
+  int C, taps;
+  const float *w, *b;  // b: [C] or nullptr
+  float* ring;
+  const long long* slots;
+  const int *row_seq, *q_start, *q_len, *positions;
+  int rows, num_seqs;
+  void* out;  // [T, C]
+};
+int launch_short_conv(const ConvArgs& a, bool is_f32, cudaStream_t st);
+
+// mamba.cu: Mamba-2. Projection rows p [T, ld] = z (H dv) | x (H dv) | B (G dn) | C (G dn) | dt (H), widths multiples of 8
+struct MambaArgs {
+  const void* p;
+  long long ld;
+  int H, dn, dv, G, dv_real, norm_groups, dt_at;
+  const void* xbc;  // convolved and activated x | B | C [T, H dv + 2 G dn] (nullptr: the decode step convolves itself)
+  int taps;
+  const float *conv_w, *conv_b;
+  float* ring;
+  const float *dt_bias, *neg_a, *D, *norm_w;  // [H] each, norm [H dv]
+  float* state;                               // [slots, H, dn, dv]
+  const long long* slots;
+  const int *q_start, *q_len, *positions;
+  int num_seqs, rows;
+  float eps;
+  float* y;   // fp32 [T, H dv]
+  void* out;  // [T, H dv], padding columns zeroed by the caller
+  float *dt, *cum;  // chunked form: fp32 [T, H]
+};
+int launch_mamba2_recurrent(const MambaArgs& a, bool is_f32, cudaStream_t st);  // xbc == nullptr: one row per sequence
+int launch_mamba2_chunked(const MambaArgs& a, const LightningChunks& c, int chunk, cudaStream_t st);
+
+// delta.cu: gated delta rule. Projection rows p [T, ld]: q (G dk) | k (G dk) | v (H dv) | beta (H) at beta_at; low [T, H dk + H dv] fp32
+struct DeltaArgs {
+  const void* p;
+  long long ld;
+  int H, G, dk, dv, dv_real, beta_at;
+  const float* low;
+  long long ld_low;
+  const void* qkv;  // convolved and activated q | k | v [T, 2 G dk + H dv] (nullptr: the decode step convolves itself)
+  int taps;
+  const float* conv_w;
+  float* ring;
+  const float *dt_bias, *neg_a, *norm_w;  // [H dk], [H], [dv]
+  float* state;                           // [slots, H, dk, dv]
+  const long long* slots;
+  const int *q_start, *q_len, *positions;
+  int num_seqs, rows;
+  float q_scale, unit_eps, eps, mult;
+  float* o;  // fp32 [T, H dv]
+  void* out;
+  long long ld_out;
+};
+struct DeltaChunks {
+  const int *seq, *row0, *len;  // per chunk
+  const int *first, *count;     // per sequence
+  int n_chunks, chunk;
+  void* qk;      // bf16 [T, H, 6, dk]: q exp(b), k exp(b_end - b), k exp(b), high and low parts
+  void* a;       // bf16 [n_chunks, H, 4, chunk, chunk]: causal matrix, (I + M)^-1 beta, high and low parts
+  float* decay;  // [n_chunks, H, dk]
+};
+int launch_delta_recurrent(const DeltaArgs& a, bool is_f32, cudaStream_t st);  // qkv == nullptr: one row per sequence, norm and gate in the launch
+int launch_delta_chunked(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t st);
+
+// mixed.cu: attention with mixed scores over wide cache rows k [pages, 1, page, KV dk], v [pages, 1, page, KV dv]
+struct MixedDecodeArgs {
+  const void* q;  // [B, H dk]
+  long long q_stride;
+  const float* mix;  // [H, H] (to, from)
+  const void *kc, *vc;
+  const int* bt;
+  int bt_stride;
+  const int* ctx;
+  void* out;
+  float *part_o, *part_ml;  // [B, H, splits, dv], [B, H, splits, 2] (splits > 1)
+  int B, H, KV, dk, dv, page;
+  float scale;
+  int window, splits;
+  AttnExtra x;
+};
+bool mixed_decode_supported(int H, int KV, int dk, int dv);
+int launch_mixed_decode(const MixedDecodeArgs& a, cudaStream_t st);
+void launch_decode_merge(const float* po, const float* pml, void* out, int B, int H, int dv, int splits, AttnExtra x, cudaStream_t st);  // attention.cu
+void launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st);
 
 // a2a.cu: expert-parallel all-to-all over peer memory (see the file comment for the protocol)
 struct A2AParams {
@@ -265,7 +351,7 @@ void launch_a2a_wait(const A2AParams* p, unsigned epoch, cudaStream_t st);
 struct LatentGeom {
   int H, dk, dn, R, Rp, dr, drp;   // heads; padded q columns per head, its unrotated part; latent size, padded; rotated size, padded in the cache
   int dv, Kp;                      // value size per head, latent columns of the value weights (32-padded)
-  int off_c, off_r, off_g;         // column offsets in the projection rows: latent, rotated key, gate (-1: no gate)
+  int off_c, off_r, off_g;         // column offsets in the projection rows: latent, rotated key (-1: queries only), gate (-1: no gate)
 };
 struct LatentPrep {
   const int* positions;
@@ -288,6 +374,7 @@ struct LatentDecodeArgs {
   const int *row_seq, *row_ctx;
   int rows, page;
   float scale;
+  const float* sink;       // [H] (nullptr: none)
   int window, splits;      // splits: a power of two
   void* o_lat;             // bf16 [rows, H, Rp]: result when the splits of a row are one cluster
   float *part_o, *part_ml; // else fp32 [rows, H, clusters, Rp] and [rows, H, clusters, 2]
@@ -299,7 +386,7 @@ void launch_latent_expand(const LatentDecodeArgs& a, const int* row_idx, const v
                           const LatentGeom& g, cudaStream_t st);
 int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, const int* row_seq, const int* row_ctx, int rows, const float* wuk,
                            const float* wuv, const float* c_cache, const float* r_cache, const int* bt, int bt_stride, float* out, int out_pitch,
-                           const LatentGeom& g, int page, float scale, int window, cudaStream_t st);
+                           const LatentGeom& g, int page, float scale, int window, const float* sink, cudaStream_t st);
 void launch_linear_f32(const float* x, int ldx, const float* w, const float* bias, float* out, int ldo, int M, int N, int K, cudaStream_t st);
 // w stacks experts [N, K]; items: work list of launch_moe_items with 64 rows per item
 void launch_grouped_linear_f32(const float* x, int ldx, const float* w, float* out, int ldo, const int* items, int n_items, int N, int K, cudaStream_t st);
@@ -316,6 +403,7 @@ struct LatentTcArgs {
   int out_pitch;
   const void* gate;
   int gate_pitch;
+  const float* sink;
   float scale;
   int window;
   int* status;
@@ -330,8 +418,8 @@ void launch_bigram_embedding(const void* table, const void* bigram, const int* i
 void launch_add_layernorm(float* residual, const float* delta, const float* w1, const float* b1, void* y1, const float* w2, const float* b2, void* y2,
                           int rows, int W, int y_pitch, float eps, bool is_f32, cudaStream_t st);
 void launch_sandwich_norm(float* residual, const void* sub, long long ld_sub, bool sub_f32, const int* pos, const float* wts, int k, const float* w_sub,
-                          float mult, const float* w_next, void* y, long long ld_y, int rows, int W, int y_width, float eps, bool vec, bool is_f32,
-                          cudaStream_t st);
+                          bool sub_one, float mult, const float* w_next, bool next_one, bool rms, void* y, long long ld_y, int rows, int W, int y_width, float eps,
+                          bool vec, bool is_f32, cudaStream_t st);
 void launch_rope_pairs_kv(void* qkv, long long ld, const int* positions, const long long* slots, const float* cos_t, const float* sin_t, void* k_cache,
                           void* v_cache, int T, int H, int KV, int dk, int dv, int page, int half, int max_pos, bool is_f32, cudaStream_t st);
 
@@ -347,6 +435,7 @@ struct RopeHeadsArgs {
   int T, H, KV, dk, dv, dim, page, half, max_pos;  // dim: real columns of a head (the norm's divisor)
   const float *q_norm, *k_norm;                    // [dk] or nullptr
   float eps;
+  int wide;             // a cache row holds all heads of a token ([pages, 1, page, KV * width])
   const void* v_first;  // values to blend with, row pitch ld_first (nullptr: none)
   long long ld_first;
   float lam;
@@ -385,6 +474,8 @@ struct LightningArgs {
   long long ld;
   int H, dk, dv, off_k, off_v, off_g;
   const float* powers;  // [H, chunk + 2]: decay^0 .. decay^chunk, then what fp32 loses of decay^1
+  int off_q, qk_div;    // first column of the queries; head h uses query / key head h / qk_div
+  const float *cum, *vscale;  // launch_decayed_chunks: [rows, H] running sums of the base-2 log decays inside a chunk, weights of the values
   int chunk;
   float* state;  // [slots, H, dk, dv]
   const long long* slots;
@@ -407,6 +498,7 @@ struct LightningChunks {
 };
 int launch_lightning_recurrent(const LightningArgs& a, bool is_f32, cudaStream_t st);
 int launch_lightning_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st);
+int launch_decayed_chunks(const LightningArgs& a, const LightningChunks& c, cudaStream_t st);  // outputs in a.o, no activation, norm or gate
 
 // gla.cu: gated linear attention. Projection rows p [T, ld] = q (H dk) | k (H dk) | v (H dv) | g (H dv) | a (rank), widths multiples of 8
 struct GlaArgs {

@@ -119,7 +119,7 @@ template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(T* __restrict__ p, long long ld, int rows, LatentPrep pr, LatentGeom g, int dn_pad) {
   pdl_wait();
   pdl_trigger();
-  if (blockIdx.y == 1) {
+  if (blockIdx.y == 1) {  // (not launched for rows without a latent)
     const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
     if (t >= rows || pr.slots[t] < 0) return;
     latent_cache_row<T>(p + t * ld, pr.slots[t], clamp_pos(pr.positions[t], pr.max_pos), pr, g, threadIdx.x & 31);
@@ -159,7 +159,7 @@ static void launch_latent_prepare_t(void* p, long long ld, int rows, const Laten
   const int dn_pad = (g.dn + 63) / 64 * 64;
   const int vec = pr.half % 8 == 0 ? 8 : 1;
   const long long rot = (static_cast<long long>(rows) * g.H * (pr.half / vec) + 255) / 256, cache = (rows + 7) / 8;
-  const dim3 grid(static_cast<unsigned>(rot > cache ? rot : cache), 2);
+  const dim3 grid(static_cast<unsigned>(rot > cache ? rot : cache), g.off_c >= 0 ? 2 : 1);
   if (vec == 8) launch_pdl(latent_prepare_kernel<T, 8>, grid, dim3(256), 0, st, static_cast<T*>(p), ld, rows, pr, g, dn_pad);
   else launch_pdl(latent_prepare_kernel<T, 1>, grid, dim3(256), 0, st, static_cast<T*>(p), ld, rows, pr, g, dn_pad);
 }
@@ -277,7 +277,7 @@ void launch_latent_absorb(const void* p, long long ld, const int* row_idx, int r
                           const LatentPrep* prep, cudaStream_t st) {
   if (rows == 0) return;
   const LatentPrep none = {};
-  launch_pdl(latent_absorb_kernel, dim3(g.H + (prep ? 1 : 0), (rows + 15) / 16, (g.Rp + 127) / 128), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(p),
+  launch_pdl(latent_absorb_kernel, dim3(g.H + (prep && g.off_c >= 0 ? 1 : 0), (rows + 15) / 16, (g.Rp + 127) / 128), dim3(128), 0, st, static_cast<const __nv_bfloat16*>(p),
              ld, row_idx, rows, static_cast<const __nv_bfloat16*>(wuk), static_cast<__nv_bfloat16*>(q_lat), g, (g.dn + 63) / 64 * 64, prep ? *prep : none,
              prep ? 1 : 0);
 }
@@ -336,7 +336,7 @@ template <int NPW, int MH, int NQ>
 __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) latent_decode_kernel(
     const __nv_bfloat16* __restrict__ q_lat, const __nv_bfloat16* __restrict__ c_cache, const __nv_bfloat16* __restrict__ r_cache, const int* __restrict__ bt,
     int bt_stride, const int* __restrict__ row_seq, const int* __restrict__ row_ctx, __nv_bfloat16* __restrict__ o_lat, float* __restrict__ part_o,
-    float* __restrict__ part_ml, LatentGeom g, int page, float scale, int window, int cs) {
+    float* __restrict__ part_ml, LatentGeom g, int page, float scale, const float* __restrict__ sink, int window, int cs) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(128) uint8_t lsm[];
@@ -593,6 +593,7 @@ __global__ void __launch_bounds__(256 * MH, (MH == 1 && NPW <= 4) ? 2 : 1) laten
         ms[s] = ms[s] == -INFINITY ? 0.f : __expf(ms[s] - m);
         l += ms[s] * (cs > 1 ? ld_cluster_f1(sL + tid, s) : sL[tid]);
       }
+    if (sink != nullptr && outer == 1 && tid < nh) l += __expf(sink[h0 + tid] - m);  // (m is finite: a row sees its own key)
     const float inv = outer > 1 ? 1.f : (l > 0.f ? 1.f / l : 0.f);
 #pragma unroll
     for (int s = 0; s < 8; ++s)
@@ -650,7 +651,7 @@ static int launch_latent_decode_t(const LatentDecodeArgs& a, const LatentGeom& g
   cfg.numAttrs = cs > 1 ? 2 : 1;
   cudaError_t e = cudaLaunchKernelEx(&cfg, latent_decode_kernel<NPW, MH, NQ>, static_cast<const __nv_bfloat16*>(a.q_lat),
                                      static_cast<const __nv_bfloat16*>(a.c_cache), static_cast<const __nv_bfloat16*>(a.r_cache), a.bt, a.bt_stride, a.row_seq,
-                                     a.row_ctx, static_cast<__nv_bfloat16*>(a.o_lat), a.part_o, a.part_ml, g, a.page, a.scale, a.window, cs);
+                                     a.row_ctx, static_cast<__nv_bfloat16*>(a.o_lat), a.part_o, a.part_ml, g, a.page, a.scale, a.sink, a.window, cs);
   if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode attention launch: ") + cudaGetErrorString(e));
   return 0;
 }
@@ -674,7 +675,8 @@ template <bool MERGE>
 __global__ void __launch_bounds__(128) latent_expand_kernel(const __nv_bfloat16* __restrict__ o_lat, const float* __restrict__ part_o,
                                                             const float* __restrict__ part_ml, int outer, const int* __restrict__ row_idx, int rows,
                                                             const __nv_bfloat16* __restrict__ wuv, const __nv_bfloat16* __restrict__ p, long long ld,
-                                                            __nv_bfloat16* __restrict__ out, int out_pitch, LatentGeom g) {
+                                                            __nv_bfloat16* __restrict__ out, int out_pitch, LatentGeom g,
+                                                            const float* __restrict__ sink) {
   const int h = blockIdx.x, i0 = blockIdx.y * 16, n0 = blockIdx.z * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, c = lane & 3;
   const int dv8 = (g.dv + 7) & ~7;
   {  // weights do not depend on the kernel in front: towards L2 while it finishes
@@ -693,7 +695,7 @@ __global__ void __launch_bounds__(128) latent_expand_kernel(const __nv_bfloat16*
       const float* ml = part_ml + (static_cast<size_t>(i0 + tid) * g.H + h) * outer * 2;
       float m = -INFINITY;
       for (int s = 0; s < outer; ++s) m = fmaxf(m, ml[2 * s]);
-      float den = 0.f;
+      float den = sink != nullptr ? __expf(sink[h] - m) : 0.f;
       for (int s = 0; s < outer; ++s) {
         const float w = ml[2 * s] == -INFINITY ? 0.f : __expf(ml[2 * s] - m);
         sW[tid * outer + s] = w;
@@ -782,8 +784,8 @@ void launch_latent_expand(const LatentDecodeArgs& a, const int* row_idx, const v
   const dim3 grid(g.H, (a.rows + 15) / 16, (g.dv + 31) / 32);
   const auto *ol = static_cast<const __nv_bfloat16*>(a.o_lat), *w = static_cast<const __nv_bfloat16*>(wuv), *pp = static_cast<const __nv_bfloat16*>(p);
   auto* o = static_cast<__nv_bfloat16*>(out);
-  if (outer > 1) launch_pdl(latent_expand_kernel<true>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g);
-  else launch_pdl(latent_expand_kernel<false>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g);
+  if (outer > 1) launch_pdl(latent_expand_kernel<true>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g, a.sink);
+  else launch_pdl(latent_expand_kernel<false>, grid, dim3(128), smem, st, ol, a.part_o, a.part_ml, outer, row_idx, a.rows, w, pp, ld, o, out_pitch, g, a.sink);
 }
 
 // ------------------------------------------------------------------------------------------------ 32-bit form
@@ -793,7 +795,7 @@ __global__ void __launch_bounds__(256) latent_rows_f32_kernel(const float* __res
                                                               const float* __restrict__ wuv, const float* __restrict__ c_cache,
                                                               const float* __restrict__ r_cache, const int* __restrict__ bt, int bt_stride,
                                                               float* __restrict__ out, int out_pitch, LatentGeom g, int dn_pad, int page, float scale,
-                                                              int window) {
+                                                              int window, const float* __restrict__ sink) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float fsm[];
@@ -849,6 +851,7 @@ __global__ void __launch_bounds__(256) latent_rows_f32_kernel(const float* __res
     }
   }
   __syncthreads();
+  if (sink != nullptr) l_run += expf(sink[h] - m_run);  // (a row sees its own key: m_run is finite)
   const int dv8 = (g.dv + 7) & ~7;
   for (int v = warp; v < g.dv; v += 8) {
     const float* w = wuv + (static_cast<size_t>(h) * dv8 + v) * g.Kp;
@@ -864,12 +867,12 @@ __global__ void __launch_bounds__(256) latent_rows_f32_kernel(const float* __res
 
 int launch_latent_rows_f32(const float* p, long long ld, const int* row_idx, const int* row_seq, const int* row_ctx, int rows, const float* wuk,
                            const float* wuv, const float* c_cache, const float* r_cache, const int* bt, int bt_stride, float* out, int out_pitch,
-                           const LatentGeom& g, int page, float scale, int window, cudaStream_t st) {
+                           const LatentGeom& g, int page, float scale, int window, const float* sink, cudaStream_t st) {
   if (rows == 0) return 0;
   const size_t smem = static_cast<size_t>(2 * g.Rp + g.drp + 64) * 4;
   if (smem > 46 * 1024 || g.H > 65535) return 1;
   launch_pdl(latent_rows_f32_kernel, dim3(rows, g.H), dim3(256), smem, st, p, ld, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, bt, bt_stride, out,
-             out_pitch, g, (g.dn + 63) / 64 * 64, page, scale, window);
+             out_pitch, g, (g.dn + 63) / 64 * 64, page, scale, window, sink);
   return 0;
 }
 

@@ -14,6 +14,8 @@
 //   What is fp32 by definition (weighted values, state, weights) enters the tensor cores as pairs of bf16 numbers (high and low part, 16 bits of
 //   mantissa) with fp32 accumulation; the activated q, k, v are exact in bf16.
 //   lightning_norm_gate_kernel  norm over all heads of a row, output gate.
+// With decays that are data (DATA: one number per token and head, running sums of their base-2 logarithms inside the chunk in `cum`, values weighted by
+// `vscale`, queries and keys shared by groups of heads) the same three kernels are the chunked form of Mamba-2 (mamba.cu), without activation and norm.
 #include "common.cuh"
 #include "gemm_api.h"
 #include "io.cuh"
@@ -194,16 +196,30 @@ constexpr int kLnPV = kLnCols + 8;  // row pitch of value and state tiles
 template <int NK>
 struct LnKv {
   static constexpr int P = NK * 16 + 8;
-  static constexpr int kBytes = (kLnChunk * P + 2 * kLnChunk * kLnPV) * 2 + (kLnChunk + 4) * 4;
+  static constexpr int kBytes = (kLnChunk * P + 2 * kLnChunk * kLnPV) * 2 + (2 * kLnChunk + 4) * 4;
 };
 template <int NK>
 struct LnOut {
   static constexpr int P = NK * 16 + 8;
-  static constexpr int kBytes = (kLnChunk * P + kLnChunk * kLnPV + 2 * NK * 16 * kLnPV) * 2 + (kLnChunk + 4) * 4;
+  static constexpr int kBytes = (kLnChunk * P + kLnChunk * kLnPV + 2 * NK * 16 * kLnPV) * 2 + (2 * kLnChunk + 4) * 4;
   static_assert(kBytes <= 227 * 1024, "tiles must fit shared memory");
 };
 
-template <int NK>
+__device__ __forceinline__ float ln_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// DATA: the chunk's running sums and value weights (zero behind its end: a weight of one that meets zero rows)
+__device__ __forceinline__ void load_decays(const LightningArgs& a, int row0, int len, int h, float* cum, float* vs) {
+  for (int i = threadIdx.x; i < kLnChunk; i += 256) {
+    const size_t at = static_cast<size_t>(row0 + (i < len ? i : 0)) * a.H + h;
+    cum[i] = i < len ? a.cum[at] : 0.f;
+    vs[i] = i < len ? a.vscale[at] : 0.f;
+  }
+}
+
+template <int NK, bool DATA>
 __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const LightningArgs a, const LightningChunks c) {
   pdl_wait();
   pdl_trigger();
@@ -211,12 +227,14 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
   extern __shared__ __align__(16) uint8_t lsm[];
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(lsm);      // [128][P]
   __nv_bfloat16* sV = sK + kLnChunk * L::P;                       // [2][128][kLnPV] decay^(len - 1 - t) v_t, high and low parts
-  float* pw = reinterpret_cast<float*>(sV + 2 * kLnChunk * kLnPV);  // decay^0 ..
+  float* pw = reinterpret_cast<float*>(sV + 2 * kLnChunk * kLnPV);  // decay^0 ..; DATA: running sums, then value weights
   const int ck = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kLnCols, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int row0 = c.row0[ck], len = c.len[ck], dk = a.dk, dv = a.dv;
   const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(a.p) + static_cast<size_t>(row0) * a.ld;
-  for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
-  copy_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
+  if constexpr (DATA) load_decays(a, row0, len, h, pw, pw + kLnChunk);
+  else
+    for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
+  copy_tile<NK>(sK, p + a.off_k + h / a.qk_div * dk, a.ld, len, dk);
   cp_commit();
   __syncthreads();
   for (int e = tid; e < kLnChunk * 8; e += 256) {
@@ -225,7 +243,7 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
     if (t < len && c0 + x < dv) {
       const uint4 u = *reinterpret_cast<const uint4*>(p + t * a.ld + a.off_v + h * dv + c0 + x);
       const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-      const float s = pw[len - 1 - t];
+      const float s = DATA ? ln_ex2(pw[len - 1] - pw[t]) * pw[kLnChunk + t] : pw[len - 1 - t];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 f = unpack_bf162(w[i]);
@@ -280,6 +298,7 @@ __global__ void __launch_bounds__(256) lightning_chunk_kv_kernel(const Lightning
 
 // a thread keeps four elements of a state and walks the sequence's chunks, four loads ahead; the state in front of every chunk is left as
 // two bf16 planes (high and low parts), the operands of the next kernel
+template <bool DATA>
 __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs a, const LightningChunks c) {
   pdl_wait();
   pdl_trigger();
@@ -289,7 +308,7 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs
   float4* slot = reinterpret_cast<float4*>(a.state + (static_cast<size_t>(a.slots[s]) * a.H + h) * per + at);
   float4 st = make_float4(0.f, 0.f, 0.f, 0.f);
   if (a.positions[a.q_start[s]] != 0) st = *slot;
-  const float* pw = a.powers + static_cast<size_t>(h) * (kLnChunk + 2);
+  const float* pw = DATA ? nullptr : a.powers + static_cast<size_t>(h) * (kLnChunk + 2);
   auto chunk = [&](int i) { return reinterpret_cast<const float4*>(c.added + (static_cast<size_t>(first + i) * a.H + h) * per + at); };
   __nv_bfloat16* planes = static_cast<__nv_bfloat16*>(c.states);
   constexpr int AHEAD = 4;
@@ -309,14 +328,15 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningArgs
       __nv_bfloat16* hi = planes + (static_cast<size_t>(first + i) * a.H + h) * 2 * per + at;
       *reinterpret_cast<uint2*>(hi) = make_uint2(h0, h1);
       *reinterpret_cast<uint2*>(hi + per) = make_uint2(l0, l1);
-      const float d = pw[c.len[first + i]];
+      const int len = c.len[first + i];
+      const float d = DATA ? ln_ex2(a.cum[static_cast<size_t>(c.row0[first + i] + len - 1) * a.H + h]) : pw[len];
       st = make_float4(fmaf(st.x, d, add.x), fmaf(st.y, d, add.y), fmaf(st.z, d, add.z), fmaf(st.w, d, add.w));
     }
   }
   *slot = st;
 }
 
-template <int NK>
+template <int NK, bool DATA>
 __global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_kernel(const LightningArgs a, const LightningChunks c) {
   pdl_wait();
   pdl_trigger();
@@ -337,21 +357,23 @@ __global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_ke
     cp16(smem_u32(sS + (plane * NK * 16 + d) * kLnPV + x), state + (ok ? (static_cast<size_t>(plane) * dk + d) * dv + c0 + x : 0), ok);
   }
   cp_commit();
-  copy_tile<NK>(sK, p + a.off_k + h * dk, a.ld, len, dk);
+  copy_tile<NK>(sK, p + a.off_k + h / a.qk_div * dk, a.ld, len, dk);
   for (int e = tid; e < kLnChunk * 8; e += 256) {
     const int t = e >> 3, x = (e & 7) * 8;
     const bool ok = t < len && c0 + x < dv;
     cp16(smem_u32(sV + t * kLnPV + x), p + (ok ? t * a.ld + a.off_v + h * dv + c0 + x : 0), ok);
   }
   cp_commit();
-  for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
+  if constexpr (DATA) load_decays(a, row0, len, h, pw, pw + kLnChunk);
+  else
+    for (int i = tid; i <= kLnChunk; i += 256) pw[i] = a.powers[static_cast<size_t>(h) * (kLnChunk + 2) + i];
   const int r0 = warp * 16, g = lane >> 2, t4 = lane & 3;  // this warp's token rows
   const bool mine = r0 < len;
   uint32_t q[NK][4];  // query fragments, straight from the rows
   {
     const bool ok0 = r0 + g < len, ok1 = r0 + g + 8 < len;
-    const __nv_bfloat16* qa = p + h * dk + static_cast<long long>(ok0 ? r0 + g : 0) * a.ld + 2 * t4;
-    const __nv_bfloat16* qb = p + h * dk + static_cast<long long>(ok1 ? r0 + g + 8 : 0) * a.ld + 2 * t4;
+    const __nv_bfloat16* qa = p + a.off_q + h / a.qk_div * dk + static_cast<long long>(ok0 ? r0 + g : 0) * a.ld + 2 * t4;
+    const __nv_bfloat16* qb = p + a.off_q + h / a.qk_div * dk + static_cast<long long>(ok1 ? r0 + g + 8 : 0) * a.ld + 2 * t4;
 #pragma unroll
     for (int kt = 0; kt < NK; ++kt) {
       const bool lo = kt * 16 < dk, hi = kt * 16 + 8 < dk;  // (widths are multiples of 8)
@@ -385,7 +407,8 @@ __global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_ke
   cp_wait<0>();
   __syncthreads();
   if (!mine) return;
-  const float d0 = pw[r0 + g + 1], d1 = pw[min(r0 + g + 9, kLnChunk)];
+  const float b0 = DATA ? pw[r0 + g] : 0.f, b1 = DATA ? pw[r0 + g + 8] : 0.f;
+  const float d0 = DATA ? ln_ex2(b0) : pw[r0 + g + 1], d1 = DATA ? ln_ex2(b1) : pw[min(r0 + g + 9, kLnChunk)];
 #pragma unroll
   for (int n = 0; n < 8; ++n) {
     o[n][0] *= d0;
@@ -409,8 +432,9 @@ __global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_ke
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int back = r0 + g + (e >> 1) * 8 - (j * 16 + n * 8 + 2 * t4 + (e & 1));
-        sc[n][e] = back >= 0 ? sc[n][e] * pw[back] : 0.f;
+        const int key = j * 16 + n * 8 + 2 * t4 + (e & 1), back = r0 + g + (e >> 1) * 8 - key;
+        if constexpr (DATA) sc[n][e] = back >= 0 ? sc[n][e] * ln_ex2(((e >> 1) ? b1 : b0) - pw[key]) * pw[kLnChunk + key] : 0.f;
+        else sc[n][e] = back >= 0 ? sc[n][e] * pw[back] : 0.f;
       }
     uint32_t ph[4], pl[4];
     split2(sc[0][0], sc[0][1], ph[0], pl[0]);
@@ -437,38 +461,49 @@ __global__ void __launch_bounds__(256, (NK <= 8 ? 2 : 1)) lightning_chunk_out_ke
   }
 }
 
-template <int NK>
+template <int NK, bool DATA>
 static cudaError_t launch_chunked_t(const LightningArgs& a, const LightningChunks& c, cudaStream_t st) {
   static PerDeviceOnce once;
   cudaError_t e = cudaSuccess;
   if (once.first()) {
-    e = cudaFuncSetAttribute(lightning_chunk_kv_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, LnKv<NK>::kBytes);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(lightning_chunk_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, LnOut<NK>::kBytes);
+    e = cudaFuncSetAttribute(lightning_chunk_kv_kernel<NK, DATA>, cudaFuncAttributeMaxDynamicSharedMemorySize, LnKv<NK>::kBytes);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(lightning_chunk_out_kernel<NK, DATA>, cudaFuncAttributeMaxDynamicSharedMemorySize, LnOut<NK>::kBytes);
     if (e != cudaSuccess) return e;
   }
-  const int n = a.off_v + a.H * a.dv;
-  const unsigned vecs = static_cast<unsigned>(n) / 8 * static_cast<unsigned>(a.rows);
-  e = launch_pdl(lightning_act_kernel, dim3((vecs + 255) / 256), dim3(256), 0, st, a, static_cast<__nv_bfloat16*>(const_cast<void*>(a.p)), n);
-  if (e != cudaSuccess) return e;
+  if constexpr (!DATA) {
+    const int n = a.off_v + a.H * a.dv;
+    const unsigned vecs = static_cast<unsigned>(n) / 8 * static_cast<unsigned>(a.rows);
+    e = launch_pdl(lightning_act_kernel, dim3((vecs + 255) / 256), dim3(256), 0, st, a, static_cast<__nv_bfloat16*>(const_cast<void*>(a.p)), n);
+    if (e != cudaSuccess) return e;
+  }
   const dim3 grid(c.n_chunks, a.H, (a.dv + kLnCols - 1) / kLnCols);
-  e = launch_pdl(lightning_chunk_kv_kernel<NK>, grid, dim3(256), LnKv<NK>::kBytes, st, a, c);
+  e = launch_pdl(lightning_chunk_kv_kernel<NK, DATA>, grid, dim3(256), LnKv<NK>::kBytes, st, a, c);
   if (e != cudaSuccess) return e;
   const unsigned blocks = static_cast<unsigned>((static_cast<size_t>(a.dk) * a.dv / 4 + 255) / 256);
-  e = launch_pdl(lightning_scan_kernel, dim3(blocks, a.H, a.num_seqs), dim3(256), 0, st, a, c);
+  e = launch_pdl(lightning_scan_kernel<DATA>, dim3(blocks, a.H, a.num_seqs), dim3(256), 0, st, a, c);
   if (e != cudaSuccess) return e;
-  return launch_pdl(lightning_chunk_out_kernel<NK>, grid, dim3(256), LnOut<NK>::kBytes, st, a, c);
+  return launch_pdl(lightning_chunk_out_kernel<NK, DATA>, grid, dim3(256), LnOut<NK>::kBytes, st, a, c);
+}
+
+template <bool DATA>
+static cudaError_t launch_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st) {
+  if (a.dk <= 32) return launch_chunked_t<2, DATA>(a, c, st);
+  if (a.dk <= 64) return launch_chunked_t<4, DATA>(a, c, st);
+  if (a.dk <= 128) return launch_chunked_t<8, DATA>(a, c, st);
+  return launch_chunked_t<16, DATA>(a, c, st);
 }
 
 int launch_lightning_chunked(const LightningArgs& a, const LightningChunks& c, cudaStream_t st) {
   if (a.rows == 0 || c.n_chunks == 0) return 0;
   if (a.off_k != a.H * a.dk || a.off_v != 2 * a.off_k || static_cast<long long>(a.rows) * (a.off_v + a.H * a.dv) / 8 > 0xffffff00ll) return 1;
   if (a.dk > 256 || a.chunk != kLnChunk || (a.dv + kLnCols - 1) / kLnCols > 65535) return 1;
-  cudaError_t e;
-  if (a.dk <= 32) e = launch_chunked_t<2>(a, c, st);
-  else if (a.dk <= 64) e = launch_chunked_t<4>(a, c, st);
-  else if (a.dk <= 128) e = launch_chunked_t<8>(a, c, st);
-  else e = launch_chunked_t<16>(a, c, st);
-  return e != cudaSuccess ? 2 : launch_norm_gate(a, false, st);
+  return launch_chunked<false>(a, c, st) != cudaSuccess ? 2 : launch_norm_gate(a, false, st);
+}
+
+int launch_decayed_chunks(const LightningArgs& a, const LightningChunks& c, cudaStream_t st) {
+  if (a.rows == 0 || c.n_chunks == 0) return 0;
+  if (a.dk > 256 || a.chunk != kLnChunk || a.cum == nullptr || a.vscale == nullptr || a.qk_div < 1) return 1;
+  return launch_chunked<true>(a, c, st) != cudaSuccess ? 2 : 0;
 }
 
 }  // namespace dlv

@@ -1,7 +1,7 @@
 """Grouped-query softmax attention with per-layer sizes: unequal query / key and value widths, partial rotation of neighbouring pairs or of
 the two halves of the rotated columns, per-head query / key norms, values that are the projected keys or a blend with another layer's,
 sliding window with kept first tokens, score soft-cap, a sink per head in the denominator (a score that has no value), an output gate per
-column or per head.
+column or per head, scores of the heads mixed by a matrix in front of the softmax.
 
 One projection row is ``[q (H * dk) | k (G * dk) | v (G * dv) | g]`` with head widths rounded up to multiples of 8 (16-byte rows everywhere);
 the columns behind the real ones carry zero weights, so scores, cache rows and outputs are exact whatever the sizes. Tied values have no
@@ -10,6 +10,10 @@ columns of their own; ``g`` is there for gated heads. CUDA forms:
 * prompts: the tcgen05 / TMA kernel (``attention_tc.cu``) over the paged cache, heads up to 256 wide;
 * decode: the split-KV tensor-core kernel (``attention.cu``), heads up to 256 wide;
 * fp32 and wider heads: one CTA per (row, head) on CUDA cores.
+
+Mixed scores (``mixed``): a cache row holds all KV heads of a token, ``k [pages, 1, page, G * dk]`` and ``v [pages, 1, page, G * dv]``. Prompts move the mixing to the
+query side: head h's mixed score against a key is the product of the whole cache row with ``[sum_(g in group 0) mix[h, g] q_g | sum_(g in group 1) .. | ..]``, so
+the prompt kernel runs with queries of ``G * dk`` columns against one wide key. Decode steps take all heads of a row in one CTA and mix the fp32 scores.
 """
 from __future__ import annotations
 
@@ -33,6 +37,7 @@ class GroupedShape:
     vdim: int
     tied: bool = False  # the values are the projected keys
     gate: str = ""  # output gate: "" | "columns" | "heads"
+    mixed: bool = False  # the heads' scores are mixed in front of the softmax
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
@@ -41,6 +46,8 @@ class GroupedShape:
             raise ValueError(f"keys of {self.dim} columns cannot be values of {self.vdim}")
         if self.gate not in ("", "columns", "heads"):
             raise ValueError(f"unknown output gate '{self.gate}'")
+        if self.mixed and self.tied:
+            raise ValueError("mixed scores with tied values are not supported")
 
     @property
     def dk(self) -> int:
@@ -87,6 +94,7 @@ class GroupedShape:
     def tensor_core(self) -> bool:
         """Widths the tensor-core kernels take (fp32 and wider heads use the CUDA-core rows form)."""
         return max(self.dk, self.dv) <= 256
+
 
 
 def pad_head_rows(w: torch.Tensor, heads: int, dim: int, padded: int) -> torch.Tensor:
@@ -136,7 +144,8 @@ def rope_heads_kv(s: GroupedShape, p, positions, slots, cos, sin, k_cache, v_cac
         v = (1.0 - lam) * v.float() + lam * v_first.float().reshape(T, s.kv_heads, s.dv)
     page = k_cache.shape[2]
     blk, off = torch.div(slots, page, rounding_mode="floor"), slots % page
-    v_cache[blk, :, off, :] = v.to(v_cache.dtype)
+    cached = lambda c, x: x.reshape(T, c.shape[1], -1).to(c.dtype)  # noqa: E731  (mixed scores: one wide head)
+    v_cache[blk, :, off, :] = cached(v_cache, v)
 
     def normed(x, w):
         if w is None:
@@ -144,19 +153,21 @@ def rope_heads_kv(s: GroupedShape, p, positions, slots, cos, sin, k_cache, v_cac
         x = x.float()
         return x * torch.rsqrt(x.pow(2).sum(dim=-1, keepdim=True) / s.dim + eps) * w
 
-    k_cache[blk, :, off, :] = ref.apply_rope(normed(k, k_norm), pos, cos, sin).to(k_cache.dtype)
+    k_cache[blk, :, off, :] = cached(k_cache, ref.apply_rope(normed(k, k_norm), pos, cos, sin))
     p[:, : s.q_width] = ref.apply_rope(normed(q, q_norm), pos, cos, sin).reshape(T, -1).to(p.dtype)
 
 
 def attention(s: GroupedShape, qkv, batch, k_cache, v_cache, scale: float, softcap: float, window: int, keep_first: int, sink, splits: int, mult: float = 1.0,
-              out=None):
+              out=None, mix=None):
     """Heads of every row of the batch, ``[T, H * dv]`` (``out``: a column range of wider rows to write to); the batch's keys and values are
-    in the cache already. ``sink``: fp32 ``[H]`` or None. Gated shapes multiply with the sigmoid of their logits in ``qkv``, all with ``mult``."""
+    in the cache already. ``sink``: fp32 ``[H]`` or None. Gated shapes multiply with the sigmoid of their logits in ``qkv``, all with ``mult``.
+    ``mix``: fp32 ``[H, H]`` of shapes with mixed scores."""
     q = qkv[:, : s.q_width]
     gate = qkv[:, s.gate_at : s.gate_at + s.gate_logits] if s.gate else None
     if not ops._cuda(qkv):
-        o = ref.paged_attention(q.reshape(-1, s.heads, s.dk), k_cache, v_cache, batch.block_tables, batch.q_start.tolist(), batch.q_len.tolist(),
-                                batch.ctx_len.tolist(), scale, softcap, window, True, keep_first, sink)
+        split = lambda c: c.reshape(c.shape[0], c.shape[2], s.kv_heads, -1).transpose(1, 2) if s.mixed else c  # noqa: E731
+        o = ref.paged_attention(q.reshape(-1, s.heads, s.dk), split(k_cache), split(v_cache), batch.block_tables, batch.q_start.tolist(), batch.q_len.tolist(),
+                                batch.ctx_len.tolist(), scale, softcap, window, True, keep_first, sink, mix)
         if gate is not None:
             o = o.float() * torch.sigmoid(gate.float()).reshape(o.shape[0], s.heads, -1)
         o = (o * mult).to(qkv.dtype).reshape(-1, s.out_width)
@@ -164,6 +175,8 @@ def attention(s: GroupedShape, qkv, batch, k_cache, v_cache, scale: float, softc
     e = ops.require_ext()
     mask = (float(scale), float(softcap), int(window))
     extra = {"keep_first": int(keep_first), "sink": sink, "gate": gate, "out_mult": float(mult), "out": out}
+    if s.mixed:
+        return _mixed_attention(s, qkv, q, mix, batch, k_cache, v_cache, mask, splits, extra)
     if qkv.dtype == torch.float32 or not s.tensor_core:
         ops._count()
         return e.attention_rows(q, k_cache, v_cache, batch.block_tables, None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask, **extra)
@@ -175,8 +188,41 @@ def attention(s: GroupedShape, qkv, batch, k_cache, v_cache, scale: float, softc
     return e.prefill_attention_tc(q, k_cache, v_cache, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_len, ts, t0, s.heads, *mask, True, **extra)
 
 
+def _mixed_attention(s: GroupedShape, qkv, q, mix, batch, k_cache, v_cache, mask: tuple, splits: int, extra: dict):
+    e = ops.require_ext()
+    if batch.is_decode and qkv.dtype == torch.bfloat16 and e.mixed_decode_ok(s.heads, s.kv_heads, s.dk, s.dv):
+        ops._count(1 if splits <= 1 else 2)
+        return e.mixed_decode(q, mix, k_cache, v_cache, batch.block_tables, batch.ctx_len, s.heads, s.kv_heads, mask[0], mask[2], splits, gate=extra["gate"],
+                              out_mult=extra["out_mult"], out=extra["out"])
+    ops._count(2)
+    folded = e.fold_heads(q, mix, s.heads, s.kv_heads)
+    rows = 0 if qkv.dtype == torch.float32 else e.prefill_wide_tile_rows(s.k_width, s.dv)
+    if not rows:
+        return e.attention_rows(folded, k_cache, v_cache, batch.block_tables, None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask,
+                                kv_heads=s.kv_heads, **extra)
+    ts, t0 = batch.tiles(rows) if not batch.is_decode else decode_tiles(batch)
+    return e.prefill_attention_tc(folded, k_cache, v_cache, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_len, ts, t0, s.heads, *mask, True,
+                                  kv_heads=s.kv_heads, **extra)
+
+
+def decode_tiles(batch):
+    """Query tiles of a decode step: one per sequence."""
+    if "decode_tiles" not in batch.plans:
+        n, dev = batch.num_seqs, batch.q_len.device
+        batch.plans["decode_tiles"] = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, dtype=torch.int32, device=dev))
+    return batch.plans["decode_tiles"]
+
+
+def mixed_splits(num_seqs: int, span: int, sms: int = 148) -> int:
+    """Split-KV factor of the decode kernel of mixed scores: one CTA per (sequence, split), at least four 32-key tiles per split."""
+    tiles = max(1, (span + 31) // 32)
+    return int(max(1, min((sms + num_seqs - 1) // max(1, num_seqs), tiles // 4 if tiles >= 8 else 1, 64)))
+
+
 def row_sequence(batch) -> torch.Tensor:
     """Sequence of every row of a batch (int32, built once per batch)."""
+    if "row_seq" not in batch.plans and batch.is_decode:
+        batch.plans["row_seq"] = torch.arange(batch.num_seqs, dtype=torch.int32, device=batch.q_len.device)
     if "row_seq" not in batch.plans:
         n = torch.tensor(batch.q_len_host)
         batch.plans["row_seq"] = torch.repeat_interleave(torch.arange(len(n)), n).to(torch.int32).to(batch.q_len.device, non_blocking=True)

@@ -2,7 +2,8 @@
 that dispatch to the kernels of ``csrc/latent.cu`` / ``csrc/attention_tc.cu`` on CUDA and to plain PyTorch statements on the CPU.
 
 A token's projection row holds ``[q of every head: unrotated | rotated] [latent] [rotated key] [gate]``. The cache keeps, per token,
-the RMS-normed latent and the rotated key; per-head keys and values are linear in the latent.
+the RMS-normed latent and the rotated key; per-head keys and values are linear in the latent. A layer without a down projection (``down`` False) has
+queries and gate only and reads the cache of another layer with the same latent and rotated sizes.
 """
 from __future__ import annotations
 
@@ -27,6 +28,7 @@ class LatentShape:
     vdim: int
     kv_rank: int
     gate: bool = True
+    down: bool = True  # the layer projects its own latent and rotated key
 
     def __post_init__(self):
         if min(self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank) < 1 or self.rot_dim % 2:
@@ -44,12 +46,14 @@ class LatentShape:
     dv8 = property(lambda s: _up(s.vdim, 8))
     off_c = property(lambda s: s.heads * s.dk)
     off_r = property(lambda s: s.off_c + s.R8)
-    off_g = property(lambda s: s.off_r + _up(s.rot_dim, 8) if s.gate else -1)
-    width = property(lambda s: s.off_r + _up(s.rot_dim, 8) + (_up(s.heads * s.vdim, 8) if s.gate else 0))
+    behind = property(lambda s: s.off_r + _up(s.rot_dim, 8) if s.down else s.off_c)
+    off_g = property(lambda s: s.behind if s.gate else -1)
+    width = property(lambda s: s.behind + (_up(s.heads * s.vdim, 8) if s.gate else 0))
     out_width = property(lambda s: s.heads * s.vdim)
 
     def geom(self) -> list[int]:
-        return [self.heads, self.dk, self.dim, self.kv_rank, self.Rp, self.rot_dim, self.drp, self.vdim, self.Kp, self.off_c, self.off_r, self.off_g]
+        return [self.heads, self.dk, self.dim, self.kv_rank, self.Rp, self.rot_dim, self.drp, self.vdim, self.Kp, self.off_c if self.down else -1,
+                self.off_r if self.down else -1, self.off_g]
 
     def prefill_dv(self) -> int:
         """Padded value width of the tensor-core prefill kernel; 0 when these head sizes are outside it."""
@@ -64,8 +68,9 @@ def pack_input(s: LatentShape, q, dkv, g, k_pad: int) -> torch.Tensor:
     qv = w[: s.off_c].view(s.heads, s.dk, k_pad)
     qv[:, : s.dim, :K] = heads[:, : s.dim]
     qv[:, s.dn : s.dn + s.rot_dim, :K] = heads[:, s.dim :]
-    w[s.off_c : s.off_c + s.kv_rank, :K] = dkv[: s.kv_rank]
-    w[s.off_r : s.off_r + s.rot_dim, :K] = dkv[s.kv_rank :]
+    if s.down:
+        w[s.off_c : s.off_c + s.kv_rank, :K] = dkv[: s.kv_rank]
+        w[s.off_r : s.off_r + s.rot_dim, :K] = dkv[s.kv_rank :]
     if s.gate:
         w[s.off_g : s.off_g + s.out_width, :K] = g
     return w
@@ -91,7 +96,8 @@ def pack_expand(s: LatentShape, uk, uv, dv: int) -> torch.Tensor:
 
 # ---------------------------------------------------------------------------------------------------------- operators
 def prepare(s: LatentShape, p, positions, slots, norm_w, cos, sin, c_cache, r_cache, eps: float) -> None:
-    """Rotate the queries in place; RMS-norm the latent, rotate the shared key and write both to the cache rows ``slots``."""
+    """Rotate the queries in place; RMS-norm the latent, rotate the shared key and write both to the cache rows ``slots`` (layers with a down
+    projection)."""
     if _cuda(p):
         _count()
         require_ext().latent_prepare(p, positions, slots, norm_w, cos, sin, c_cache, r_cache, s.geom(), eps)
@@ -99,6 +105,8 @@ def prepare(s: LatentShape, p, positions, slots, norm_w, cos, sin, c_cache, r_ca
     T, pos = p.shape[0], positions.long()
     q = p[:, : s.off_c].view(T, s.heads, s.dk)
     q[:, :, s.dn : s.dn + s.rot_dim] = ref.apply_rope(q[:, :, s.dn : s.dn + s.rot_dim], pos, cos, sin)
+    if not s.down:
+        return
     c = ref.rmsnorm(p[:, s.off_c : s.off_c + s.kv_rank], norm_w[: s.kv_rank], eps)
     r = ref.apply_rope(p[:, s.off_r : s.off_r + s.rot_dim].unsqueeze(1), pos, cos, sin).squeeze(1)
     c_cache.view(-1, s.Rp)[slots.long()] = F.pad(c, (0, s.Rp - s.kv_rank)).to(c_cache.dtype)
@@ -106,20 +114,20 @@ def prepare(s: LatentShape, p, positions, slots, norm_w, cos, sin, c_cache, r_ca
 
 
 def rows_attention(s: LatentShape, p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, scale: float, window: int,
-                   splits: int = 1, write=None) -> None:
+                   splits: int = 1, write=None, sink=None) -> None:
     """Rows of ``p`` one by one against the cache (decode, short portions), absorbed form. Row ``i`` is ``p[row_idx[i]]`` of block-table
     row ``row_seq[i]`` and sees the last ``window`` of its first ``row_ctx[i]`` keys; ``None`` index arrays mean ``i``. Writes the gated
     heads to columns ``[0, H * vdim)`` of the rows of ``out``. ``write`` = the arguments of :func:`prepare` behind ``p``, for a decode batch
-    whose rows were not prepared yet (on CUDA in bf16 that work rides in the first launch)."""
+    whose rows were not prepared yet (on CUDA in bf16 that work rides in the first launch). ``sink`` fp32 ``[H]``: a score per head without a value."""
     if write is not None and (not _cuda(p) or p.dtype == torch.float32):
         prepare(s, p, *write)
     if _cuda(p):
         if p.dtype == torch.float32:
             _count()
-            require_ext().latent_rows_f32(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window)
+            require_ext().latent_rows_f32(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window, sink)
         else:
             _count(3)
-            require_ext().latent_decode(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window, splits,
+            require_ext().latent_decode(p, row_idx, row_seq, row_ctx, wuk, wuv, c_cache, r_cache, block_tables, out, s.geom(), scale, window, splits, sink,
                                         *(() if write is None else (*write[:5], write[7])))
         return
     n = row_ctx.shape[0]
@@ -135,7 +143,9 @@ def rows_attention(s: LatentShape, p, row_idx, row_seq, row_ctx, wuk, wuv, c_cac
         q = p[t, : s.off_c].view(s.heads, s.dk).float()
         ql = torch.einsum("hd,hrd->hr", q[:, : s.dn], wuk.float())
         sc = (ql @ c.t() + q[:, s.dn : s.dn + s.drp] @ r.t()) * scale
-        o = torch.softmax(sc, dim=-1) @ c
+        if sink is not None:
+            sc = torch.cat([sc, sink.view(-1, 1)], dim=1)
+        o = torch.softmax(sc, dim=-1)[:, : c.shape[0]] @ c
         o = torch.einsum("hr,hvr->hv", o, wuv[:, : s.vdim, : s.Rp].float()).reshape(-1)
         if s.gate:
             o = o * torch.sigmoid(p[t, s.off_g : s.off_g + s.out_width].float())
@@ -148,10 +158,10 @@ def gather(s: LatentShape, c_cache, r_cache, block_tables, seq, key0, n_keys, ro
     return require_ext().latent_gather(c_cache, r_cache, block_tables, seq, key0, n_keys, row0, max_rows, total, s.R8, s.dk - s.dn)
 
 
-def prefill_attention(s: LatentShape, p, kv, kr, q_start, q_len, ctx, row0, tile_seq, tile_q0, out, scale: float, window: int) -> None:
+def prefill_attention(s: LatentShape, p, kv, kr, q_start, q_len, ctx, row0, tile_seq, tile_q0, out, scale: float, window: int, sink=None) -> None:
     """Prompt rows against expanded keys and values (CUDA, tcgen05): gated heads to columns ``[0, H * vdim)`` of ``out``."""
     _count()
-    require_ext().latent_prefill(p, kv, kr, q_start, q_len, ctx, row0, tile_seq, tile_q0, out, s.geom(), scale, window)
+    require_ext().latent_prefill(p, kv, kr, q_start, q_len, ctx, row0, tile_seq, tile_q0, out, s.geom(), scale, window, sink)
 
 
 def prefill_tile_rows(dv: int) -> int:

@@ -28,6 +28,8 @@ def act_fn(name: str):
         return F.gelu
     if name == "relu":
         return F.relu
+    if name == "relu2":
+        return lambda x: F.relu(x).square()
     if name == "tanh":
         return torch.tanh
     raise ValueError(f"unknown activation '{name}'")
@@ -153,14 +155,14 @@ def qk_prepare_and_cache(qkv, positions, slots, n_heads, n_kv, head_dim, q_norm_
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, scale, softcap=0.0, window=0,
-                    causal=True, keep_first=0, sink=None):
+                    causal=True, keep_first=0, sink=None, mix=None):
     """Attention of ragged query rows against paged K/V.
 
     q ``[T, H, D]``; sequence ``i`` owns query rows ``[q_start[i], q_start[i] + q_len[i])`` which are the *last*
     ``q_len[i]`` positions of a context of ``ctx_len[i]`` cached tokens. Row at position ``p`` sees keys ``j <= p``
     (and ``j > p - window`` or ``j < keep_first`` when ``window > 0``). Score = ``softmax(softcap * tanh(scale * q.k / softcap))``;
-    ``sink`` ``[H]``: a further score per head without a value takes part in the softmax (neither scaled nor capped). Values may be wider or
-    narrower than keys.
+    ``sink`` ``[H]``: a further score per head without a value takes part in the softmax (neither scaled nor capped). ``mix`` ``[H, H]`` (to, from):
+    the heads' scores are mixed in front of the softmax. Values may be wider or narrower than keys.
     """
     T, H, D = q.shape
     nb, KV, bs, _ = k_cache.shape
@@ -179,6 +181,8 @@ def paged_attention(q, k_cache, v_cache, block_tables, q_start, q_len, ctx_len, 
         k = k.repeat_interleave(group, dim=0)
         v = v.repeat_interleave(group, dim=0)
         s = torch.matmul(qi, k.transpose(1, 2)) * scale
+        if mix is not None:
+            s = torch.einsum("hg,gtj->htj", mix.float(), s)
         if softcap and softcap > 0:
             s = torch.tanh(s / softcap) * softcap
         pos = torch.arange(cl - ql, cl, device=q.device).unsqueeze(1)
@@ -228,10 +232,11 @@ def add_layernorm(residual, delta, norm1, norm2, eps, pitch, dtype):
     return tuple(None if nb is None else F.pad(n * nb[0] + nb[1], (0, pad)).to(dtype) for nb in (norm1, norm2))
 
 
-def sandwich_norm(residual, sub, w_sub, mult, w_next, eps):
-    """fp32 ``residual += mult * LayerNorm(sub; w_sub)`` in place, then ``LayerNorm(residual; w_next)`` (the plain residual without it)."""
+def sandwich_norm(residual, sub, w_sub, mult, w_next, eps, rms=False):
+    """fp32 ``residual += mult * norm(sub; w_sub)`` in place, then ``norm(residual; w_next)`` (the plain residual without it); ``rms``: RMS norms
+    instead of LayerNorms."""
     def norm(v, w):
-        d = v - v.mean(dim=-1, keepdim=True)
+        d = v if rms else v - v.mean(dim=-1, keepdim=True)
         return d * torch.rsqrt(d.pow(2).mean(dim=-1, keepdim=True) + eps) * w
 
     if sub is not None:
@@ -294,47 +299,46 @@ def moe_experts(x, weights, idx, gate_up_fn, down_fn, num_experts, act, gated_fn
 
 
 # ---- Mamba2 ----------------------------------------------------------------------------------------------------------
-def mamba2_sequential(zxbcdt, conv_w, conv_b, dt_bias, A_log, D, norm_w, eps, n_heads, d_head, n_groups, d_state,
-                      conv_state, ssm_state, act="silu"):
-    """Token-by-token Mamba2 mixer core for ONE sequence (reference GraniteMoeHybridMambaLayer.java:130-252).
+def short_conv(x, weight, bias, ring, start: int):
+    """Causal convolution per channel over the rows ``x [n, C]`` of ONE sequence, whose first row is position ``start``, then silu; fp32 result.
+    ``weight [C, taps]`` (last column: the current token's). ``ring [taps, C]`` keeps the inputs of the last positions, position ``p`` at row ``p
+    mod taps``, and is advanced."""
+    n, taps = x.shape[0], weight.shape[1]
+    rows = [ring[p % taps].clone() if p >= 0 else torch.zeros_like(ring[0]) for p in range(start - taps + 1, start)]
+    x = x.float()
+    seen = torch.cat([torch.stack(rows), x]) if rows else x
+    acc = sum(seen[j : j + n] * weight[:, j].float() for j in range(taps))
+    if bias is not None:
+        acc = acc + bias.float()
+    for i in range(max(0, n - taps), n):
+        ring[(start + i) % taps] = x[i]
+    return F.silu(acc)
 
-    zxbcdt ``[T, I + convDim + H]`` laid out ``[gate (I) | x (I) | B (G*S) | C (G*S) | dt (H)]``;
-    conv_state ``[convDim, K-1]``, ssm_state ``[H, d_head, S]`` are updated in place. Returns ``[T, I]`` (after the
-    gated RMSNorm over the whole intermediate), fp32 math.
-    """
-    T = zxbcdt.shape[0]
-    I = n_heads * d_head
-    GS = n_groups * d_state
-    conv_dim = I + 2 * GS
-    Kc = conv_w.shape[-1]
-    f = act_fn(act)
-    A = -torch.exp(A_log.float())
-    out = torch.empty(T, I, dtype=torch.float32, device=zxbcdt.device)
-    cw = conv_w.float().reshape(conv_dim, Kc)
-    for t in range(T):
-        row = zxbcdt[t].float()
-        gate = row[:I]
-        xbc = row[I : I + conv_dim]
-        dt = F.softplus(row[I + conv_dim :] + dt_bias.float())
-        window = torch.cat([conv_state.float(), xbc.unsqueeze(1)], dim=1)  # convDim, K
-        conv = (window * cw).sum(dim=1)
-        if conv_b is not None:
-            conv = conv + conv_b.float()
-        conv_state.copy_(window[:, 1:].to(conv_state.dtype))
-        conv = f(conv)
-        x = conv[:I].reshape(n_heads, d_head)
-        B = conv[I : I + GS].reshape(n_groups, d_state)
-        C = conv[I + GS :].reshape(n_groups, d_state)
-        hpg = n_heads // n_groups
-        Bh = B.repeat_interleave(hpg, dim=0)  # H, S
-        Ch = C.repeat_interleave(hpg, dim=0)
-        decay = torch.exp(dt * A)  # H
-        st = ssm_state.float() * decay.view(-1, 1, 1) + (dt.view(-1, 1) * x).unsqueeze(2) * Bh.unsqueeze(1)
-        ssm_state.copy_(st.to(ssm_state.dtype))
-        y = (st * Ch.unsqueeze(1)).sum(dim=2) + D.float().view(-1, 1) * x
-        y = y.reshape(I) * f(gate)
-        y = y * torch.rsqrt(y.pow(2).mean() + eps) * norm_w.float()
-        out[t] = y
+
+def ssd_sequential(x, B, C, dt, neg_a, D, state):
+    """Token-by-token state-space recurrence of ONE sequence, fp32: ``S <- exp(neg_a dt) S + dt B x^T``, ``y = S^T C + D x``. x ``[T, H, dv]``, B and C
+    ``[T, G, N]`` (head h uses group h // (H / G)), dt ``[T, H]`` positive, neg_a and D ``[H]``; ``state [H, N, dv]`` is updated in place."""
+    x, group = x.float(), x.shape[1] // B.shape[1]
+    B, C = B.float().repeat_interleave(group, dim=1), C.float().repeat_interleave(group, dim=1)
+    y = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    decay = torch.exp(neg_a * dt)
+    for t in range(x.shape[0]):
+        state.mul_(decay[t].view(-1, 1, 1)).addcmul_((dt[t].unsqueeze(-1) * B[t]).unsqueeze(-1), x[t].unsqueeze(-2))
+        y[t] = (state * C[t].unsqueeze(-1)).sum(dim=-2) + D.view(-1, 1) * x[t]
+    return y
+
+
+# ---- gated delta rule --------------------------------------------------------------------------------------------------
+def delta_sequential(q, k, v, log_a, beta, state):
+    """Token-by-token gated delta rule of ONE sequence, fp32: ``S <- diag(exp(log_a)) S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q``.
+    q, k, log_a ``[T, H, dk]``, v ``[T, H, dv]``, beta ``[T, H]``; ``state [H, dk, dv]`` is updated in place. Returns ``[T, H, dv]``."""
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    a = torch.exp(log_a)
+    for t in range(v.shape[0]):
+        state.mul_(a[t].unsqueeze(-1))
+        u = beta[t].unsqueeze(-1) * (v[t] - (state * k[t].unsqueeze(-1)).sum(dim=-2))
+        state.addcmul_(k[t].unsqueeze(-1), u.unsqueeze(-2))
+        out[t] = (state * q[t].unsqueeze(-1)).sum(dim=-2)
     return out
 
 

@@ -110,7 +110,7 @@ def run_mixer(mixer, kv, h, portions, pages, run):
     for n in portions:
         b = make_batch([{"tokens": [0] * n, "start": at, "pages": pages}], kv.page_size, device)
         y = torch.zeros(n, (mixer.shape.out_width + 7) // 8 * 8, dtype=dtype, device=device)
-        mixer.forward(torch.nn.functional.pad(h[at : at + n], (0, pad)).to(device, dtype), b, kv.layer(0), y, lambda _: _Stage())
+        mixer.heads(torch.nn.functional.pad(h[at : at + n], (0, pad)).to(device, dtype), b, kv.layer(0), y, lambda _: _Stage())
         out.append(y[:, : mixer.shape.out_width].float().cpu())
         at += n
     return torch.cat(out)
@@ -201,7 +201,7 @@ def test_mixed_rows_and_prompts_in_one_batch(run):
     b = make_batch([{"tokens": [0] * n, "start": s, "pages": pg} for n, s, pg in zip(lens, starts, own)], kv.page_size, device)
     x = torch.cat([h[s:] for h, s in zip(hs, starts)]).to(device, dtype)
     y = torch.zeros(sum(lens), 40, dtype=dtype, device=device)
-    mixer.forward(x, b, kv.layer(0), y, lambda _: _Stage())
+    mixer.heads(x, b, kv.layer(0), y, lambda _: _Stage())
     row = 0
     for h, s, n in zip(hs, starts, lens):
         want = plain.latent_attention(W, m, "", h.double(), 1e-5)[s:]
@@ -504,7 +504,7 @@ def test_groups_of_16_heads_give_the_same_decode_result():
                 for t in range(697, 700):
                     b = make_batch([{"tokens": [0], "start": t, "pages": pages}], kv.page_size, "cuda")
                     y = torch.zeros(1, s.out_width, dtype=torch.bfloat16, device="cuda")
-                    mixer.forward(h[t : t + 1].cuda(), b, kv.layer(0), y, lambda _: _Stage())
+                    mixer.heads(h[t : t + 1].cuda(), b, kv.layer(0), y, lambda _: _Stage())
                     out.append(y.float().cpu())
                 assert rel(torch.cat(out), want) < tol(torch.bfloat16), (groups, splits)
         finally:
