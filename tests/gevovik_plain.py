@@ -64,13 +64,12 @@ def frequencies(rot):
 def rotate(x, rot, pairs):
     """x [T, heads, d], row t at position t. ``pairs``: entries 2 i and 2 i + 1 turn together, else i and i + dims / 2."""
     f, mult = frequencies(rot)
-    n, out = rot["dims"] // 2, x.clone()
-    for t in range(x.shape[0]):
-        for i in range(n):
-            a, b = (2 * i, 2 * i + 1) if pairs else (i, i + n)
-            c, s = math.cos(t * f[i]) * mult, math.sin(t * f[i]) * mult
-            out[t, :, a] = x[t, :, a] * c - x[t, :, b] * s
-            out[t, :, b] = x[t, :, b] * c + x[t, :, a] * s
+    n, out, t = rot["dims"] // 2, x.clone(), torch.arange(x.shape[0], dtype=real).unsqueeze(1)
+    for i in range(n):
+        a, b = (2 * i, 2 * i + 1) if pairs else (i, i + n)
+        c, s = torch.cos(t * f[i]) * mult, torch.sin(t * f[i]) * mult
+        out[..., a] = x[..., a] * c - x[..., b] * s
+        out[..., b] = x[..., b] * c + x[..., a] * s
     return out
 
 
@@ -79,10 +78,9 @@ def causal_conv(x, w, bias=None):
     """Per channel over time: x [T, C], w [C, taps], the last column is the current token's, zeros in front of the sequence."""
     T, taps = x.shape[0], w.shape[1]
     out = torch.zeros_like(x)
-    for t in range(T):
-        for j in range(taps):
-            if t - (taps - 1 - j) >= 0:
-                out[t] += w[:, j].to(real) * x[t - (taps - 1 - j)]
+    for j in range(taps):
+        back = taps - 1 - j
+        out[back:] += w[:, j].to(real) * x[: T - back] if back < T else 0
     return out if bias is None else out + bias.to(real)
 
 
@@ -92,11 +90,11 @@ def ssd(x, B, C, dt, A_log, D):
     T, H, dv = x.shape
     G, N = B.shape[1:]
     S, y = torch.zeros(H, N, dv, dtype=real), torch.zeros(T, H, dv, dtype=real)
+    group = [h // (H // G) for h in range(H)]
     for t in range(T):
-        for h in range(H):
-            g = h // (H // G)
-            S[h] = torch.exp(-torch.exp(A_log[h]) * dt[t, h]) * S[h] + dt[t, h] * torch.outer(B[t, g], x[t, h])
-            y[t, h] = S[h].T @ C[t, g] + D[h] * x[t, h]
+        decay, b, c = torch.exp(-torch.exp(A_log) * dt[t]), B[t, group], C[t, group]
+        S = decay.view(H, 1, 1) * S + dt[t].view(H, 1, 1) * b.unsqueeze(2) * x[t].unsqueeze(1)
+        y[t] = (S * c.unsqueeze(2)).sum(dim=1) + D.view(H, 1) * x[t]
     return y
 
 
@@ -117,12 +115,12 @@ def mixed_head_attention(q, k, v, scale, temp, talk, window):
     to, from), in front of a softmax over the last ``window`` keys."""
     T, H, G = q.shape[0], q.shape[1], k.shape[1]
     out = torch.zeros(T, H, v.shape[2], dtype=real)
+    own = [n // (H // G) for n in range(H)]
     for t in range(T):
         lo = max(0, t - window + 1) if window else 0
-        raw = torch.stack([k[lo : t + 1, n // (H // G)] @ q[t, n] * scale * temp[n] for n in range(H)])
+        raw = (k[lo : t + 1, own] * q[t]).sum(dim=-1).T * scale * temp.unsqueeze(1)  # [H, keys]
         s = torch.softmax(talk @ raw, dim=-1)
-        for n in range(H):
-            out[t, n] = s[n] @ v[lo : t + 1, n // (H // G)]
+        out[t] = (s.T.unsqueeze(2) * v[lo : t + 1, own]).sum(dim=0)
     return out
 
 
@@ -142,11 +140,10 @@ def delta_rule(q, k, v, a, beta):
     T, H, d = q.shape
     S, out = torch.zeros(H, d, v.shape[2], dtype=real), torch.zeros(v.shape, dtype=real)
     for t in range(T):
-        for n in range(H):
-            S[n] = a[t, n].unsqueeze(-1) * S[n]
-            u = beta[t, n] * (v[t, n] - S[n].T @ k[t, n])
-            S[n] = S[n] + torch.outer(k[t, n], u)
-            out[t, n] = S[n].T @ q[t, n]
+        S = a[t].unsqueeze(2) * S
+        u = beta[t].unsqueeze(1) * (v[t] - (S * k[t].unsqueeze(2)).sum(dim=1))
+        S = S + k[t].unsqueeze(2) * u.unsqueeze(1)
+        out[t] = (S * q[t].unsqueeze(2)).sum(dim=1)
     return out
 
 
@@ -180,10 +177,10 @@ def latent_rows(W, m, p, h, eps):
 
 
 def sink_softmax(s, sink):
-    """Weights of scores s [n] beside a sink that has neither key nor value."""
-    top = max(s.max().item(), sink)
+    """Weights of scores s [H, n] beside a sink per head that has neither key nor value."""
+    top = torch.maximum(s.max(dim=-1).values, sink).unsqueeze(1)
     e = torch.exp(s - top)
-    return e / (e.sum() + math.exp(sink - top))
+    return e / (e.sum(dim=-1, keepdim=True) + torch.exp(sink.unsqueeze(1) - top))
 
 
 def latent_attention(W, m, p, h, c, r):
@@ -194,9 +191,8 @@ def latent_attention(W, m, p, h, c, r):
     k, v = (c @ g("uk").T).reshape(T, H, d), (c @ g("uv").T).reshape(T, H, dv)
     out = torch.zeros(T, H, dv, dtype=real)
     for t in range(T):
-        for n in range(H):
-            s = (k[: t + 1, n] @ q[t, n, :d] + r[: t + 1] @ qr[t, n]) * m["scale"]
-            out[t, n] = sink_softmax(s, g("sink").reshape(-1)[n].item()) @ v[: t + 1, n]
+        s = ((k[: t + 1] * q[t, :, :d]).sum(dim=-1).T + qr[t] @ r[: t + 1].T) * m["scale"]
+        out[t] = (sink_softmax(s, g("sink").reshape(-1)).T.unsqueeze(2) * v[: t + 1]).sum(dim=0)
     return out.reshape(T, -1) @ g("o").T
 
 
