@@ -155,7 +155,7 @@ def main() -> int:
     ap.add_argument("--parallelism", default="auto", choices=["auto", "dp", "tp"],
                     help="N > 1: tp (default) = one engine over N GPUs (tensor parallel, --batch sequences in total, strong scaling); "
                          "dp = one engine replica per GPU, --batch sequences each (weak scaling, no communication)")
-    ap.add_argument("--design", default=None, choices=["fatotar", "fopivik", "dubozen"],
+    ap.add_argument("--design", default=None, choices=["fatotar", "fopivik", "dubozen", "gevovik"],
                     help="instead of the headline workload: prefill / decode throughput and kernel times of this design beside the closest decoder of equal size (1 GPU)")
     ap.add_argument("--sizes", default="small,1b,3b", help="--design: sizes to run")
     ap.add_argument("--no-kernels", action="store_true", help="--design: throughput only")
@@ -165,6 +165,8 @@ def main() -> int:
             from deliverance_b200.bench.fopivik_bench import main as design_main
         elif args.design == "dubozen":
             from deliverance_b200.bench.dubozen_bench import main as design_main
+        elif args.design == "gevovik":
+            from deliverance_b200.bench.gevovik_bench import main as design_main
         else:
             from deliverance_b200.bench.design_bench import main as design_main
 

@@ -45,28 +45,27 @@ def moe_shape(z: dict) -> dict:
 
 
 class Mamba:
-    """The Mamba2 mixer core (scan, convolution, gated norm) with a state as large as the linear-attention layer's."""
+    """The Mamba-2 mixer core (convolution, recurrence, gated norm) with a state as large as the linear-attention layer's."""
 
     def __init__(self, z: dict, dev):
+        from ..ops.mamba import Mamba2Shape, Mamba2Weights
+
         self.S, self.dh = 128, 64
         self.H = z["gla_heads"] * z["gla_dim"] * z["gla_vdim"] // (self.S * self.dh)
         self.I = self.H * self.dh
-        self.conv = self.I + 2 * self.S
-        r = lambda *s: torch.randn(*s, device=dev)  # noqa: E731
-        self.par = (r(self.conv * 4) * 0.3, None, r(self.H), r(self.H) * 0.3, r(self.H), 1 + 0.1 * r(self.I))
-        self.width = self.I + self.conv + self.H
+        self.shape = Mamba2Shape(self.H, self.dh, self.S, 1, 4)
+        r = lambda *s: torch.randn(*s)  # noqa: E731
+        C = self.shape.conv_width
+        self.w = Mamba2Weights.pack(self.shape, r(C, 4) * 0.3, None, r(self.H), r(self.H) * 0.3, r(self.H), 1 + 0.1 * r(self.I), dev)
+        self.width = self.shape.dt_at + self.H
 
     def states(self, slots, dev):
-        return torch.zeros(slots, self.conv, 3, device=dev), torch.zeros(slots, self.H, self.dh, self.S, device=dev)
+        return tuple(torch.zeros((slots,) + s, device=dev) for s in self.shape.state_shapes().values())
 
     def run(self, zx, st, b):
-        from .. import ops
-        from ..models.mamba import _chunk_meta
+        from ..ops.mamba import mamba2
 
-        m = _chunk_meta(b, zx.device)
-        return ops.require_ext().mamba2_forward(zx, *self.par, *st, b.state_slots, b.q_start, b.q_len, b.positions, m["row_seq"], m["chunk_seq"], m["chunk_row0"],
-                                                m["chunk_len"], m["chunk_first"], m["chunk_last"], m["seq_chunk0"], m["seq_nchunks"], m["multi"], self.H, self.dh,
-                                                1, self.S, 1e-5)
+        return mamba2(self.shape, zx, self.w, *st, b, 1e-5)
 
 
 def kernel_times(fop, moe, z: dict, t: Timer, peaks: dict) -> list:

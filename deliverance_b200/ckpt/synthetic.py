@@ -19,7 +19,7 @@ from .tiny import build_tensors, dubozen_shapes, dubozen_value, fatotar_is_norm,
 
 
 def _shapes(cfg: dict) -> dict[str, tuple]:
-    """name -> shape for decoder families (llama, mistral, qwen2, qwen3, gemma2, gemma3, mixtral, qwen3_moe)."""
+    """name -> shape for decoder families (llama, mistral, qwen2, qwen3, gemma2, gemma3, mixtral, qwen3_moe, granitemoehybrid without routed experts)."""
     mt = config_model_type(cfg)
     if mt == "fatotar":
         return fatotar_shapes(cfg)
@@ -40,6 +40,16 @@ def _shapes(cfg: dict) -> dict[str, tuple]:
         p = f"model.layers.{i}."
         s[p + "input_layernorm.weight"] = (h,)
         s[p + "post_attention_layernorm.weight"] = (h,)
+        if mt == "granitemoehybrid":
+            F = cfg["shared_intermediate_size"]
+            s[p + "shared_mlp.input_linear.weight"], s[p + "shared_mlp.output_linear.weight"] = (2 * F, h), (h, F)
+            if cfg["layer_types"][i] == "mamba":
+                H, inner = cfg["mamba_n_heads"], cfg["mamba_n_heads"] * cfg["mamba_d_head"]
+                conv, m = inner + 2 * cfg["mamba_n_groups"] * cfg["mamba_d_state"], p + "mamba."
+                s.update({m + "in_proj.weight": (inner + conv + H, h), m + "out_proj.weight": (h, inner), m + "conv1d.weight": (conv, 1, cfg["mamba_d_conv"]),
+                          m + "conv1d.bias": (conv,), m + "norm.weight": (inner,)})
+                s.update({m + n: (H,) for n in ("dt_bias", "A_log", "D")})
+                continue
         s[p + "self_attn.q_proj.weight"] = (nh * hd, h)
         s[p + "self_attn.k_proj.weight"] = (nkv * hd, h)
         s[p + "self_attn.v_proj.weight"] = (nkv * hd, h)
@@ -64,7 +74,7 @@ def _shapes(cfg: dict) -> dict[str, tuple]:
             for e in range(E):
                 ep = p + f"mlp.experts.{e}."
                 s[ep + "gate_proj.weight"], s[ep + "up_proj.weight"], s[ep + "down_proj.weight"] = (MI, h), (MI, h), (h, MI)
-        else:
+        elif mt != "granitemoehybrid":
             s[p + "mlp.gate_proj.weight"], s[p + "mlp.up_proj.weight"], s[p + "mlp.down_proj.weight"] = (I, h), (I, h), (h, I)
     return s
 
@@ -116,6 +126,8 @@ class SyntheticLoader:
         if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
             base = 0.0 if self.cfg["model_type"] in ("gemma2", "gemma3_text") else 1.0
             return (base + torch.randn(shape, generator=g, device=self.device) * 0.02).to(self.dtype)
+        if name.endswith("conv1d.weight") or name.endswith((".dt_bias", ".A_log")):  # filters and decays that do something
+            return (torch.randn(shape, generator=g, device=self.device) * 0.5 - (0 if "conv1d" in name else 1.0)).to(self.dtype)
         if name.endswith(".gate.weight"):  # routers: wider spread so that top-k choices are well separated
             return (torch.randn(shape, generator=g, device=self.device) * 0.5).to(self.dtype)
         return (torch.randn(shape, generator=g, device=self.device) * self.std).to(self.dtype)

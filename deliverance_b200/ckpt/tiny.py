@@ -323,7 +323,7 @@ def gevovik_value(name: str, r, cfg: dict):
     if name.endswith("conv.b"):
         return 0.3 * r
     if len(r.shape) == 2 and name not in ("embed", "bigram"):
-        return r * r.shape[1] ** -0.5 * (3.0 if name.endswith("left.q") or name.endswith("mix.q") else 1.0)
+        return r * r.shape[1] ** -0.5 * (2.0 if name.endswith("mix.q") else 1.0)
     return r
 
 

@@ -454,7 +454,8 @@ def test_sink_levels(run, scale, level):
     for splits, portions in ((None, [T]), (None, [1] * T), (None, [2, 40, 2, 46]), (4, [80] + [1] * 10), (32, [80] + [1] * 10)):
         if splits:
             mixer._splits = lambda rows, span: splits  # noqa: B023
-        assert rel(run_mixer(mixer, kv, h, portions, pages, run), want) < tol(run[1], 5e-5, 0.05), (splits, portions)
+        # (below a sink that outweighs everything, an output's relative error is the scores' absolute one)
+        assert rel(run_mixer(mixer, kv, h, portions, pages, run), want) < tol(run[1], 5e-5, 0.1 if level > 20 else 0.05), (splits, portions)
 
 
 @pytest.mark.parametrize("run", RUNS)
