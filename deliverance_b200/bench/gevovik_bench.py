@@ -92,7 +92,7 @@ def kernel_times(gev, hyb, z: dict, t: Timer, peaks: dict) -> list:
         gemm("Mamba-2 output projection", M, lm.mixer.w_out, hm.mamba["out_proj"])
         gemm("side-by-side input projection (against q|k|v)", M, px.w_in, ha.qkv)
         gemm("side-by-side output projection (against o)", M, px.w_out, ha.o)
-        gemm("low-rank projections (against o)", M, right.w_low, ha.o, out_f32=True)
+        gemm("low-rank projection(s) (against o)", M, right.w_low if M < 8192 else right.w_decay, ha.o, out_f32=True)
         gemm("latent input projection (against q|k|v)", M, lat.w_in, ha.qkv)
         gemm("queries on a shared cache (against q|k|v)", M, ls.mixer.w_in, ha.qkv)
         gemm("latent output projection", M, lat.w_out, ha.o)
@@ -142,7 +142,7 @@ def kernel_times(gev, hyb, z: dict, t: Timer, peaks: dict) -> list:
         kv = SimpleNamespace(state={"conv": {0: ring}, "delta": {0: st}})
         state, fl = B * d.heads * d.dk * d.dv * 8, 6.0 * T * d.heads * d.dk * d.dv
         add(f"gated delta rule: low-rank projections, convolution, recurrence, norm, gate {tag} (against gated linear attention)",
-            lambda: right.heads(pd[:, s.width :], b, kv, 0, row[:, s.out_width :], stage), (state + right.w_low.nbytes() + T * (d.width + d.out_width) * 2, fl * 4 / 3),
+            lambda: right.heads(pd[:, s.width :], b, kv, 0, row[:, s.out_width :], stage), (state + (right.w_decay.nbytes() + right.w_gate.nbytes()) + T * (d.width + d.out_width) * 2, fl * 4 / 3),
             lambda: gla_op.gla(gs, pg, a2, a2b, gn, sg, b, gs.dim ** -0.5, 16.0, 1e-5), (state + a2.numel() * 4 + T * (gs.width + gs.out_width) * 2, fl))
         del st, sg
         # ---- attention with mixed scores

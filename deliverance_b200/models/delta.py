@@ -1,6 +1,6 @@
 """Gated-delta-rule mixer (``ops/delta.py``): any decoder can use it, alone or beside another mixer. It works on a column range of projection rows, keeps
 a ring of convolution inputs and one fp32 state per sequence in the cache manager's state slots and writes its gated heads into a column range of
-the rows that the output projection reads. The two low-rank projections (decays, output gate) are one GEMM with fp32 results."""
+the rows that the output projection reads. The two low-rank projections (decays, output gate) are one GEMM in decode steps."""
 from __future__ import annotations
 
 import torch
@@ -40,7 +40,8 @@ class GatedDeltaNet:
         w = torch.cat([heads(t, h, d) for _, t, h, d in pieces] + [rows(b), rows(a1), rows(g1)])
         ra, rg = up8(s.rank_a), up8(s.rank_g)
         decay, gate = pad(heads(a2, H, s.dim), (0, ra - s.rank_a + rg)), pad(heads(g2, H, s.vdim), (ra, rg - s.rank_g))
-        self.w_low = LinearWeight(torch.cat([decay, gate]).to(device=self.device, dtype=self.dtype).contiguous())
+        put = lambda t: LinearWeight(t.to(device=self.device, dtype=self.dtype).contiguous())  # noqa: E731
+        self.w_low, self.w_decay, self.w_gate = put(torch.cat([decay, gate])), put(decay[:, :ra]), put(gate[:, ra:])
         dev = lambda t: t.float().to(self.device).contiguous()  # noqa: E731
         self.conv = dev(torch.cat([heads(c.reshape(h * d, s.taps), h, d) for (_, _, h, d), c in zip(pieces, convs)]).t())
         self.dt_bias = dev(heads(dt_bias.reshape(-1, 1), H, s.dim).reshape(-1))
@@ -49,15 +50,19 @@ class GatedDeltaNet:
         return w, pad_head_columns(o, H, s.vdim, s.dv)
 
     def nbytes(self) -> int:
-        return self.w_low.nbytes() + (self.conv.numel() + self.dt_bias.numel() + self.norm.numel()) * 4
+        return self.w_low.nbytes() + self.w_decay.nbytes() + self.w_gate.nbytes() + (self.conv.numel() + self.dt_bias.numel() + self.norm.numel()) * 4
 
     def heads(self, p, batch: ForwardBatch, kv, run: int, out, stage) -> None:
         """``p [T, shape.width]``: this mixer's columns of the projection rows; the heads go to ``out [T, H * dv]``."""
         s = self.shape
         with stage("delta.low_rank_projections"):
-            low = ops.linear(p[:, s.low_at :], self.w_low, out_f32=True)
+            if dop.fused_step(s, batch):  # one launch, block diagonal
+                z, gate = ops.linear(p[:, s.low_at :], self.w_low, out_f32=True).split([s.heads * s.dk, s.out_width], dim=1)
+            else:
+                z = ops.linear(p[:, s.low_at : s.low_at + self.w_decay.K], self.w_decay, out_f32=True)
+                gate = ops.linear(p[:, s.low_at + self.w_decay.K : s.width], self.w_gate)
         with stage("delta.recurrence"):
-            dop.delta(s, p, low, self.conv, self.dt_bias, self.neg_a, self.norm, kv.state["conv"][run], kv.state["delta"][run], batch, self.q_scale, self.eps, self.mult,
+            dop.delta(s, p, z, gate, self.conv, self.dt_bias, self.neg_a, self.norm, kv.state["conv"][run], kv.state["delta"][run], batch, self.q_scale, self.eps, self.mult,
                       out)
 
     def state_shapes(self) -> dict:

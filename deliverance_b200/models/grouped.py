@@ -120,7 +120,7 @@ class GroupedAttention:
         if self.window > 0:
             span = min(span, self.window + self.keep_first)
         if self.shape.mixed:  # (a CTA takes all heads)
-            return gop.mixed_splits(batch.num_seqs, span)
+            return gop.mixed_splits(self.shape, batch.num_seqs, span)
         return ops.decode_splits(batch.num_seqs, self.shape.kv_heads * ((self.shape.heads // self.shape.kv_heads + 15) // 16), span)
 
     def cache_layout(self) -> dict:

@@ -37,7 +37,8 @@
 // Wide rows (paged layout, `wide`): a cache row holds the heads of all KV heads side by side, and a query head's keys are the WHOLE row (attention with
 // mixed scores: the mixing has moved to the query side, see ops/grouped.py), its values the dv columns of its own KV head. Rows of more than 256 key
 // columns go by in pieces of 128 columns (KM = 1: the query tile of up to 512 columns stays in shared memory; KM = 2: wider rows, the query's pieces
-// travel with the keys' pieces, from L2). KM = 0: whole key tiles.
+// travel with the keys' pieces, from L2). KM = 0: whole key tiles. With KM > 0 and QT = 2 there is ONE query tile, and the two softmax groups take its key
+// tiles in turn, each with an accumulator, maximum and sum of its own; they meet in the epilogue (one group alone cannot keep up with the tensor cores).
 //
 // Replaces the reference's packed prefill attention (core/.../generator/CausalSelfAttention.java:458-502: per head QK^T GEMM over
 // the visible pages, causal scaled softmax with optional soft-cap, saxpy with V).
@@ -117,7 +118,7 @@ constexpr int kAtBM = 128, kAtBN = 64;  // query rows per score tile / keys per 
 constexpr int kAtPiece = 2, kAtResident = 8;  // KM > 0: 64-column blocks per piece of a key row; most blocks of a query tile that stays in shared memory
 
 // KM > 0 (one query tile): a K stage is one piece of a key tile, with KM = 2 behind the query's piece
-template <int DV, int KM>
+template <int DV, int QT, int KM>
 struct AttnTcWideSmem {
   static constexpr int kTileQ = kAtBM * 128 * kAtPiece;  // bytes of a query piece
   static constexpr int kTileK = kAtBN * 128 * kAtPiece + (KM == 2 ? kTileQ : 0);
@@ -131,9 +132,9 @@ struct AttnTcWideSmem {
   static constexpr int kOffV = kOffK + kStages * kTileK;
   static constexpr int kOffCtrl = kOffV + kStagesV * kTileV;
   static constexpr int kBytes = kOffCtrl + 512 + 1024;
-  static constexpr int kThreads = 256;
+  static constexpr int kThreads = 128 + 128 * QT;
   static constexpr int kSubK = 0, kSubV = DV / 64;
-  static_assert(kStages >= 2 && DV % 64 == 0 && kBytes > 118 * 1024 && kBytes <= 227 * 1024 && 256 + DV <= 512, "attention tile does not fit");
+  static_assert(kStages >= 2 && DV % 64 == 0 && kBytes > 118 * 1024 && kBytes <= 227 * 1024 && 256 + QT * DV <= 512, "attention tile does not fit");
 };
 
 template <int DK, int DV, int QT>
@@ -208,9 +209,9 @@ template <int DK, int DV, int QT, int KM>
 struct AttnTcLayout {
   using T = AttnTcSmem<DK, DV, QT>;
 };
-template <int DV, int KM>
-struct AttnTcLayout<0, DV, 1, KM> {
-  using T = AttnTcWideSmem<DV, KM>;
+template <int DV, int QT, int KM>
+struct AttnTcLayout<0, DV, QT, KM> {
+  using T = AttnTcWideSmem<DV, QT, KM>;
 };
 
 template <int DK, int DV, int QT, bool LATENT, int KM = 0>
@@ -236,7 +237,8 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
   uint64_t* bar_pv_done = bar_p_full + 4;  // [2][2] the P V that read the slot's probabilities has retired
   uint64_t* bar_o_final = bar_pv_done + 4;
   uint64_t* bar_drain = bar_o_final + 1;    // [2] an issuing thread's MMAs have retired (only used when a wait ran out)
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_drain + 2);
+  uint64_t* bar_ml = bar_drain + 2;         // SPLIT: maxima and sums of both softmax groups are in shared memory
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_ml + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -249,14 +251,16 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
   const int kvh = h / (p.H / p.KV);
   const int qs = p.q_start[seq], ql = p.q_len[seq], ctx = p.ctx_lens[seq];
   const int pos0 = ctx - ql;  // position of the sequence's first query row
-  const int rows_all = min(QT * kAtBM, ql - q0);
-  const bool two = QT == 2 && rows_all > kAtBM;  // two query tiles share every K / V tile
+  constexpr bool SPLIT = KM > 0 && QT == 2;  // one query tile, its key tiles alternate between the softmax groups
+  const int rows_all = min((SPLIT ? 1 : QT) * kAtBM, ql - q0);
+  const bool two = QT == 2 && (SPLIT || rows_all > kAtBM);  // two query tiles share every K / V tile
   // key tiles [a, b) each query tile sees
   int rows_q[2], first_q[2], a_q[2], b_q[2];
 #pragma unroll
   for (int q = 0; q < 2; ++q) {
-    rows_q[q] = max(0, min(kAtBM, rows_all - q * kAtBM));
-    first_q[q] = pos0 + q0 + q * kAtBM;
+    const int behind = SPLIT ? 0 : q * kAtBM;
+    rows_q[q] = max(0, min(kAtBM, rows_all - behind));
+    first_q[q] = pos0 + q0 + behind;
     const int last_pos = p.causal ? first_q[q] + rows_q[q] - 1 : ctx - 1;
     const int key_hi = min(ctx, last_pos + 1);
     const int key_lo = p.window > 0 ? max(0, first_q[q] - p.window + 1) : 0;
@@ -285,6 +289,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     mbar_init(smem_u32(&bar_drain[0]), 1);
     mbar_init(smem_u32(&bar_drain[1]), 1);
     mbar_init(smem_u32(bar_o_final), 1);
+    mbar_init(smem_u32(bar_ml), 8);
     *abort_flag = 0;
     mbar_fence_init();
     tma_prefetch_desc(&map_q);
@@ -432,6 +437,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     constexpr uint32_t idesc_s = umma_idesc_bf16(kAtBM, kAtBN);
     constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(kAtBM, DV);
     auto valid = [&](int u, int q) {
+      if (SPLIT) return (u & 1) == q;
       const int j = tile_at(u);
       return q == 0 ? ((j >= a0 || j < kept_tiles) && j < b0) : ((j >= a1 || j < kept_tiles) && j < b1);
     };
@@ -441,9 +447,10 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
         else { q = 0; ++u; }
       } while (u < n_tiles && !valid(u, q));
     };
-    auto last_of_tile = [&](int u, int q) { return !two || q == 1 || !valid(u, 1); };
+    auto last_of_tile = [&](int u, int q) { return SPLIT || !two || q == 1 || !valid(u, 1); };
     // key tiles of query tile q before tile j (the same count its softmax warps keep)
     auto count_at = [&](int u, int q) {
+      if (SPLIT) return u >> 1;
       const int j = tile_at(u), a = q == 0 ? a0 : a1;
       return j < kept_tiles ? j : j - max(a, kept_tiles) + kept_tiles;
     };
@@ -543,21 +550,23 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const int my_rows = q == 0 ? rows_q[0] : rows_q[1], my_first = q == 0 ? first_q[0] : first_q[1];
     const int ja = q == 0 ? a0 : a1, jb = q == 0 ? b0 : b1;
-    const int my_kept = min(kept_tiles, ja), my_tiles = my_kept + jb - ja;  // this query tile's key tiles: [0, my_kept), then [ja, jb)
+    // this query tile's key tiles: [0, my_kept), then [ja, jb) (SPLIT: every other one)
+    const int my_kept = min(kept_tiles, ja), my_tiles = SPLIT ? (n_tiles - q + 1) / 2 : my_kept + jb - ja;
     const int my_pos = my_first + r;
     const float c_log2 = 1.4426950408889634f;
     // scores stay in the units the tensor core delivers; kf turns a difference of scores into a base-2 exponent
     const float kf = p.softcap > 0.f ? c_log2 : p.scale * c_log2;
     float m_run = -INFINITY, l_run = 0.f;
     // gate logits of this row; threads behind the last row read that row's (every branch around tensor-memory accesses stays warp-uniform)
-    const size_t gate_row = static_cast<size_t>(qs + q0 + q * kAtBM + max(0, min(r, my_rows - 1)));
+    const int q_rows = SPLIT ? 0 : q * kAtBM;  // rows in front of this group's
+    const size_t gate_row = static_cast<size_t>(qs + q0 + q_rows + max(0, min(r, my_rows - 1)));
     const __nv_bfloat16* grow = p.gate != nullptr && !p.gate_heads ? p.gate + gate_row * p.gate_pitch + static_cast<size_t>(h) * p.dv : nullptr;
     const bool gate_vec = grow != nullptr && (p.dv & 7) == 0;  // (then rows, heads and the gate are 16-byte aligned)
     if (grow != nullptr)
       for (int c = 0; c < p.dv; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + c));
     bool ok = true;
     for (int t = 0; t < my_tiles && ok; ++t) {
-      const int j = t < my_kept ? t : ja + t - my_kept;
+      const int j = SPLIT ? lo + 2 * t + q : (t < my_kept ? t : ja + t - my_kept);
       const uint32_t slot = q * 2 + (t & 1);
       const uint32_t sb = lane_addr + kColS + slot * kAtBN;
       // warp-uniform: the loop holds warp-collective TMEM accesses
@@ -647,15 +656,36 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     // ---------------- epilogue ----------------
     if (ok) ok = mbar_wait(smem_u32(bar_o_final), 0, abort_flag, p.status);
     ok = __all_sync(0xffffffffu, ok && *abort_flag == 0);
+    if constexpr (SPLIT) {
+      if (ok) {  // every copy has landed and every MMA has retired: the maxima and sums pass through the key stages
+        float* ml = reinterpret_cast<float*>(smem + L::kOffK) + q * 256;
+        ml[r] = m_run;
+        ml[128 + r] = l_run;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(bar_ml));
+        ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(bar_ml), 0, abort_flag, p.status));
+      }
+    }
     if (ok) {
       tc_fence_after();
+      float w_mine = 1.f, w_other = 0.f;  // SPLIT: weights of this group's and the other one's accumulator
+      if constexpr (SPLIT) {
+        const float* ml = reinterpret_cast<const float*>(smem + L::kOffK) + (1 - q) * 256;
+        const float m2 = ml[r], l2 = ml[128 + r], m = fmaxf(m_run, m2);
+        w_mine = m_run == -INFINITY ? 0.f : ex2_approx((m_run - m) * kf);
+        w_other = m2 == -INFINITY ? 0.f : ex2_approx((m2 - m) * kf);
+        l_run = l_run * w_mine + l2 * w_other;
+        m_run = m;
+      }
       if (p.sink != nullptr) l_run += ex2_approx(p.sink[h] * c_log2 - m_run * kf);  // relative to the running maximum
       float inv = l_run > 0.f ? p.out_mult / l_run : 0.f;
-      const size_t trow = static_cast<size_t>(qs + q0 + q * kAtBM + r);
+      const size_t trow = static_cast<size_t>(qs + q0 + q_rows + r);
       __nv_bfloat16* orow = p.out + trow * p.out_pitch + static_cast<size_t>(h) * p.dv;
       if (!LATENT && p.gate_heads) inv /= 1.f + __expf(-bf2f(p.gate[gate_row * p.gate_pitch + h]));
+      // SPLIT: each group stores half of the columns, from both accumulators
+      const int c_first = SPLIT ? q * (DV / 2) : 0, c_last = SPLIT ? c_first + DV / 2 : DV;
 #pragma unroll 1
-      for (int c0 = 0; c0 < DV; c0 += 32) {
+      for (int c0 = c_first; c0 < c_last; c0 += 32) {
         uint4 gv[4];  // the gate logits of this step, all on their way before the first is used
         if (gate_vec) {
 #pragma unroll
@@ -669,6 +699,17 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = 0u;
+        }
+        if constexpr (SPLIT) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * w_mine);
+          if (n_tiles > 1 - q) {  // the other group has had a tile
+            uint32_t v2[32];
+            tmem_ld_x32(lane_addr + kColO + (1 - q) * DV + c0, v2);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) + __uint_as_float(v2[i]) * w_other);
+          }
         }
         if (LATENT) {
           if (r < my_rows) {
@@ -808,7 +849,7 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
 int prefill_attention_tc_tile_rows(int D) { return D <= 128 ? 256 : 128; }
 int prefill_attention_wide_tile_rows(int k_width, int dv) {
   if (k_width <= 0 || dv <= 0 || k_width % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
-  return k_width > 256 ? kAtBM : prefill_attention_tc_tile_rows(k_width > dv ? k_width : dv);
+  return k_width > 256 || dv > 128 ? kAtBM : 2 * kAtBM;
 }
 
 // tile arrays: prefill_attention_tc_tile_rows(max(dk, dv)) query rows per tile. page_size must be 32, 64 or 128. Returns 1 for an unsupported
@@ -852,17 +893,21 @@ int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, 
   p.k_subs = (dk + 63) / 64;
   const long long cache_rows = num_pages * (wide ? 1 : KV) * page;
   if (pieces) {
-#define DLV_WIDE(DVV)                                                                                                               \
-  return p.k_subs <= kAtResident ? launch_prefill_tc_t<0, DVV, 1, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)          \
-                                 : launch_prefill_tc_t<0, DVV, 1, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
-    if (dv <= 64) DLV_WIDE(64);
-    if (dv <= 128) DLV_WIDE(128);
-    DLV_WIDE(256);
+#define DLV_WIDE(DVV, QTV)                                                                                                            \
+  return p.k_subs <= kAtResident ? launch_prefill_tc_t<0, DVV, QTV, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)          \
+                                 : launch_prefill_tc_t<0, DVV, QTV, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
+    if (dv <= 64) DLV_WIDE(64, 2);
+    if (dv <= 128) DLV_WIDE(128, 2);
+    DLV_WIDE(256, 1);
 #undef DLV_WIDE
   }
   if (D <= 64) return launch_prefill_tc_t<64, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128 && dv <= 64) return launch_prefill_tc_t<128, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128) return launch_prefill_tc_t<128, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (wide && dv <= 64) return dk <= 192 ? launch_prefill_tc_t<192, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
+                                         : launch_prefill_tc_t<256, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
+  if (wide && dv <= 128) return dk <= 192 ? launch_prefill_tc_t<192, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
+                                          : launch_prefill_tc_t<256, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   return launch_prefill_tc_t<256, 256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
 }
 

@@ -1645,6 +1645,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mixed_decode_ok", [](int64_t H, int64_t KV, int64_t dk, int64_t dv) {
     return dlv::mixed_decode_supported(static_cast<int>(H), static_cast<int>(KV), static_cast<int>(dk), static_cast<int>(dv));
   });
+  m.def("mixed_decode_ctas", [](int64_t H, int64_t KV, int64_t dk, int64_t dv) {
+    return dlv::mixed_decode_ctas(static_cast<int>(H), static_cast<int>(KV), static_cast<int>(dk), static_cast<int>(dv));
+  });
   m.def("mixed_decode", &mixed_decode, py::arg("q"), py::arg("mix"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("ctx_lens"),
         py::arg("H"), py::arg("KV"), py::arg("scale"), py::arg("window"), py::arg("splits"), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
         py::arg("out") = py::none());

@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a)
   }
   for (int t = 0; t < n; ++t) {
     const TIO* row = p + static_cast<size_t>(row0 + t) * a.ld;
-    const float* low = a.low + static_cast<size_t>(row0 + t) * a.ld_low;
+    const float* z = a.z + static_cast<size_t>(row0 + t) * a.ld_z + h * a.dk;
     float qq = 0.f, kk = 0.f;
     if constexpr (STEP) {
       // (ring rows of a query / key head are written by its first CTA, those of value columns by their own)
@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a)
       }
       if (tid < kDnCols) sv[tid] = c_first + tid < a.dv ? io_ld(in + off_v + h * a.dv + c_first + tid) : 0.f;
     }
-    for (int d = tid; d < RPT * 16; d += 256) sa[d] = d < a.dk ? expf(neg_a * dn_softplus(low[h * a.dk + d] + a.dt_bias[h * a.dk + d])) : 0.f;
+    for (int d = tid; d < RPT * 16; d += 256) sa[d] = d < a.dk ? expf(neg_a * dn_softplus(z[d] + a.dt_bias[h * a.dk + d])) : 0.f;
     const float fq = rsqrtf(block_sum(qq, redq) + a.unit_eps) * a.q_scale, fk = rsqrtf(block_sum(kk, redk) + a.unit_eps);
     // ---- decay, what the state returns for the key
     float r[4] = {0.f, 0.f, 0.f, 0.f};
@@ -187,7 +187,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a)
     const int c = c_first + tid;
     if (tid < kDnCols && c < a.dv && n > 0) {
       const float inv = rsqrtf(ss / a.dv_real + a.eps) * a.mult;
-      const float z = a.low[static_cast<size_t>(row0) * a.ld_low + a.H * a.dk + h * a.dv + c];
+      const float z = static_cast<const float*>(a.gate)[static_cast<size_t>(row0) * a.ld_gate + h * a.dv + c];
       io_st(static_cast<TIO*>(a.out) + static_cast<size_t>(row0) * a.ld_out + h * a.dv + c, red[0][tid] * inv * a.norm_w[c] * dn_sigmoid(z));
     }
     cluster.sync();  // no CTA leaves while another one may still read its sum
@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(256) delta_norm_gate_kernel(const DeltaArgs a)
   if (w >= static_cast<long long>(a.rows) * a.H) return;
   const int t = static_cast<int>(w / a.H), h = static_cast<int>(w % a.H);
   const float* o = a.o + static_cast<size_t>(t) * (a.H * a.dv) + h * a.dv;
-  const float* z = a.low + static_cast<size_t>(t) * a.ld_low + a.H * a.dk + h * a.dv;
+  const TIO* z = static_cast<const TIO*>(a.gate) + static_cast<size_t>(t) * a.ld_gate + h * a.dv;
   float ss = 0.f;
   for (int c = lane * 4; c < a.dv; c += 128) {
     const float4 v = *reinterpret_cast<const float4*>(o + c);
@@ -269,30 +269,33 @@ constexpr float kDnMaxLogDecay = 86.f;  // 2^(+-86) and its products with unit v
 
 template <int C>
 struct DeltaPrepareSmem {
-  int P, off_q, off_m, off_f, bytes;
+  int P, off_m, off_t, off_f, bytes;
   __host__ __device__ explicit DeltaPrepareSmem(int dk) {
     P = (dk + 15) / 16 * 16 + 8;
-    off_q = C * dk * 4;                  // [3][2][C][P]: q exp(b), k exp(-b), k exp(b)
-    off_m = off_q + 6 * C * P * 2;       // [C][C + 1] M, then its inverse
-    off_f = off_m + 2 * C * (C + 1) * 4; // [3][C] unit factors of q and k, beta
-    bytes = off_f + 3 * C * 4;
+    off_m = 6 * C * P * 2;               // [3][2][C][P]: q exp(b), k exp(-b), k exp(b); term by term: running sums [C][dk]
+    off_t = off_m + 2 * C * (C + 1) * 4; // [C][C + 1] M, then its inverse
+    off_f = off_t + C / 8 * dk * 4;      // [C / 8][dk] sums of the log decays of eight rows
+    bytes = off_f + 3 * C * 4;           // [3][C] unit factors of q and k, beta
   }
 };
 
+// A thread keeps two channels of eight rows.
 template <int C>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, const DeltaChunks c) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) uint8_t dsm[];
   const DeltaPrepareSmem<C> L(a.dk);
+  constexpr int R = 8, NG = C / R;
   const int ck = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int dk = a.dk, dk16 = (dk + 15) / 16 * 16, P = L.P;
-  float* sb = reinterpret_cast<float*>(dsm);  // [C][dk] decay logarithms, then their running sums
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dsm + L.off_q);
+  const int dk = a.dk, dk16 = (dk + 15) / 16 * 16, P = L.P, half = dk / 2;
+  float* sb = reinterpret_cast<float*>(dsm);
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dsm);
   __nv_bfloat16* sK = sQ + 2 * C * P;
   __nv_bfloat16* sB = sK + 2 * C * P;
   float* sM = reinterpret_cast<float*>(dsm + L.off_m);
   float* sX = sM + C * (C + 1);
+  float* sT = reinterpret_cast<float*>(dsm + L.off_t);
   float* fq = reinterpret_cast<float*>(dsm + L.off_f);
   float* fk = fq + C;
   float* beta = fk + C;
@@ -300,27 +303,47 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
   const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.qkv) + static_cast<size_t>(row0) * width + g * dk;
   const __nv_bfloat16* kp = qp + a.G * dk;
   const float la = a.neg_a[h] * 1.4426950408889634f;
-  // ---- decay logarithms; unit factors, one warp per row
-  for (int e = tid; e < C * dk / 4; e += 256) {
-    const int t = e / (dk / 4), d = (e % (dk / 4)) * 4;
-    float z[4] = {0.f, 0.f, 0.f, 0.f};
-    if (t < len) {
-      float bias[4];
-      io_ld4(a.low + static_cast<size_t>(row0 + t) * a.ld_low + h * dk + d, z);
-      io_ld4(a.dt_bias + h * dk + d, bias);
+  const int d = (tid % half) * 2, grp = tid / half, t0 = grp * R;
+  const bool active = grp < NG;
+  // ---- decay logarithms and their running sums inside the thread's rows
+  float2 b[R];
+  uint32_t qu[R], ku[R];
+  if (active) {
+    const float2 bias = *reinterpret_cast<const float2*>(a.dt_bias + h * dk + d);
+    const float* zp = a.z + static_cast<size_t>(row0 + t0) * a.ld_z + h * dk + d;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) z[i] = la * dn_softplus(z[i] + bias[i]);
+    for (int i = 0; i < R; ++i) {
+      const bool ok = t0 + i < len;
+      b[i] = ok ? *reinterpret_cast<const float2*>(zp + i * a.ld_z) : make_float2(0.f, 0.f);
+      qu[i] = ok ? *reinterpret_cast<const uint32_t*>(qp + static_cast<size_t>(t0 + i) * width + d) : 0u;
+      ku[i] = ok ? *reinterpret_cast<const uint32_t*>(kp + static_cast<size_t>(t0 + i) * width + d) : 0u;
     }
-    *reinterpret_cast<float4*>(sb + t * dk + d) = make_float4(z[0], z[1], z[2], z[3]);
+    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      if (t0 + i < len) {
+        acc.x += la * dn_softplus(b[i].x + bias.x);
+        acc.y += la * dn_softplus(b[i].y + bias.y);
+      }
+      b[i] = acc;
+    }
+    *reinterpret_cast<float2*>(sT + grp * dk + d) = acc;
   }
-  for (int t = warp; t < C; t += 8) {
+  // ---- unit factors, one warp per row
+#pragma unroll
+  for (int i = 0; i < C / 8; ++i) {
+    const int t = warp + 8 * i;
     float qq = 0.f, kk = 0.f;
     if (t < len)
-      for (int d = lane * 2; d < dk; d += 64) {
-        const float2 q = unpack_bf162(*reinterpret_cast<const uint32_t*>(qp + static_cast<size_t>(t) * width + d));
-        const float2 k = unpack_bf162(*reinterpret_cast<const uint32_t*>(kp + static_cast<size_t>(t) * width + d));
-        qq += q.x * q.x + q.y * q.y;
-        kk += k.x * k.x + k.y * k.y;
+      for (int x = lane * 4; x < dk; x += 128) {
+        float q[4], k[4];
+        io_ld4(qp + static_cast<size_t>(t) * width + x, q);
+        io_ld4(kp + static_cast<size_t>(t) * width + x, k);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          qq += q[e] * q[e];
+          kk += k[e] * k[e];
+        }
       }
     qq = warp_sum(qq);
     kk = warp_sum(kk);
@@ -331,39 +354,45 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     }
   }
   __syncthreads();
-  for (int d = tid; d < dk; d += 256) {
-    float acc = 0.f;
-#pragma unroll 8
-    for (int t = 0; t < C; ++t) {
-      acc += sb[t * dk + d];
-      sb[t * dk + d] = acc;
-    }
-  }
-  __syncthreads();
-  const float* b_end = sb + (C - 1) * dk;
+  float2 be = make_float2(0.f, 0.f);
   bool small = true;
-  for (int d = tid; d < dk; d += 256) small = small && b_end[d] > -kDnMaxLogDecay;
+  if (active) {
+    float2 before = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      const float2 v = *reinterpret_cast<const float2*>(sT + i * dk + d);
+      if (i < grp) {
+        before.x += v.x;
+        before.y += v.y;
+      }
+      be.x += v.x;
+      be.y += v.y;
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      b[i].x += before.x;
+      b[i].y += before.y;
+    }
+    small = fminf(be.x, be.y) > -kDnMaxLogDecay;
+    if (grp == 0) *reinterpret_cast<float2*>(c.decay + (static_cast<size_t>(ck) * a.H + h) * dk + d) = make_float2(dn_ex2(be.x), dn_ex2(be.y));
+  }
   const bool fast = __syncthreads_and(small);
   // ---- scaled queries and keys
-  {
-    const int half = dk / 2;
-    uint32_t* dst = reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(c.qk) + (static_cast<size_t>(row0) * a.H + h) * 6 * dk);
-    for (int e = tid; e < C * half; e += 256) {
-      const int t = e / half, d = (e % half) * 2;
-      uint32_t qu = 0u, ku = 0u;
-      if (t < len) {
-        qu = *reinterpret_cast<const uint32_t*>(qp + static_cast<size_t>(t) * width + d);
-        ku = *reinterpret_cast<const uint32_t*>(kp + static_cast<size_t>(t) * width + d);
-      }
-      const float2 q = unpack_bf162(qu), k0 = unpack_bf162(ku), b = *reinterpret_cast<const float2*>(sb + t * dk + d), be = *reinterpret_cast<const float2*>(b_end + d);
-      const float2 k = make_float2(k0.x * fk[t], k0.y * fk[t]);
-      const float ex = dn_ex2(b.x), ey = dn_ex2(b.y);
+  if (active) {
+    uint32_t* o = reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(c.qk) + (static_cast<size_t>(row0 + t0) * a.H + h) * 6 * dk + d);
+    const size_t step = static_cast<size_t>(a.H) * 6 * half;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int t = t0 + i;
+      const float2 q = unpack_bf162(qu[i]), k0 = unpack_bf162(ku[i]);
+      const float uq = fq[t], uk = fk[t];
+      const float2 k = make_float2(k0.x * uk, k0.y * uk);
+      const float ex = dn_ex2(b[i].x), ey = dn_ex2(b[i].y);
       uint32_t qh, ql, bh, bl, kh, kl;
-      split2(q.x * fq[t] * ex, q.y * fq[t] * ey, qh, ql);
+      split2(q.x * uq * ex, q.y * uq * ey, qh, ql);
       split2(k.x * ex, k.y * ey, bh, bl);
-      split2(k.x * dn_ex2(be.x - b.x), k.y * dn_ex2(be.y - b.y), kh, kl);
+      split2(k.x * dn_ex2(be.x - b[i].x), k.y * dn_ex2(be.y - b[i].y), kh, kl);
       if (t < len) {
-        uint32_t* o = dst + static_cast<size_t>(t) * a.H * 6 * half + d / 2;
         o[0] = qh;
         o[half] = ql;
         o[2 * half] = kh;
@@ -371,20 +400,22 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
         o[4 * half] = bh;
         o[5 * half] = bl;
       }
+      o += step;
       if (fast) {
         *reinterpret_cast<uint32_t*>(sQ + t * P + d) = qh;
         *reinterpret_cast<uint32_t*>(sQ + (C + t) * P + d) = ql;
         *reinterpret_cast<uint32_t*>(sB + t * P + d) = bh;
         *reinterpret_cast<uint32_t*>(sB + (C + t) * P + d) = bl;
-        split2(k.x * dn_ex2(-b.x), k.y * dn_ex2(-b.y), kh, kl);
+        split2(k.x * dn_ex2(-b[i].x), k.y * dn_ex2(-b[i].y), kh, kl);
         *reinterpret_cast<uint32_t*>(sK + t * P + d) = kh;
         *reinterpret_cast<uint32_t*>(sK + (C + t) * P + d) = kl;
+      } else {
+        *reinterpret_cast<float2*>(sb + t * dk + d) = b[i];
       }
     }
-    if (dk16 != dk)  // (widths are multiples of 8)
-      for (int e = tid; e < 6 * C * 4; e += 256) reinterpret_cast<uint32_t*>(sQ + (e >> 2) * P + dk)[e & 3] = 0u;
   }
-  for (int d = tid; d < dk; d += 256) c.decay[(static_cast<size_t>(ck) * a.H + h) * dk + d] = dn_ex2(b_end[d]);
+  if (fast && dk16 != dk)  // (widths are multiples of 8)
+    for (int e = tid; e < 6 * C * 4; e += 256) reinterpret_cast<uint32_t*>(sQ + (e >> 2) * P + dk)[e & 3] = 0u;
   __syncthreads();
   // ---- causal matrix of the queries (to memory) and M (to shared memory): the 16 x 16 blocks on and below the diagonal
   __nv_bfloat16* am = static_cast<__nv_bfloat16*>(c.a) + (static_cast<size_t>(ck) * a.H + h) * 4 * C * C;
@@ -440,10 +471,10 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
           if (s + j > t) continue;
           const __nv_bfloat16* k = kp + static_cast<size_t>(s + j) * width;
           float acc = 0.f, accm = 0.f;
-          for (int d = 0; d < dk; ++d) {
-            const float kd = bf2f(k[d]) * dn_ex2(sb[t * dk + d] - sb[(s + j) * dk + d]);
-            acc += bf2f(q[d]) * kd;
-            accm += bf2f(kt[d]) * kd;
+          for (int x = 0; x < dk; ++x) {
+            const float kd = bf2f(k[x]) * dn_ex2(sb[t * dk + x] - sb[(s + j) * dk + x]);
+            acc += bf2f(q[x]) * kd;
+            accm += bf2f(kt[x]) * kd;
           }
           v[j] = acc * fq[t] * fk[s + j];
           m[j] = s + j < t ? accm * fk[t] * fk[s + j] * beta[t] : 0.f;

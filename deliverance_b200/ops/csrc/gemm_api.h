@@ -278,13 +278,16 @@ struct MambaArgs {
 int launch_mamba2_recurrent(const MambaArgs& a, bool is_f32, cudaStream_t st);  // xbc == nullptr: one row per sequence
 int launch_mamba2_chunked(const MambaArgs& a, const LightningChunks& c, int chunk, cudaStream_t st);
 
-// delta.cu: gated delta rule. Projection rows p [T, ld]: q (G dk) | k (G dk) | v (H dv) | beta (H) at beta_at; low [T, H dk + H dv] fp32
+// delta.cu: gated delta rule. Projection rows p [T, ld]: q (G dk) | k (G dk) | v (H dv) | beta (H) at beta_at; z [T, H dk] fp32: argument of the decays without dt_bias;
+// gate [T, H dv]: logits of the output gate, fp32 in the decode step, else of the rows' type
 struct DeltaArgs {
   const void* p;
   long long ld;
   int H, G, dk, dv, dv_real, beta_at;
-  const float* low;
-  long long ld_low;
+  const float* z;
+  long long ld_z;
+  const void* gate;
+  long long ld_gate;
   const void* qkv;  // convolved and activated q | k | v [T, 2 G dk + H dv] (nullptr: the decode step convolves itself)
   int taps;
   const float* conv_w;
@@ -327,9 +330,10 @@ struct MixedDecodeArgs {
   AttnExtra x;
 };
 bool mixed_decode_supported(int H, int KV, int dk, int dv);
+int mixed_decode_ctas(int H, int KV, int dk, int dv);  // CTAs per SM
 int launch_mixed_decode(const MixedDecodeArgs& a, cudaStream_t st);
 void launch_decode_merge(const float* po, const float* pml, void* out, int B, int H, int dv, int splits, AttnExtra x, cudaStream_t st);  // attention.cu
-void launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st);
+int launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st);
 
 // a2a.cu: expert-parallel all-to-all over peer memory (see the file comment for the protocol)
 struct A2AParams {

@@ -9,53 +9,53 @@
 
 namespace dlv {
 
-constexpr int kConvRows = 16;  // rows per thread: the inputs of the taps stay in registers
+constexpr int kConvRows = 8;  // rows per thread (of four channels): their inputs are loaded at once
 
 template <typename TIO, int TAPS>
 __global__ void __launch_bounds__(128) short_conv_kernel(const ConvArgs a) {
   pdl_wait();
   pdl_trigger();
-  const int vecs = a.C / 8, c = (blockIdx.x * 128 + threadIdx.x) * 8;
-  if (c >= vecs * 8) return;
-  const int r0 = blockIdx.y * kConvRows, r1 = min(r0 + kConvRows, a.rows);
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 4;
+  if (c >= a.C) return;
+  const int r0 = blockIdx.y * kConvRows, n = min(kConvRows, a.rows - r0);
   const TIO* p = static_cast<const TIO*>(a.p) + c;
   TIO* out = static_cast<TIO*>(a.out) + c;
-  float w[TAPS][8], b[8] = {}, x[TAPS][8];  // x[j]: the input that filter row j multiplies
+  float w[TAPS][4], b[4] = {};
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j) io_ld8(a.w + static_cast<size_t>(j) * a.C + c, w[j]);
-  if (a.b != nullptr) io_ld8(a.b + c, b);
-  int seq = -1;
-  for (int r = r0; r < r1; ++r) {
-    const int s = a.row_seq[r];
-    if (s != seq) {  // first row of the block or of a sequence: the inputs in front of it
-      seq = s;
-      const int first = a.q_start[s], pos = a.positions[first] + r - first;
-      const float* ring = a.ring + static_cast<size_t>(a.slots[s]) * TAPS * a.C + c;
+  for (int j = 0; j < TAPS; ++j) io_ld4(a.w + static_cast<size_t>(j) * a.C + c, w[j]);
+  if (a.b != nullptr) io_ld4(a.b + c, b);
+  auto put = [&](int r, const float (&x)[TAPS][4]) {  // x[j]: the input that filter row j multiplies
+    float y[4];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
-        const int back = TAPS - 1 - j;
-        if (r - back >= first) io_ld8(p + static_cast<long long>(r - back) * a.ld, x[j]);
-        else if (pos - back >= 0) io_ld8(ring + static_cast<size_t>((pos - back) % TAPS) * a.C, x[j]);
-        else {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) x[j][e] = 0.f;
-        }
-      }
-    }
-    io_ld8(p + static_cast<long long>(r) * a.ld, x[TAPS - 1]);
-    float y[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) {
+    for (int e = 0; e < 4; ++e) {
       float acc = b[e];
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) acc += w[j][e] * x[j][e];
-      y[e] = acc / (1.f + __expf(-acc));
+      y[e] = __fdividef(acc, 1.f + __expf(-acc));
     }
-    io_st8(out + static_cast<size_t>(r) * a.C, y);
+    io_st4(out + static_cast<size_t>(r) * a.C, y);
+  };
+  const int seq0 = a.row_seq[r0], first0 = a.q_start[seq0];
+  if (n == kConvRows && a.row_seq[r0 + n - 1] == seq0 && r0 - (TAPS - 1) >= first0) {  // all inputs are rows of this batch
+    float x[kConvRows + TAPS - 1][4];
 #pragma unroll
-    for (int j = 0; j + 1 < TAPS; ++j)
+    for (int i = 0; i < kConvRows + TAPS - 1; ++i) io_ld4(p + static_cast<long long>(r0 - (TAPS - 1) + i) * a.ld, x[i]);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[j][e] = x[j + 1][e];
+    for (int i = 0; i < kConvRows; ++i) put(r0 + i, reinterpret_cast<const float (&)[TAPS][4]>(x[i]));
+    return;
+  }
+  for (int r = r0; r < r0 + n; ++r) {
+    const int s = a.row_seq[r], first = a.q_start[s], pos = a.positions[first] + r - first;
+    const float* ring = a.ring + static_cast<size_t>(a.slots[s]) * TAPS * a.C + c;
+    float x[TAPS][4];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const int back = TAPS - 1 - j;
+      if (r - back >= first) io_ld4(p + static_cast<long long>(r - back) * a.ld, x[j]);
+      else if (pos - back >= 0) io_ld4(ring + static_cast<size_t>((pos - back) % TAPS) * a.C, x[j]);
+      else x[j][0] = x[j][1] = x[j][2] = x[j][3] = 0.f;
+    }
+    put(r, x);
   }
 }
 
@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(128) short_conv_ring_kernel(const ConvArgs a) 
 template <typename TIO>
 static cudaError_t launch_short_conv_t(const ConvArgs& a, cudaStream_t st) {
   const unsigned gx = static_cast<unsigned>((a.C / 8 + 127) / 128);
-  const dim3 grid(gx, static_cast<unsigned>((a.rows + kConvRows - 1) / kConvRows));
+  const dim3 grid(static_cast<unsigned>((a.C / 4 + 127) / 128), static_cast<unsigned>((a.rows + kConvRows - 1) / kConvRows));
   cudaError_t e = cudaErrorInvalidValue;
 #define DLV_CONV(N) case N: e = launch_pdl(short_conv_kernel<TIO, N>, grid, dim3(128), 0, st, a); break
   switch (a.taps) {

@@ -92,15 +92,20 @@ class DeltaShape:
         return [self.heads, self.kv_heads, self.dk, self.dv, self.vdim, self.beta_at]
 
 
-def delta(s: DeltaShape, p, low, conv_w, dt_bias, neg_a, norm_w, ring, state, batch, q_scale: float, eps: float, mult: float, out) -> None:
-    """Rows of the projection -> normed, gated heads times ``mult`` in ``out [T, H * dv]`` (a column range of wider rows). ``low [T, H * dk + H * dv]``: results
-    of the low-rank projections (decay argument without ``dt_bias``, gate logits). ``low``, ``conv_w [taps, C]``, ``dt_bias [H * dk]``, ``neg_a [H]`` = -exp(A_log),
+def fused_step(s: DeltaShape, batch) -> bool:
+    """A decode step of which one launch does everything (its gate logits are fp32)."""
+    return batch.is_decode and s.dv <= MAX_DV_FUSED
+
+
+def delta(s: DeltaShape, p, z, gate, conv_w, dt_bias, neg_a, norm_w, ring, state, batch, q_scale: float, eps: float, mult: float, out) -> None:
+    """Rows of the projection -> normed, gated heads times ``mult`` in ``out [T, H * dv]`` (a column range of wider rows). ``z [T, H * dk]``: the decays'
+    argument without ``dt_bias``, ``gate [T, H * dv]``: logits of the output gate (results of the low-rank projections). ``z``, ``conv_w [taps, C]``, ``dt_bias [H * dk]``, ``neg_a [H]`` = -exp(A_log),
     ``norm_w [dv]``, ``ring`` and ``state`` are fp32; the slots of the batch's sequences are advanced (one at position 0 starts from zero)."""
     if ops._cuda(p):
         e = ops.require_ext()
-        args = (low, conv_w, dt_bias, neg_a, norm_w, ring, state, batch.state_slots, batch.q_start, batch.q_len, batch.positions, s.geometry(), q_scale, UNIT_EPS, eps,
+        args = (z, gate, conv_w, dt_bias, neg_a, norm_w, ring, state, batch.state_slots, batch.q_start, batch.q_len, batch.positions, s.geometry(), q_scale, UNIT_EPS, eps,
                 mult, out)
-        if batch.is_decode and s.dv <= MAX_DV_FUSED:
+        if fused_step(s, batch):
             ops._count()
             e.delta_decode(p, *args)
             return
@@ -115,7 +120,6 @@ def delta(s: DeltaShape, p, low, conv_w, dt_bias, neg_a, norm_w, ring, state, ba
     unit = lambda x: x * torch.rsqrt(x.pow(2).sum(dim=-1, keepdim=True) + UNIT_EPS)  # noqa: E731
     q, k = (unit(x.reshape(T, G, s.dk)).repeat_interleave(H // G, dim=1) for x in (q, k))
     beta = torch.sigmoid(p[:, s.beta_at : s.beta_at + H].float())
-    z, gate = low.split([H * s.dk, H * s.dv], dim=-1)
     log_a = neg_a.view(1, H, 1) * torch.nn.functional.softplus(z + dt_bias).reshape(T, H, s.dk)
     o = torch.empty(T, H, s.dv, dtype=torch.float32)
     for slot, lo, n in zip(batch.state_slots.tolist(), batch.q_start.tolist(), batch.q_len.tolist()):
@@ -126,4 +130,4 @@ def delta(s: DeltaShape, p, low, conv_w, dt_bias, neg_a, norm_w, ring, state, ba
         r = slice(lo, lo + n)
         o[r] = ref.delta_sequential(q[r] * q_scale, k[r], v[r].reshape(n, H, s.dv), log_a[r], beta[r], state[slot])
     o = o * torch.rsqrt(o.pow(2).sum(dim=-1, keepdim=True) / s.vdim + eps) * norm_w
-    out.copy_(o.reshape(T, -1) * torch.sigmoid(gate) * mult)
+    out.copy_(o.reshape(T, -1) * torch.sigmoid(gate.float()) * mult)

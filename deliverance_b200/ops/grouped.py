@@ -213,10 +213,12 @@ def decode_tiles(batch):
     return batch.plans["decode_tiles"]
 
 
-def mixed_splits(num_seqs: int, span: int, sms: int = 148) -> int:
-    """Split-KV factor of the decode kernel of mixed scores: one CTA per (sequence, split), at least four 32-key tiles per split."""
+def mixed_splits(s: GroupedShape, num_seqs: int, span: int, sms: int = 148) -> int:
+    """Split-KV factor of the decode kernel of mixed scores: one CTA per (sequence, split), as many as run at once, at least two 32-key tiles per split."""
+    e = ops.ext()
+    ctas = e.mixed_decode_ctas(s.heads, s.kv_heads, s.dk, s.dv) if e is not None else 1
     tiles = max(1, (span + 31) // 32)
-    return int(max(1, min((sms + num_seqs - 1) // max(1, num_seqs), tiles // 4 if tiles >= 8 else 1, 64)))
+    return int(max(1, min(sms * max(1, ctas) // max(1, num_seqs), tiles // 2, 64)))
 
 
 def row_sequence(batch) -> torch.Tensor:
