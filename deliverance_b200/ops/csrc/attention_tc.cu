@@ -22,7 +22,7 @@
 // Every wait is bounded (common.cuh); on expiry the CTA records a status word, skips its stores, lets its copies and MMAs drain
 // (bounded), frees tensor memory and returns; CTAs that start after a recorded failure leave at once.
 //
-// Two layouts share the kernel (template parameter LATENT):
+// Three layouts share the kernel (template parameters LATENT, KM):
 //   paged   q [T, H * dk], K and V rows in the paged cache, GQA groups; the real widths dk and dv may be smaller than DK and DV (multiples
 //           of 8): tensor-map bounds fill the columns behind a cache row with zeros, and query columns that reach into the next head meet
 //           zeros. The first `keep_first` keys stay visible beside a sliding window (their key tiles are listed in front of the window's),
@@ -34,11 +34,13 @@
 //           with a sigmoid output gate and stores the dv real columns of every head.
 // Both take DK (query / key columns) and DV (value columns) as multiples of 64.
 //
-// Wide rows (paged layout, `wide`): a cache row holds the heads of all KV heads side by side, and a query head's keys are the WHOLE row (attention with
-// mixed scores: the mixing has moved to the query side, see ops/grouped.py), its values the dv columns of its own KV head. Rows of more than 256 key
-// columns go by in pieces of 128 columns (KM = 1: the query tile of up to 512 columns stays in shared memory; KM = 2: wider rows, the query's pieces
-// travel with the keys' pieces, from L2). KM = 0: whole key tiles. With KM > 0 and QT = 2 there is ONE query tile, and the two softmax groups take its key
-// tiles in turn, each with an accumulator, maximum and sum of its own; they meet in the epilogue (one group alone cannot keep up with the tensor cores).
+//   wide    (KM > 0) attention with mixed scores, the mixing moved to the query side (ops/grouped.py): a row holds the heads of all KV heads side by side,
+//           a query head's keys are the WHOLE row, its values the dv columns of its own KV head. The visible cache rows have been gathered into flat
+//           buffers (key 0 of a sequence is row kv_row0), key rows padded with zeros to 64-column blocks, so that one copy fetches 64 keys x several
+//           blocks: with a copy per cache page and block the copy engine sets the pace (20 copies per tile of 512 columns: 3.4 us). KM = 3: whole key
+//           tiles, rows of up to 256 columns. Wider rows go by in pieces of 128 columns: KM = 1, the query tile of up to 512 columns stays in shared
+//           memory; KM = 2, the query's pieces travel with the keys' pieces, from L2. With KM = 1, 2 and QT = 2 there is ONE query tile, and the two
+//           softmax groups take its key tiles in turn, each with an accumulator, maximum and sum of its own; they meet in the epilogue.
 //
 // Replaces the reference's packed prefill attention (core/.../generator/CausalSelfAttention.java:458-502: per head QK^T GEMM over
 // the visible pages, causal scaled softmax with optional soft-cap, saxpy with V).
@@ -50,6 +52,7 @@
 
 namespace dlv {
 
+void encode_map_kchunks(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint64_t pitch_bytes, uint32_t box_rows, uint32_t chunks = 2);
 void encode_map_2d(CUtensorMap* map, int dtype_code, const void* base, uint64_t rows, uint64_t cols, uint64_t pitch_bytes, uint32_t box_rows,
                    uint32_t box_cols, int swizzle_code);
 
@@ -77,8 +80,7 @@ struct AttnTcParams {
   long long gate_pitch;
   int gate_heads;
   float out_mult;
-  int wide;                    // cache rows hold all KV heads, keys are whole rows
-  int k_subs;                  // KM > 0: 64-column blocks of a key row
+  int k_subs;                  // wide layout: 64-column blocks of a key row
 };
 
 // MN-major shared-memory descriptor (128-byte swizzle): the operand tile is stored as rows of the K dimension, each row 64 elements of
@@ -115,9 +117,9 @@ __device__ __forceinline__ void tmem_st_x32(uint32_t taddr, const uint32_t* r) {
 }
 
 constexpr int kAtBM = 128, kAtBN = 64;  // query rows per score tile / keys per tile
-constexpr int kAtPiece = 2, kAtResident = 8;  // KM > 0: 64-column blocks per piece of a key row; most blocks of a query tile that stays in shared memory
+constexpr int kAtPiece = 2, kAtResident = 8;  // KM = 1, 2: 64-column blocks per piece of a key row; most blocks of a query tile that stays in shared memory
 
-// KM > 0 (one query tile): a K stage is one piece of a key tile, with KM = 2 behind the query's piece
+// KM = 1, 2 (one query tile): a K stage is one piece of a key tile, with KM = 2 behind the query's piece
 template <int DV, int QT, int KM>
 struct AttnTcWideSmem {
   static constexpr int kTileQ = kAtBM * 128 * kAtPiece;  // bytes of a query piece
@@ -223,7 +225,8 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
                            const AttnTcParams p) {
   using L = typename AttnTcLayout<DK, DV, QT, KM>::T;
   constexpr int NS = L::kStages, NSV = L::kStagesV, SUBK = L::kSubK, SUBV = L::kSubV;
-  const int pieces = KM > 0 ? (p.k_subs + kAtPiece - 1) / kAtPiece : 1;  // K stages per key tile
+  constexpr bool PIECES = KM == 1 || KM == 2;
+  const int pieces = PIECES ? (p.k_subs + kAtPiece - 1) / kAtPiece : 1;  // K stages per key tile
   constexpr int kProducer = 1, kIssuer = 0, kIssuerPV = 2;
   extern __shared__ uint8_t at_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(at_raw) + 1023) & ~uintptr_t(1023));
@@ -251,7 +254,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
   const int kvh = h / (p.H / p.KV);
   const int qs = p.q_start[seq], ql = p.q_len[seq], ctx = p.ctx_lens[seq];
   const int pos0 = ctx - ql;  // position of the sequence's first query row
-  constexpr bool SPLIT = KM > 0 && QT == 2;  // one query tile, its key tiles alternate between the softmax groups
+  constexpr bool SPLIT = PIECES && QT == 2;  // one query tile, its key tiles alternate between the softmax groups
   const int rows_all = min((SPLIT ? 1 : QT) * kAtBM, ql - q0);
   const bool two = QT == 2 && (SPLIT || rows_all > kAtBM);  // two query tiles share every K / V tile
   // key tiles [a, b) each query tile sees
@@ -312,50 +315,35 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     // One thread can start a tensor copy only every few hundred nanoseconds, whatever its size, and a key tile is several copies
     // (pages x D / 64 column blocks, for K and for V): the copies of a tile are spread over the lanes of the warp.
     if (KM == 1) {
-      if (lane == 0) mbar_expect_tx(smem_u32(bar_q), p.k_subs * kAtBM * 128);
+      if (lane == 0) mbar_expect_tx(smem_u32(bar_q), pieces * L::kTileQ);
       __syncwarp();
-      for (int c = lane; c < p.k_subs; c += 32)
-        tma_load_2d(smem_u32(smem + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0);
+      if (lane < pieces) tma_load_3d(smem_u32(smem + lane * L::kTileQ), &map_q, smem_u32(bar_q), 0, qs + q0, h * p.k_subs + lane * kAtPiece);
     }
-    if (KM == 0 && lane == 0) {
+    if (!PIECES && lane == 0) {
       mbar_expect_tx(smem_u32(bar_q), (two ? 2 : 1) * L::kTileQ);
       for (int q = 0; q < (two ? 2 : 1); ++q)
-        for (int c = 0; c < SUBK; ++c)
+        if (KM == 3) tma_load_3d(smem_u32(smem + q * L::kTileQ), &map_q, smem_u32(bar_q), 0, qs + q0 + q * kAtBM, h * p.k_subs);
+        else for (int c = 0; c < SUBK; ++c)
           tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0 + q * kAtBM);
     }
     const int box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;  // page_size is 32, 64 or 128
-    int issued = 0, issued_k = 0;  // key tiles; KM > 0: pieces of key tiles
+    int issued = 0, issued_k = 0;  // key tiles; pieces of key tiles
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t, ++issued) {
       const int s = t % NS;
       const int kt = tile_at(t);
-      if constexpr (KM > 0) {
-        // the cache pages of the tile (64 keys: one or two of them), then the pieces of its key rows, then its values
-        const int n_pg = kAtBN / box_rows;
-        long long row_of[2] = {0, 0};
-        for (int pg = 0; pg < n_pg; ++pg) {
-          const int key0 = kt * kAtBN + pg * box_rows;
-          const int page = key0 < ctx ? p.block_tables[static_cast<long long>(seq) * p.bt_stride + key0 / p.page_size] : 0;
-          row_of[pg] = static_cast<long long>(page) * p.page_size + key0 % p.page_size;
-        }
+      if constexpr (PIECES) {  // the pieces of the tile's key rows, then its values
+        const int row = p.kv_row0[seq] + kt * kAtBN;
         for (int pc = 0; pc < pieces; ++pc, ++issued_k) {
           const int st = issued_k % NS;
           if (issued_k >= NS) ok = mbar_wait(smem_u32(&bar_k_empty[st]), ((issued_k / NS) - 1) & 1, abort_flag, p.status);
           ok = __all_sync(0xffffffffu, ok);
           if (!ok) break;
-          const int subs = min(kAtPiece, p.k_subs - pc * kAtPiece);
-          if (lane == 0) mbar_expect_tx(smem_u32(&bar_k_full[st]), subs * (kAtBN * 128 + (KM == 2 ? kAtBM * 128 : 0)));
+          if (lane == 0) mbar_expect_tx(smem_u32(&bar_k_full[st]), L::kTileK);
           __syncwarp();
           uint8_t* dst = smem + L::kOffK + st * L::kTileK;
-          const int n_k = n_pg * subs;
-          if (lane < n_k) {
-            const int pg = lane / subs, c = lane - pg * subs;
-            tma_load_2d(smem_u32(dst + L::kOffKeys + c * (kAtBN * 128) + pg * box_rows * 128), &map_k, smem_u32(&bar_k_full[st]), (pc * kAtPiece + c) * 64,
-                        static_cast<int>(row_of[pg]));
-          } else if (KM == 2 && lane < n_k + subs) {
-            const int c = lane - n_k;
-            tma_load_2d(smem_u32(dst + c * (kAtBM * 128)), &map_q, smem_u32(&bar_k_full[st]), h * p.dk + (pc * kAtPiece + c) * 64, qs + q0);
-          }
+          if (lane == 0) tma_load_3d(smem_u32(dst + L::kOffKeys), &map_k, smem_u32(&bar_k_full[st]), 0, row, pc * kAtPiece);
+          if (KM == 2 && lane == 1) tma_load_3d(smem_u32(dst), &map_q, smem_u32(&bar_k_full[st]), 0, qs + q0, h * p.k_subs + pc * kAtPiece);
         }
         if (!ok) break;
         const int sv = t % NSV;
@@ -364,11 +352,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(smem_u32(&bar_v_full[sv]), L::kTileV);
         __syncwarp();
-        for (int i = lane; i < n_pg * SUBV; i += 32) {
-          const int pg = i / SUBV, c = i - pg * SUBV;
-          tma_load_2d(smem_u32(smem + L::kOffV + sv * L::kTileV + c * (kAtBN * 128) + pg * box_rows * 128), &map_v, smem_u32(&bar_v_full[sv]),
-                      kvh * p.dv + c * 64, static_cast<int>(row_of[pg]));
-        }
+        if (lane < SUBV) tma_load_2d(smem_u32(smem + L::kOffV + sv * L::kTileV + lane * (kAtBN * 128)), &map_v, smem_u32(&bar_v_full[sv]), kvh * p.dv + lane * 64, row);
         continue;
       }
       for (int kv = 0; kv < 2; ++kv) {
@@ -381,6 +365,12 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
         __syncwarp();
         uint8_t* dst = smem + (kv == 0 ? L::kOffK + s * L::kTileK : L::kOffV + s * L::kTileV);
         const int sub = kv == 0 ? SUBK : SUBV;
+        if constexpr (KM == 3) {
+          const int row = p.kv_row0[seq] + kt * kAtBN;
+          if (kv == 0 && lane == 0) tma_load_3d(smem_u32(dst), &map_k, smem_u32(full), 0, row, 0);
+          if (kv == 1 && lane < SUBV) tma_load_2d(smem_u32(dst + lane * (kAtBN * 128)), &map_v, smem_u32(full), kvh * p.dv + lane * 64, row);
+          continue;
+        }
         if constexpr (LATENT) {
           // rows behind the sequence's last key belong to the next sequence, or lie outside the buffer and arrive as zeros
           const int row = p.kv_row0[seq] + kt * kAtBN;
@@ -397,26 +387,26 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
           const int key0 = kt * kAtBN + pg * box_rows;
           // pages past the context are never read by an unmasked score; the scratch page 0 keeps the copy inside the cache
           const int page = key0 < ctx ? p.block_tables[static_cast<long long>(seq) * p.bt_stride + key0 / p.page_size] : 0;
-          const int row = (p.wide ? page : page * p.KV + kvh) * p.page_size + (key0 % p.page_size);
+          const int row = (page * p.KV + kvh) * p.page_size + (key0 % p.page_size);
           const uint32_t off = c * (kAtBN * 128) + pg * box_rows * 128;
-          tma_load_2d(smem_u32(dst + off), kv == 0 ? &map_k : &map_v, smem_u32(full), (p.wide && kv == 1 ? kvh * p.dv : 0) + c * 64, row);
+          tma_load_2d(smem_u32(dst + off), kv == 0 ? &map_k : &map_v, smem_u32(full), c * 64, row);
         }
       }
       if (!ok) break;
     }
     if (lane == 0 && *abort_flag) {
       // a wait ran out somewhere in the CTA: before shared memory goes away let the copies already issued land (bounded)
-      for (int t = issued_k > NS ? issued_k - NS : 0; KM > 0 && t < issued_k; ++t) {
+      for (int t = issued_k > NS ? issued_k - NS : 0; PIECES && t < issued_k; ++t) {
         const unsigned long long t0 = globaltimer_ns();
         while (!mbar_try_wait(smem_u32(&bar_k_full[t % NS]), (t / NS) & 1) && globaltimer_ns() - t0 < 20000000ull) {
         }
       }
-      for (int t = issued > NSV ? issued - NSV : 0; KM > 0 && t < issued; ++t) {
+      for (int t = issued > NSV ? issued - NSV : 0; PIECES && t < issued; ++t) {
         const unsigned long long t0 = globaltimer_ns();
         while (!mbar_try_wait(smem_u32(&bar_v_full[t % NSV]), (t / NSV) & 1) && globaltimer_ns() - t0 < 20000000ull) {
         }
       }
-      for (int t = issued > NS ? issued - NS : 0; KM == 0 && t < issued; ++t) {
+      for (int t = issued > NS ? issued - NS : 0; !PIECES && t < issued; ++t) {
         const unsigned long long t0 = globaltimer_ns();
         while (!(mbar_try_wait(smem_u32(&bar_k_full[t % NS]), (t / NS) & 1) && mbar_try_wait(smem_u32(&bar_v_full[t % NS]), (t / NS) & 1)) &&
                globaltimer_ns() - t0 < 20000000ull) {
@@ -460,7 +450,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
       if (n_tiles > 0 && !valid(u, q)) advance(u, q);
       if (warp == kIssuer) {
         if (KM != 2) ok = mbar_wait(smem_u32(bar_q), 0, abort_flag, p.status);
-        int piece = 0;  // KM > 0: pieces of key tiles so far
+        int piece = 0;  // pieces of key tiles so far
         const uint64_t desc_q0 = umma_desc_k_sw128(smem_u32(smem)), desc_k0 = umma_desc_k_sw128(smem_u32(smem + L::kOffK));
         int k_seen = -1;  // key tiles whose K has been waited for
         while (ok && u < n_tiles) {
@@ -468,7 +458,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
           const int s = u % NS;
           const uint32_t slot = q * 2 + (t & 1);
           if (t >= 2) ok = mbar_wait(smem_u32(&bar_pv_done[slot]), ((t >> 1) - 1) & 1, abort_flag, p.status);
-          if constexpr (KM > 0) {
+          if constexpr (PIECES) {
             const uint32_t d_w = tmem_base + kColS + slot * kAtBN;
             for (int pc = 0; ok && pc < pieces; ++pc, ++piece) {
               const int st = piece % NS;
@@ -777,16 +767,15 @@ static int launch_prefill_tc_maps(const CUtensorMap& mq, const CUtensorMap& mk, 
   return 0;
 }
 
-template <int DK, int DV, int QT, int KM = 0>
+template <int DK, int DV, int QT>
 static int launch_prefill_tc_t(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long cache_rows, const AttnTcParams& p,
                                int num_tiles, cudaStream_t st) {
   CUtensorMap mq, mk, mv;
   encode_map_2d(&mq, 0, q, static_cast<uint64_t>(T), static_cast<uint64_t>(p.H) * p.dk, static_cast<uint64_t>(q_stride) * 2, kAtBM, 64, 128);
   const uint32_t box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;
   encode_map_2d(&mk, 0, kc, static_cast<uint64_t>(cache_rows), p.dk, static_cast<uint64_t>(p.dk) * 2, box_rows, 64, 128);
-  const uint64_t v_width = static_cast<uint64_t>(p.dv) * (p.wide ? p.KV : 1);
-  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), v_width, v_width * 2, box_rows, 64, 128);
-  return launch_prefill_tc_maps<DK, DV, QT, false, KM>(mq, mk, mv, mv, p, num_tiles, st);
+  encode_map_2d(&mv, 0, vc, static_cast<uint64_t>(cache_rows), p.dv, static_cast<uint64_t>(p.dv) * 2, box_rows, 64, 128);
+  return launch_prefill_tc_maps<DK, DV, QT, false>(mq, mk, mv, mv, p, num_tiles, st);
 }
 
 // ---- latent layout -----------------------------------------------------------------------------------------------------
@@ -844,24 +833,80 @@ int launch_prefill_latent_tc(const LatentTcArgs& a, cudaStream_t st) {
   return 1;
 }
 
-// Query rows one CTA of the tcgen05 prefill kernel covers: two 128-row tiles share the K / V tiles where their two accumulators fit
-// tensor memory beside the two score slots.
-int prefill_attention_tc_tile_rows(int D) { return D <= 128 ? 256 : 128; }
+// ---- wide rows ---------------------------------------------------------------------------------------------------------
 int prefill_attention_wide_tile_rows(int k_width, int dv) {
   if (k_width <= 0 || dv <= 0 || k_width % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
   return k_width > 256 || dv > 128 ? kAtBM : 2 * kAtBM;
 }
+
+template <int DK, int DV, int QT, int KM>
+static int launch_wide_t(const WideTcArgs& a, const AttnTcParams& p, cudaStream_t st) {
+  CUtensorMap mq, mk, mv;
+  const uint64_t width = static_cast<uint64_t>(p.k_subs) * 64, rows = static_cast<uint64_t>(a.kv_rows), v_width = static_cast<uint64_t>(p.KV) * p.dv;
+  const uint32_t blocks = KM == 3 ? DK / 64 : kAtPiece;
+  encode_map_kchunks(&mq, a.q, static_cast<uint64_t>(a.T), p.H * width, p.H * width * 2, kAtBM, blocks);
+  encode_map_kchunks(&mk, a.k, rows, width, width * 2, kAtBN, blocks);
+  encode_map_2d(&mv, 0, a.v, rows, v_width, v_width * 2, kAtBN, 64, 128);
+  return launch_prefill_tc_maps<DK, DV, QT, false, KM>(mq, mk, mv, mv, p, a.num_tiles, st);
+}
+
+int launch_prefill_wide_tc(const WideTcArgs& a, AttnExtra x, cudaStream_t st) {
+  if (a.num_tiles == 0) return 0;
+  const int subs = (a.k_width + 63) / 64;
+  if (prefill_attention_wide_tile_rows(a.k_width, a.dv) == 0 || x.keep_first != 0 || x.sink != nullptr) return 1;
+  AttnTcParams p = {};
+  p.q_start = a.q_start;
+  p.q_len = a.q_len;
+  p.ctx_lens = a.ctx;
+  p.tile_seq = a.tile_seq;
+  p.tile_q0 = a.tile_q0;
+  p.kv_row0 = a.kv_row0;
+  p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.H = a.H;
+  p.KV = a.KV;
+  p.page_size = kAtBN;
+  p.scale = a.scale;
+  p.window = a.window;
+  p.causal = 1;
+  p.dk = subs * 64;
+  p.dv = a.dv;
+  p.k_subs = subs;
+  p.gate = static_cast<const __nv_bfloat16*>(x.gate);
+  p.gate_pitch = x.gate_pitch;
+  p.gate_heads = x.gate_heads;
+  p.out_mult = x.out_mult;
+  p.out_pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(a.H) * a.dv;
+  p.status = a.status;
+  if (subs <= 4) {
+    if (a.dv <= 64) {
+      if (subs <= 2) return launch_wide_t<128, 64, 2, 3>(a, p, st);
+      return subs <= 3 ? launch_wide_t<192, 64, 2, 3>(a, p, st) : launch_wide_t<256, 64, 2, 3>(a, p, st);
+    }
+    if (a.dv <= 128) {
+      if (subs <= 2) return launch_wide_t<128, 128, 2, 3>(a, p, st);
+      return subs <= 3 ? launch_wide_t<192, 128, 2, 3>(a, p, st) : launch_wide_t<256, 128, 2, 3>(a, p, st);
+    }
+    return launch_wide_t<256, 256, 1, 3>(a, p, st);
+  }
+#define DLV_WIDE(DVV, QTV) return subs <= kAtResident ? launch_wide_t<0, DVV, QTV, 1>(a, p, st) : launch_wide_t<0, DVV, QTV, 2>(a, p, st)
+  if (a.dv <= 64) DLV_WIDE(64, 2);
+  if (a.dv <= 128) DLV_WIDE(128, 2);
+  DLV_WIDE(256, 1);
+#undef DLV_WIDE
+}
+
+// Query rows one CTA of the tcgen05 prefill kernel covers: two 128-row tiles share the K / V tiles where their two accumulators fit
+// tensor memory beside the two score slots.
+int prefill_attention_tc_tile_rows(int D) { return D <= 128 ? 256 : 128; }
 
 // tile arrays: prefill_attention_tc_tile_rows(max(dk, dv)) query rows per tile. page_size must be 32, 64 or 128. Returns 1 for an unsupported
 // head size (multiples of 8 up to 256) or page size.
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                                 int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
-                                bool wide, AttnExtra x, int* status, cudaStream_t st) {
+                                AttnExtra x, int* status, cudaStream_t st) {
   if (num_tiles == 0) return 0;
-  if (wide && (prefill_attention_wide_tile_rows(dk, dv) == 0 || x.keep_first != 0)) return 1;
-  const bool pieces = wide && dk > 256;
-  const int D = pieces ? dv : (dk > dv ? dk : dv);
+  const int D = dk > dv ? dk : dv;
   if ((page != 32 && page != 64 && page != 128) || dk % 8 != 0 || dv % 8 != 0 || dk <= 0 || dv <= 0 || D > 256) return 1;
   AttnTcParams p = {};
   p.block_tables = bt;
@@ -889,25 +934,10 @@ int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, 
   p.dv = dv;
   p.out_pitch = x.out_pitch > 0 ? x.out_pitch : static_cast<long long>(H) * dv;
   p.status = status;
-  p.wide = wide ? 1 : 0;
-  p.k_subs = (dk + 63) / 64;
-  const long long cache_rows = num_pages * (wide ? 1 : KV) * page;
-  if (pieces) {
-#define DLV_WIDE(DVV, QTV)                                                                                                            \
-  return p.k_subs <= kAtResident ? launch_prefill_tc_t<0, DVV, QTV, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)          \
-                                 : launch_prefill_tc_t<0, DVV, QTV, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
-    if (dv <= 64) DLV_WIDE(64, 2);
-    if (dv <= 128) DLV_WIDE(128, 2);
-    DLV_WIDE(256, 1);
-#undef DLV_WIDE
-  }
+  const long long cache_rows = num_pages * KV * page;
   if (D <= 64) return launch_prefill_tc_t<64, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128 && dv <= 64) return launch_prefill_tc_t<128, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   if (D <= 128) return launch_prefill_tc_t<128, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-  if (wide && dv <= 64) return dk <= 192 ? launch_prefill_tc_t<192, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
-                                         : launch_prefill_tc_t<256, 64, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
-  if (wide && dv <= 128) return dk <= 192 ? launch_prefill_tc_t<192, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st)
-                                          : launch_prefill_tc_t<256, 128, 2>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
   return launch_prefill_tc_t<256, 256, 1>(q, q_stride, T, kc, vc, cache_rows, p, num_tiles, st);
 }
 

@@ -833,7 +833,7 @@ Tensor prefill_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v
 Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& q_start,
                             const Tensor& q_len, const Tensor& ctx_lens, const Tensor& tile_seq, const Tensor& tile_q0, int64_t H, double scale,
                             double softcap, int64_t window, bool causal, int64_t keep_first, c10::optional<Tensor> sink, c10::optional<Tensor> gate,
-                            double out_mult, c10::optional<Tensor> out_opt, int64_t kv_heads) {
+                            double out_mult, c10::optional<Tensor> out_opt) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 2 && q.stride(1) == 1, "q must be bf16 [T, H*D]");
   TORCH_CHECK(q.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0, "q rows must be 16-byte aligned");
   check_bf16(k_cache, "k_cache");
@@ -843,15 +843,11 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
     TORCH_CHECK(t->scalar_type() == at::kInt, "index tensors must be int32");
   }
   const int T = static_cast<int>(q.size(0));
-  // kv_heads > 0: wide rows, keys [pages, 1, page, D], values [pages, 1, page, kv_heads * DV]
-  const bool wide = kv_heads > 0;
-  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && v_cache.size(1) == k_cache.size(1) && (!wide || (k_cache.size(1) == 1 && v_cache.size(3) % kv_heads == 0)),
-              "shape mismatch");
-  const int KV = static_cast<int>(wide ? kv_heads : k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
-  const int DV = static_cast<int>(wide ? v_cache.size(3) / KV : v_cache.size(3));
-  TORCH_CHECK(v_cache.size(0) == k_cache.size(0) && v_cache.size(2) == page && q.size(1) == H * D && H % KV == 0 && k_cache.size(0) * KV * page < (int64_t(1) << 31),
-              "shape mismatch");
-  TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && (D <= 256 || wide) && DV % 8 == 0 && DV <= 256,
+  const int KV = static_cast<int>(k_cache.size(1)), page = static_cast<int>(k_cache.size(2)), D = static_cast<int>(k_cache.size(3));
+  const int DV = static_cast<int>(v_cache.size(3));
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == KV && v_cache.size(2) == page &&
+                  q.size(1) == H * D && H % KV == 0, "shape mismatch");
+  TORCH_CHECK((page == 32 || page == 64 || page == 128) && D % 8 == 0 && D <= 256 && DV % 8 == 0 && DV <= 256,
               "page size 32 / 64 / 128 and head widths that are multiples of 8 up to 256");
   TORCH_CHECK(tile_seq.numel() == tile_q0.numel(), "tile arrays differ in length");
   c10::cuda::CUDAGuard guard(q.device());
@@ -862,7 +858,7 @@ Tensor prefill_attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor
                                             static_cast<int>(block_tables.stride(0)), q_start.data_ptr<int>(), q_len.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                             tile_seq.data_ptr<int>(), tile_q0.data_ptr<int>(), static_cast<int>(tile_seq.numel()), out.data_ptr(),
                                             static_cast<int>(H), KV, D, DV, page, static_cast<float>(scale), static_cast<float>(softcap),
-                                            static_cast<int>(window), causal ? 1 : 0, wide, x, s.status.data_ptr<int>(), cur_stream());
+                                            static_cast<int>(window), causal ? 1 : 0, x, s.status.data_ptr<int>(), cur_stream());
   TORCH_CHECK(rc == 0, "prefill attention (tcgen05): unsupported shape");
   check_last_error("prefill_attention_tc");
   return out;
@@ -1561,7 +1557,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("prefill_attention_tc", &prefill_attention_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("q_start"),
         py::arg("q_len"), py::arg("ctx_lens"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"),
         py::arg("causal"), py::arg("keep_first") = 0, py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
-        py::arg("out") = py::none(), py::arg("kv_heads") = 0);
+        py::arg("out") = py::none());
   m.def("attention_rows", &attention_rows, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_tables"), py::arg("row_seq"), py::arg("positions"),
         py::arg("H"), py::arg("scale"), py::arg("softcap"), py::arg("window"), py::arg("keep_first") = 0, py::arg("sink") = py::none(),
         py::arg("gate") = py::none(), py::arg("out_mult") = 1.0, py::arg("out") = py::none(), py::arg("kv_heads") = 0);
@@ -1641,6 +1637,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("delta_decode", &delta_decode);
   m.def("delta_prompt", &delta_prompt);
   m.def("fold_heads", &fold_heads);
+  m.def("prefill_wide", &prefill_wide, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("q_start"), py::arg("q_len"), py::arg("ctx"), py::arg("row0"), py::arg("tile_seq"),
+        py::arg("tile_q0"), py::arg("H"), py::arg("KV"), py::arg("scale"), py::arg("window"), py::arg("gate") = py::none(), py::arg("out_mult") = 1.0,
+        py::arg("out") = py::none());
   m.def("prefill_wide_tile_rows", [](int64_t k_width, int64_t dv) { return dlv::prefill_attention_wide_tile_rows(static_cast<int>(k_width), static_cast<int>(dv)); });
   m.def("mixed_decode_ok", [](int64_t H, int64_t KV, int64_t dk, int64_t dv) {
     return dlv::mixed_decode_supported(static_cast<int>(H), static_cast<int>(KV), static_cast<int>(dk), static_cast<int>(dv));

@@ -578,7 +578,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) decode_chain_kernel(const __g
 }
 
 // ------------------------------------------------------------------------------------------------ host side
-void encode_map_kchunks(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint64_t pitch_bytes, uint32_t box_rows);
+void encode_map_kchunks(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint64_t pitch_bytes, uint32_t box_rows, uint32_t chunks = 2);
 int gemm_num_sms();
 
 int chain_smax(int n_tiles, int kbt, int P) {

@@ -51,15 +51,15 @@ void encode_map_2d(CUtensorMap* map, int dtype_code, const void* base, uint64_t 
   if (r != CUDA_SUCCESS) throw std::runtime_error("cuTensorMapEncodeTiled failed with code " + std::to_string(static_cast<int>(r)));
 }
 
-// bf16 matrix [rows, K] (K % 64 == 0) seen as [K / 64 chunks][rows][64]: one box = `box_rows` rows x 2 chunks lands in shared
+// bf16 matrix [rows, K] (K % 64 == 0) seen as [K / 64 chunks][rows][64]: one box = `box_rows` rows x `chunks` (2) chunks lands in shared
 // memory as two consecutive 128B-swizzled 64-wide sub-tiles, i.e. a whole 128-k pipeline stage with ONE copy instruction
 // (a single thread can only issue a copy every ~0.3 us, whatever its size).
-void encode_map_kchunks(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint64_t pitch_bytes, uint32_t box_rows) {
+void encode_map_kchunks(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint64_t pitch_bytes, uint32_t box_rows, uint32_t chunks = 2) {
   if ((reinterpret_cast<uintptr_t>(base) & 15) != 0) throw std::runtime_error("TMA base address must be 16-byte aligned");
   if (pitch_bytes % 16 != 0 || K % 64 != 0) throw std::runtime_error("chunked TMA map needs K % 64 == 0 and a 16-byte row pitch");
   cuuint64_t dims[3] = {64, rows, K / 64};
   cuuint64_t strides[2] = {pitch_bytes, 128};
-  cuuint32_t box[3] = {64, box_rows, 2};
+  cuuint32_t box[3] = {64, box_rows, chunks};
   cuuint32_t estr[3] = {1, 1, 1};
   CUresult r = get_encode()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
                             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

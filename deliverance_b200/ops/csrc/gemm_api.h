@@ -178,9 +178,22 @@ extern bool g_gemv_simt_only;  // gemm.cu: grouped JQ4 GEMV on CUDA cores instea
 int launch_prefill_attention_tc(const void* q, long long q_stride, long long T, const void* kc, const void* vc, long long num_pages, const int* bt,
                                 int bt_stride, const int* q_start, const int* q_len, const int* ctx, const int* tile_seq, const int* tile_q0,
                                 int num_tiles, void* out, int H, int KV, int dk, int dv, int page, float scale, float cap, int window, int causal,
-                                bool wide, AttnExtra x, int* status, cudaStream_t st);
+                                AttnExtra x, int* status, cudaStream_t st);
 // wide rows: query tile height for keys of k_width columns and values of dv columns per head, 0 when the kernel does not take them
 int prefill_attention_wide_tile_rows(int k_width, int dv);
+// q [T, H * W], gathered keys k [kv_rows, W] (W: k_width padded with zeros to a multiple of 64) and values v [kv_rows, KV * dv]
+struct WideTcArgs {
+  const void *q, *k, *v;
+  long long T, kv_rows;
+  int H, KV, k_width, dv;
+  const int *q_start, *q_len, *ctx, *kv_row0, *tile_seq, *tile_q0;  // ctx: keys of a sequence in k / v (its query rows are the last q_len)
+  int num_tiles;
+  void* out;
+  float scale;
+  int window;
+  int* status;
+};
+int launch_prefill_wide_tc(const WideTcArgs& a, AttnExtra x, cudaStream_t st);
 
 // sampling.cu
 void launch_argmax(const float* logits, int ld, int B, int V, const uint32_t* mask, int mask_ld, float softcap, float inv_scale,
@@ -333,7 +346,8 @@ bool mixed_decode_supported(int H, int KV, int dk, int dv);
 int mixed_decode_ctas(int H, int KV, int dk, int dv);  // CTAs per SM
 int launch_mixed_decode(const MixedDecodeArgs& a, cudaStream_t st);
 void launch_decode_merge(const float* po, const float* pml, void* out, int B, int H, int dv, int splits, AttnExtra x, cudaStream_t st);  // attention.cu
-int launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st);
+// out [T, H * pitch], pitch >= KV * dk (columns behind it are the caller's)
+int launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int pitch, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st);
 
 // a2a.cu: expert-parallel all-to-all over peer memory (see the file comment for the protocol)
 struct A2AParams {

@@ -413,11 +413,11 @@ int launch_mixed_decode(const MixedDecodeArgs& a, cudaStream_t st) {
   return 1;
 }
 
-// out [T, H, KV dk]. A thread takes eight columns of one (row, KV head): the group's queries stay in registers (PER > 0 of them) while it goes over the
+// out [T, H, pitch >= KV dk]. A thread takes eight columns of one (row, KV head): the group's queries stay in registers (PER > 0 of them) while it goes over the
 // heads; PER = 0: groups of any size, read again for every head.
 template <typename TIO, int PER>
-__global__ void __launch_bounds__(256) fold_heads_kernel(const TIO* __restrict__ q, long long q_stride, const float* __restrict__ mix, TIO* __restrict__ out, int H,
-                                                         int KV, int dk, int rows) {
+__global__ void __launch_bounds__(256) fold_heads_kernel(const TIO* __restrict__ q, long long q_stride, const float* __restrict__ mix, TIO* __restrict__ out,
+                                                         int pitch, int H, int KV, int dk, int rows) {
   extern __shared__ float fsm[];  // [H][H]
   pdl_wait();
   pdl_trigger();
@@ -433,8 +433,7 @@ __global__ void __launch_bounds__(256) fold_heads_kernel(const TIO* __restrict__
 #pragma unroll
     for (int g = 0; g < PER; ++g) io_ld8(src + g * dk, v[g]);
   }
-  TIO* dst = out + (static_cast<long long>(t) * H * KV + kvh) * dk + x;
-  const long long step = static_cast<long long>(KV) * dk;
+  TIO* dst = out + static_cast<long long>(t) * H * pitch + kvh * dk + x;
   const float* m = fsm + kvh * per;
 #pragma unroll 2
   for (int h = 0; h < H; ++h) {
@@ -455,16 +454,16 @@ __global__ void __launch_bounds__(256) fold_heads_kernel(const TIO* __restrict__
       }
     }
     io_st8(dst, acc);
-    dst += step;
+    dst += pitch;
     m += H;
   }
 }
 
 template <typename TIO>
-static void launch_fold_heads_t(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, cudaStream_t st) {
+static void launch_fold_heads_t(const void* q, long long q_stride, const float* mix, void* out, int pitch, int T, int H, int KV, int dk, cudaStream_t st) {
   const dim3 grid(static_cast<unsigned>((static_cast<long long>(T) * KV * (dk / 8) + 255) / 256));
   const size_t smem = static_cast<size_t>(H) * H * 4;
-#define DLV_FOLD(N) launch_pdl(fold_heads_kernel<TIO, N>, grid, dim3(256), smem, st, static_cast<const TIO*>(q), q_stride, mix, static_cast<TIO*>(out), H, KV, dk, T)
+#define DLV_FOLD(N) launch_pdl(fold_heads_kernel<TIO, N>, grid, dim3(256), smem, st, static_cast<const TIO*>(q), q_stride, mix, static_cast<TIO*>(out), pitch, H, KV, dk, T)
   switch (H / KV) {
     case 1: DLV_FOLD(1); break;
     case 2: DLV_FOLD(2); break;
@@ -477,11 +476,11 @@ static void launch_fold_heads_t(const void* q, long long q_stride, const float* 
   }
 #undef DLV_FOLD
 }
-int launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st) {
+int launch_fold_heads(const void* q, long long q_stride, const float* mix, void* out, int pitch, int T, int H, int KV, int dk, bool is_f32, cudaStream_t st) {
   if (T == 0) return 0;
   if (H > 108 || static_cast<long long>(T) * KV * (dk / 8) > 0x7fffff00ll) return 1;  // (the matrix fits 48 KB of shared memory)
-  if (is_f32) launch_fold_heads_t<float>(q, q_stride, mix, out, T, H, KV, dk, st);
-  else launch_fold_heads_t<__nv_bfloat16>(q, q_stride, mix, out, T, H, KV, dk, st);
+  if (is_f32) launch_fold_heads_t<float>(q, q_stride, mix, out, pitch, T, H, KV, dk, st);
+  else launch_fold_heads_t<__nv_bfloat16>(q, q_stride, mix, out, pitch, T, H, KV, dk, st);
   return 0;
 }
 

@@ -13,7 +13,7 @@ columns of their own; ``g`` is there for gated heads. CUDA forms:
 
 Mixed scores (``mixed``): a cache row holds all KV heads of a token, ``k [pages, 1, page, G * dk]`` and ``v [pages, 1, page, G * dv]``. Prompts move the mixing to the
 query side: head h's mixed score against a key is the product of the whole cache row with ``[sum_(g in group 0) mix[h, g] q_g | sum_(g in group 1) .. | ..]``, so
-the prompt kernel runs with queries of ``G * dk`` columns against one wide key. Decode steps take all heads of a row in one CTA and mix the fp32 scores.
+the prompt kernel runs with queries of ``G * dk`` columns against one wide key (gathered rows). Decode steps take all heads of a row in one CTA and mix the fp32 scores.
 """
 from __future__ import annotations
 
@@ -194,23 +194,34 @@ def _mixed_attention(s: GroupedShape, qkv, q, mix, batch, k_cache, v_cache, mask
         ops._count(1 if splits <= 1 else 2)
         return e.mixed_decode(q, mix, k_cache, v_cache, batch.block_tables, batch.ctx_len, s.heads, s.kv_heads, mask[0], mask[2], splits, gate=extra["gate"],
                               out_mult=extra["out_mult"], out=extra["out"])
-    ops._count(2)
-    folded = e.fold_heads(q, mix, s.heads, s.kv_heads)
-    rows = 0 if qkv.dtype == torch.float32 else e.prefill_wide_tile_rows(s.k_width, s.dv)
+    rows = 0 if batch.is_decode or qkv.dtype == torch.float32 else e.prefill_wide_tile_rows(s.k_width, s.dv)
     if not rows:
-        return e.attention_rows(folded, k_cache, v_cache, batch.block_tables, None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask,
-                                kv_heads=s.kv_heads, **extra)
-    ts, t0 = batch.tiles(rows) if not batch.is_decode else decode_tiles(batch)
-    return e.prefill_attention_tc(folded, k_cache, v_cache, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_len, ts, t0, s.heads, *mask, True,
-                                  kv_heads=s.kv_heads, **extra)
+        ops._count(2)
+        return e.attention_rows(e.fold_heads(q, mix, s.heads, s.kv_heads, s.k_width), k_cache, v_cache, batch.block_tables,
+                                None if batch.is_decode else row_sequence(batch), batch.positions, s.heads, *mask, kv_heads=s.kv_heads, **extra)
+    ops._count(3)
+    pitch = (s.k_width + 63) // 64 * 64
+    plan = wide_plan(batch, mask[2])
+    keys, values = e.latent_gather(k_cache, v_cache, batch.block_tables, plan["seq"], plan["key0"], plan["n_keys"], plan["row0"], plan["max_rows"], plan["total"], pitch,
+                                   s.v_width)
+    ts, t0 = batch.tiles(rows)
+    return e.prefill_wide(e.fold_heads(q, mix, s.heads, s.kv_heads, pitch), keys, values, batch.q_start, batch.q_len, plan["n_keys"], plan["row0"], ts, t0, s.heads,
+                          s.kv_heads, mask[0], mask[2], gate=extra["gate"], out_mult=extra["out_mult"], out=extra["out"])
 
 
-def decode_tiles(batch):
-    """Query tiles of a decode step: one per sequence."""
-    if "decode_tiles" not in batch.plans:
-        n, dev = batch.num_seqs, batch.q_len.device
-        batch.plans["decode_tiles"] = (torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, dtype=torch.int32, device=dev))
-    return batch.plans["decode_tiles"]
+def wide_plan(batch, window: int) -> dict:
+    """Visible key range of every sequence of a batch and its place in the gathered rows (built once per batch and window)."""
+    key = ("wide", window)
+    if key not in batch.plans:
+        dev = batch.q_len.device
+        n, ctx = torch.tensor(batch.q_len_host), torch.tensor(batch.ctx_len_host)
+        first = (ctx - n - window + 1).clamp(min=0) if window > 0 else torch.zeros_like(ctx)
+        keys = torch.where(n > 0, ctx - first, torch.zeros_like(ctx))
+        row0 = torch.cumsum(keys, 0) - keys
+        put = lambda t: t.to(torch.int32).to(dev, non_blocking=True)  # noqa: E731
+        batch.plans[key] = {"seq": put(torch.arange(len(n))), "key0": put(first), "n_keys": put(keys), "row0": put(row0), "max_rows": int(keys.max()),
+                            "total": int(keys.sum())}
+    return batch.plans[key]
 
 
 def mixed_splits(s: GroupedShape, num_seqs: int, span: int, sms: int = 148) -> int:
