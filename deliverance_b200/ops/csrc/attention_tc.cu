@@ -40,7 +40,9 @@
 //           blocks: with a copy per cache page and block the copy engine sets the pace (20 copies per tile of 512 columns: 3.4 us). KM = 3: whole key
 //           tiles, rows of up to 256 columns. Wider rows go by in pieces of 128 columns: KM = 1, the query tile of up to 512 columns stays in shared
 //           memory; KM = 2, the query's pieces travel with the keys' pieces, from L2. With KM = 1, 2 and QT = 2 there is ONE query tile, and the two
-//           softmax groups take its key tiles in turn, each with an accumulator, maximum and sum of its own; they meet in the epilogue.
+//           softmax groups take its key tiles in turn, each with an accumulator, maximum and sum of its own; they meet in the epilogue. Warps 0 and 3
+//           then issue the Q K^T of one group's tiles each, from halves of the key ring: a group of eight MMAs behind a wait costs its thread about a
+//           thousand cycles, twice the MMAs themselves (one thread 337 us for 16 heads over rows of 512 columns, whatever the depth of the ring).
 //
 // Replaces the reference's packed prefill attention (core/.../generator/CausalSelfAttention.java:458-502: per head QK^T GEMM over
 // the visible pages, causal scaled softmax with optional soft-cap, saxpy with V).
@@ -136,7 +138,7 @@ struct AttnTcWideSmem {
   static constexpr int kBytes = kOffCtrl + 512 + 1024;
   static constexpr int kThreads = 128 + 128 * QT;
   static constexpr int kSubK = 0, kSubV = DV / 64;
-  static_assert(kStages >= 2 && DV % 64 == 0 && kBytes > 118 * 1024 && kBytes <= 227 * 1024 && 256 + QT * DV <= 512, "attention tile does not fit");
+  static_assert(kStages >= 2 && (QT == 1 || kStages == 4) && DV % 64 == 0 && kBytes > 118 * 1024 && kBytes <= 227 * 1024 && 256 + QT * DV <= 512, "attention tile does not fit");
 };
 
 template <int DK, int DV, int QT>
@@ -227,7 +229,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
   constexpr int NS = L::kStages, NSV = L::kStagesV, SUBK = L::kSubK, SUBV = L::kSubV;
   constexpr bool PIECES = KM == 1 || KM == 2;
   const int pieces = PIECES ? (p.k_subs + kAtPiece - 1) / kAtPiece : 1;  // K stages per key tile
-  constexpr int kProducer = 1, kIssuer = 0, kIssuerPV = 2;
+  constexpr int kProducer = 1, kIssuer = 0, kIssuerPV = 2, kIssuer2 = 3;  // (kIssuer2: SPLIT, the second softmax group's Q K^T)
   extern __shared__ uint8_t at_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(at_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bar_q = reinterpret_cast<uint64_t*>(smem + L::kOffCtrl);
@@ -239,8 +241,8 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
   uint64_t* bar_p_full = bar_s_full + 4;   // [2][2] probabilities written over the scores
   uint64_t* bar_pv_done = bar_p_full + 4;  // [2][2] the P V that read the slot's probabilities has retired
   uint64_t* bar_o_final = bar_pv_done + 4;
-  uint64_t* bar_drain = bar_o_final + 1;    // [2] an issuing thread's MMAs have retired (only used when a wait ran out)
-  uint64_t* bar_ml = bar_drain + 2;         // SPLIT: maxima and sums of both softmax groups are in shared memory
+  uint64_t* bar_drain = bar_o_final + 1;    // [3] an issuing thread's MMAs have retired (only used when a wait ran out)
+  uint64_t* bar_ml = bar_drain + 3;         // SPLIT: maxima and sums of both softmax groups are in shared memory
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_ml + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
@@ -291,6 +293,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     }
     mbar_init(smem_u32(&bar_drain[0]), 1);
     mbar_init(smem_u32(&bar_drain[1]), 1);
+    mbar_init(smem_u32(&bar_drain[2]), 1);
     mbar_init(smem_u32(bar_o_final), 1);
     mbar_init(smem_u32(bar_ml), 8);
     *abort_flag = 0;
@@ -327,32 +330,40 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
           tma_load_2d(smem_u32(smem + q * L::kTileQ + c * (kAtBM * 128)), &map_q, smem_u32(bar_q), h * p.dk + c * 64, qs + q0 + q * kAtBM);
     }
     const int box_rows = p.page_size < kAtBN ? p.page_size : kAtBN;  // page_size is 32, 64 or 128
-    int issued = 0, issued_k = 0;  // key tiles; pieces of key tiles
+    int issued = 0, issued_k[2] = {0, 0};  // key tiles; pieces of key tiles (SPLIT: of either group, which has half of the ring)
+    constexpr int NSK = SPLIT ? NS / 2 : NS;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t, ++issued) {
       const int s = t % NS;
       const int kt = tile_at(t);
-      if constexpr (PIECES) {  // the pieces of the tile's key rows, then its values
-        const int row = p.kv_row0[seq] + kt * kAtBN;
-        for (int pc = 0; pc < pieces; ++pc, ++issued_k) {
-          const int st = issued_k % NS;
-          if (issued_k >= NS) ok = mbar_wait(smem_u32(&bar_k_empty[st]), ((issued_k / NS) - 1) & 1, abort_flag, p.status);
-          ok = __all_sync(0xffffffffu, ok);
+      if constexpr (PIECES) {  // the pieces of the tile's key rows (SPLIT: of two tiles in turn), then its values
+        if (!SPLIT || (t & 1) == 0) {
+          const int n_q = SPLIT && t + 1 < n_tiles ? 2 : 1;
+          for (int i = 0; ok && i < pieces * n_q; ++i) {
+            const int pc = i / n_q, q = i % n_q, n = q == 0 ? issued_k[0] : issued_k[1];
+            const int st = q * NSK + n % NSK;
+            if (n >= NSK) ok = mbar_wait(smem_u32(&bar_k_empty[st]), ((n / NSK) - 1) & 1, abort_flag, p.status);
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            if (lane == 0) mbar_expect_tx(smem_u32(&bar_k_full[st]), L::kTileK);
+            __syncwarp();
+            uint8_t* dst = smem + L::kOffK + st * L::kTileK;
+            if (lane == 0) tma_load_3d(smem_u32(dst + L::kOffKeys), &map_k, smem_u32(&bar_k_full[st]), 0, p.kv_row0[seq] + (kt + q) * kAtBN, pc * kAtPiece);
+            if (KM == 2 && lane == 1) tma_load_3d(smem_u32(dst), &map_q, smem_u32(&bar_k_full[st]), 0, qs + q0, h * p.k_subs + pc * kAtPiece);
+            if (q == 0) ++issued_k[0];
+            else ++issued_k[1];
+          }
           if (!ok) break;
-          if (lane == 0) mbar_expect_tx(smem_u32(&bar_k_full[st]), L::kTileK);
-          __syncwarp();
-          uint8_t* dst = smem + L::kOffK + st * L::kTileK;
-          if (lane == 0) tma_load_3d(smem_u32(dst + L::kOffKeys), &map_k, smem_u32(&bar_k_full[st]), 0, row, pc * kAtPiece);
-          if (KM == 2 && lane == 1) tma_load_3d(smem_u32(dst), &map_q, smem_u32(&bar_k_full[st]), 0, qs + q0, h * p.k_subs + pc * kAtPiece);
         }
-        if (!ok) break;
         const int sv = t % NSV;
         if (t >= NSV) ok = mbar_wait(smem_u32(&bar_v_empty[sv]), ((t / NSV) - 1) & 1, abort_flag, p.status);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(smem_u32(&bar_v_full[sv]), L::kTileV);
         __syncwarp();
-        if (lane < SUBV) tma_load_2d(smem_u32(smem + L::kOffV + sv * L::kTileV + lane * (kAtBN * 128)), &map_v, smem_u32(&bar_v_full[sv]), kvh * p.dv + lane * 64, row);
+        if (lane < SUBV)
+          tma_load_2d(smem_u32(smem + L::kOffV + sv * L::kTileV + lane * (kAtBN * 128)), &map_v, smem_u32(&bar_v_full[sv]), kvh * p.dv + lane * 64,
+                      p.kv_row0[seq] + kt * kAtBN);
         continue;
       }
       for (int kv = 0; kv < 2; ++kv) {
@@ -396,11 +407,12 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
     }
     if (lane == 0 && *abort_flag) {
       // a wait ran out somewhere in the CTA: before shared memory goes away let the copies already issued land (bounded)
-      for (int t = issued_k > NS ? issued_k - NS : 0; PIECES && t < issued_k; ++t) {
-        const unsigned long long t0 = globaltimer_ns();
-        while (!mbar_try_wait(smem_u32(&bar_k_full[t % NS]), (t / NS) & 1) && globaltimer_ns() - t0 < 20000000ull) {
+      for (int q = 0; PIECES && q < 2; ++q)
+        for (int n = issued_k[q] > NSK ? issued_k[q] - NSK : 0; n < issued_k[q]; ++n) {
+          const unsigned long long t0 = globaltimer_ns();
+          while (!mbar_try_wait(smem_u32(&bar_k_full[q * NSK + n % NSK]), (n / NSK) & 1) && globaltimer_ns() - t0 < 20000000ull) {
+          }
         }
-      }
       for (int t = issued > NSV ? issued - NSV : 0; PIECES && t < issued; ++t) {
         const unsigned long long t0 = globaltimer_ns();
         while (!mbar_try_wait(smem_u32(&bar_v_full[t % NSV]), (t / NSV) & 1) && globaltimer_ns() - t0 < 20000000ull) {
@@ -414,7 +426,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
       }
     }
     __syncwarp();
-  } else if (warp == kIssuer || warp == kIssuerPV) {
+  } else if (warp == kIssuer || warp == kIssuerPV || (SPLIT && warp == kIssuer2)) {
     // ---------------- MMA issuers ----------------
     // Work items (key tile j, query tile q) in order: (j, 0), (j, 1) for every j the query tile sees. Each query tile has two score
     // slots, used by its key tiles in turn.
@@ -448,9 +460,14 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
       bool ok = true;
       int u = 0, q = 0;
       if (n_tiles > 0 && !valid(u, q)) advance(u, q);
-      if (warp == kIssuer) {
+      if (warp != kIssuerPV) {
         if (KM != 2) ok = mbar_wait(smem_u32(bar_q), 0, abort_flag, p.status);
-        int piece = 0;  // pieces of key tiles so far
+        if (warp == kIssuer2) {
+          u = 1;
+          q = 1;
+        }
+        constexpr int NSK = SPLIT ? NS / 2 : NS;
+        int piece = 0;  // pieces of this thread's key tiles so far
         const uint64_t desc_q0 = umma_desc_k_sw128(smem_u32(smem)), desc_k0 = umma_desc_k_sw128(smem_u32(smem + L::kOffK));
         int k_seen = -1;  // key tiles whose K has been waited for
         while (ok && u < n_tiles) {
@@ -461,8 +478,8 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
           if constexpr (PIECES) {
             const uint32_t d_w = tmem_base + kColS + slot * kAtBN;
             for (int pc = 0; ok && pc < pieces; ++pc, ++piece) {
-              const int st = piece % NS;
-              ok = mbar_wait(smem_u32(&bar_k_full[st]), (piece / NS) & 1, abort_flag, p.status);
+              const int st = (SPLIT ? q * NSK : 0) + piece % NSK;
+              ok = mbar_wait(smem_u32(&bar_k_full[st]), (piece / NSK) & 1, abort_flag, p.status);
               if (!ok) break;
               tc_fence_after();
               const uint64_t desc_q = umma_desc_k_sw128(smem_u32(smem + (KM == 1 ? pc * L::kTileQ : L::kOffK + st * L::kTileK)));
@@ -477,7 +494,8 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
             }
             if (!ok) break;
             umma_commit(smem_u32(&bar_s_full[slot]));
-            advance(u, q);
+            if (SPLIT) u += 2;
+            else advance(u, q);
             continue;
           }
           if (ok && u > k_seen) {
@@ -525,7 +543,7 @@ __global__ void __launch_bounds__(AttnTcLayout<DK, DV, QT, KM>::T::kThreads, 1)
       }
       if (!ok) {
         // a wait ran out: let this thread's outstanding MMAs retire (bounded) before tensor memory is released
-        uint64_t* drain = &bar_drain[warp == kIssuer ? 0 : 1];
+        uint64_t* drain = &bar_drain[warp == kIssuer ? 0 : (warp == kIssuerPV ? 1 : 2)];
         umma_commit(smem_u32(drain));
         const unsigned long long t0 = globaltimer_ns();
         while (!mbar_try_wait(smem_u32(drain), 0) && globaltimer_ns() - t0 < 20000000ull) {
