@@ -13,7 +13,8 @@
 //   delta_chunks_kernel     one CTA per (64 value columns, head, sequence) walks the chunks: U^T = (V^T - S^T K'^T) T^T, O^T = S^T Q^T + U^T A^T, then
 //                           S^T = S^T diag(exp(b_end)) + U^T K. S^T is the accumulator of the last product and, converted in registers, the left operand of
 //                           the first two; eight warps = 4 x 16 value columns x 2 halves of the key channels. The halves' shares of S^T K'^T meet in
-//                           shared memory (both then hold the whole U^T), those of O on their way out. Chunk tiles arrive by cp.async in two stages.
+//                           shared memory (both then hold the whole U^T), those of O on their way out. Two stages; the prepare kernel writes what
+//                           a chunk needs as it lies in shared memory, so a stage is one contiguous copy.
 //   delta_norm_gate_kernel  norm and gate of prompt rows.
 #include <cooperative_groups.h>
 
@@ -29,6 +30,11 @@ namespace {
 
 constexpr int kDnCols = 64;  // value columns per CTA
 __device__ __forceinline__ float dn_softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+// softplus of prepared chunks: the series of log(1 + e) where 1 + e would round e away
+__device__ __forceinline__ float dn_softplus_fast(float v) {
+  const float e = __expf(-fabsf(v));
+  return fmaxf(v, 0.f) + (e < 0.04f ? e * (1.f - e * (0.5f - e * (0.33333333f - e * (0.25f - e * 0.2f)))) : __logf(1.f + e));
+}
 __device__ __forceinline__ float dn_sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
 __device__ __forceinline__ float dn_ex2(float x) {
   float y;
@@ -265,28 +271,45 @@ int launch_delta_recurrent(const DeltaArgs& a, bool is_f32, cudaStream_t st) {
 // =====================================================================================================================
 // Chunked form (decay logarithms in base 2)
 // =====================================================================================================================
+// What the walk reads of one (chunk, head), as it lies in shared memory: q exp(b), k exp(b_end - b), k exp(b) high | low [6][C][P], A and T high | low
+// [4][C][PA], decay [16 NK] fp32. NK: 16-channel tiles of the key width (2, 4, 8 or 16); columns and rows behind the real ones are zero.
+template <int C>
+struct DeltaImage {
+  int P, off_a, off_dec, bytes;
+  static constexpr int PA = C + 8;
+  __host__ __device__ constexpr explicit DeltaImage(int nk) : P(nk * 16 + 8), off_a(6 * C * (nk * 16 + 8) * 2), off_dec(0), bytes(0) {
+    off_dec = off_a + 4 * C * PA * 2;
+    bytes = off_dec + nk * 16 * 4;
+  }
+};
+static int delta_tiles(int dk) { return dk <= 32 ? 2 : dk <= 64 ? 4 : dk <= 128 ? 8 : 16; }
+
+int64_t delta_image_bytes(int dk, int chunk) { return chunk == 16 ? DeltaImage<16>(delta_tiles(dk)).bytes : DeltaImage<32>(delta_tiles(dk)).bytes; }
+
 constexpr float kDnMaxLogDecay = 86.f;  // 2^(+-86) and its products with unit vectors stay inside fp32
 
-template <int C>
+template <int C, int R>
 struct DeltaPrepareSmem {
   int P, off_m, off_t, off_f, bytes;
   __host__ __device__ explicit DeltaPrepareSmem(int dk) {
     P = (dk + 15) / 16 * 16 + 8;
     off_m = 6 * C * P * 2;               // [3][2][C][P]: q exp(b), k exp(-b), k exp(b); term by term: running sums [C][dk]
     off_t = off_m + 2 * C * (C + 1) * 4; // [C][C + 1] M, then its inverse
-    off_f = off_t + C / 8 * dk * 4;      // [C / 8][dk] sums of the log decays of eight rows
+    off_f = off_t + C / R * dk * 4;      // [C / R][dk] sums of the log decays of R rows
     bytes = off_f + 3 * C * 4;           // [3][C] unit factors of q and k, beta
   }
 };
 
-// A thread keeps two channels of eight rows.
-template <int C>
+// A thread keeps two channels of R rows.
+template <int C, int R>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, const DeltaChunks c) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) uint8_t dsm[];
-  const DeltaPrepareSmem<C> L(a.dk);
-  constexpr int R = 8, NG = C / R;
+  const DeltaPrepareSmem<C, R> L(a.dk);
+  constexpr int NG = C / R;
+  const DeltaImage<C> I(c.tiles);
+  uint8_t* image = static_cast<uint8_t*>(c.images) + (static_cast<size_t>(blockIdx.x) * a.H + blockIdx.y) * I.bytes;
   const int ck = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int dk = a.dk, dk16 = (dk + 15) / 16 * 16, P = L.P, half = dk / 2;
   float* sb = reinterpret_cast<float*>(dsm);
@@ -322,8 +345,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       if (t0 + i < len) {
-        acc.x += la * dn_softplus(b[i].x + bias.x);
-        acc.y += la * dn_softplus(b[i].y + bias.y);
+        acc.x += la * dn_softplus_fast(b[i].x + bias.x);
+        acc.y += la * dn_softplus_fast(b[i].y + bias.y);
       }
       b[i] = acc;
     }
@@ -374,13 +397,13 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       b[i].y += before.y;
     }
     small = fminf(be.x, be.y) > -kDnMaxLogDecay;
-    if (grp == 0) *reinterpret_cast<float2*>(c.decay + (static_cast<size_t>(ck) * a.H + h) * dk + d) = make_float2(dn_ex2(be.x), dn_ex2(be.y));
+    if (grp == 0) *reinterpret_cast<float2*>(image + I.off_dec + d * 4) = make_float2(dn_ex2(be.x), dn_ex2(be.y));
   }
   const bool fast = __syncthreads_and(small);
   // ---- scaled queries and keys
   if (active) {
-    uint32_t* o = reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(c.qk) + (static_cast<size_t>(row0 + t0) * a.H + h) * 6 * dk + d);
-    const size_t step = static_cast<size_t>(a.H) * 6 * half;
+    uint32_t* o = reinterpret_cast<uint32_t*>(image) + (t0 * I.P + d) / 2;
+    const int plane = C * I.P / 2;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int t = t0 + i;
@@ -392,15 +415,13 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       split2(q.x * uq * ex, q.y * uq * ey, qh, ql);
       split2(k.x * ex, k.y * ey, bh, bl);
       split2(k.x * dn_ex2(be.x - b[i].x), k.y * dn_ex2(be.y - b[i].y), kh, kl);
-      if (t < len) {
-        o[0] = qh;
-        o[half] = ql;
-        o[2 * half] = kh;
-        o[3 * half] = kl;
-        o[4 * half] = bh;
-        o[5 * half] = bl;
-      }
-      o += step;
+      o[0] = qh;
+      o[plane] = ql;
+      o[2 * plane] = kh;
+      o[3 * plane] = kl;
+      o[4 * plane] = bh;
+      o[5 * plane] = bl;
+      o += I.P / 2;
       if (fast) {
         *reinterpret_cast<uint32_t*>(sQ + t * P + d) = qh;
         *reinterpret_cast<uint32_t*>(sQ + (C + t) * P + d) = ql;
@@ -414,11 +435,15 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       }
     }
   }
+  if (const int pad = (I.P - 8 - dk) / 8; pad > 0) {
+    for (int e = tid; e < 6 * C * pad; e += 256) *reinterpret_cast<uint4*>(image + ((e / pad) * I.P + dk + (e % pad) * 8) * 2) = make_uint4(0, 0, 0, 0);
+    if (tid < pad * 8) reinterpret_cast<float*>(image + I.off_dec)[dk + tid] = 0.f;
+  }
   if (fast && dk16 != dk)  // (widths are multiples of 8)
     for (int e = tid; e < 6 * C * 4; e += 256) reinterpret_cast<uint32_t*>(sQ + (e >> 2) * P + dk)[e & 3] = 0u;
   __syncthreads();
   // ---- causal matrix of the queries (to memory) and M (to shared memory): the 16 x 16 blocks on and below the diagonal
-  __nv_bfloat16* am = static_cast<__nv_bfloat16*>(c.a) + (static_cast<size_t>(ck) * a.H + h) * 4 * C * C;
+  __nv_bfloat16* am = reinterpret_cast<__nv_bfloat16*>(image + I.off_a);
   constexpr int NB = C / 16;
   const int gq = lane >> 2, t4 = lane & 3;
   if (fast) {
@@ -454,8 +479,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
           } else {
             uint32_t hi, lw;
             split2(s <= t ? acc[n][2 * r] : 0.f, s + 1 <= t ? acc[n][2 * r + 1] : 0.f, hi, lw);
-            *reinterpret_cast<uint32_t*>(am + t * C + s) = hi;
-            *reinterpret_cast<uint32_t*>(am + C * C + t * C + s) = lw;
+            *reinterpret_cast<uint32_t*>(am + t * I.PA + s) = hi;
+            *reinterpret_cast<uint32_t*>(am + (C + t) * I.PA + s) = lw;
           }
         }
     }
@@ -482,8 +507,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       }
       uint32_t hi, lw;
       split2(v[0], v[1], hi, lw);
-      *reinterpret_cast<uint32_t*>(am + t * C + s) = hi;
-      *reinterpret_cast<uint32_t*>(am + C * C + t * C + s) = lw;
+      *reinterpret_cast<uint32_t*>(am + t * I.PA + s) = hi;
+      *reinterpret_cast<uint32_t*>(am + (C + t) * I.PA + s) = lw;
       sM[t * (C + 1) + s] = m[0];
       sM[t * (C + 1) + s + 1] = m[1];
     }
@@ -527,20 +552,17 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     if (s / 16 > t / 16) continue;
     uint32_t hi, lw;
     split2(s <= t ? sX[t * W + s] * beta[s] : 0.f, s + 1 <= t ? sX[t * W + s + 1] * beta[s + 1] : 0.f, hi, lw);
-    *reinterpret_cast<uint32_t*>(am + 2 * C * C + t * C + s) = hi;
-    *reinterpret_cast<uint32_t*>(am + 3 * C * C + t * C + s) = lw;
+    *reinterpret_cast<uint32_t*>(am + (2 * C + t) * I.PA + s) = hi;
+    *reinterpret_cast<uint32_t*>(am + (3 * C + t) * I.PA + s) = lw;
   }
 }
 
-// NK: 16-channel tiles of the key width (padded). Stage layout in shared memory: q, k, k' high | low [6][C][P], v [C][72], A and T high | low
-// [4][C][C + 8], decay [16 NK] fp32.
+// A stage: the image of a chunk, then v [C][72].
 template <int C, int NK>
 struct DeltaStage {
   static constexpr int P = NK * 16 + 8, PV = kDnCols + 8, PA = C + 8;
-  static constexpr int kV = 6 * C * P * 2;
-  static constexpr int kA = kV + C * PV * 2;
-  static constexpr int kDec = kA + 4 * C * PA * 2;
-  static constexpr int kBytes = (kDec + NK * 16 * 4 + 127) / 128 * 128;
+  static constexpr int kA = DeltaImage<C>(NK).off_a, kDec = DeltaImage<C>(NK).off_dec, kV = DeltaImage<C>(NK).bytes;
+  static constexpr int kBytes = (kV + C * PV * 2 + 127) / 128 * 128;
   static constexpr int PO = kDnCols + 4;
   static constexpr int kOut = 2 * kBytes;                        // both halves' shares of the outputs [2][C][PO]
   static constexpr int kR = kOut + 2 * C * PO * 4;               // shares of S^T K'^T: [8 warps][C / 2][32 lanes]
@@ -549,7 +571,7 @@ struct DeltaStage {
 };
 
 template <int C, int NK>
-__global__ void __launch_bounds__(256, 1) delta_chunks_kernel(const DeltaArgs a, const DeltaChunks c) {
+__global__ void __launch_bounds__(256, C == 16 && NK <= 8 ? 2 : 1) delta_chunks_kernel(const DeltaArgs a, const DeltaChunks c) {
   pdl_wait();
   pdl_trigger();
   using L = DeltaStage<C, NK>;
@@ -563,32 +585,19 @@ __global__ void __launch_bounds__(256, 1) delta_chunks_kernel(const DeltaArgs a,
   if (n_chunks == 0) return;
   const int dk = a.dk, dv = a.dv, width = 2 * a.G * dk + a.H * dv;
   const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.qkv) + 2 * a.G * dk + h * dv;
-  const __nv_bfloat16* qk = static_cast<const __nv_bfloat16*>(c.qk);
-  const __nv_bfloat16* am = static_cast<const __nv_bfloat16*>(c.a);
   float* state = a.state + (static_cast<size_t>(a.slots[s]) * a.H + h) * dk * dv;
   const bool fresh = a.positions[a.q_start[s]] == 0;
 
   auto load = [&](int i, int stage) {
     const int ck = first + i, row0 = c.row0[ck], len = c.len[ck];
     const uint32_t base = smem_u32(dsm + stage * L::kBytes);
-    constexpr int CH = NK * 2;  // 16-byte pieces per row and plane
-    for (int e = tid; e < 6 * C * CH; e += 256) {
-      const int x = e % CH, t = (e / CH) % C, plane = e / (CH * C);
-      const bool ok = t < len && x * 8 < dk;
-      const __nv_bfloat16* src = qk + ((static_cast<size_t>(row0 + (ok ? t : 0)) * a.H + h) * 6 + plane) * dk + (ok ? x * 8 : 0);
-      cp16(base + ((plane * C + t) * L::P + x * 8) * 2, src, ok);
-    }
+    const uint8_t* image = static_cast<const uint8_t*>(c.images) + (static_cast<size_t>(ck) * a.H + h) * L::kV;
+    for (int e = tid * 16; e < L::kV; e += 256 * 16) cp16(base + e, image + e, true);
     for (int e = tid; e < C * 8; e += 256) {
       const int t = e >> 3, x = (e & 7) * 8;
       const bool ok = t < len && c0 + x < dv;
       cp16(base + L::kV + (t * L::PV + x) * 2, vp + static_cast<size_t>(row0 + (ok ? t : 0)) * width + (ok ? c0 + x : 0), ok);
     }
-    const __nv_bfloat16* ap = am + (static_cast<size_t>(ck) * a.H + h) * 4 * C * C;
-    for (int e = tid; e < 4 * C * (C / 8); e += 256) {
-      const int r = e / (C / 8), x = (e % (C / 8)) * 8;
-      cp16(base + L::kA + (r * L::PA + x) * 2, ap + r * C + x, true);
-    }
-    for (int e = tid; e < NK * 4; e += 256) cp16(base + L::kDec + e * 16, c.decay + (static_cast<size_t>(ck) * a.H + h) * dk + (e * 4 < dk ? e * 4 : 0), e * 4 < dk);
     cp_commit();
   };
 
@@ -604,13 +613,9 @@ __global__ void __launch_bounds__(256, 1) delta_chunks_kernel(const DeltaArgs a,
       st[j][e] = (!fresh && d < dk && col < dv) ? state[static_cast<size_t>(d) * dv + col] : 0.f;
     }
   for (int i = 0; i < n_chunks; ++i) {
-    if (i + 1 < n_chunks) {
-      load(i + 1, (i + 1) & 1);
-      cp_wait<1>();
-    } else {
-      cp_wait<0>();
-    }
-    __syncthreads();
+    cp_wait<0>();
+    __syncthreads();  // the chunk has arrived, and all warps are done with the one in front of it
+    if (i + 1 < n_chunks) load(i + 1, (i + 1) & 1);
     const uint32_t base = smem_u32(dsm + (i & 1) * L::kBytes);
     const float* dec = reinterpret_cast<const float*>(dsm + (i & 1) * L::kBytes + L::kDec);
     const __nv_bfloat16* sv = reinterpret_cast<const __nv_bfloat16*>(dsm + (i & 1) * L::kBytes + L::kV);
@@ -737,10 +742,11 @@ __global__ void __launch_bounds__(256, 1) delta_chunks_kernel(const DeltaArgs a,
         mma16816(st[2 * jp], uh[ks], b[0], b[1]);
         mma16816(st[2 * jp + 1], uh[ks], b[2], b[3]);
       }
-    __syncthreads();  // the stage is refilled by the next iteration's load; both shares of the outputs are complete
+    asm volatile("bar.sync %0, 64;" ::"r"(1 + wd) : "memory");  // both shares of these 16 columns are there
     const int row0 = c.row0[first + i], len = c.len[first + i];
-    for (int e = tid; e < C * (kDnCols / 4); e += 256) {
-      const int t = e / (kDnCols / 4), x = (e % (kDnCols / 4)) * 4;
+#pragma unroll
+    for (int e = hk * 32 + lane; e < C * 4; e += 64) {
+      const int t = e >> 2, x = wd * 16 + (e & 3) * 4;
       if (t >= len || c0 + x >= dv) continue;
       const float4 p = *reinterpret_cast<const float4*>(so + t * L::PO + x), w = *reinterpret_cast<const float4*>(so + (C + t) * L::PO + x);
       *reinterpret_cast<float4*>(a.o + static_cast<size_t>(row0 + t) * (a.H * dv) + h * dv + c0 + x) = make_float4(p.x + w.x, p.y + w.y, p.z + w.z, p.w + w.w);
@@ -766,28 +772,28 @@ static cudaError_t launch_chunks_t(const DeltaArgs& a, const DeltaChunks& c, cud
   return launch_pdl(delta_chunks_kernel<C, NK>, dim3((a.dv + kDnCols - 1) / kDnCols, a.H, a.num_seqs), dim3(256), L::kTotal, st, a, c);
 }
 
-template <int C>
+template <int C, int R>
 static cudaError_t launch_prepare_t(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t st) {
-  const size_t smem = static_cast<size_t>(DeltaPrepareSmem<C>(a.dk).bytes);
+  const size_t smem = static_cast<size_t>(DeltaPrepareSmem<C, R>(a.dk).bytes);
   static PerDeviceOnce once;
   if (once.first()) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_prepare_kernel<C>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(delta_prepare_kernel<C, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
     if (e != cudaSuccess) return e;
   }
-  return launch_pdl(delta_prepare_kernel<C>, dim3(c.n_chunks, a.H), dim3(256), smem, st, a, c);
+  return launch_pdl(delta_prepare_kernel<C, R>, dim3(c.n_chunks, a.H), dim3(256), smem, st, a, c);
 }
 
-int launch_delta_chunked(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t st) {
+int launch_delta_chunked(const DeltaArgs& a, DeltaChunks c, cudaStream_t st) {
   if (a.rows == 0 || c.n_chunks == 0) return 0;
+  c.tiles = delta_tiles(a.dk);
   cudaError_t e;
-  if (c.chunk == 32 && a.dk <= 128) e = launch_prepare_t<32>(a, c, st);
-  else if (c.chunk == 16 && a.dk <= 256) e = launch_prepare_t<16>(a, c, st);
+  if (c.chunk == 32 && a.dk <= 128) e = launch_prepare_t<32, 8>(a, c, st);
+  else if (c.chunk == 16 && a.dk <= 128) e = launch_prepare_t<16, 4>(a, c, st);
+  else if (c.chunk == 16 && a.dk <= 256) e = launch_prepare_t<16, 8>(a, c, st);
   else return 1;
   if (e == cudaSuccess) {
-    if (c.chunk == 32 && a.dk <= 32) e = launch_chunks_t<32, 2>(a, c, st);
-    else if (c.chunk == 32 && a.dk <= 64) e = launch_chunks_t<32, 4>(a, c, st);
-    else if (c.chunk == 32) e = launch_chunks_t<32, 8>(a, c, st);
-    else e = launch_chunks_t<16, 16>(a, c, st);
+    if (c.chunk == 16) e = c.tiles == 16 ? launch_chunks_t<16, 16>(a, c, st) : c.tiles == 8 ? launch_chunks_t<16, 8>(a, c, st) : c.tiles == 4 ? launch_chunks_t<16, 4>(a, c, st) : launch_chunks_t<16, 2>(a, c, st);
+    else e = c.tiles == 8 ? launch_chunks_t<32, 8>(a, c, st) : c.tiles == 4 ? launch_chunks_t<32, 4>(a, c, st) : launch_chunks_t<32, 2>(a, c, st);
   }
   if (e == cudaSuccess) e = launch_norm_gate(a, false, st);
   return e == cudaSuccess ? 0 : 2;

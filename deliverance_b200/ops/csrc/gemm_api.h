@@ -319,12 +319,12 @@ struct DeltaChunks {
   const int *seq, *row0, *len;  // per chunk
   const int *first, *count;     // per sequence
   int n_chunks, chunk;
-  void* qk;      // bf16 [T, H, 6, dk]: q exp(b), k exp(b_end - b), k exp(b), high and low parts
-  void* a;       // bf16 [n_chunks, H, 4, chunk, chunk]: causal matrix, (I + M)^-1 beta, high and low parts
-  float* decay;  // [n_chunks, H, dk]
+  void* images;  // [n_chunks, H, delta_image_bytes]: scaled queries and keys, causal matrix, (I + M)^-1 beta, decay over the chunk
+  int tiles;     // (set by the launch)
 };
 int launch_delta_recurrent(const DeltaArgs& a, bool is_f32, cudaStream_t st);  // qkv == nullptr: one row per sequence, norm and gate in the launch
-int launch_delta_chunked(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t st);
+int64_t delta_image_bytes(int dk, int chunk);
+int launch_delta_chunked(const DeltaArgs& a, DeltaChunks c, cudaStream_t st);
 
 // mixed.cu: attention with mixed scores over wide cache rows k [pages, 1, page, KV dk], v [pages, 1, page, KV dv]
 struct MixedDecodeArgs {

@@ -27,6 +27,7 @@ from .short_conv import ring_shape, short_conv
 
 MAX_DK = 512  # key channels per head the CUDA kernels take
 MAX_DK_CHUNKED = 256
+MAX_DK_CHUNK32 = 128  # wider keys: chunks of 16 tokens
 MAX_DV_FUSED = 512  # one cluster of eight CTAs per head norms and gates inside the decode launch
 UNIT_EPS = 1e-6  # under the root of the unit vectors' length
 
@@ -80,10 +81,11 @@ class DeltaShape:
     def out_width(self) -> int:
         return self.heads * self.dv
 
-    @property
-    def chunk(self) -> int:
-        """Tokens per chunk of the chunked form (shared memory of two stages bounds it)."""
-        return 32 if self.dk <= 128 else 16
+    def chunk(self, lengths, sms: int = 148) -> int:
+        """Tokens per chunk of the chunked form: 32 where shared memory holds two stages of them, unless the walks of the batch's prompts are more than
+        the processors; two walks over chunks of 16 fit one processor."""
+        walks = sum(n > 32 for n in lengths) * self.heads * ((self.dv + 63) // 64)
+        return 32 if self.dk <= MAX_DK_CHUNK32 and walks <= sms else 16
 
     def state_shapes(self) -> dict:
         return {"conv": ring_shape(self.taps, self.conv_width), "delta": (self.heads, self.dk, self.dv)}
@@ -112,7 +114,8 @@ def delta(s: DeltaShape, p, z, gate, conv_w, dt_bias, neg_a, norm_w, ring, state
         qkv = short_conv(p, 0, conv_w, None, ring, batch)
         chunked = not batch.is_decode and p.dtype == torch.bfloat16 and s.dk <= MAX_DK_CHUNKED
         ops._count(3 if chunked else 2)
-        e.delta_prompt(p, qkv, *args, s.chunk, list(chunk_plan(batch, s.chunk)) if chunked else [])
+        chunk = s.chunk(batch.q_len_host) if chunked else 0
+        e.delta_prompt(p, qkv, *args, chunk, list(chunk_plan(batch, chunk)) if chunked else [])
         return
     qkv = short_conv(p, 0, conv_w, None, ring, batch)
     T, H, G = p.shape[0], s.heads, s.kv_heads

@@ -799,12 +799,16 @@ def test_prompt_kernels_agree_with_the_row_forms_on_cuda():
         finally:
             gop.ops.require_ext, mop.MAX_STATE_CHUNKED, dop.MAX_DK_CHUNKED = old
 
+    wide = dop.MAX_DK_CHUNK32
     ops.set_bounds_check(True)
     try:
         cases = [("attention",) + attention_case(run, *a) for a in ((8, 2, 64, 64, 100), (16, 4, 128, 128, 256), (24, 4, 128, 128, 0), (16, 8, 128, 64, 300), (8, 1, 40, 256, 77))]
         cases += [("ssm",) + mamba_case(run, *a) for a in ((8, 64, 128, 1, 4, 1), (4, 96, 64, 2, 4, 2), (2, 40, 200, 1, 3, 1))]
         cases += [("delta",) + delta_case(run, *a)[:5] for a in ((4, 2, 128, 128, 4, 16, 16), (2, 2, 64, 192, 4, 8, 8), (2, 1, 256, 64, 3, 8, 8))]
+        cases += [("delta 16",) + delta_case(run, *a)[:5] for a in ((4, 2, 128, 128, 4, 16, 16), (2, 2, 24, 48, 4, 8, 8), (2, 1, 56, 64, 3, 8, 8))]
         for name, mixer, m, W, kv, pages in cases:
+            name, _, short = name.partition(" ")  # chunks of 16 tokens where the batch would get 32
+            dop.MAX_DK_CHUNK32 = 0 if short else wide
             a = run_mixer(mixer, kv, h, [256, 424] + [1] * 20, pages, run)
             b = row_forms(lambda: run_mixer(mixer, kv, h, [256, 444], pages[::-1], run, 2))  # noqa: B023
             e = rows_rel(a, b)
@@ -819,4 +823,5 @@ def test_prompt_kernels_agree_with_the_row_forms_on_cuda():
             ops.check_guards()
         ops.check_status()
     finally:
+        dop.MAX_DK_CHUNK32 = wide
         ops.set_bounds_check(False)
