@@ -134,7 +134,7 @@ def kernel_times(fop, moe, z: dict, t: Timer, peaks: dict) -> list:
             (T * (H * (z["dim"] // 2) + 2 * KV * D) * 4, 0),
             lambda: ops.rope_kv(qkv, b.positions, b.slots, None, None, moe.cos, moe.sin, kc, vc, H, KV, D, 1e-5), (T * (H + 2 * KV) * D * 4, 0))
         win, keep = z["window"], z["keep"]
-        att = (sx.scale, sx.softcap, win, keep, True)
+        att = (sx.scale, sx.softcap, win, keep, sx.sink)
         if n == 1:
             span = min(2048, win + keep)
             sp = ops.decode_splits(B, KV, span)
@@ -145,7 +145,7 @@ def kernel_times(fop, moe, z: dict, t: Timer, peaks: dict) -> list:
             pairs = lambda w: B * (n * (n + 1) / 2 if w >= n else w * (n - w) + w * (w + 1) / 2)  # noqa: E731
             for cap in (50.0, 0.0):
                 tail = " soft-capped" if cap else " no cap"
-                add(f"prompt attention {tag}{tail}", lambda: gop.attention(s, qkv, b, kc, vc, sx.scale, cap, win, keep, True, 1),
+                add(f"prompt attention {tag}{tail}", lambda: gop.attention(s, qkv, b, kc, vc, sx.scale, cap, win, keep, sx.sink, 1),
                     (0, 4.0 * (pairs(win) + B * keep * max(0, n - win - keep)) * H * D),
                     lambda: ops.prefill_attention(q, kc, vc, b.block_tables, b.q_start, b.q_len, b.ctx_len, H, D ** -0.5, cap, win, True, b.tile_seq, b.tile_q0,
                                                   tiles_for=b.tiles), (0, 4.0 * pairs(win) * H * D))
