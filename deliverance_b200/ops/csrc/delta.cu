@@ -205,9 +205,9 @@ template <typename TIO>
 __global__ void __launch_bounds__(256) delta_norm_gate_kernel(const DeltaArgs a) {
   pdl_wait();
   pdl_trigger();
-  const long long w = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  const unsigned w = blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (w >= static_cast<long long>(a.rows) * a.H) return;
+  if (w >= static_cast<unsigned>(a.rows) * a.H) return;
   const int t = static_cast<int>(w / a.H), h = static_cast<int>(w % a.H);
   const float* o = a.o + static_cast<size_t>(t) * (a.H * a.dv) + h * a.dv;
   const TIO* z = static_cast<const TIO*>(a.gate) + static_cast<size_t>(t) * a.ld_gate + h * a.dv;
@@ -224,12 +224,13 @@ __global__ void __launch_bounds__(256) delta_norm_gate_kernel(const DeltaArgs a)
     io_ld4(a.norm_w + c, nw);
     io_ld4(z + c, zv);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) v[e] *= inv * nw[e] * dn_sigmoid(zv[e]);
+    for (int e = 0; e < 4; ++e) v[e] *= inv * nw[e] * (sizeof(TIO) == 2 ? __fdividef(1.f, 1.f + __expf(-zv[e])) : dn_sigmoid(zv[e]));
     io_st4(out + c, v);
   }
 }
 
 static cudaError_t launch_norm_gate(const DeltaArgs& a, bool is_f32, cudaStream_t st) {
+  if (static_cast<long long>(a.rows) * a.H > (1ll << 31)) return cudaErrorInvalidValue;
   const dim3 grid(static_cast<unsigned>((static_cast<long long>(a.rows) * a.H + 7) / 8));
   return is_f32 ? launch_pdl(delta_norm_gate_kernel<float>, grid, dim3(256), 0, st, a) : launch_pdl(delta_norm_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a);
 }
