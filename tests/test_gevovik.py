@@ -111,7 +111,7 @@ def test_squared_relu_feed_forward(run, ff, width, T):
 YARN = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 2.0}
 
 
-@pytest.mark.parametrize("dims,base,scaling", [(16, 10000.0, None), (12, 500.0, YARN), (64, 5e5, dict(YARN, original=512, fast=32.0, slow=1.0)), (2, 100.0, YARN),
+@pytest.mark.parametrize("dims,base,scaling", [(16, 10000.0, None), (12, 500.0, YARN), (64, 3e5, dict(YARN, original=700, fast=24.0, slow=1.0)), (2, 100.0, YARN),
                                                (24, 700.0, dict(YARN, fast=1.0, slow=1.0, factor=3.0))])
 def test_rotations(dims, base, scaling):
     rot, extra = {"dims": dims, "base": base, "scaling": scaling}, 3
@@ -342,7 +342,7 @@ def attention_case(run, H, G, dk, dv, window, rot=None, scale=None, width=WIDTH,
 
 # heads, kv heads, dim, vdim, window, rotated: odd widths, one head, more than 16 heads per KV head, as many KV heads as heads, cache rows of every form of the
 # prompt kernel (64 / 128 / 256 columns, pieces of rows up to 512 and beyond), values narrower and wider than keys, sizes outside the decode kernel
-MIXED = [(1, 1, 2, 1, 5, 2), (6, 2, 20, 12, 40, 6), (4, 1, 64, 64, 33, 64), (6, 3, 64, 64, 64, 32), (20, 1, 16, 24, 50, 16), (36, 2, 24, 40, 100, 8), (8, 8, 40, 40, 32, 20),
+MIXED = [(1, 1, 2, 1, 5, 2), (6, 2, 20, 12, 40, 6), (4, 1, 64, 64, 33, 64), (6, 3, 72, 64, 64, 32), (20, 1, 16, 24, 50, 16), (36, 2, 24, 40, 100, 8), (8, 8, 40, 40, 32, 20),
          (4, 4, 128, 128, 70, 128), (5, 5, 104, 72, 45, 24), (6, 6, 128, 64, 96, 64), (10, 10, 64, 200, 31, 64), (2, 2, 264, 24, 20, 16), (3, 1, 24, 300, 60, 24), (66, 2, 8, 8, 40, 8)]
 
 
